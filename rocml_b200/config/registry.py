@@ -27,7 +27,8 @@ def register_architecture(name: str, config_from_dict: Callable) -> None:
     """Make ``name`` (the string in config.json's ``architectures``) loadable.
 
     ``config_from_dict(d)`` returns the typed configuration; it must offer
-    ``to_model_spec() -> ModelSpec`` and ``to_dict() -> dict``.
+    ``to_model_spec() -> ModelSpec`` and ``to_dict() -> dict``, and may offer ``with_tensor_shapes(shape_of)``:
+    the configuration completed by sizes that only the tensors' shapes tell.
     """
     _ARCHITECTURES[name] = config_from_dict
 
@@ -68,7 +69,7 @@ def load_config(folder: str):
         raise ConfigError(f"{path} is not valid JSON: {e}") from e
     if not isinstance(d, dict):
         raise ConfigError(f"{path} does not hold a JSON object")
-    cfg = config_from_dict(d)
+    cfg = _with_tensor_shapes(config_from_dict(d), os.path.dirname(path))
     gen = os.path.join(os.path.dirname(path), "generation_config.json")
     extra_stop = ()
     if os.path.isfile(gen):
@@ -80,6 +81,19 @@ def load_config(folder: str):
         except (json.JSONDecodeError, OSError):
             extra_stop = ()
     return cfg, extra_stop
+
+
+def _with_tensor_shapes(cfg, folder: str):
+    """A configuration that leaves some sizes to the tensors (it has ``with_tensor_shapes``) reads them from the folder's
+    files; without files it stays as it is."""
+    if not hasattr(cfg, "with_tensor_shapes"):
+        return cfg
+    from ..weights.safetensors_io import ModelFiles
+    try:
+        with ModelFiles(folder) as files:
+            return cfg.with_tensor_shapes(lambda name: tuple(files.shape(name)) if name in files else None)
+    except ModelFileMissing:
+        return cfg
 
 
 def load_model_spec(folder: str) -> ModelSpec:

@@ -34,7 +34,8 @@ def tensor_names(params: Mapping[str, Any], defaults: Mapping[str, str]) -> dict
 @dataclass(frozen=True)
 class NormSpec:
     """A normalisation over the last axis.  kind "rmsnorm": x * rsqrt(mean(x^2) + eps) * (w + weight_offset);
-    ``weight_offset`` 1 is a weight that the files store around zero."""
+    ``weight_offset`` 1 is a weight that the files store around zero.  kind "layernorm": (x - mean) / sqrt(variance + eps) * w + b,
+    with a bias tensor beside the weight."""
 
     kind: str = "rmsnorm"
     eps: float = 1e-6
@@ -52,7 +53,8 @@ class PositionSpec:
     ({factor, original, fast, slow}: frequencies blended between f and f / factor along a ramp over
     the pair index, and cosines and sines times 0.1 ln(factor) + 1); kind "none": nothing.
     As a model's ``input_position`` (added to the embedding output, not applied inside a mixer):
-    kind "sinusoid": entry 2i of the vector is sin(pos * theta^(-2i / width)), entry 2i + 1 the cosine.
+    kind "sinusoid": entry 2i of the vector is sin(pos * theta^(-2i / width)), entry 2i + 1 the cosine; kind "learned": row pos of a table with
+    the parameter ``rows`` rows.
     """
 
     kind: str = "rope_neox"
@@ -86,7 +88,9 @@ class MixerSpec:
     root mean square over the head, without a weight, after the position encoding; eps is
     qk_norm_eps), value_mix ("source": this layer's values as projected are kept for the step;
     "mix": what is cached and read is (1 - lambda) v + lambda v_source, lambda the layer's scalar
-    tensor of role value_mix, v_source the values of the same token in the step's source layer).
+    tensor of role value_mix, v_source the values of the same token in the step's source layer), sink "per_head" (a tensor of
+    role sink with a score for every query head), q_temperature ({coef, every}: the query at position p is multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1)).
     """
 
     kind: str
@@ -97,6 +101,11 @@ class MixerSpec:
     # size a sequence): n_heads, head_dim, v_head_dim, decay (one number a head), qk_activation and v_activation
     # ("none" | "silu"), k_scale, out_norm ("per_head" | "all_heads") with out_norm_eps and out_norm_weight (bool),
     # gate_activation ("silu" | "sigmoid"), names (roles q, k, v, gate, o, out_norm).
+    # Kind "gated_delta" (the gated delta rule; see parts/gated_delta.py): n_heads, n_kv_heads, head_dim, v_head_dim, conv_taps,
+    # decay ("per_head" | "per_channel" with decay_rank), gate ("silu" | "sigmoid_low_rank" with gate_rank), out_norm_eps,
+    # unit_eps, names.
+    # Kind "side_by_side" (two mixers on one input; see parts/side_by_side.py): left and right (MixerSpecs), left_scale,
+    # right_scale, prefixes (the tensor-name prefixes of the sides under the layer's mixer prefix).
     # Kind "latent_attention" (keys and values unfolded from one cached latent vector a token): n_heads, head_dim
     # (queries and keys), v_head_dim, kv_rank, latent_norm_eps, window, scale, gated (a sigmoid gate per head on the
     # attention's output, read from the mixer's input), names (roles q, down, latent_norm, up_k, up_v, gate, o).
@@ -119,7 +128,8 @@ class FeedForwardSpec:
     up, down; default gate_proj, up_proj, down_proj).
 
     routed_mlp (a router and ``experts`` small gated feed-forwards, ``top`` of them a token) params: experts, top,
-    intermediate, activation ("silu" or "clamped_swish" with ``limit`` and ``alpha``), score ("sigmoid"),
+    intermediate, activation ("silu" or "clamped_swish" with ``limit`` and ``alpha``), score ("sigmoid" or "softmax" over all
+    experts), identity (so many more experts that have no tensors and give their input back),
     choice_bias (a per-expert vector added to the scores for the choice only), renormalize, names (roles router,
     choice_bias, expert (a pattern with {e}), gate, up, down).
     """
@@ -149,6 +159,8 @@ class LayerSpec:
     sum and the sublayers read the stream itself.  Its constants are ``arrangement_items``: alpha (default 1),
     layer_scale (the vectors g1, g2 exist; default False), token_shift (h_t = x_t + (x_(t-1) - x_t) * mu with a vector mu,
     the row before kept per sequence; default False: h = x), names (roles mixer_scale, ff_scale, shift).
+    arrangement "output_norm": x += m * norm1(mixer(x)); x += m * norm2(ff(x)), no norm before a sublayer; its constant in
+    ``arrangement_items`` is multiplier (m, default 1); ``feed_forward`` None leaves the second half out.
     ``prefix`` is the layer's tensor-name prefix in the weight files; under it the four parts'
     tensors are named ``<prefix>.<mixer_norm_name>.weight``, ``<prefix>.<mixer_name><stem>...``,
     ``<prefix>.<ff_norm_name>.weight`` and ``<prefix>.<ff_name><stem>...`` (the defaults are the
@@ -219,6 +231,8 @@ class ModelSpec:
     bias_suffix: str = ".bias"                         # the same for a part's '<stem>.bias'
     embedding_norm: Optional[NormSpec] = None          # a norm of the embedding output, before the first layer
     embedding_norm_name: str = "model.embed_norm.weight"
+    input_position_name: str = "model.embed_positions.weight"   # the table of an input position that has one
+    logit_softcap: Optional[float] = None              # logits <- cap * tanh(logits / cap), after logit_scale
 
     def __post_init__(self):
         n = len(self.layers)

@@ -18,9 +18,10 @@ int rb_silu_mul(const void* in, int in_dtype, int n_in, long long in_stride, voi
                 int I, int paired, void* stream);
 
 // Embedding rows times `scale` plus, when inv_freq is given, a sinusoid position vector (even entries sine, odd
-// cosine of positions[t] * inv_freq[i / 2]); `copy` (optional) receives the same rows.
+// cosine of positions[t] * inv_freq[i / 2]), or, when pos_table is given, its row positions[t]; `copy` (optional) receives the same rows.
 int rb_embedding_pos(const int* ids, const void* table, int table_dtype, float* out, float* copy, int T, int H,
-                     int vocab, float scale, const int* positions, const float* inv_freq, int* status, void* stream);
+                     int vocab, float scale, const int* positions, const float* inv_freq, const void* pos_table,
+                     int pos_dtype, int pos_rows, int* status, void* stream);
 
 // resid += sum of delta partial sums (+ other) (+ vec, broadcast over the rows); each may be absent.
 int rb_residual_inject(float* resid, const float* delta, int n_delta, long long delta_stride, const float* other,
@@ -40,6 +41,8 @@ int rb_gated_act(const void* in, int in_dtype, int n_in, long long in_stride, lo
                  long long out_ld, int rows, int I, int kind, float limit, float alpha, int paired, void* stream);
 
 int rb_scale(float* x, long long n, float factor, void* stream);
+// x <- cap * tanh(factor * x / cap), in place, 32-bit.
+int rb_softcap(float* x, long long n, float factor, float cap, void* stream);
 
 // out[t, h, :out_w] = in[t, h, :out_w] * gate for heads of in_w (>= out_w) values; gate float32 [T, heads * gate_w]
 // (gate_w 1: one a head, out_w: one a value), or the sigmoid of `raw` (such columns of projection rows, n_in
@@ -59,18 +62,20 @@ int rb_latent_prep(const void* in, int in_dtype, int n_in, long long in_stride, 
 int rb_router_logits(const void* x, int x_dtype, long long ldx, const float* w, float* z, int ldz, int T, int E, int K,
                      void* stream);
 // n_groups > 1: only experts of the keep_groups best groups of neighbours can be chosen (a group's score: its two
-// largest scores added); renormalize: weights divided by their sum + norm_eps.
+// largest scores added); renormalize: weights divided by their sum + norm_eps.  score 0: sigmoid, 1: softmax over all
+// E.  The last `identity` of the E are identity experts: a choice of one gets no row (id -1), its weight is summed into
+// self_weight[t].
 int rb_moe_route(const float* z, int ldz, const void* bias, int bias_dtype, const int* slot_of_token, int T, int E,
                  int top, int* ids, float* weights, int* place, int* counts, int n_groups, int keep_groups,
-                 int renormalize, float norm_eps, void* stream);
+                 int renormalize, float norm_eps, int score, int identity, float* self_weight, void* stream);
 int rb_moe_plan(const int* counts, int E, int tile_rows, int max_tiles, int* starts, int* tile_group, void* stream);
 int rb_moe_gather(const void* x, int dtype, int H, const int* ids, const int* place, const int* starts, int T, int top,
                   void* rows, int* row_of, void* stream);
 // extra (optional): [n_extra][T, H] partial sums added to every token's row, times sigmoid(extra_gate[t * ld]) when
-// extra_gate is given.
+// extra_gate is given; self_weight (optional): plus self_weight[t] * self_x[t].
 int rb_moe_combine(const float* y, long long ldy, const int* row_of, const float* weights, int T, int top, float* out,
                    int H, const float* extra, int n_extra, long long extra_stride, const float* extra_gate,
-                   int extra_gate_ld, void* stream);
+                   int extra_gate_ld, const float* self_weight, const void* self_x, int self_dtype, void* stream);
 
 // Linear attention with a fixed decay per head (linear_attention.cu).  The step's tokens go through
 // S = decay[h] * S + k v^T, o = S^T q per (sequence, head), the state [slots, heads, dim, vdim] float32 read and
@@ -111,7 +116,7 @@ int rb_qk_norm_rope_cache(const void* in, int in_dtype, int n_in, long long in_s
                           const int* positions, const int* slot_of_token, const int* block_table, int max_pages,
                           void* k_cache, void* v_cache, int write_kv, const void* cos_sin, int vd, int hdp,
                           int interleaved, int n_gate, float* gate_out, int post_norm, const float* v_first,
-                          const float* v_lambda, float* v_out, void* stream);
+                          const float* v_lambda, float* v_out, float temp_coef, float temp_every, void* stream);
 
 int rb_rope_table(const int* positions, const float* inv_freq, int T, int half, float mag, void* out, void* stream);
 
@@ -154,23 +159,23 @@ int rb_gemm_tcgen05_add(const void* x, const void* w, const float* bias, float* 
 int rb_attention_generic(const void* q, int q_stride, void* out, int o_stride, int dtype, const void* k_cache,
                          const void* v_cache, const int* block_table, int max_pages, const int* seq_slot,
                          const int* cu_q, const int* kv_len, int B, int max_q_len, int nq, int nkv, int hd,
-                         float scale, int window, int keep, float sink, int chunk, int n_chunks, float* part_acc,
+                         float scale, int window, int keep, float sink, const float* sinks, int chunk, int n_chunks, float* part_acc,
                          float* part_ml, int cross, void* stream);
 
 int rb_attention_prefill(const void* q, int q_stride, void* out, int o_stride, const void* k_cache,
                          const void* v_cache, const int* block_table, int max_pages, const int* seq_slot,
                          const int* cu_q, const int* kv_len, int B, int max_q_len, int nq, int nkv, int hd, float scale,
-                         int window, int keep, float sink, void* stream);
+                         int window, int keep, float sink, const float* sinks, void* stream);
 
 int rb_attention_prefill_tc5(const void* q, int q_stride, int T, void* out, int o_stride, const void* k_cache,
                              const void* v_cache, int n_pages, const int* block_table, int max_pages,
                              const int* seq_slot, const int* cu_q, const int* kv_len, int B, int max_q_len, int nq,
-                             int nkv, int hd, float scale, int window, int keep, float sink, int heads_first, int* status,
+                             int nkv, int hd, float scale, int window, int keep, float sink, const float* sinks, int heads_first, int* status,
                              const void* gate, long long gate_row_stride, int cross, void* stream);
 
 int rb_attention_decode(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                         const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
-                        const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window, int keep, float sink,
+                        const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window, int keep, float sink, const float* sinks,
                         int n_chunks, int pages_per_block, float* part_acc, float* part_ml, int* counters, void* out,
                         int o_stride, const void* gate, int gate_f32, int gate_n_in, long long gate_in_stride,
                         long long gate_row_stride, int cross, void* stream);
@@ -181,13 +186,14 @@ int rb_attention_decode_fused(const float* proj, int n_in, long long in_stride, 
                               int row_width, void* k_cache, void* v_cache, const int* block_table, int max_pages, const int* seq_slot,
                               const int* cu_q, const int* kv_len, int B, int nq, int nkv, int hd, float scale,
                               int window, int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
-                              int* counters, void* out, int o_stride, int keep, float sink, int rot_dim, int post_norm,
+                              int* counters, void* out, int o_stride, int keep, float sink, const float* sinks, float temp_coef,
+                              float temp_every, int rot_dim, int post_norm,
                               const float* v_first, const float* v_lambda, float* v_keep, const void* gate, int gate_f32,
                               int gate_n_in, long long gate_in_stride, long long gate_row_stride, void* stream);
 
 int rb_attention_merge(const float* part_acc, const float* part_ml, void* out, int o_stride, int dtype,
                        const int* positions, const int* slot_of_token, int T, int nq, int hd, int chunk,
-                       int n_chunks, int window, int keep, float sink, void* stream);
+                       int n_chunks, int window, int keep, float sink, const float* sinks, void* stream);
 
 int rb_argmax(const float* logits, long long row_stride, int rows, int V, int* out, float* scratch_v,
               int* scratch_i, int slices, void* stream);
@@ -248,6 +254,38 @@ int rb_latent_rot_prep(const void* in, int in_dtype, int n_in, long long in_stri
                        const int* slot_of_token, const int* block_table, int max_pages, int T, void* stream);
 int rb_latent_q_rot(const void* q, int q_stride, int heads, int dim, int rot, int rank, int dp, const float* cos_sin,
                     void* folded, int f_stride, int dtype, const int* slot_of_token, int T, void* stream);
+
+// Layer norms and norms of a sublayer's result (outnorm.cu).  rb_add_layernorm: as rb_add_rmsnorm with
+// out = (r - mean) / sqrt(variance + eps) * w + b; w and b float32.
+int rb_add_layernorm(float* resid, const float* delta, int n_delta, long long delta_stride, const float* w, const float* b,
+                     void* out, int out_dtype, const int* rows, int n_rows, int H, float eps, int write_back, void* stream);
+// resid += mult * norm(d), in place; d = d_scale * (sum of the delta partial sums), or, with row_of, d_scale * (the weighted
+// sum of a token's rows of delta plus self_weight[t] * self_x[t]).  layer 1: layer norm, 0: RMS norm; b may be absent.  out
+// (optional) receives the new rows in its own type.
+int rb_out_norm(float* resid, const float* delta, int n_delta, long long delta_stride, float d_scale, const int* row_of,
+                const float* weights, int top, const float* self_weight, const void* self_x, int self_dtype, int layer,
+                const float* w, const float* b, float eps, float mult, void* out, int out_dtype, int n_rows, int H,
+                void* stream);
+
+// The gated delta rule (gated_delta.cu).  rb_delta_prep: from a layer's projection rows, the short convolutions with silu,
+// the unit norms of q and k, step sizes and decays, into rows of u (float32, row stride ld_u): q at uq, k at uk (kv_heads *
+// dim each), v at uv (heads * vdim), decays at ug (heads, or heads * dim when per_channel), step sizes at ub (heads), q . k
+// at ud (kv_heads).  conv_w float32 [taps][q | k | v channels], kept float32 [slots][taps - 1][channels]; z: what the decays
+// are made from, columns z_off.. of rows of its own.
+int rb_delta_prep(const void* in, int in_dtype, int n_in, long long in_stride, int row_stride, int q_off, int k_off, int v_off,
+                  int b_off, int heads, int kv_heads, int dim, int vdim, int taps, const float* conv_w, float* kept,
+                  const void* z, int z_dtype, int z_n_in, long long z_in_stride, int z_row_stride, const float* dt_bias,
+                  const float* a_log, int per_channel, float unit_eps, float q_scale, const int* seq_slot, const int* cu_q,
+                  int n_seqs, int max_q_len, float* u, int ld_u, int uq, int uk, int uv, int ug, int ub, int ud, void* stream);
+// S <- g S; w = beta (v - S^T k); S <- S + k w^T; o = S^T q over the step's tokens; state float32 [slots][heads][vdim][dim].
+int rb_delta_scan(const float* u, int ld_u, int uq, int uk, int uv, int ug, int ub, int ud, int heads, int kv_heads, int dim,
+                  int vdim, int per_channel, float* state, const int* seq_slot, const int* cu_q, int n_seqs, float* out,
+                  int ld_out, void* stream);
+// out[t, n] = sum_r w_i[n, r] * x_i[t, r] for up to two matrices w_i [n_i, rank_i] and column blocks x_off_i of the rows (n_in
+// partial sums added first); results side by side, float32.
+int rb_low_rank(const void* in, int in_dtype, int n_in, long long in_stride, int row_stride, int x_off0, int rank0,
+                const void* w0, int n0, int x_off1, int rank1, const void* w1, int n1, int w_dtype, int T, float* out,
+                int ld_out, void* stream);
 
 // Attention with a norm over the whole q and k projections and head weights mixed after the softmax (talking_heads.cu).
 int rb_wide_norm_rope_cache(const void* in, int in_dtype, int n_in, long long in_stride, int row_stride, int nq, int nkv,

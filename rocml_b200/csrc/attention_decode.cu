@@ -96,12 +96,16 @@ struct Projections {
     // every stored head.  nkv = n * n then counts (key head, value head) pairs and nq = n * query heads the results; pair
     // (a, m) sits at a * n + m, is read by the queries of key head a, and q holds nq / n heads.
     int cross;
+    const float* sinks;       // one sink score a query head (float32 [nq]) instead of one for all; null: `sink`
+    // temp_coef != 0: the query of a token at position p is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1),
+    // after everything else that happens to it
+    float temp_coef, temp_every;
 };
 
 // One head of 128 values, 4 per lane: the sum of the partial sums, then (what != 2) RMSNorm with `w`
 // and the rotation by the token's angles.  what: 0 query, 1 key, 2 value.
 __device__ __forceinline__ void project_head(const Projections& pj, const float* src, int what, int t, int lane,
-                                             float sumsq_share, float* v) {
+                                             float sumsq_share, float* v, int pos) {
     v[0] = v[1] = v[2] = v[3] = 0.f;
     // the norm's weights and the token's angles do not depend on the sums: their loads go out first
     const void* w = what == 0 ? pj.q_norm_w : (what == 1 ? pj.k_norm_w : nullptr);
@@ -161,6 +165,11 @@ __device__ __forceinline__ void project_head(const Projections& pj, const float*
         const float inv = rsqrtf(ss / 128.f + pj.eps);
 #pragma unroll
         for (int j = 0; j < 4; ++j) v[j] *= inv;
+    }
+    if (what == 0 && pj.temp_coef != 0.f) {
+        const float f = query_temperature(pos, pj.temp_coef, pj.temp_every);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] *= f;
     }
 }
 __device__ __forceinline__ uint2 pack4_bf16(const float* v) {
@@ -346,7 +355,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                     float v[4];
                     const bool is_k = warp == WARPS - 2;
                     const int head = is_k ? nq + kvh : nq + nkv + kvh;
-                    project_head(pj, row + (size_t)head * HD + lane * 4, is_k ? 1 : 2, t, lane, share, v);
+                    project_head(pj, row + (size_t)head * HD + lane * 4, is_k ? 1 : 2, t, lane, share, v, pos);
                     if (!is_k && (pj.v_keep || pj.v_first)) {
                         const size_t vrow = ((size_t)t * nkv + kvh) * HD + lane * 4;
                         if (pj.v_keep) *reinterpret_cast<float4*>(pj.v_keep + vrow) = make_float4(v[0], v[1], v[2], v[3]);
@@ -369,7 +378,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         if (!early1) issue(page_first + 1, 1);              // commits an empty group beyond page_last
         for (int r = warp; r < ROWS; r += WARPS) {          // the query heads of this block
             float v[4] = {0.f, 0.f, 0.f, 0.f};
-            if (r < rows_valid) project_head(pj, row + (size_t)(h0 + r) * HD + lane * 4, 0, t, lane, share, v);
+            if (r < rows_valid) project_head(pj, row + (size_t)(h0 + r) * HD + lane * 4, 0, t, lane, share, v, pos);
             const int chunk = lane >> 1;                    // 8 values per 16-byte chunk, 4 per lane
             *reinterpret_cast<uint2*>(reinterpret_cast<uint8_t*>(Qs) + r * (HD * 2) + ((chunk ^ (r & 7)) << 4) +
                                       (lane & 1) * 8) = pack4_bf16(v);
@@ -627,7 +636,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             part_acc[pidx * HD + d] = A;
             if (d == 0) { part_ml[pidx * 2] = M; part_ml[pidx * 2 + 1] = L; }
         } else {
-            float y = finished(A, L, M, sink);
+            float y = finished(A, L, M, pj.sinks ? pj.sinks[head] : sink);
             if (pj.gate.raw) y *= gate_factor(pj.gate, (size_t)t, (size_t)head * HD + d);
             out[(size_t)t * o_stride + (size_t)head * HD + d] = __float2bfloat16_rn(y);
         }
@@ -667,7 +676,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                     A = fmaf(wt, pa[i], A);
                 }
             }
-            float y = finished(A, L, MM, sink);
+            float y = finished(A, L, MM, pj.sinks ? pj.sinks[h0 + r] : sink);
             if (pj.gate.raw) y *= gate_factor(pj.gate, (size_t)t, (size_t)(h0 + r) * HD + d);
             out[(size_t)t * o_stride + (size_t)(h0 + r) * HD + d] = __float2bfloat16_rn(y);
         }
@@ -718,7 +727,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             L = fmaf(wt, pl[i], L);
             A = fmaf(wt, __ldcg(pa + (size_t)i * HD), A);
         }
-        float y = finished(A, L, MM, sink);
+        float y = finished(A, L, MM, pj.sinks ? pj.sinks[h0 + r] : sink);
         if (pj.gate.raw) y *= gate_factor(pj.gate, (size_t)t, (size_t)(h0 + r) * HD + d);
         out[(size_t)t * o_stride + (size_t)(h0 + r) * HD + d] = __float2bfloat16_rn(y);
     }
@@ -841,12 +850,13 @@ static int decode_entry(const void* q, int q_stride, const void* k_cache, const 
 extern "C" int rb_attention_decode(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                                    const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                                    const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window,
-                                   int keep, float sink, int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
+                                   int keep, float sink, const float* sinks, int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
                                    int* counters, void* out, int o_stride, const void* gate, int gate_f32, int gate_n_in,
                                    long long gate_in_stride, long long gate_row_stride, int cross, void* stream) {
     Projections none = {};
     if (cross < 0 || (cross > 1 && (nkv != cross * cross || gate != nullptr))) return RB_ERR_BAD_SIZE;
     none.cross = cross;
+    none.sinks = sinks;
     if (gate != nullptr) {      // nq * hd columns of the projection rows: the result times their sigmoid
         if (gate_n_in < 1) return RB_ERR_BAD_SIZE;
         none.gate = GateCols{gate, gate_f32, gate_n_in, gate_in_stride, gate_row_stride};
@@ -874,12 +884,13 @@ extern "C" int rb_attention_decode_fused(const float* proj, int n_in, long long 
                                          const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                                          const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window,
                                          int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
-                                         int* counters, void* out, int o_stride, int keep, float sink, int rot_dim,
-                                         int post_norm, const float* v_first, const float* v_lambda, float* v_keep,
+                                         int* counters, void* out, int o_stride, int keep, float sink, const float* sinks,
+                                         float temp_coef, float temp_every, int rot_dim, int post_norm, const float* v_first, const float* v_lambda, float* v_keep,
                                          const void* gate, int gate_f32, int gate_n_in, long long gate_in_stride,
                                          long long gate_row_stride, void* stream) {
     if (hd != 128 || proj == nullptr || n_in < 1) return RB_ERR_BAD_SIZE;
     if (((uintptr_t)proj & 15) || (in_stride % 4) || (row_stride % 4) || ((uintptr_t)cos_sin & 15)) return RB_ERR_BAD_ALIGN;
+    if (temp_coef != 0.f && !(temp_every > 0.f)) return RB_ERR_BAD_SIZE;
     if (rot_dim <= 0) rot_dim = 128;
     if (rot_dim > 128 || rot_dim % 8 || (v_first && !v_lambda) || ((v_first || v_keep) && !write_kv) || (gate && gate_n_in < 1))
         return RB_ERR_BAD_SIZE;
@@ -896,6 +907,7 @@ extern "C" int rb_attention_decode_fused(const float* proj, int n_in, long long 
     pj.row_eps = row_eps; pj.row_inv_width = row_width > 0 ? 1.f / (float)row_width : 0.f;
     if (row_sumsq != nullptr && (row_groups < 1 || row_width < 1)) return RB_ERR_BAD_SIZE;
     pj.rot_dim = rot_dim; pj.post_norm = post_norm;
+    pj.sinks = sinks; pj.temp_coef = temp_coef; pj.temp_every = temp_every;
     pj.v_first = v_first; pj.v_lambda = v_lambda; pj.v_keep = v_keep;
     if (gate != nullptr) pj.gate = GateCols{gate, gate_f32, gate_n_in, gate_in_stride, gate_row_stride};
     return decode_entry(nullptr, 0, k_cache, v_cache, block_table, max_pages, seq_slot, cu_q, kv_len, B, nq, nkv, hd,
@@ -966,6 +978,6 @@ extern "C" int rb_attention_decode_static(const void* q, int q_stride, const voi
     cudaError_t e = cudaMemsetAsync(sc->counters, 0, n_counters * sizeof(int), (cudaStream_t)stream);
     if (e != cudaSuccess) return (int)e;
     return rb_attention_decode(q, q_stride, k_cache, v_cache, block_table, max_pages, seq_slot, cu_q, kv_len, n_seqs,
-                               nq, nkv, hd, scale, window, 0, RB_NO_SINK, n_chunks, 1, sc->acc, sc->ml, sc->counters, out, o_stride,
+                               nq, nkv, hd, scale, window, 0, RB_NO_SINK, nullptr, n_chunks, 1, sc->acc, sc->ml, sc->counters, out, o_stride,
                                nullptr, 0, 0, 0, 0, 0, stream);
 }

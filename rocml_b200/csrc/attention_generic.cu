@@ -47,7 +47,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
                          const int* __restrict__ block_table, int max_pages,
                          const int* __restrict__ seq_slot, const int* __restrict__ cu_q,
                          const int* __restrict__ kv_len, int nq, int nkv, int hd, float scale, int window,
-                         int keep, float sink, int chunk, int n_chunks, float* __restrict__ part_acc,
+                         int keep, float sink, const float* __restrict__ sinks, int chunk, int n_chunks, float* __restrict__ part_acc,
                          float* __restrict__ part_ml, int cross) {
     pdl_trigger();
     pdl_wait();
@@ -261,7 +261,8 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
             }
         } else {
             float lsum = l[i];
-            const float a = has_sink(sink) ? add_sink(m[i], lsum, sink) : 1.f;
+            const float sk = sinks ? sinks[head] : sink;
+            const float a = has_sink(sk) ? add_sink(m[i], lsum, sk) : 1.f;
             const float inv = lsum > 0.f ? a / lsum : 0.f;
 #pragma unroll
             for (int dd = 0; dd < DPL; ++dd) {
@@ -279,7 +280,8 @@ template <typename T>
 __global__ void attention_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                        T* __restrict__ out, int o_stride, const int* __restrict__ positions,
                                        const int* __restrict__ slot_of_token, int T_tokens, int nq, int hd,
-                                       int chunk, int n_chunks, int window, int keep, float sink) {
+                                       int chunk, int n_chunks, int window, int keep, float sink,
+                                       const float* __restrict__ sinks) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float w_s[];   // [warps][n_chunks]
@@ -311,7 +313,8 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_acc, const
     }
     L = warp_sum(L);
     __syncwarp();
-    const float a_sink = has_sink(sink) ? add_sink(M, L, sink) : 1.f;
+    const float sk = sinks ? sinks[head] : sink;
+    const float a_sink = has_sink(sk) ? add_sink(M, L, sk) : 1.f;
     const float inv = L > 0.f ? a_sink / L : 0.f;
     for (int d = lane; d < hd; d += 32) {
         float a = 0.f;
@@ -332,7 +335,7 @@ template <typename T>
 int launch_attn(const void* q, int q_stride, void* out, int o_stride, const void* k_cache, const void* v_cache,
                 const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                 const int* kv_len, int B, int max_q_len, int nq, int nkv, int hd, float scale, int window,
-                int keep, float sink, int chunk, int n_chunks, float* part_acc, float* part_ml, int cross, cudaStream_t s) {
+                int keep, float sink, const float* sinks, int chunk, int n_chunks, float* part_acc, float* part_ml, int cross, cudaStream_t s) {
     const int g = nq / nkv;
     const int HG = g < ROWS ? g : ROWS;
     const int QB = ROWS / HG;
@@ -348,7 +351,7 @@ int launch_attn(const void* q, int q_stride, void* out, int o_stride, const void
     dim3 grid((unsigned)gx, nkv * head_chunks, B);
     RB_LAUNCH((k), dim3(grid), dim3(128), smem, s, (const T*)q, q_stride, (T*)out, o_stride, (const T*)k_cache, (const T*)v_cache,
                               block_table, max_pages, seq_slot, cu_q, kv_len, nq, nkv, hd, scale, window,
-                              keep, sink, chunk, n_chunks, part_acc, part_ml, cross);
+                              keep, sink, sinks, chunk, n_chunks, part_acc, part_ml, cross);
     RB_LAUNCH_CHECK();
     return RB_OK;
 }
@@ -358,8 +361,8 @@ extern "C" int rb_attention_generic(const void* q, int q_stride, void* out, int 
                                     const void* k_cache, const void* v_cache, const int* block_table,
                                     int max_pages, const int* seq_slot, const int* cu_q, const int* kv_len,
                                     int B, int max_q_len, int nq, int nkv, int hd, float scale, int window,
-                                    int keep, float sink, int chunk, int n_chunks, float* part_acc, float* part_ml,
-                                    int cross, void* stream) {
+                                    int keep, float sink, const float* sinks, int chunk, int n_chunks, float* part_acc,
+                                    float* part_ml, int cross, void* stream) {
     if (B <= 0 || max_q_len <= 0) return RB_OK;
     if (keep < 0 || (keep > 0 && window < 0)) return RB_ERR_BAD_SIZE;
     if (hd <= 0 || hd > 32 * MAX_DPL || nkv <= 0 || nq % nkv) return RB_ERR_BAD_SIZE;
@@ -370,17 +373,17 @@ extern "C" int rb_attention_generic(const void* q, int q_stride, void* out, int 
     if (dtype == RB_BF16)
         return launch_attn<__nv_bfloat16>(q, q_stride, out, o_stride, k_cache, v_cache, block_table, max_pages,
                                           seq_slot, cu_q, kv_len, B, max_q_len, nq, nkv, hd, scale, window,
-                                          keep, sink, chunk, n_chunks, part_acc, part_ml, cross, s);
+                                          keep, sink, sinks, chunk, n_chunks, part_acc, part_ml, cross, s);
     if (dtype == RB_F32)
         return launch_attn<float>(q, q_stride, out, o_stride, k_cache, v_cache, block_table, max_pages, seq_slot,
-                                  cu_q, kv_len, B, max_q_len, nq, nkv, hd, scale, window, keep, sink, chunk, n_chunks,
+                                  cu_q, kv_len, B, max_q_len, nq, nkv, hd, scale, window, keep, sink, sinks, chunk, n_chunks,
                                   part_acc, part_ml, cross, s);
     return RB_ERR_BAD_DTYPE;
 }
 
 extern "C" int rb_attention_merge(const float* part_acc, const float* part_ml, void* out, int o_stride,
                                   int dtype, const int* positions, const int* slot_of_token, int T, int nq,
-                                  int hd, int chunk, int n_chunks, int window, int keep, float sink, void* stream) {
+                                  int hd, int chunk, int n_chunks, int window, int keep, float sink, const float* sinks, void* stream) {
     if (T <= 0) return RB_OK;
     if (chunk <= 0 || n_chunks <= 0) return RB_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
@@ -392,11 +395,11 @@ extern "C" int rb_attention_merge(const float* part_acc, const float* part_ml, v
     if (dtype == RB_BF16)
         RB_LAUNCH((attention_merge_kernel<__nv_bfloat16>), dim3((int)blocks), dim3(warps * 32), smem, s, part_acc, part_ml, (__nv_bfloat16*)out, o_stride,
                                                                   positions, slot_of_token, T, nq, hd, chunk,
-                                                                  n_chunks, window, keep, sink);
+                                                                  n_chunks, window, keep, sink, sinks);
     else if (dtype == RB_F32)
         RB_LAUNCH((attention_merge_kernel<float>), dim3((int)blocks), dim3(warps * 32), smem, s, part_acc, part_ml, (float*)out, o_stride,
                                                                   positions, slot_of_token, T, nq, hd, chunk,
-                                                                  n_chunks, window, keep, sink);
+                                                                  n_chunks, window, keep, sink, sinks);
     else
         return RB_ERR_BAD_DTYPE;
     RB_LAUNCH_CHECK();

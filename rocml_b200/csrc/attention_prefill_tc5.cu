@@ -115,7 +115,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                              const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, int o_stride,
                              const int* __restrict__ block_table, int max_pages, const int* __restrict__ seq_slot,
                              const int* __restrict__ cu_q, const int* __restrict__ kv_len, int nq, int nkv,
-                             float scale, int window, int keep, float sink, int heads_first, int strict_order,
+                             float scale, int window, int keep, float sink, const float* __restrict__ sinks, int heads_first, int strict_order,
                              int* __restrict__ status, const __nv_bfloat16* __restrict__ gate, long long gate_row_stride,
                              int cross) {
     using Z = Sizes<HD>;
@@ -394,6 +394,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
         if (alive) {
             tc_fence_after();
             // one more term in the denominator: O and the sum carry the factor 2^-m_used, so the term does too
+            if (sinks) sink = sinks[head];
             if (rb::has_sink(sink)) l_sum += exp2f(fminf(sink * LOG2E - m_used, 126.f));
             const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
             __nv_bfloat16* orow = out + (size_t)(q0 + m0 + r) * o_stride + (size_t)head * HD;
@@ -489,7 +490,7 @@ template <int HD>
 int launch_tc5(const void* q, int q_stride, int T, void* out, int o_stride, const void* k_cache, const void* v_cache,
                int n_pages, const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                const int* kv_len, int B, int max_q_len, int nq, int nkv, float scale, int window, int keep, float sink,
-               int heads_first, int* status, const void* gate, long long gate_row_stride, int cross, cudaStream_t stream) {
+               const float* sinks, int heads_first, int* status, const void* gate, long long gate_row_stride, int cross, cudaStream_t stream) {
     // RB_PREFILL_STRICT_ORDER=0: see `strict_order` in the kernel's MMA thread
     static const int strict_order = [] { const char* e = getenv("RB_PREFILL_STRICT_ORDER"); return (e && e[0] == '0') ? 0 : 1; }();
     CUtensorMap mq, mk, mv;
@@ -509,7 +510,7 @@ int launch_tc5(const void* q, int q_stride, int T, void* out, int o_stride, cons
     dim3 grid = heads_first ? dim3(nq, B, q_tiles) : dim3(q_tiles, nq, B);
     if (grid.y > 65535 || grid.z > 65535) return RB_ERR_BAD_SIZE;
     RB_LAUNCH((k), grid, dim3(192), Sizes<HD>::SMEM_BYTES, stream, mq, mk, mv, (__nv_bfloat16*)out, o_stride,
-              block_table, max_pages, seq_slot, cu_q, kv_len, nq, nkv, scale, window, keep, sink, heads_first, strict_order,
+              block_table, max_pages, seq_slot, cu_q, kv_len, nq, nkv, scale, window, keep, sink, sinks, heads_first, strict_order,
               status, (const __nv_bfloat16*)gate, gate_row_stride, cross);
     return RB_OK;
 }
@@ -517,7 +518,8 @@ int launch_tc5(const void* q, int q_stride, int T, void* out, int o_stride, cons
 
 // q rows [T, q_stride] bfloat16 (T = tokens of the step), caches [n_pages, nkv, 64, hd].  heads_first: the order
 // in which blocks start (see the kernel); it changes no result.  keep: beside a window the keys at positions below
-// it stay visible; sink: a score whose exponential joins every row's denominator (RB_NO_SINK: none).  Head sizes 64, 128 and 256;
+// it stay visible; sink: a score whose exponential joins every row's denominator (RB_NO_SINK: none);
+// sinks: one such score a query head instead.  Head sizes 64, 128 and 256;
 // RB_ERR_BAD_SIZE / RB_ERR_BAD_ALIGN otherwise (the caller then uses the mma.sync kernel).  gate: nq * hd bfloat16 columns of
 // the tokens' projection rows (gate_row_stride elements apart), or null: the result is multiplied by their sigmoid.
 // cross (n > 1, the caches' own number of heads): every query head's weights on the values of every stored head; nkv = n * n
@@ -526,7 +528,7 @@ extern "C" int rb_attention_prefill_tc5(const void* q, int q_stride, int T, void
                                         const void* k_cache, const void* v_cache, int n_pages,
                                         const int* block_table, int max_pages, const int* seq_slot,
                                         const int* cu_q, const int* kv_len, int B, int max_q_len, int nq, int nkv,
-                                        int hd, float scale, int window, int keep, float sink, int heads_first,
+                                        int hd, float scale, int window, int keep, float sink, const float* sinks, int heads_first,
                                         int* status, const void* gate, long long gate_row_stride, int cross, void* stream) {
     if (B <= 0 || max_q_len <= 0 || T <= 0) return RB_OK;
     if (cross < 0 || (cross > 1 && (nkv != cross * cross || gate))) return RB_ERR_BAD_SIZE;
@@ -537,7 +539,7 @@ extern "C" int rb_attention_prefill_tc5(const void* q, int q_stride, int T, void
         (q_stride % 8) || (o_stride % 8))
         return RB_ERR_BAD_ALIGN;
 #define RB_TC5_ARGS q, q_stride, T, out, o_stride, k_cache, v_cache, n_pages, block_table, max_pages, seq_slot, cu_q, kv_len, \
-                    B, max_q_len, nq, nkv, scale, window, keep, sink, heads_first, status, gate, gate_row_stride, cross, (cudaStream_t)stream
+                    B, max_q_len, nq, nkv, scale, window, keep, sink, sinks, heads_first, status, gate, gate_row_stride, cross, (cudaStream_t)stream
     if (hd == 64) return launch_tc5<64>(RB_TC5_ARGS);
     if (hd == 128) return launch_tc5<128>(RB_TC5_ARGS);
     return launch_tc5<256>(RB_TC5_ARGS);

@@ -95,6 +95,10 @@ __device__ __forceinline__ int span_lo(int pos, int window) {
 // sum to less than one.
 #define RB_NO_SINK (-3.0e38f)
 __device__ __forceinline__ bool has_sink(float sink) { return sink > -1.0e38f; }
+// A temperature that grows with the query's position p (>= 0): 1 + coef * ln(floor((p + 1) / every) + 1), 32-bit.
+__device__ __forceinline__ float query_temperature(int pos, float coef, float every) {
+    return 1.f + coef * logf(floorf((float)(pos + 1) / every) + 1.f);
+}
 // What the sink does to a finished row: with running maximum m and sum l, the factor for the accumulated values
 // (returned) and the new sum (through l): m' = max(m, sink), l' = l e^(m - m') + e^(sink - m').
 __device__ __forceinline__ float add_sink(float m, float& l, float sink) {

@@ -409,25 +409,29 @@ extern "C" int rb_cast(const void* in, int in_dtype, void* out, int out_dtype, l
 // inv_freq (float32 [ceil(H / 2)]) may be absent: then nothing is added.  `copy` (optional) receives the
 // same rows (a model that adds its embedding output back in later keeps them).  Angle, sine and cosine
 // are 32-bit and full precision.
+// With pos_table ([pos_rows, H]) its row positions[t] is added instead of a sinusoid.
 template <typename WT>
 __global__ void embedding_pos_kernel(const int* __restrict__ ids, const WT* __restrict__ table, float* __restrict__ out,
                                      float* __restrict__ copy, int H, int vocab, float scale,
                                      const int* __restrict__ positions, const float* __restrict__ inv_freq,
-                                     int* __restrict__ status) {
+                                     const WT* __restrict__ pos_table, int pos_rows, int* __restrict__ status) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
     const int id = ids[t];
-    const bool bad = id < 0 || id >= vocab;
+    const int p = positions[t];
+    const bool bad = id < 0 || id >= vocab || (pos_table && (p < 0 || p >= pos_rows));
     if (bad && threadIdx.x == 0 && status) atomicExch(status, RB_ERR_BAD_SIZE);
     const WT* row = table + (size_t)(bad ? 0 : id) * H;
-    const float pos = (float)positions[t];
+    const float pos = (float)p;
+    const WT* prow = pos_table ? pos_table + (size_t)(bad ? 0 : p) * H : nullptr;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = bad ? 0.f : to_f32(row[i]) * scale;
         if (inv_freq) {
             const float a = pos * inv_freq[i >> 1];
             v += (i & 1) ? cosf(a) : sinf(a);
         }
+        if (prow && !bad) v += to_f32(prow[i]);
         out[(size_t)t * H + i] = v;
         if (copy) copy[(size_t)t * H + i] = v;
     }
@@ -435,16 +439,18 @@ __global__ void embedding_pos_kernel(const int* __restrict__ ids, const WT* __re
 
 extern "C" int rb_embedding_pos(const int* ids, const void* table, int table_dtype, float* out, float* copy, int T,
                                 int H, int vocab, float scale, const int* positions, const float* inv_freq,
-                                int* status, void* stream) {
+                                const void* pos_table, int pos_dtype, int pos_rows, int* status, void* stream) {
     if (T <= 0) return RB_OK;
+    if (pos_table && (inv_freq || pos_rows <= 0)) return RB_ERR_BAD_SIZE;
+    if (pos_table && pos_dtype != table_dtype) return RB_ERR_BAD_DTYPE;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = H >= 1024 ? 256 : 128;
     if (table_dtype == RB_BF16)
         RB_LAUNCH((embedding_pos_kernel<__nv_bfloat16>), dim3(T), dim3(threads), 0, s, ids, (const __nv_bfloat16*)table, out,
-                  copy, H, vocab, scale, positions, inv_freq, status);
+                  copy, H, vocab, scale, positions, inv_freq, (const __nv_bfloat16*)pos_table, pos_rows, status);
     else if (table_dtype == RB_F32)
         RB_LAUNCH((embedding_pos_kernel<float>), dim3(T), dim3(threads), 0, s, ids, (const float*)table, out, copy, H, vocab,
-                  scale, positions, inv_freq, status);
+                  scale, positions, inv_freq, (const float*)pos_table, pos_rows, status);
     else
         return RB_ERR_BAD_DTYPE;
     RB_LAUNCH_CHECK();
@@ -750,5 +756,23 @@ extern "C" int rb_scale(float* x, long long n, float factor, void* stream) {
     const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
     RB_LAUNCH((scale_kernel), dim3(blocks), dim3(threads), 0, (cudaStream_t)stream, x, (size_t)n, factor);
     RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+// ---- x <- cap * tanh(factor * x / cap) (32-bit, in place) ------------------------------------------------------
+__global__ void softcap_kernel(float* __restrict__ x, size_t n, float factor, float cap) {
+    pdl_trigger();
+    pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
+        x[i] = cap * tanhf(x[i] * factor / cap);
+}
+
+extern "C" int rb_softcap(float* x, long long n, float factor, float cap, void* stream) {
+    if (n <= 0) return RB_OK;
+    if (!(cap > 0.f)) return RB_ERR_BAD_SIZE;
+    const int threads = 256;
+    const long long want = (n + threads - 1) / threads;
+    const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+    RB_LAUNCH((softcap_kernel), dim3(blocks), dim3(threads), 0, (cudaStream_t)stream, x, (size_t)n, factor, cap);
     return RB_OK;
 }

@@ -1,0 +1,536 @@
+// The gated delta rule: a state per head that forgets by a decay and is corrected, token by token, towards v along k.
+//
+//   S <- g S;   w = beta (v - S^T k);   S <- S + k w^T;   o = S^T q          S [dim, vdim] per (sequence, head), 32-bit
+//
+// with g one number a head or one a key channel (a row of S).  With k and q the token's vectors and P = g S the decayed
+// state, o = P^T q + w (k . q), so both sums over the rows are formed in one pass over the state and meet in one exchange.
+//
+//   delta_prep   everything between the projections and the recurrence: the short causal convolutions over time with
+//                silu, q and k divided by their length (q times a constant as well), their dot product, the step size
+//                beta = sigmoid(.), the decay g = exp(-exp(A) softplus(z + bias)); all 32-bit, into rows that the
+//                recurrence copies straight to shared memory.  A block is (sequence, 32 tokens, unit), a unit the q and k
+//                of one key head or one head's v, beta and g; a warp takes a token at a time.  What lies before a
+//                sequence's first token of the step comes from its slot; the block of a sequence's first tokens
+//                is the only one that reads the slot, and it leaves the step's last inputs there after its reads.
+//   delta_scan   the recurrence.  A head's columns do not depend on one another: a warp owns four of them, sixteen lanes
+//                each pair, and keeps its part of the state in registers from the step's first token to its last, so the
+//                state is read and written once a step whatever the number of tokens.  A block has eight warps (or fewer, for
+//                few columns); the tokens' q, k, g and v arrive in shared memory by cp.async, a batch of tokens ahead.
+//                The order of a token's operations depends neither on how the prompt was cut nor on the batch: one
+//                token a step gives the bits of the whole prompt.
+//   low_rank     a narrow product through few inner values for few tokens (a decode step's W2 (W1 h)), 32-bit FMA.
+#include "common.cuh"
+#include "api.h"
+
+using namespace rb;
+
+namespace {
+template <typename IT>
+__device__ __forceinline__ float sum_in(const IT* p, int n_in, size_t in_stride) {
+    float v = 0.f;
+    for (int s = 0; s < n_in; ++s) v += to_f32(p[(size_t)s * in_stride]);
+    return v;
+}
+template <int VEC, typename IT>
+__device__ __forceinline__ void sum_vec(const IT* p, int n_in, size_t in_stride, float* x) {
+    if constexpr (VEC == 4) {
+        x[0] = x[1] = x[2] = x[3] = 0.f;
+        for (int s = 0; s < n_in; ++s) {
+            float y[4];
+            load4(p + (size_t)s * in_stride, y);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) x[u] += y[u];
+        }
+    } else {
+        x[0] = sum_in(p, n_in, in_stride);
+    }
+}
+template <int VEC>
+__device__ __forceinline__ void load_vec(const float* p, float* x) {
+    if constexpr (VEC == 4) load4(p, x);
+    else x[0] = p[0];
+}
+template <int VEC>
+__device__ __forceinline__ void store_vec(float* p, const float* x) {
+    if constexpr (VEC == 4) store4(p, x);
+    else p[0] = x[0];
+}
+__device__ __forceinline__ float softplus_f32(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+constexpr int PREP_TOK = 32;          // tokens a block; more than a convolution's kept inputs
+constexpr int PREP_MAX_TAPS = PREP_TOK;
+
+struct PrepArgs {
+    size_t in_stride;
+    int n_in, row_stride, q_off, k_off, v_off, b_off;
+    int heads, kv_heads, dim, vdim, taps, channels;
+    const float* conv_w;              // [taps][channels]
+    float* kept;                      // [slots][taps - 1][channels]
+    size_t z_in_stride;
+    int z_n_in, z_row_stride;
+    const float *dt_bias, *a_log;
+    int per_channel;
+    float unit_eps, q_scale;
+    const int *seq_slot, *cu_q;
+    float* u;
+    int ld_u, uq, uk, uv, ug, ub, ud;
+};
+
+// silu(convolution) of VEC neighbouring channels of token t: `col` their column in the projection rows, `c` their place among
+// the convolution's channels.
+template <int VEC, typename IT>
+__device__ __forceinline__ void conv_silu(const PrepArgs& a, const IT* in, const float* mine, int t, int t_begin, int col, int c,
+                                          float* acc) {
+#pragma unroll
+    for (int u = 0; u < VEC; ++u) acc[u] = 0.f;
+    const int back = a.taps - 1;
+    for (int j = 0; j < a.taps; ++j) {
+        const int r = t - back + j;
+        float x[VEC], w[VEC];
+        if (r >= t_begin) sum_vec<VEC>(in + (size_t)r * a.row_stride + col, a.n_in, a.in_stride, x);
+        else load_vec<VEC>(mine + (size_t)(back + (r - t_begin)) * a.channels + c, x);
+        load_vec<VEC>(a.conv_w + (size_t)j * a.channels + c, w);
+#pragma unroll
+        for (int u = 0; u < VEC; ++u) acc[u] = fmaf(w[u], x[u], acc[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < VEC; ++u) acc[u] = silu(acc[u]);
+}
+
+// The slot's new rows for channels [c0, c0 + n): the last taps - 1 of (old rows, the step's rows).  A channel is one thread's,
+// which reads every row before it overwrites it (a row comes from the same or a later place).
+template <typename IT>
+__device__ __forceinline__ void keep_inputs(const PrepArgs& a, const IT* in, float* mine, int t_begin, int len, int col0, int c0,
+                                            int n) {
+    const int back = a.taps - 1;
+    for (int i = threadIdx.x; i < n; i += blockDim.x)
+        for (int j = 0; j < back; ++j) {
+            const int at = len + j;
+            mine[(size_t)j * a.channels + c0 + i] =
+                at < back ? mine[(size_t)at * a.channels + c0 + i]
+                          : sum_in(in + (size_t)(t_begin + at - back) * a.row_stride + col0 + i, a.n_in, a.in_stride);
+        }
+}
+
+template <typename IT, typename ZT, int VEC>
+__global__ void __launch_bounds__(128)
+delta_prep_kernel(const IT* __restrict__ in, const ZT* __restrict__ z, const PrepArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const int b = blockIdx.z, slot = a.seq_slot[b];
+    if (slot < 0) return;
+    const int t_begin = a.cu_q[b], t_end = a.cu_q[b + 1];
+    const int t0 = t_begin + blockIdx.y * PREP_TOK;
+    if (t0 >= t_end) return;
+    const int n = min(PREP_TOK, t_end - t0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    float* mine = a.taps > 1 ? a.kept + (size_t)slot * (a.taps - 1) * a.channels : nullptr;
+    const int kd = a.kv_heads * a.dim;
+    if ((int)blockIdx.x < a.kv_heads) {
+        const int h = blockIdx.x, c = h * a.dim;
+        for (int tt = warp; tt < n; tt += warps) {
+            const int t = t0 + tt;
+            float* uq = a.u + (size_t)t * a.ld_u + a.uq + c;
+            float* uk = a.u + (size_t)t * a.ld_u + a.uk + c;
+            float qq = 0.f, kk = 0.f, qk = 0.f;
+            for (int i = lane * VEC; i < a.dim; i += 32 * VEC) {
+                float q[VEC], k[VEC];
+                conv_silu<VEC>(a, in, mine, t, t_begin, a.q_off + c + i, c + i, q);
+                conv_silu<VEC>(a, in, mine, t, t_begin, a.k_off + c + i, kd + c + i, k);
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) { qq = fmaf(q[u], q[u], qq); kk = fmaf(k[u], k[u], kk); qk = fmaf(q[u], k[u], qk); }
+                store_vec<VEC>(uq + i, q);
+                store_vec<VEC>(uk + i, k);
+            }
+            const float fq = a.q_scale / sqrtf(warp_sum(qq) + a.unit_eps), fk = 1.f / sqrtf(warp_sum(kk) + a.unit_eps);
+            qk = warp_sum(qk);
+            for (int i = lane * VEC; i < a.dim; i += 32 * VEC) {      // each lane its own values
+                float q[VEC], k[VEC];
+                load_vec<VEC>(uq + i, q);
+                load_vec<VEC>(uk + i, k);
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) { q[u] *= fq; k[u] *= fk; }
+                store_vec<VEC>(uq + i, q);
+                store_vec<VEC>(uk + i, k);
+            }
+            if (lane == 0) a.u[(size_t)t * a.ld_u + a.ud + h] = qk * fq * fk;
+        }
+        if (blockIdx.y == 0 && a.taps > 1) {
+            __syncthreads();
+            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.q_off + c, c, a.dim);
+            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.k_off + c, kd + c, a.dim);
+        }
+        return;
+    }
+    const int h = blockIdx.x - a.kv_heads, c = h * a.vdim;
+    const float rate = expf(a.a_log[h]);
+    for (int tt = warp; tt < n; tt += warps) {
+        const int t = t0 + tt;
+        float* row = a.u + (size_t)t * a.ld_u;
+        for (int i = lane * VEC; i < a.vdim; i += 32 * VEC) {
+            float v[VEC];
+            conv_silu<VEC>(a, in, mine, t, t_begin, a.v_off + c + i, 2 * kd + c + i, v);
+            store_vec<VEC>(row + a.uv + c + i, v);
+        }
+        if (a.per_channel) {
+            for (int i = lane * VEC; i < a.dim; i += 32 * VEC) {
+                float g[VEC], bias[VEC];
+                sum_vec<VEC>(z + (size_t)t * a.z_row_stride + (size_t)h * a.dim + i, a.z_n_in, a.z_in_stride, g);
+                load_vec<VEC>(a.dt_bias + (size_t)h * a.dim + i, bias);
+#pragma unroll
+                for (int u = 0; u < VEC; ++u) g[u] = expf(-rate * softplus_f32(g[u] + bias[u]));
+                store_vec<VEC>(row + a.ug + (size_t)h * a.dim + i, g);
+            }
+        } else if (lane == 1) {
+            row[a.ug + h] = expf(-rate * softplus_f32(sum_in(z + (size_t)t * a.z_row_stride + h, a.z_n_in, a.z_in_stride) + a.dt_bias[h]));
+        }
+        if (lane == 0) row[a.ub + h] = sigmoid_f32(sum_in(in + (size_t)t * a.row_stride + a.b_off + h, a.n_in, a.in_stride));
+    }
+    if (blockIdx.y == 0 && a.taps > 1) {
+        __syncthreads();
+        keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.v_off + c, 2 * kd + c, a.vdim);
+    }
+}
+
+// ---- the recurrence ---------------------------------------------------------------------------------------------
+constexpr int RL = 16;                // lanes that share a column's rows
+constexpr int WCOLS = 4;              // columns a warp owns: two for each half of the warp
+
+struct ScanArgs {
+    const float* u;
+    int ld_u, uq, uk, uv, ug, ub, ud;
+    int heads, kv_heads, dim, vdim;
+    float* state;                     // [slots][heads][vdim][dim]
+    const int *seq_slot, *cu_q;
+    float* out;
+    int ld_out;
+    int vec;                          // rows and pieces of them start on 16 bytes
+};
+
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+// R4: groups of four rows a lane holds (dim <= 64 R4).  CH: a decay per key channel.  TB: tokens staged at a time.
+template <int R4, bool CH, int TB>
+__global__ void __launch_bounds__(256)
+delta_scan_kernel(const ScanArgs a) {
+    pdl_trigger();
+    extern __shared__ __align__(16) float sm[];
+    constexpr int DP = 64 * R4;                         // rows of a staged vector, zeros beyond dim
+    constexpr int NV = CH ? 3 : 2;                      // q, k (, g)
+    const int warps = blockDim.x >> 5;
+    const int cols = warps * WCOLS;
+    const int tok = NV * DP + cols + 4;                 // a staged token: q | k (| g) | v of this block's columns | beta, q.k, g
+    float* outs = sm + 2 * TB * tok;                    // [TB][cols]
+    const int b = blockIdx.z, h = blockIdx.y, j0 = blockIdx.x * cols;
+    const int slot = a.seq_slot[b];
+    if (slot < 0) return;
+    const int t_begin = a.cu_q[b], t_end = a.cu_q[b + 1];
+    if (t_end <= t_begin) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane & 15, half = lane >> 4;
+    const int kvh = h / (a.heads / a.kv_heads);
+    const int jl = warp * WCOLS + half * 2;             // this lane's two columns: jl, jl + 1 of the block's
+
+    // the state: written by an earlier step, so it is read before this step's kernels are waited for
+    float S[2][R4][4];
+    float* st = a.state + ((size_t)slot * a.heads + h) * a.vdim * a.dim;
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const int j = j0 + jl + c;
+#pragma unroll
+        for (int r = 0; r < R4; ++r) {
+            const int i = (r * RL + l) * 4;
+            S[c][r][0] = S[c][r][1] = S[c][r][2] = S[c][r][3] = 0.f;
+            if (j < a.vdim) {
+                if ((a.dim & 3) == 0) {
+                    if (i < a.dim) load4(st + (size_t)j * a.dim + i, S[c][r]);
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) if (i + e < a.dim) S[c][r][e] = st[(size_t)j * a.dim + i + e];
+                }
+            }
+        }
+    }
+    if (a.dim < DP || j0 + cols > a.vdim)               // what no copy fills stays zero
+        for (int i = threadIdx.x; i < 2 * TB * tok; i += blockDim.x) sm[i] = 0.f;
+    __syncthreads();
+    pdl_wait();
+
+    const int nv = min(cols, a.vdim - j0);
+    auto stage = [&](int t0, int buf) {
+        const int nb = min(TB, t_end - t0);
+        float* base = sm + buf * TB * tok;
+        const float* u0 = a.u + (size_t)t0 * a.ld_u;
+        if (a.vec) {
+            const int d4 = a.dim >> 2, v4 = nv >> 2, per = NV * d4 + v4;
+            for (int i = threadIdx.x; i < nb * per; i += blockDim.x) {
+                const int tt = i / per;
+                int x = i - tt * per;
+                const float* row = u0 + (size_t)tt * a.ld_u;
+                float* dst = base + tt * tok;
+                if (x < d4) cp_async16(dst + 4 * x, row + a.uq + kvh * a.dim + 4 * x);
+                else if ((x -= d4) < d4) cp_async16(dst + DP + 4 * x, row + a.uk + kvh * a.dim + 4 * x);
+                else if (CH && (x -= d4) < d4) cp_async16(dst + 2 * DP + 4 * x, row + a.ug + (size_t)h * a.dim + 4 * x);
+                else {
+                    cp_async16(dst + NV * DP + 4 * (x - d4), row + a.uv + (size_t)h * a.vdim + j0 + 4 * (x - d4));
+                }
+            }
+        } else {
+            const int per = NV * a.dim + nv;
+            for (int i = threadIdx.x; i < nb * per; i += blockDim.x) {
+                const int tt = i / per, x = i - tt * per;
+                const float* row = u0 + (size_t)tt * a.ld_u;
+                float* dst = base + tt * tok;
+                const int what = x / a.dim, e = x - what * a.dim;
+                if (what == 0) cp_async4(dst + e, row + a.uq + kvh * a.dim + e);
+                else if (what == 1) cp_async4(dst + DP + e, row + a.uk + kvh * a.dim + e);
+                else if (CH && what == 2) cp_async4(dst + 2 * DP + e, row + a.ug + (size_t)h * a.dim + e);
+                else cp_async4(dst + NV * DP + (x - NV * a.dim), row + a.uv + (size_t)h * a.vdim + j0 + (x - NV * a.dim));
+            }
+        }
+        for (int i = threadIdx.x; i < nb; i += blockDim.x) {
+            const float* row = u0 + (size_t)i * a.ld_u;
+            float* dst = base + i * tok + NV * DP + cols;
+            cp_async4(dst, row + a.ub + h);
+            cp_async4(dst + 1, row + a.ud + kvh);
+            if (!CH) cp_async4(dst + 2, row + a.ug + h);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+
+    stage(t_begin, 0);
+    int buf = 0;
+    for (int t0 = t_begin; t0 < t_end; t0 += TB, buf ^= 1) {
+        const int nb = min(TB, t_end - t0);
+        if (t0 + TB < t_end) {
+            stage(t0 + TB, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const float* base = sm + buf * TB * tok;
+        for (int tt = 0; tt < nb; ++tt) {
+            const float* x = base + tt * tok;
+            const float* sc = x + NV * DP + cols;
+            const float beta = sc[0], dot = sc[1];
+            const float gh = CH ? 0.f : sc[2];
+            const float v0 = x[NV * DP + jl], v1 = x[NV * DP + jl + 1];
+            float k[R4][4];
+            float ak0 = 0.f, ak1 = 0.f, aq0 = 0.f, aq1 = 0.f;
+#pragma unroll
+            for (int r = 0; r < R4; ++r) {
+                const int i = (r * RL + l) * 4;
+                float q[4], g[4];
+                load4(x + i, q);
+                load4(x + DP + i, k[r]);
+                if (CH) load4(x + 2 * DP + i, g);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float f = CH ? g[e] : gh;
+                    const float s0 = f * S[0][r][e], s1 = f * S[1][r][e];
+                    S[0][r][e] = s0;
+                    S[1][r][e] = s1;
+                    ak0 = fmaf(k[r][e], s0, ak0);
+                    ak1 = fmaf(k[r][e], s1, ak1);
+                    aq0 = fmaf(q[e], s0, aq0);
+                    aq1 = fmaf(q[e], s1, aq1);
+                }
+            }
+            // four sums over sixteen lanes: halves exchange what the other keeps; lanes 0-3 end with k . column 0, 4-7 with
+            // k . column 1, 8-11 and 12-15 with q's
+            const bool up8 = (lane & 8) != 0, up4 = (lane & 4) != 0;
+            float x0 = up8 ? aq0 : ak0, x1 = up8 ? aq1 : ak1;
+            x0 += __shfl_xor_sync(0xffffffffu, up8 ? ak0 : aq0, 8);
+            x1 += __shfl_xor_sync(0xffffffffu, up8 ? ak1 : aq1, 8);
+            float y = up4 ? x1 : x0;
+            y += __shfl_xor_sync(0xffffffffu, up4 ? x0 : x1, 4);
+            y += __shfl_xor_sync(0xffffffffu, y, 2);
+            y += __shfl_xor_sync(0xffffffffu, y, 1);
+            const float w0 = beta * (v0 - __shfl_sync(0xffffffffu, y, lane & 16));
+            const float w1 = beta * (v1 - __shfl_sync(0xffffffffu, y, (lane & 16) | 4));
+            if (l == 8) outs[tt * cols + jl] = fmaf(w0, dot, y);
+            if (l == 12) outs[tt * cols + jl + 1] = fmaf(w1, dot, y);
+#pragma unroll
+            for (int r = 0; r < R4; ++r)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    S[0][r][e] = fmaf(k[r][e], w0, S[0][r][e]);
+                    S[1][r][e] = fmaf(k[r][e], w1, S[1][r][e]);
+                }
+        }
+        __syncthreads();                                // the results are there, and the buffer may be filled again
+        for (int i = threadIdx.x; i < nb * cols; i += blockDim.x) {
+            const int tt = i / cols, j = i - tt * cols;
+            if (j < nv) a.out[(size_t)(t0 + tt) * a.ld_out + (size_t)h * a.vdim + j0 + j] = outs[i];
+        }
+    }
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const int j = j0 + jl + c;
+        if (j >= a.vdim) continue;
+#pragma unroll
+        for (int r = 0; r < R4; ++r) {
+            const int i = (r * RL + l) * 4;
+            if ((a.dim & 3) == 0) {
+                if (i < a.dim) store4(st + (size_t)j * a.dim + i, S[c][r]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) if (i + e < a.dim) st[(size_t)j * a.dim + i + e] = S[c][r][e];
+            }
+        }
+    }
+}
+
+template <int R4, bool CH, int TB>
+int launch_scan(const ScanArgs& a, int n_seqs, cudaStream_t s) {
+    // columns a block takes: few (16) while the grid would not fill the device otherwise, 32 beyond
+    int warps = 8;
+    const long long heads = (long long)n_seqs * a.heads;
+    while (warps > 1 && (heads * ((a.vdim + warps * WCOLS - 1) / (warps * WCOLS)) < 148 || (warps - 1) * WCOLS >= a.vdim)) warps >>= 1;
+    if (warps < 4 && a.vdim > 2 * WCOLS) warps = a.vdim > 8 ? 4 : 2;
+    const int cols = warps * WCOLS;
+    const size_t smem = ((size_t)2 * TB * ((CH ? 3 : 2) * 64 * R4 + cols + 4) + (size_t)TB * cols) * sizeof(float);
+    if (smem > 200 * 1024) return RB_ERR_BAD_SIZE;
+    auto k = delta_scan_kernel<R4, CH, TB>;
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    RB_LAUNCH((k), dim3((a.vdim + cols - 1) / cols, a.heads, n_seqs), dim3(warps * 32), smem, s, a);
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+// ---- W2 x for few tokens ------------------------------------------------------------------------------------------
+constexpr int LR_TOK = 8;
+struct LowRank {
+    const void *w0, *w1;
+    int x0, rank0, n0, x1, rank1, n1;
+};
+
+template <typename IT, typename WT>
+__global__ void __launch_bounds__(128)
+low_rank_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, int row_stride, const LowRank p, int T,
+                float* __restrict__ out, int ld_out) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float xs[];        // [rank][LR_TOK]
+    const int blocks0 = (p.n0 + 127) / 128;
+    const bool second = (int)blockIdx.x >= blocks0;
+    const int rank = second ? p.rank1 : p.rank0, n = second ? p.n1 : p.n0, x_off = second ? p.x1 : p.x0;
+    const WT* w = static_cast<const WT*>(second ? p.w1 : p.w0);
+    const int row = ((int)blockIdx.x - (second ? blocks0 : 0)) * 128 + threadIdx.x;
+    const int t0 = blockIdx.y * LR_TOK;
+    for (int i = threadIdx.x; i < rank * LR_TOK; i += 128) {
+        const int tt = i / rank, r = i - tt * rank;
+        xs[r * LR_TOK + tt] = t0 + tt < T ? sum_in(in + (size_t)(t0 + tt) * row_stride + x_off + r, n_in, in_stride) : 0.f;
+    }
+    __syncthreads();
+    if (row >= n) return;
+    float acc[LR_TOK] = {};
+    const WT* wr = w + (size_t)row * rank;
+    auto add = [&](float wv, int r) {
+        const float4 lo = *reinterpret_cast<const float4*>(xs + r * LR_TOK), hi = *reinterpret_cast<const float4*>(xs + r * LR_TOK + 4);
+        acc[0] = fmaf(wv, lo.x, acc[0]); acc[1] = fmaf(wv, lo.y, acc[1]); acc[2] = fmaf(wv, lo.z, acc[2]); acc[3] = fmaf(wv, lo.w, acc[3]);
+        acc[4] = fmaf(wv, hi.x, acc[4]); acc[5] = fmaf(wv, hi.y, acc[5]); acc[6] = fmaf(wv, hi.z, acc[6]); acc[7] = fmaf(wv, hi.w, acc[7]);
+    };
+    int r = 0;
+    if ((rank & 3) == 0 && ((uintptr_t)w & (4 * sizeof(WT) - 1)) == 0) {
+        for (; r + 16 <= rank; r += 16) {               // sixteen weights in flight
+            float wv[16];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) load4(wr + r + 4 * u, wv + 4 * u);
+#pragma unroll
+            for (int u = 0; u < 16; ++u) add(wv[u], r + u);
+        }
+    }
+    for (; r < rank; ++r) add(to_f32(wr[r]), r);
+    float* o = out + (size_t)t0 * ld_out + (second ? p.n0 : 0) + row;
+#pragma unroll
+    for (int tt = 0; tt < LR_TOK; ++tt)
+        if (t0 + tt < T) o[(size_t)tt * ld_out] = acc[tt];
+}
+}  // namespace
+
+extern "C" int rb_delta_prep(const void* in, int in_dtype, int n_in, long long in_stride, int row_stride, int q_off, int k_off,
+                             int v_off, int b_off, int heads, int kv_heads, int dim, int vdim, int taps, const float* conv_w,
+                             float* kept, const void* z, int z_dtype, int z_n_in, long long z_in_stride, int z_row_stride,
+                             const float* dt_bias, const float* a_log, int per_channel, float unit_eps, float q_scale,
+                             const int* seq_slot, const int* cu_q, int n_seqs, int max_q_len, float* u, int ld_u, int uq, int uk,
+                             int uv, int ug, int ub, int ud, void* stream) {
+    if (n_seqs <= 0 || max_q_len <= 0) return RB_OK;
+    if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || n_in < 1 || z_n_in < 1 || n_seqs > 65535 ||
+        taps < 1 || taps > PREP_MAX_TAPS || (taps > 1 && !kept))
+        return RB_ERR_BAD_SIZE;
+    const PrepArgs a{(size_t)in_stride, n_in, row_stride, q_off, k_off, v_off, b_off, heads, kv_heads, dim, vdim, taps,
+                     2 * kv_heads * dim + heads * vdim, conv_w, kept, (size_t)z_in_stride, z_n_in, z_row_stride, dt_bias, a_log,
+                     per_channel, unit_eps, q_scale, seq_slot, cu_q, u, ld_u, uq, uk, uv, ug, ub, ud};
+    const dim3 grid(kv_heads + heads, (max_q_len + PREP_TOK - 1) / PREP_TOK, n_seqs);
+    if (grid.y > 65535) return RB_ERR_BAD_SIZE;
+    const dim3 block(max_q_len == 1 ? 32 : 128);
+    const size_t isz = in_dtype == RB_F32 ? 4 : 2, zsz = z_dtype == RB_F32 ? 4 : 2;
+    const bool vec = ((dim | vdim | row_stride | q_off | k_off | v_off | ld_u | uq | uk | uv) & 3) == 0 && (in_stride & 3) == 0 &&
+                     ((uintptr_t)in & (4 * isz - 1)) == 0 && (((uintptr_t)u | (uintptr_t)conv_w | (uintptr_t)kept) & 15) == 0 &&
+                     (!per_channel || (((ug | z_row_stride) & 3) == 0 && (z_in_stride & 3) == 0 && ((uintptr_t)z & (4 * zsz - 1)) == 0 &&
+                                       ((uintptr_t)dt_bias & 15) == 0));
+    cudaStream_t s = (cudaStream_t)stream;
+    typedef __nv_bfloat16 bf;
+#define RB_DP(IT, ZT)                                                                                          \
+    do {                                                                                                       \
+        if (vec) RB_LAUNCH((delta_prep_kernel<IT, ZT, 4>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a); \
+        else RB_LAUNCH((delta_prep_kernel<IT, ZT, 1>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a);     \
+    } while (0)
+    if (in_dtype == RB_F32 && z_dtype == RB_F32) RB_DP(float, float);
+    else if (in_dtype == RB_BF16 && z_dtype == RB_F32) RB_DP(bf, float);
+    else if (in_dtype == RB_BF16 && z_dtype == RB_BF16) RB_DP(bf, bf);
+    else return RB_ERR_BAD_DTYPE;
+#undef RB_DP
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+extern "C" int rb_delta_scan(const float* u, int ld_u, int uq, int uk, int uv, int ug, int ub, int ud, int heads, int kv_heads,
+                             int dim, int vdim, int per_channel, float* state, const int* seq_slot, const int* cu_q, int n_seqs,
+                             float* out, int ld_out, void* stream) {
+    if (n_seqs <= 0) return RB_OK;
+    if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || n_seqs > 65535 || heads > 65535)
+        return RB_ERR_BAD_SIZE;
+    if ((dim & 3) == 0 && ((uintptr_t)state & 15)) return RB_ERR_BAD_ALIGN;
+    ScanArgs a{u, ld_u, uq, uk, uv, ug, ub, ud, heads, kv_heads, dim, vdim, state, seq_slot, cu_q, out, ld_out, 0};
+    a.vec = ((dim | vdim | ld_u | uq | uk | uv) & 3) == 0 && (!per_channel || (ug & 3) == 0) && ((uintptr_t)u & 15) == 0;
+    cudaStream_t s = (cudaStream_t)stream;
+#define RB_DS(R4, TB) return per_channel ? launch_scan<R4, true, TB>(a, n_seqs, s) : launch_scan<R4, false, TB>(a, n_seqs, s)
+    if (dim <= 64) RB_DS(1, 16);
+    if (dim <= 128) RB_DS(2, 16);
+    if (dim <= 256) RB_DS(4, 8);
+    if (dim <= 512) RB_DS(8, 4);
+#undef RB_DS
+    return RB_ERR_BAD_SIZE;
+}
+
+extern "C" int rb_low_rank(const void* in, int in_dtype, int n_in, long long in_stride, int row_stride, int x_off0, int rank0,
+                           const void* w0, int n0, int x_off1, int rank1, const void* w1, int n1, int w_dtype, int T, float* out,
+                           int ld_out, void* stream) {
+    if (T <= 0) return RB_OK;
+    if (rank0 <= 0 || n0 <= 0 || n_in < 1 || n1 < 0 || (n1 > 0 && rank1 <= 0)) return RB_ERR_BAD_SIZE;
+    const int rank = n1 > 0 && rank1 > rank0 ? rank1 : rank0;
+    const size_t smem = (size_t)rank * LR_TOK * sizeof(float);
+    if (smem > 48 * 1024) return RB_ERR_BAD_SIZE;
+    const LowRank p{w0, w1, x_off0, rank0, n0, x_off1, rank1, n1};
+    const dim3 grid((n0 + 127) / 128 + (n1 + 127) / 128, (T + LR_TOK - 1) / LR_TOK);
+    if (grid.y > 65535) return RB_ERR_BAD_SIZE;
+    cudaStream_t s = (cudaStream_t)stream;
+    typedef __nv_bfloat16 bf;
+#define RB_LR(IT, WT) RB_LAUNCH((low_rank_kernel<IT, WT>), grid, dim3(128), smem, s, (const IT*)in, n_in, (size_t)in_stride, row_stride, p, T, out, ld_out)
+    if (in_dtype == RB_F32 && w_dtype == RB_BF16) RB_LR(float, bf);
+    else if (in_dtype == RB_F32 && w_dtype == RB_F32) RB_LR(float, float);
+    else if (in_dtype == RB_BF16 && w_dtype == RB_BF16) RB_LR(bf, bf);
+    else if (in_dtype == RB_BF16 && w_dtype == RB_F32) RB_LR(bf, float);
+    else return RB_ERR_BAD_DTYPE;
+#undef RB_LR
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}

@@ -19,7 +19,7 @@
 // general kernel: `post_norm`, queries and keys divided by their root mean square over the head after the rotation
 // (no weight); `v_out`, the value heads as they came from the projection, 32-bit [T, nkv * vd], for later layers;
 // `v_first` and `v_lambda`, such rows of an earlier layer and a factor on the device: what is stored is
-// (1 - lambda) v + lambda v_first.  The table of cosines and sines may carry a common factor (the position
+// (1 - lambda) v + lambda v_first; `temp_coef` != 0: queries times 1 + temp_coef ln(floor((pos + 1) / temp_every) + 1).  The table of cosines and sines may carry a common factor (the position
 // encoding's magnitude); the kernel's own sincosf path has none.
 #include "common.cuh"
 #include "api.h"
@@ -41,7 +41,7 @@ __global__ void qk_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, s
                                           const float2* __restrict__ cs_table, int vd, int hdp, int interleaved,
                                           int n_gate, float* __restrict__ gate_out, int post_norm,
                                           const float* __restrict__ v_first, const float* __restrict__ v_lambda,
-                                          float* __restrict__ v_out) {
+                                          float* __restrict__ v_out, float temp_coef, float temp_every) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float smem[];
@@ -153,7 +153,8 @@ __global__ void qk_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, s
         ss2 += x * x;
     }
     __syncwarp();
-    const float inv2 = post_norm ? rsqrtf(warp_sum(ss2) / (float)hd + eps) : 1.f;
+    float inv2 = post_norm ? rsqrtf(warp_sum(ss2) / (float)hd + eps) : 1.f;
+    if (kind == 0 && temp_coef != 0.f) inv2 *= query_temperature(pos, temp_coef, temp_every);
     for (int i = lane; i < hd; i += 32) dst[i] = from_f32<AT>(buf[i] * inv2);
 }
 
@@ -188,6 +189,7 @@ struct RotateExt {
     const float* v_first;
     const float* v_lambda;
     float* v_out;
+    float temp_coef, temp_every;
 };
 
 template <typename IT, typename AT, typename WT, bool EXT>
@@ -323,6 +325,11 @@ qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_s
 #pragma unroll
                 for (int i = 0; i < 4; ++i) x[i] *= inv;
             }
+            if (EXT && kind == 0 && ext.temp_coef != 0.f) {
+                const float f = query_temperature(pos, ext.temp_coef, ext.temp_every);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) x[i] *= f;
+            }
         }
         if (sizeof(AT) == 4) {
             *reinterpret_cast<float4*>(dst + lane * 4) = make_float4(x[0], x[1], x[2], x[3]);
@@ -342,7 +349,7 @@ static int launch_qk(const void* in, int n_in, long long in_stride, int row_stri
                      const float* inv_freq, int rot_dim, const int* positions, const int* slot_of_token,
                      const int* block_table, int max_pages, void* k_cache, void* v_cache, int write_kv,
                      const float2* cs_table, int vd, int hdp, int interleaved, int n_gate, float* gate_out, int post_norm,
-                     const float* v_first, const float* v_lambda, float* v_out, cudaStream_t s) {
+                     const float* v_first, const float* v_lambda, float* v_out, float temp_coef, float temp_every, cudaStream_t s) {
     const int warps = 4;
     const long long items = (long long)T * (nq + (write_kv ? 2 * nkv : 0) + (n_gate > 0 ? 1 : 0));
     const long long blocks = (items + warps - 1) / warps;
@@ -354,8 +361,8 @@ static int launch_qk(const void* in, int n_in, long long in_stride, int row_stri
                                                           (uintptr_t)cs_table | (uintptr_t)v_first | (uintptr_t)v_out) & 15) == 0 &&
         (row_stride * esz) % 16 == 0 && ((size_t)in_stride * esz) % 16 == 0 && (q_stride * sizeof(AT)) % 16 == 0) {
         const long long groups = (long long)T * ((nq + (write_kv ? 2 * nkv : 0) + HPW - 1) / HPW);
-        const bool ext = post_norm || v_first || v_out || (inv_freq && rot_dim != 128);
-        const RotateExt e{inv_freq ? rot_dim : 128, post_norm, v_first, v_lambda, v_out};
+        const bool ext = post_norm || v_first || v_out || temp_coef != 0.f || (inv_freq && rot_dim != 128);
+        const RotateExt e{inv_freq ? rot_dim : 128, post_norm, v_first, v_lambda, v_out, temp_coef, temp_every};
 #define RB_QK128(EXT)                                                                                                          \
         RB_LAUNCH((qk_norm_rope_cache_hd128_kernel<IT, AT, WT, EXT>), dim3((int)((groups + 3) / 4)), dim3(128), 0, s, (const IT*)in, \
                   n_in, (size_t)in_stride, row_stride, (AT*)q_out, q_stride, T, nq, nkv, (const WT*)qw, (const WT*)kw, eps,    \
@@ -371,7 +378,7 @@ static int launch_qk(const void* in, int n_in, long long in_stride, int row_stri
               n_in, (size_t)in_stride, row_stride, (AT*)q_out, q_stride, T, nq, nkv, hd, (const WT*)qw,
               (const WT*)kw, eps, inv_freq, rot_dim, positions, slot_of_token, block_table, max_pages,
               (AT*)k_cache, (AT*)v_cache, write_kv, cs_table, vd, hdp, interleaved, n_gate, gate_out, post_norm,
-              v_first, v_lambda, v_out);
+              v_first, v_lambda, v_out, temp_coef, temp_every);
     return RB_OK;
 }
 
@@ -382,8 +389,9 @@ extern "C" int rb_qk_norm_rope_cache(const void* in, int in_dtype, int n_in, lon
                                      const int* slot_of_token, const int* block_table, int max_pages,
                                      void* k_cache, void* v_cache, int write_kv, const void* cos_sin, int vd, int hdp,
                                      int interleaved, int n_gate, float* gate_out, int post_norm, const float* v_first,
-                                     const float* v_lambda, float* v_out, void* stream) {
+                                     const float* v_lambda, float* v_out, float temp_coef, float temp_every, void* stream) {
     if (T <= 0) return RB_OK;
+    if (temp_coef != 0.f && !(temp_every > 0.f)) return RB_ERR_BAD_SIZE;
     if (vd <= 0) vd = hd;
     if (hdp <= 0) hdp = hd > vd ? hd : vd;
     if (hd <= 0 || n_in < 1 || hdp < hd || hdp < vd || (inv_freq && (rot_dim <= 0 || rot_dim % 2 || rot_dim > hd)) ||
@@ -393,7 +401,7 @@ extern "C" int rb_qk_norm_rope_cache(const void* in, int in_dtype, int n_in, lon
     typedef __nv_bfloat16 bf;
 #define RB_QK_ARGS in, n_in, in_stride, row_stride, q_out, q_stride, T, nq, nkv, hd, q_norm_w, k_norm_w, eps, \
                    inv_freq, rot_dim, positions, slot_of_token, block_table, max_pages, k_cache, v_cache, write_kv, \
-                   (const float2*)cos_sin, vd, hdp, interleaved, n_gate, gate_out, post_norm, v_first, v_lambda, v_out, s
+                   (const float2*)cos_sin, vd, hdp, interleaved, n_gate, gate_out, post_norm, v_first, v_lambda, v_out, temp_coef, temp_every, s
     if (in_dtype == RB_BF16 && act_dtype == RB_BF16 && w_dtype == RB_BF16) return launch_qk<bf, bf, bf>(RB_QK_ARGS);
     if (in_dtype == RB_BF16 && act_dtype == RB_BF16 && w_dtype == RB_F32) return launch_qk<bf, bf, float>(RB_QK_ARGS);
     if (in_dtype == RB_F32 && act_dtype == RB_BF16 && w_dtype == RB_BF16) return launch_qk<float, bf, bf>(RB_QK_ARGS);

@@ -8,12 +8,15 @@
 //            With `n_groups` > 1 the experts form that many equal groups of neighbours; a group's score is the
 //            sum of its two largest s_e + bias_e (of its only one, in groups of one), and only experts of the
 //            `keep_groups` best groups (ties: the lower number) can be chosen.  With `renormalize` the weights
-//            are divided by their sum + norm_eps.
+//            are divided by their sum + norm_eps.  The scores can also be the softmax of the logits over all experts, and
+//            the last `identity` experts may be identity experts: a choice of one takes no row (its id is -1), and its
+//            weight joins the token's self weight, by which the sum multiplies the token's own row.
 //   plan     one block: every expert's rows start at a multiple of `tile_rows`; tile i of the row buffer
 //            belongs to expert tile_group[i] (-1: unused).
 //   gather   a token's normalised row is copied to each of its `top` places; row_of[t, j] names the place.
 //   combine  out[t] = sum_j weight[t, j] * y[row_of[t, j]] in 32-bit, j ascending; optionally plus
-//            sigmoid(extra_gate[t]) * (sum of the partial sums extra[s][t]): an expert that every token uses.
+//            sigmoid(extra_gate[t]) * (sum of the partial sums extra[s][t]): an expert that every token uses; and plus
+//            self_weight[t] * self_x[t]: what the identity experts give.
 #include "common.cuh"
 #include "api.h"
 
@@ -126,7 +129,8 @@ template <typename BT>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bias, const int* __restrict__ slot_of_token,
                  int T, int E, int top, int* __restrict__ ids, float* __restrict__ weights, int* __restrict__ place,
-                 int* __restrict__ counts, int n_groups, int keep_groups, int renormalize, float norm_eps) {
+                 int* __restrict__ counts, int n_groups, int keep_groups, int renormalize, float norm_eps, int score, int identity,
+                 float* __restrict__ self_weight) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float route_s[];           // [warps][E + n_groups] when groups are cut, else unused
@@ -135,19 +139,36 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bi
     if (t >= T) return;
     if (slot_of_token[t] < 0) {
         for (int j = lane; j < top; j += 32) { ids[(size_t)t * top + j] = -1; weights[(size_t)t * top + j] = 0.f; place[(size_t)t * top + j] = 0; }
+        if (lane == 0 && self_weight) self_weight[t] = 0.f;
         return;
     }
     float s[MAX_EPL], c[MAX_EPL];
+    float top_z = -INFINITY;
 #pragma unroll
     for (int i = 0; i < MAX_EPL; ++i) {
         const int e = lane + i * 32;
-        if (e < E) {
-            s[i] = 1.f / (1.f + expf(-z[(size_t)t * ldz + e]));
-            c[i] = s[i] + (bias ? to_f32(bias[e]) : 0.f);
-        } else {
-            s[i] = 0.f;
-            c[i] = -INFINITY;
+        s[i] = e < E ? z[(size_t)t * ldz + e] : -INFINITY;
+        top_z = fmaxf(top_z, s[i]);
+    }
+    if (score == 1) {          // softmax over all of them
+        top_z = warp_max(top_z);
+        float sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < MAX_EPL; ++i) {
+            s[i] = lane + i * 32 < E ? expf(s[i] - top_z) : 0.f;
+            sum += s[i];
         }
+        sum = warp_sum(sum);
+#pragma unroll
+        for (int i = 0; i < MAX_EPL; ++i) s[i] /= sum;
+    } else {
+#pragma unroll
+        for (int i = 0; i < MAX_EPL; ++i) s[i] = lane + i * 32 < E ? 1.f / (1.f + expf(-s[i])) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < MAX_EPL; ++i) {
+        const int e = lane + i * 32;
+        c[i] = e < E ? s[i] + (bias ? to_f32(bias[e]) : 0.f) : -INFINITY;
     }
     if (n_groups > 1 && keep_groups < n_groups) {
         // the groups' cut: scores to shared memory, a lane scores whole groups, the best groups are marked
@@ -188,7 +209,8 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bi
             if (e < E && gs[e / per] != -INFINITY) c[i] = -INFINITY;       // its group was not kept
         }
     }
-    float picked_sum = 0.f;
+    float picked_sum = 0.f, self_sum = 0.f;
+    const int real = E - identity;           // the experts that have rows
     for (int j = 0; j < top; ++j) {
         float best = -INFINITY, best_s = 0.f;
         int best_e = 0x7fffffff;
@@ -209,16 +231,19 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bi
             if (lane + i * 32 == best_e) c[i] = -INFINITY;
         if (best_e >= E) best_e = E - 1;      // scores that compare with nothing (NaN): stay inside the tables
         picked_sum += best_s;
+        if (best_e >= real) self_sum += best_s;
         if (lane == 0) {
-            ids[(size_t)t * top + j] = best_e;
+            ids[(size_t)t * top + j] = best_e < real ? best_e : -1;
             weights[(size_t)t * top + j] = best_s;
-            place[(size_t)t * top + j] = atomicAdd(&counts[best_e], 1);
+            place[(size_t)t * top + j] = best_e < real ? atomicAdd(&counts[best_e], 1) : 0;
         }
     }
     if (renormalize && lane == 0) {
         const float d = picked_sum + norm_eps;
         for (int j = 0; j < top; ++j) weights[(size_t)t * top + j] /= d;
+        self_sum /= d;
     }
+    if (self_weight && lane == 0) self_weight[t] = self_sum;
 }
 
 __global__ void __launch_bounds__(256)
@@ -265,10 +290,12 @@ moe_gather_kernel(const AT* __restrict__ x, int H, const int* __restrict__ ids, 
     }
 }
 
+template <typename XT>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, long long ldy, const int* __restrict__ row_of, const float* __restrict__ weights,
                    int top, float* __restrict__ out, int H, const float* __restrict__ extra, int n_extra,
-                   long long extra_stride, const float* __restrict__ extra_gate, int extra_gate_ld) {
+                   long long extra_stride, const float* __restrict__ extra_gate, int extra_gate_ld,
+                   const float* __restrict__ self_weight, const XT* __restrict__ self_x) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -279,6 +306,7 @@ moe_combine_kernel(const float* __restrict__ y, long long ldy, const int* __rest
             const int r = row_of[(size_t)t * top + j];
             if (r >= 0) v = fmaf(weights[(size_t)t * top + j], y[(size_t)r * ldy + i], v);
         }
+        if (self_weight) v = fmaf(self_weight[t], to_f32(self_x[(size_t)t * H + i]), v);
         if (extra) {
             float x = 0.f;
             for (int s = 0; s < n_extra; ++s) x += extra[(size_t)s * extra_stride + (size_t)t * H + i];
@@ -313,9 +341,11 @@ extern "C" int rb_router_logits(const void* x, int x_dtype, long long ldx, const
 
 extern "C" int rb_moe_route(const float* z, int ldz, const void* bias, int bias_dtype, const int* slot_of_token, int T,
                             int E, int top, int* ids, float* weights, int* place, int* counts, int n_groups,
-                            int keep_groups, int renormalize, float norm_eps, void* stream) {
+                            int keep_groups, int renormalize, float norm_eps, int score, int identity, float* self_weight,
+                            void* stream) {
     if (T <= 0) return RB_OK;
     if (E <= 0 || E > 32 * MAX_EPL || top <= 0 || top > E) return RB_ERR_BAD_SIZE;
+    if (identity < 0 || identity >= E || (identity > 0 && !self_weight) || score < 0 || score > 1) return RB_ERR_BAD_SIZE;
     if (n_groups < 1) n_groups = 1;
     if (keep_groups < 1 || keep_groups > n_groups) keep_groups = n_groups;
     if (E % n_groups || (long long)keep_groups * (E / n_groups) < top) return RB_ERR_BAD_SIZE;
@@ -325,10 +355,10 @@ extern "C" int rb_moe_route(const float* z, int ldz, const void* bias, int bias_
     const size_t smem = (n_groups > 1 && keep_groups < n_groups) ? (size_t)warps * (E + n_groups) * sizeof(float) : 0;
     if (!bias || bias_dtype == RB_F32)
         RB_LAUNCH((moe_route_kernel<float>), grid, dim3(warps * 32), smem, s, z, ldz, (const float*)bias, slot_of_token, T, E, top,
-                  ids, weights, place, counts, n_groups, keep_groups, renormalize, norm_eps);
+                  ids, weights, place, counts, n_groups, keep_groups, renormalize, norm_eps, score, identity, self_weight);
     else if (bias_dtype == RB_BF16)
         RB_LAUNCH((moe_route_kernel<__nv_bfloat16>), grid, dim3(warps * 32), smem, s, z, ldz, (const __nv_bfloat16*)bias,
-                  slot_of_token, T, E, top, ids, weights, place, counts, n_groups, keep_groups, renormalize, norm_eps);
+                  slot_of_token, T, E, top, ids, weights, place, counts, n_groups, keep_groups, renormalize, norm_eps, score, identity, self_weight);
     else
         return RB_ERR_BAD_DTYPE;
     RB_LAUNCH_CHECK();
@@ -361,10 +391,18 @@ extern "C" int rb_moe_gather(const void* x, int dtype, int H, const int* ids, co
 
 extern "C" int rb_moe_combine(const float* y, long long ldy, const int* row_of, const float* weights, int T, int top,
                               float* out, int H, const float* extra, int n_extra, long long extra_stride,
-                              const float* extra_gate, int extra_gate_ld, void* stream) {
+                              const float* extra_gate, int extra_gate_ld, const float* self_weight, const void* self_x,
+                              int self_dtype, void* stream) {
     if (T <= 0) return RB_OK;
-    RB_LAUNCH((moe_combine_kernel), dim3(T), dim3(256), 0, (cudaStream_t)stream, y, ldy, row_of, weights, top, out, H,
-              extra, n_extra, extra_stride, extra_gate, extra_gate_ld);
+    if (self_weight && !self_x) return RB_ERR_BAD_SIZE;
+    if (!self_weight || self_dtype == RB_F32)
+        RB_LAUNCH((moe_combine_kernel<float>), dim3(T), dim3(256), 0, (cudaStream_t)stream, y, ldy, row_of, weights, top, out, H,
+                  extra, n_extra, extra_stride, extra_gate, extra_gate_ld, self_weight, (const float*)self_x);
+    else if (self_dtype == RB_BF16)
+        RB_LAUNCH((moe_combine_kernel<__nv_bfloat16>), dim3(T), dim3(256), 0, (cudaStream_t)stream, y, ldy, row_of, weights, top,
+                  out, H, extra, n_extra, extra_stride, extra_gate, extra_gate_ld, self_weight, (const __nv_bfloat16*)self_x);
+    else
+        return RB_ERR_BAD_DTYPE;
     RB_LAUNCH_CHECK();
     return RB_OK;
 }

@@ -74,6 +74,8 @@ class Model:
         out = [TensorDecl(self.spec.embedding_name, (self.vocab, self.hidden), "matrix")]
         if self.embedding_norm is not None:
             out += self.embedding_norm.declare(self.spec.embedding_norm_name[: -len(".weight")])
+        if self.input_position is not None:
+            out += self.input_position.declare(self.spec.input_position_name[: -len(".weight")])
         for name, rows in self.added_rows.items():
             out.append(TensorDecl(name, (rows, self.hidden), "matrix"))
         for b in self.blocks:
@@ -100,6 +102,8 @@ class Model:
         self.embed = tensors[self.spec.embedding_name]
         if self.embedding_norm is not None:
             self.embedding_norm.load(tensors, self.spec.embedding_norm_name[: -len(".weight")])
+        if self.input_position is not None:
+            self.input_position.load(tensors, self.spec.input_position_name[: -len(".weight")])
         self.added = {name: tensors[name] for name in self.added_rows}
         for b in self.blocks:
             b.load(tensors)
@@ -181,7 +185,8 @@ class Model:
             else:
                 kernels.embedding_pos(batch.token_ids, self.embed, rows, self.spec.embedding_scale, batch.positions,
                                       self.input_position.inv_freq if self.input_position is not None else None,
-                                      copy=x0 if rows is resid else None, status=self.status)
+                                      copy=x0 if rows is resid else None, status=self.status,
+                                      pos_table=getattr(self.input_position, "table", None))
         if self.embedding_norm is not None:
             with scope(op="embedding_norm"):
                 kernels.add_rmsnorm(rows, None, self.embedding_norm.weight, self.embedding_norm.eps, resid, n_rows=T,
@@ -221,7 +226,10 @@ class Model:
             xn = self.final_norm.forward(resid, pending, n_rows=batch.n_want, rows=batch.want_rows, write_back=False)
         logits = torch.empty((batch.n_want, self.vocab), dtype=torch.float32, device=self.env.device)
         self.head.forward(xn, logits, batch.n_want)
-        if self.spec.logit_scale != 1.0:
+        if self.spec.logit_softcap is not None:
+            with scope(op="logit_softcap"):
+                kernels.softcap_(logits, self.spec.logit_softcap, self.spec.logit_scale)
+        elif self.spec.logit_scale != 1.0:
             with scope(op="logit_scale"):
                 kernels.scale_(logits, self.spec.logit_scale)
         return logits

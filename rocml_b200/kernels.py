@@ -131,23 +131,23 @@ def _lib():
         lib.rb_cast.argtypes = [_vp, _i, _vp, _i, _ll, _vp]
         lib.rb_qk_norm_rope_cache.argtypes = [_vp, _i, _i, _ll, _i, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _f,
                                               _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _i, _i, _vp, _i, _vp,
-                                              _vp, _vp, _vp]
+                                              _vp, _vp, _f, _f, _vp]
         lib.rb_rope_table.argtypes = [_vp, _vp, _i, _i, _f, _vp, _vp]
         lib.rb_gemm_generic.argtypes = [_vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _ll, _ll, _i, _ll, _vp]
         lib.rb_attention_generic.argtypes = [_vp, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i,
-                                             _i, _i, _i, _f, _i, _i, _f, _i, _i, _vp, _vp, _i, _vp]
-        lib.rb_attention_merge.argtypes = [_vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp]
+                                             _i, _i, _i, _f, _i, _i, _f, _vp, _i, _i, _vp, _vp, _i, _vp]
+        lib.rb_attention_merge.argtypes = [_vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp]
         lib.rb_argmax.argtypes = [_vp, _ll, _i, _i, _vp, _vp, _vp, _i, _vp]
         lib.rb_attention_prefill.argtypes = [_vp, _i, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i,
-                                             _f, _i, _i, _f, _vp]
+                                             _f, _i, _i, _f, _vp, _vp]
         lib.rb_attention_prefill_tc5.argtypes = [_vp, _i, _i, _vp, _i, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i,
-                                                 _i, _i, _i, _f, _i, _i, _f, _i, _vp, _vp, _ll, _i, _vp]
-        lib.rb_attention_decode.argtypes = [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _f, _i,
+                                                 _i, _i, _i, _f, _i, _i, _f, _vp, _i, _vp, _vp, _ll, _i, _vp]
+        lib.rb_attention_decode.argtypes = [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _f, _vp, _i,
                                             _i, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _ll, _ll, _i, _vp]
         lib.rb_attention_decode_fused.argtypes = [_vp, _i, _ll, _i, _vp, _vp, _i, _f, _vp, _i, _vp, _i, _ll, _f, _i,
                                                   _vp, _vp, _vp, _i, _vp, _vp,
                                                   _vp, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _vp, _vp, _vp, _i,
-                                                  _i, _f, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _ll, _ll, _vp]
+                                                  _i, _f, _vp, _f, _f, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _ll, _ll, _vp]
         lib.rb_sample.argtypes = [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp]
         lib.rb_gemm_tcgen05.argtypes = [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _ll, _ll, _i, _ll, _i, _i, _vp, _vp]
         lib.rb_gemm_tcgen05_add.argtypes = [_vp, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _i, _vp, _vp]
@@ -157,7 +157,7 @@ def _lib():
         lib.rb_gemm_tcgen05_residual.argtypes = [_vp, _vp, _vp, _i, _i, _i, _ll, _i, _vp, _ll, _vp, _i, _vp, _ll, _vp,
                                                  _ll, _i, _vp, _vp]
         lib.rb_hold.argtypes = [_ll, _vp]
-        lib.rb_embedding_pos.argtypes = [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _vp, _vp, _vp, _vp]
+        lib.rb_embedding_pos.argtypes = [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _vp, _vp, _vp, _i, _i, _vp, _vp]
         lib.rb_residual_inject.argtypes = [_vp, _vp, _i, _ll, _vp, _vp, _i, _i, _i, _vp]
         lib.rb_postnorm_add_norm.argtypes = [_vp, _vp, _i, _ll, _vp, _vp, _i, _vp, _f, _vp, _f, _i, _vp, _i, _i, _i, _vp]
         lib.rb_gated_act.argtypes = [_vp, _i, _i, _ll, _ll, _vp, _i, _ll, _i, _i, _i, _f, _f, _i, _vp]
@@ -166,10 +166,10 @@ def _lib():
         lib.rb_scale.argtypes = [_vp, _ll, _f, _vp]
         lib.rb_latent_prep.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _vp, _i, _f, _vp, _i, _vp, _vp, _i, _vp, _vp,
                                        _vp, _i, _i, _vp]
-        lib.rb_moe_route.argtypes = [_vp, _i, _vp, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _vp]
+        lib.rb_moe_route.argtypes = [_vp, _i, _vp, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _vp, _vp]
         lib.rb_moe_plan.argtypes = [_vp, _i, _i, _i, _vp, _vp, _vp]
         lib.rb_moe_gather.argtypes = [_vp, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _vp]
-        lib.rb_moe_combine.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _vp, _i, _vp, _i, _ll, _vp, _i, _vp]
+        lib.rb_moe_combine.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _vp, _i, _vp, _i, _ll, _vp, _i, _vp, _vp, _i, _vp]
         lib.rb_grouped_matmul.argtypes = [_vp, _i, _ll, _i, _vp, _i, _ll, _vp, _i, _ll, _i, _i, _i, _i, _i, _vp, _i,
                                           _vp, _i, _i, _f, _f, _vp]
         lib.rb_head_gate.argtypes = [_vp, _ll, _i, _vp, _ll, _i, _vp, _i, _vp, _i, _i, _ll, _ll, _i, _i, _i, _vp]
@@ -194,6 +194,13 @@ def _lib():
         lib.rb_wide_norm_rope_cache.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _vp, _vp, _i, _i, _vp,
                                                 _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _vp]
         lib.rb_talk_mix.argtypes = [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp]
+        lib.rb_softcap.argtypes = [_vp, _ll, _f, _f, _vp]
+        lib.rb_add_layernorm.argtypes = [_vp, _vp, _i, _ll, _vp, _vp, _vp, _i, _vp, _i, _i, _f, _i, _vp]
+        lib.rb_out_norm.argtypes = [_vp, _vp, _i, _ll, _f, _vp, _vp, _i, _vp, _vp, _i, _i, _vp, _vp, _f, _f, _vp, _i, _i, _i, _vp]
+        lib.rb_delta_prep.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _ll, _i, _vp,
+                                      _vp, _i, _f, _f, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]
+        lib.rb_delta_scan.argtypes = [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp]
+        lib.rb_low_rank.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _vp, _i, _i, _i, _vp, _i, _i, _i, _vp, _i, _vp]
         lib.rb_gemm_tcgen05_set_wait.argtypes = [_ll, _i]
         lib.rb_gemm_tcgen05_set_wait.restype = None
         _sigs_done = True
@@ -315,7 +322,7 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_out: torch.Tensor, n_tokens: int, n
                        padded_head_dim: Optional[int] = None, interleaved: bool = False,
                        gates: Optional[torch.Tensor] = None, post_norm: bool = False,
                        v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None,
-                       v_out: Optional[torch.Tensor] = None):
+                       v_out: Optional[torch.Tensor] = None, q_temp=None):
     """``cos_sin`` (from rope_table, float32 [T, rot_dim / 2, 2]) replaces the kernel's own sincosf.
     proj [T, nq*hd (+ nkv*hd + nkv*vd) (+ gates)] (or [S, T, ...] partial sums): q normalised and rotated into
     q_out (rows of nq*hdp, any row stride; it may be ``proj`` itself when nothing is padded); k (normalised,
@@ -325,7 +332,8 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_out: torch.Tensor, n_tokens: int, n
     (float32 [T, n]): the sigmoid of the row's last n columns.  ``post_norm``: q and k are divided by their root
     mean square over the head (eps inside the root, no weight) after the rotation.  ``v_out`` (float32 [T, nkv * vd])
     receives the value heads as projected; ``v_first`` (such rows of an earlier layer) and ``v_lambda`` (float32,
-    one number on the device): the cache receives (1 - lambda) v + lambda v_first."""
+    one number on the device): the cache receives (1 - lambda) v + lambda v_first.  ``q_temp`` (coef, every): queries are
+    multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p, after everything else."""
     vd = hd if v_head_dim is None else int(v_head_dim)
     hdp = max(hd, vd) if padded_head_dim is None else int(padded_head_dim)
     n_gate = 0 if gates is None else gates.shape[-1]
@@ -365,7 +373,7 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_out: torch.Tensor, n_tokens: int, n
         rot_dim, _i32(positions, "positions"), _i32(slot_of_token, "slot_of_token"),
         None if block_table is None else _i32(block_table, "block_table"), max_pages, _ptr(k_cache), _ptr(v_cache),
         1 if write_kv else 0, _ptr(cos_sin), vd, hdp, 1 if interleaved else 0, n_gate, _ptr(gates),
-        1 if post_norm else 0, _ptr(v_first), _ptr(v_lambda), _ptr(v_out), _stream())
+        1 if post_norm else 0, _ptr(v_first), _ptr(v_lambda), _ptr(v_out), *_temperature(q_temp), _stream())
     _check(rc, "qk_norm_rope_cache")
 
 
@@ -417,10 +425,10 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                       block_table: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                       n_seqs: int, max_q_len: int, nq: int, nkv: int, hd: int, scale: float, window: int = 0,
                       chunk: int = 0, n_chunks: int = 1, part_acc: Optional[torch.Tensor] = None,
-                      part_ml: Optional[torch.Tensor] = None, keep: int = 0, sink: Optional[float] = None, cross: int = 0):
+                      part_ml: Optional[torch.Tensor] = None, keep: int = 0, sink=None, cross: int = 0):
     """q rows [T, >= nq*hd] (row stride free) -> out rows [T, >= nq*hd]; keys and values from the pages.
     ``keep``: the keys at positions below it stay visible beside the window; ``sink``: a score that adds
-    exp(sink) to every row's denominator and brings no value (None: no such term).  ``cross`` (n > 1, the cache's
+    exp(sink) to every row's denominator and brings no value (None: no such term; a float32 tensor [nq]: one a query head).  ``cross`` (n > 1, the cache's
     own number of key/value heads): every query head's weights are applied to the values of EVERY stored head;
     ``nkv`` = n * n then counts (key head, value head) pairs, ``nq`` = n * query heads the results, pair
     (a, m) at a * n + m with the results of key head a's queries in their order, and q holds nq / n heads."""
@@ -432,7 +440,7 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     rc = _lib().rb_attention_generic(
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), dtype_code(q.dtype), _ptr(k_cache), _ptr(v_cache),
         _i32(block_table, "block_table"), block_table.shape[1], _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"),
-        _i32(kv_len, "kv_len"), n_seqs, max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), _sink(sink),
+        _i32(kv_len, "kv_len"), n_seqs, max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), *_sink(sink, nq),
         int(chunk), int(n_chunks), _ptr(part_acc), _ptr(part_ml), int(cross), _stream())
     _check(rc, "attention_generic")
 
@@ -440,8 +448,24 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
 NO_SINK = -3.0e38     # RB_NO_SINK of csrc/common.cuh
 
 
-def _sink(sink: Optional[float]) -> float:
-    return NO_SINK if sink is None else float(sink)
+def _sink(sink, nq: int):
+    """A layer's sink as the kernels take it: (one score for all heads, one score a query head).  ``sink``: None, a number,
+    or a float32 tensor [nq]."""
+    if sink is None:
+        return NO_SINK, None
+    if isinstance(sink, torch.Tensor):
+        return NO_SINK, _f32vec(sink, nq, "sink")
+    return float(sink), None
+
+
+def _temperature(q_temp):
+    """(coef, every) of a temperature that grows with the query's position: 1 + coef ln(floor((p + 1) / every) + 1)."""
+    if q_temp is None:
+        return 0.0, 1.0
+    coef, every = float(q_temp[0]), float(q_temp[1])
+    if not every > 0:
+        raise KernelError("the query temperature's 'every' must be positive")
+    return coef, every
 
 
 PREFILL_L2_BYTES = 96 << 20     # keys and values that stay in the 126 MB L2 cache beside everything else
@@ -460,7 +484,7 @@ def prefill_heads_first(n_seqs: int, nkv: int, hd: int, max_kv_len: int, window:
 def attention_prefill_tc5(q: torch.Tensor, n_tokens: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                           block_table: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                           n_seqs: int, max_q_len: int, nq: int, nkv: int, hd: int, scale: float, window: int = 0,
-                          max_kv_len: Optional[int] = None, keep: int = 0, sink: Optional[float] = None,
+                          max_kv_len: Optional[int] = None, keep: int = 0, sink=None,
                           gate: Optional[torch.Tensor] = None, cross: int = 0) -> bool:
     """bfloat16 flash attention with tcgen05 (accumulators in tensor memory, TMA loads), head sizes 64, 128 and 256.
     ``cross`` (n > 1, the cache's own number of key/value heads): as in ``attention_generic``.
@@ -483,7 +507,7 @@ def attention_prefill_tc5(q: torch.Tensor, n_tokens: int, out: torch.Tensor, k_c
     rc = _lib().rb_attention_prefill_tc5(
         _ptr(q), q.stride(0), n_tokens, _ptr(out), out.stride(0), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0],
         _i32(block_table, "block_table"), block_table.shape[1], _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"),
-        _i32(kv_len, "kv_len"), n_seqs, max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), _sink(sink),
+        _i32(kv_len, "kv_len"), n_seqs, max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), *_sink(sink, nq),
         1 if prefill_heads_first(n_seqs, nkv, hd, max_q_len if max_kv_len is None else max_kv_len, window) else 0,
         _ptr(status_word(q.device)), _ptr(gate), gate.stride(0) if gate is not None else 0, int(cross), _stream())
     if rc in (10001, 10003):
@@ -496,7 +520,7 @@ def attention_prefill_tc5(q: torch.Tensor, n_tokens: int, out: torch.Tensor, k_c
 def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       block_table: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                       n_seqs: int, max_q_len: int, nq: int, nkv: int, hd: int, scale: float, window: int = 0,
-                      keep: int = 0, sink: Optional[float] = None) -> bool:
+                      keep: int = 0, sink=None) -> bool:
     """bfloat16 flash attention on the tensor cores for any number of query tokens per sequence.
     ``keep``: beside a window the keys at positions below it stay visible; ``sink``: a score whose exponential
     joins every row's denominator.
@@ -509,7 +533,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     rc = _lib().rb_attention_prefill(
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_cache), _ptr(v_cache), _i32(block_table, "block_table"),
         block_table.shape[1], _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), _i32(kv_len, "kv_len"), n_seqs,
-        max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), _sink(sink), _stream())
+        max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), *_sink(sink, nq), _stream())
     if rc in (10001, 10003):
         return False
     _check(rc, "attention_prefill")
@@ -578,7 +602,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
                      block_table: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                      n_seqs: int, nq: int, nkv: int, hd: int, scale: float, window: int, n_chunks: int,
                      part_acc: Optional[torch.Tensor], part_ml: Optional[torch.Tensor],
-                     pages_per_block: int = 1, keep: int = 0, sink: Optional[float] = None,
+                     pages_per_block: int = 1, keep: int = 0, sink=None,
                      gate: Optional[torch.Tensor] = None, cross: int = 0) -> bool:
     """``cross`` (n > 1, the cache's own number of key/value heads): as in ``attention_generic``.  ``keep``: the keys at positions below it stay visible beside the window (not with ``pages_per_block`` 0);
     ``sink``: a score whose exponential joins every row's denominator.  ``gate``: [T, nq * hd] or [S, T, nq * hd]
@@ -608,7 +632,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
     rc = _lib().rb_attention_decode(
         _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _i32(block_table, "block_table"), block_table.shape[1],
         _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), _i32(kv_len, "kv_len"), n_seqs, nq, nkv, hd, float(scale),
-        int(window), int(keep), _sink(sink), int(n_chunks), int(pages_per_block), _ptr(part_acc), _ptr(part_ml),
+        int(window), int(keep), *_sink(sink, nq), int(n_chunks), int(pages_per_block), _ptr(part_acc), _ptr(part_ml),
         _ptr(decode_counters(q.device)), _ptr(out),
         out.stride(0), _ptr(gate), 1 if gate is not None and gate.dtype == torch.float32 else 0, g_n, g_in, g_row, int(cross),
         _stream())
@@ -626,9 +650,9 @@ def attention_decode_fused(proj: torch.Tensor, out: torch.Tensor, k_cache: torch
                            write_kv: bool, scale: float, window: int, n_chunks: int,
                            part_acc: Optional[torch.Tensor], part_ml: Optional[torch.Tensor],
                            pages_per_block: int = 1, rowscale=None, row_width: int = 0, keep: int = 0,
-                           sink: Optional[float] = None, rot_dim: int = 0, post_norm: bool = False,
+                           sink=None, rot_dim: int = 0, post_norm: bool = False,
                            v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None,
-                           v_keep: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> bool:
+                           v_keep: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, q_temp=None) -> bool:
     """attention_decode for head size 128 that takes the step's projections as the matrix product left
     them: ``proj`` float32 [S, T, (nq + 2 nkv) * 128] partial sums (or [T, ...]; only the nq query heads
     when ``write_kv`` is off).  The kernel adds them, applies the per-head norm and the rotation
@@ -639,7 +663,8 @@ def attention_decode_fused(proj: torch.Tensor, out: torch.Tensor, k_cache: torch
     ``keep``, ``sink`` and ``gate`` as in attention_decode.  ``rot_dim`` (0: the whole head): only the first
     rot_dim dimensions of a head turn and ``cos_sin`` is [T, rot_dim / 2, 2]; ``post_norm``: queries and keys are divided
     by their root mean square after the rotation; ``v_keep``: float32 [T, nkv * 128], receives the new values as projected;
-    ``v_first`` and ``v_lambda`` (float32 [1]): such rows of an earlier layer, blended into what is cached.  With any
+    ``v_first`` and ``v_lambda`` (float32 [1]): such rows of an earlier layer, blended into what is cached; ``q_temp``
+    (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1) at position p.  With any
     of these the rows may hold further columns after the heads.
     Returns False when the kernel does not take the sizes (use the two kernels)."""
     if hd != 128 or proj.dtype != torch.float32 or k_cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 \
@@ -681,7 +706,7 @@ def attention_decode_fused(proj: torch.Tensor, out: torch.Tensor, k_cache: torch
         _ptr(k_cache), _ptr(v_cache), _i32(block_table, "block_table"), block_table.shape[1],
         _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), _i32(kv_len, "kv_len"), n_seqs, nq, nkv, hd, float(scale),
         int(window), int(n_chunks), int(pages_per_block), _ptr(part_acc), _ptr(part_ml),
-        _ptr(decode_counters(out.device)), _ptr(out), out.stride(0), int(keep), _sink(sink), rot, 1 if post_norm else 0,
+        _ptr(decode_counters(out.device)), _ptr(out), out.stride(0), int(keep), *_sink(sink, nq), *_temperature(q_temp), rot, 1 if post_norm else 0,
         _ptr(v_first), _ptr(v_lambda), _ptr(v_keep), _ptr(gate), 1 if gate is not None and gate.dtype == torch.float32 else 0,
         g_n, g_in, g_row, _stream())
     if rc in (10001, 10003):
@@ -693,10 +718,10 @@ def attention_decode_fused(proj: torch.Tensor, out: torch.Tensor, k_cache: torch
 @_profiled(lambda a, facts: (a["part_acc"].numel() * 4 + a["part_ml"].numel() * 4 + a["n_tokens"] * a["nq"] * a["hd"] * _esz(a["out"]), 0))
 def attention_merge(part_acc: torch.Tensor, part_ml: torch.Tensor, out: torch.Tensor, positions: torch.Tensor,
                     slot_of_token: torch.Tensor, n_tokens: int, nq: int, hd: int, chunk: int, n_chunks: int,
-                    window: int = 0, keep: int = 0, sink: Optional[float] = None):
+                    window: int = 0, keep: int = 0, sink=None):
     rc = _lib().rb_attention_merge(_ptr(part_acc), _ptr(part_ml), _ptr(out), out.stride(0), dtype_code(out.dtype),
                                    _i32(positions, "positions"), _i32(slot_of_token, "slot_of_token"), n_tokens,
-                                   nq, hd, chunk, n_chunks, int(window), int(keep), _sink(sink), _stream())
+                                   nq, hd, chunk, n_chunks, int(window), int(keep), *_sink(sink, nq), _stream())
     _check(rc, "attention_merge")
 
 
@@ -986,9 +1011,10 @@ def gemm_tcgen05_qkv_rope(x: torch.Tensor, w: torch.Tensor, q_out: torch.Tensor,
 @_profiled(lambda a, facts: _cost.embedding(a["out"].shape[0], a["out"].shape[1], _esz(a["table"])))
 def embedding_pos(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float, positions: torch.Tensor,
                   inv_freq: Optional[torch.Tensor], copy: Optional[torch.Tensor] = None,
-                  status: Optional[torch.Tensor] = None):
+                  status: Optional[torch.Tensor] = None, pos_table: Optional[torch.Tensor] = None):
     """out[t, i] = float32(table[ids[t], i]) * scale + (sin | cos)(positions[t] * inv_freq[i // 2]) for even | odd i
-    (nothing is added without ``inv_freq``); ``copy`` receives the same rows."""
+    (nothing is added without ``inv_freq``); with ``pos_table`` [rows, H] of the table's type its row positions[t] is added
+    instead; ``copy`` receives the same rows."""
     T, H = out.shape
     if out.dtype != torch.float32 or not out.is_contiguous() or not table.is_contiguous() or table.shape[1] != H:
         raise KernelError("embedding_pos: out must be contiguous float32 [T, H], table contiguous [vocab, H]")
@@ -996,9 +1022,13 @@ def embedding_pos(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, sca
         raise KernelError("embedding_pos: copy must look like out")
     if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() < (H + 1) // 2):
         raise KernelError("embedding_pos: inv_freq must be float32 [ceil(H / 2)]")
+    if pos_table is not None and (pos_table.dtype != table.dtype or not pos_table.is_contiguous() or pos_table.dim() != 2 or
+                                  pos_table.shape[1] != H or inv_freq is not None):
+        raise KernelError("embedding_pos: pos_table must be contiguous [rows, H] of the table's type, without inv_freq")
     rc = _lib().rb_embedding_pos(_i32(ids, "ids"), _ptr(table), dtype_code(table.dtype), _ptr(out), _ptr(copy), T, H,
-                                 table.shape[0], float(scale), _i32(positions, "positions"), _ptr(inv_freq),
-                                 _ptr(status), _stream())
+                                 table.shape[0], float(scale), _i32(positions, "positions"), _ptr(inv_freq), _ptr(pos_table),
+                                 dtype_code(pos_table.dtype) if pos_table is not None else F32,
+                                 pos_table.shape[0] if pos_table is not None else 0, _ptr(status), _stream())
     _check(rc, "embedding_pos")
 
 
@@ -1092,6 +1122,14 @@ def scale_(x: torch.Tensor, factor: float):
     _check(_lib().rb_scale(_ptr(x), x.numel(), float(factor), _stream()), "scale_")
 
 
+@_profiled(lambda a, facts: (a["x"].numel() * 8, a["x"].numel() * 4))
+def softcap_(x: torch.Tensor, cap: float, factor: float = 1.0):
+    """x <- cap * tanh(factor * x / cap) in place (contiguous float32)."""
+    if x.dtype != torch.float32 or not x.is_contiguous() or not cap > 0:
+        raise KernelError("softcap_: x must be contiguous float32 and the cap positive")
+    _check(_lib().rb_softcap(_ptr(x), x.numel(), float(factor), float(cap), _stream()), "softcap_")
+
+
 # ---- latent attention: between the projection and the attention ---------------------------------------------------
 
 @_profiled(lambda a, facts: (a["n_tokens"] * (a["proj"].shape[-1] * _esz(a["proj"]) * _n_in(a["proj"])
@@ -1137,16 +1175,22 @@ def router_logits(x: torch.Tensor, w: torch.Tensor, z: torch.Tensor, n_tokens: i
                                    _stream()), "router_logits")
 
 
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
+
+
 @_profiled(lambda a, facts: (a["n_tokens"] * (a["z"].shape[1] * 4 + a["top"] * 12), a["n_tokens"] * a["z"].shape[1] * 8))
 def moe_route(z: torch.Tensor, bias: Optional[torch.Tensor], slot_of_token: torch.Tensor, n_tokens: int, top: int,
               ids: torch.Tensor, weights: torch.Tensor, place: torch.Tensor, counts: torch.Tensor,
-              n_groups: int = 1, keep_groups: int = 1, renormalize: bool = False, norm_eps: float = 0.0):
+              n_groups: int = 1, keep_groups: int = 1, renormalize: bool = False, norm_eps: float = 0.0, score: str = "sigmoid",
+              identity: int = 0, self_weight: Optional[torch.Tensor] = None):
     """z float32 [T, >= E] router logits -> per token the ``top`` experts by sigmoid(z) + bias (``ids`` int32 [T, top],
     -1 for padding tokens), their weights sigmoid(z) (float32 [T, top]) and each choice's place among its expert's
     rows (``place``); ``counts`` int32 [E], zero on entry, ends as the rows of every expert (E is its length; z may
     have more columns).  ``n_groups`` > 1: the experts form equal groups of neighbours, a group's score is the sum of
     its two largest scores, and only experts of the ``keep_groups`` best groups can be chosen.  ``renormalize``: the
-    weights are divided by their sum + ``norm_eps``."""
+    weights are divided by their sum + ``norm_eps``.  ``score`` "softmax": the scores are the softmax over all E.  The last
+    ``identity`` of the E are identity experts: a choice of one has no row (its id is -1), and its weight is summed into
+    ``self_weight`` float32 [T]."""
     E = counts.numel()
     if z.shape[1] < E:
         raise KernelError("moe_route: fewer router logits than experts")
@@ -1159,10 +1203,15 @@ def moe_route(z: torch.Tensor, bias: Optional[torch.Tensor], slot_of_token: torc
         raise KernelError("moe_route: weights must be contiguous float32 [T, top]")
     if counts.dtype != torch.int32 or counts.numel() != E or (bias is not None and bias.numel() != E):
         raise KernelError("moe_route: counts (int32) and bias must be [E]")
+    if score not in ROUTER_SCORES:
+        raise KernelError(f"moe_route: score {score!r} is not built (known: {sorted(ROUTER_SCORES)})")
+    if identity and (self_weight is None or self_weight.dtype != torch.float32 or self_weight.numel() < n_tokens or
+                     not self_weight.is_contiguous()):
+        raise KernelError("moe_route: identity experts need self_weight, contiguous float32 [T]")
     rc = _lib().rb_moe_route(_ptr(z), z.stride(0), _ptr(bias), dtype_code(bias.dtype) if bias is not None else F32,
                              _i32(slot_of_token, "slot_of_token"), n_tokens, E, top, _ptr(ids), _ptr(weights),
                              _ptr(place), _ptr(counts), int(n_groups), int(keep_groups), 1 if renormalize else 0,
-                             float(norm_eps), _stream())
+                             float(norm_eps), ROUTER_SCORES[score], int(identity), _ptr(self_weight), _stream())
     _check(rc, "moe_route")
 
 
@@ -1188,12 +1237,24 @@ def moe_gather(x: torch.Tensor, ids: torch.Tensor, place: torch.Tensor, starts: 
                                 top, _ptr(rows), _ptr(row_of), _stream()), "moe_gather")
 
 
+def _self_rows(self_weight, self_x, n_tokens: int, H: int, what: str):
+    """(weights, rows, the rows' type) of what identity experts give."""
+    if self_weight is None:
+        return None, None, F32
+    if self_weight.dtype != torch.float32 or self_weight.numel() < n_tokens or self_x is None or not self_x.is_contiguous() or \
+            self_x.shape[-1] != H or self_x.shape[0] < n_tokens:
+        raise KernelError(f"{what}: self_weight must be float32 [T], self_x contiguous [T, H]")
+    return _ptr(self_weight), _ptr(self_x), dtype_code(self_x.dtype)
+
+
 @_profiled(lambda a, facts: (a["n_tokens"] * a["out"].shape[1] * 4 * (1 + a["top"]), a["n_tokens"] * a["out"].shape[1] * 2 * a["top"]))
 def moe_combine(y: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, n_tokens: int, top: int, out: torch.Tensor,
-                extra: Optional[torch.Tensor] = None, extra_gate: Optional[torch.Tensor] = None):
+                extra: Optional[torch.Tensor] = None, extra_gate: Optional[torch.Tensor] = None,
+                self_weight: Optional[torch.Tensor] = None, self_x: Optional[torch.Tensor] = None):
     """out [T, H] float32 = sum over a token's choices j of weights[t, j] * y[row_of[t, j]] (y float32 [R, H]), plus,
     with ``extra`` (float32 [S, T, H] partial sums), sigmoid(extra_gate[t]) * sum_s extra[s, t] (``extra_gate``: a
-    float32 column, one logit a token, any row stride; None: no gate)."""
+    float32 column, one logit a token, any row stride; None: no gate), plus, with ``self_weight`` (float32 [T]),
+    self_weight[t] * self_x[t] (``self_x`` [T, H] bfloat16 or float32)."""
     if y.dtype != torch.float32 or out.dtype != torch.float32 or y.stride(1) != 1 or not out.is_contiguous() or \
             y.shape[1] != out.shape[1]:
         raise KernelError("moe_combine: y and out must be float32 of one width")
@@ -1209,7 +1270,8 @@ def moe_combine(y: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, n_
             gate_ld = extra_gate.stride(0)
     _check(_lib().rb_moe_combine(_ptr(y), y.stride(0), _ptr(row_of), _ptr(weights), n_tokens, top, _ptr(out),
                                  out.shape[1], _ptr(extra), n_extra, stride,
-                                 _ptr(extra_gate) if extra is not None else None, gate_ld, _stream()), "moe_combine")
+                                 _ptr(extra_gate) if extra is not None else None, gate_ld, *_self_rows(self_weight, self_x, n_tokens,
+                                 out.shape[1], "moe_combine"), _stream()), "moe_combine")
 
 
 # ---- linear attention with a fixed decay per head ------------------------------------------------------------------
@@ -1667,3 +1729,153 @@ def talk_mix(o: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, nq: int, nkv
     rc = _lib().rb_talk_mix(_ptr(o), o.stride(0), _f32vec(mix, nq * nq, "talk_mix: mix"), _ptr(out), out.stride(0), nq, nkv, hdp, vd,
                             dtype_code(o.dtype), _i32(slot_of_token, "slot_of_token"), n_tokens, _stream())
     _check(rc, "talk_mix")
+
+
+# ---- layer norms, and norms of a sublayer's result ----------------------------------------------------------------------------
+
+@_profiled(lambda a, facts: _cost.add_norm(
+    a["n_rows"] if a["n_rows"] is not None else (a["rows"].numel() if a["rows"] is not None else a["resid"].shape[0]),
+    a["resid"].shape[1], _n_partials(a["delta"]), _esz(a["out"]), bool(a["write_back"]) and a["delta"] is not None, 8))
+def add_layernorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                  out: torch.Tensor, rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, write_back: bool = True):
+    """``add_rmsnorm`` with a layer norm: out[i] = (r - mean) / sqrt(variance + eps) * weight + bias with r = resid[row] (+ the
+    sum of delta [S, >= T, H] float32, written back if ``write_back``); weight and bias float32 [H]."""
+    T, H = resid.shape
+    if resid.dtype != torch.float32 or not resid.is_contiguous() or not out.is_contiguous():
+        raise KernelError("add_layernorm: resid must be contiguous float32, out contiguous")
+    n_delta, stride = 0, 0
+    if delta is not None:
+        if delta.dtype != torch.float32 or not delta.is_contiguous() or delta.dim() != 3 or delta.shape[1] < T or delta.shape[2] != H:
+            raise KernelError("add_layernorm: delta must be contiguous float32 [S, >= T, H]")
+        n_delta, stride = delta.shape[0], delta.stride(0)
+    n = (rows.numel() if rows is not None else T) if n_rows is None else n_rows
+    if out.shape[-1] != H or out.numel() < n * H:
+        raise KernelError("add_layernorm: shapes do not fit")
+    rc = _lib().rb_add_layernorm(_ptr(resid), _ptr(delta), n_delta, stride, _f32vec(weight, H, "add_layernorm: weight"),
+                                 _f32vec(bias, H, "add_layernorm: bias"), _ptr(out), dtype_code(out.dtype),
+                                 None if rows is None else _i32(rows, "rows"), n, H, float(eps), 1 if write_back else 0, _stream())
+    _check(rc, "add_layernorm")
+
+
+@_profiled(lambda a, facts: _cost.add_norm(a["n_rows"] or a["resid"].shape[0], a["resid"].shape[1],
+                                           a["top"] if a["row_of"] is not None else a["delta"].shape[0],
+                                           _esz(a["out"]) if a["out"] is not None else 0, True, 8))
+def out_norm(resid: torch.Tensor, delta: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, mult: float,
+             layer: bool, out: Optional[torch.Tensor] = None, scale: float = 1.0, row_of: Optional[torch.Tensor] = None,
+             weights: Optional[torch.Tensor] = None, top: int = 0, self_weight: Optional[torch.Tensor] = None,
+             self_x: Optional[torch.Tensor] = None, n_rows: Optional[int] = None):
+    """resid [T, H] float32 += mult * norm(d) in place; ``out`` [T, H] also receives the new rows in its own type.  norm: a layer
+    norm (``layer``) or an RMS norm, weight (and bias) float32 [H].  d = ``scale`` * (the sum of ``delta`` [S, >= T, H] float32), or,
+    with ``row_of`` (int32 [T, top], -1: none) and ``weights`` (float32 [T, top]), scale * (row t's weighted sum of the rows of
+    ``delta`` [R, H] it names plus ``self_weight``[t] * ``self_x``[t])."""
+    T, H = resid.shape
+    n = T if n_rows is None else n_rows
+    if resid.dtype != torch.float32 or not resid.is_contiguous():
+        raise KernelError("out_norm: resid must be contiguous float32")
+    if row_of is not None:
+        if delta.dtype != torch.float32 or delta.dim() != 2 or delta.shape[1] != H or delta.stride(1) != 1 or weights is None or \
+                weights.dtype != torch.float32 or top < 1 or row_of.numel() < n * top or weights.numel() < n * top or \
+                not weights.is_contiguous():
+            raise KernelError("out_norm: rows to sum must be float32 [R, H] with int32 places and float32 weights [T, top]")
+        n_delta, stride = 1, delta.stride(0)
+    else:
+        if delta.dtype != torch.float32 or delta.dim() != 3 or delta.shape[1] < n or delta.shape[2] != H or \
+                delta.stride(2) != 1 or delta.stride(1) != H:
+            raise KernelError("out_norm: delta must be float32 [S, >= T, H] with dense rows")
+        n_delta, stride = delta.shape[0], delta.stride(0)
+    if out is not None and (not out.is_contiguous() or out.shape[-1] != H or out.numel() < n * H):
+        raise KernelError("out_norm: out must be contiguous [T, H]")
+    rc = _lib().rb_out_norm(_ptr(resid), _ptr(delta), n_delta, stride, float(scale), None if row_of is None else _i32(row_of, "row_of"),
+                            _ptr(weights), int(top), *_self_rows(self_weight, self_x, n, H, "out_norm"), 1 if layer else 0,
+                            _f32vec(weight, H, "out_norm: weight"), _f32vec(bias, H, "out_norm: bias"), float(eps), float(mult),
+                            _ptr(out), dtype_code(out.dtype) if out is not None else F32, n, H, _stream())
+    _check(rc, "out_norm")
+
+
+# ---- the gated delta rule -------------------------------------------------------------------------------------------------------
+
+DELTA_MAX_TAPS = 32       # PREP_MAX_TAPS of csrc/gated_delta.cu
+DELTA_MAX_DIM = 512       # rows of a head's state that fit the registers of delta_scan
+LOW_RANK_MAX = 1536       # inner values of low_rank
+
+
+class DeltaRows:
+    """Where a token's inputs of the recurrence sit in its row: q | k | v | decays | step sizes | q . k, every part on four
+    numbers."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool):
+        at, offs = 0, []
+        for n in (kv_heads * dim, kv_heads * dim, heads * vdim, heads * dim if per_channel else heads, heads, kv_heads):
+            offs.append(at)
+            at += -(-n // 4) * 4
+        self.offsets, self.width = tuple(offs), at
+
+
+@_profiled(lambda a, facts: (a["n_tokens"] * ((2 * a["kv_heads"] * a["dim"] + a["heads"] * a["vdim"]) * (4 + _esz(a["proj"]) * _n_in(a["proj"]))
+                                              + (a["heads"] * a["dim"] * (4 + _esz(a["z"])) if a["per_channel"] else a["heads"] * 8)),
+                             a["n_tokens"] * (2 * a["kv_heads"] * a["dim"] + a["heads"] * a["vdim"]) * (2 * a["taps"] + 6)))
+def delta_prep(proj: torch.Tensor, n_tokens: int, q_off: int, k_off: int, v_off: int, b_off: int, heads: int, kv_heads: int, dim: int,
+               vdim: int, taps: int, conv_w: torch.Tensor, kept: Optional[torch.Tensor], z: torch.Tensor, dt_bias: torch.Tensor,
+               a_log: torch.Tensor, per_channel: bool, unit_eps: float, q_scale: float, seq_slot: torch.Tensor, cu_q: torch.Tensor,
+               n_seqs: int, max_q_len: int, u: torch.Tensor, rows: DeltaRows):
+    """Everything between a layer's projections and the recurrence S <- g S; w = beta (v - S^T k); S <- S + k w^T, written to the
+    rows ``u`` float32 [T, rows.width] at ``rows.offsets``: q, k and v through a causal convolution over ``taps`` tokens and silu
+    (``conv_w`` float32 [taps, q | k | v channels], ``kept`` float32 [slots, taps - 1, channels]: the inputs before the step's first
+    token, replaced by the step's last), q and k divided by sqrt(sum of squares + unit_eps), q times ``q_scale``, their dot product
+    per key head, beta = sigmoid(column b_off + h), g = exp(-exp(a_log[h]) softplus(z + dt_bias)) with ``z`` [T, heads] or, when
+    ``per_channel``, [T, heads * dim] (a view of the projection rows or rows of its own, partial sums added first)."""
+    n_in, in_stride, row_stride = _partials(proj, "delta_prep")
+    z_n, z_stride, z_row = _partials(z, "delta_prep: z")
+    channels = 2 * kv_heads * dim + heads * vdim
+    n_z = heads * dim if per_channel else heads
+    if taps < 1 or taps > DELTA_MAX_TAPS or max(q_off, k_off) + kv_heads * dim > proj.shape[-1] or \
+            v_off + heads * vdim > proj.shape[-1] or b_off + heads > proj.shape[-1] or z.shape[-1] < n_z:
+        raise KernelError(f"delta_prep: 1 to {DELTA_MAX_TAPS} taps, and all columns inside the rows")
+    if taps > 1 and (kept is None or kept.dtype != torch.float32 or not kept.is_contiguous() or tuple(kept.shape[1:]) != (taps - 1, channels)):
+        raise KernelError("delta_prep: kept must be contiguous float32 [slots, taps - 1, channels]")
+    if u.dtype != torch.float32 or u.stride(-1) != 1 or u.shape[-1] < rows.width or u.shape[0] < n_tokens:
+        raise KernelError("delta_prep: u must be float32 [T, rows.width]")
+    rc = _lib().rb_delta_prep(_ptr(proj), dtype_code(proj.dtype), n_in, in_stride, row_stride, q_off, k_off, v_off, b_off, heads,
+                              kv_heads, dim, vdim, taps, _f32vec(conv_w, taps * channels, "delta_prep: conv_w"), _ptr(kept), _ptr(z),
+                              dtype_code(z.dtype), z_n, z_stride, z_row, _f32vec(dt_bias, n_z, "delta_prep: dt_bias"),
+                              _f32vec(a_log, heads, "delta_prep: a_log"), 1 if per_channel else 0, float(unit_eps), float(q_scale),
+                              _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, max_q_len, _ptr(u), u.stride(0), *rows.offsets,
+                              _stream())
+    _check(rc, "delta_prep")
+
+
+@_profiled(lambda a, facts: _cost.delta_scan(a["n_tokens"], a["n_seqs"], a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["per_channel"]))
+def delta_scan(u: torch.Tensor, n_tokens: int, rows: DeltaRows, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool,
+               state: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, n_seqs: int, out: torch.Tensor):
+    """The step's tokens through S <- g S; w = beta (v - S^T k); S <- S + k w^T; o = S^T q for every (sequence, head), from the rows
+    ``delta_prep`` made.  ``state`` float32 [slots, heads, vdim, dim] (a head's S transposed), read and written in place; ``out``
+    float32 [T, heads * vdim]."""
+    if u.dtype != torch.float32 or u.stride(-1) != 1 or u.shape[-1] < rows.width or u.shape[0] < n_tokens:
+        raise KernelError("delta_scan: u must be float32 [T, rows.width]")
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (heads, vdim, dim):
+        raise KernelError("delta_scan: state must be contiguous float32 [slots, heads, vdim, dim]")
+    if out.dtype != torch.float32 or out.stride(-1) != 1 or out.shape[-1] != heads * vdim or out.shape[0] < n_tokens:
+        raise KernelError("delta_scan: out must be float32 [T, heads * vdim]")
+    rc = _lib().rb_delta_scan(_ptr(u), u.stride(0), *rows.offsets, heads, kv_heads, dim, vdim, 1 if per_channel else 0, _ptr(state),
+                              _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, _ptr(out), out.stride(0), _stream())
+    _check(rc, "delta_scan")
+
+
+@_profiled(lambda a, facts: (a["w0"].numel() * _esz(a["w0"]) + (a["w1"].numel() * _esz(a["w1"]) if a["w1"] is not None else 0)
+                             + a["n_tokens"] * a["out"].shape[1] * 4,
+                             2 * a["n_tokens"] * (a["w0"].numel() + (a["w1"].numel() if a["w1"] is not None else 0))))
+def low_rank(proj: torch.Tensor, n_tokens: int, x_off0: int, w0: torch.Tensor, x_off1: int, w1: Optional[torch.Tensor],
+             out: torch.Tensor):
+    """out [T, n0 (+ n1)] float32 = [w0 x0 | w1 x1] for few tokens: x_i are the columns x_off_i .. + rank_i of the projection rows
+    (partial sums added first), w_i [n_i, rank_i] of one type; 32-bit FMA."""
+    n_in, in_stride, row_stride = _partials(proj, "low_rank")
+    n0, r0 = w0.shape
+    n1, r1 = w1.shape if w1 is not None else (0, 0)
+    if not w0.is_contiguous() or (w1 is not None and (not w1.is_contiguous() or w1.dtype != w0.dtype)) or max(r0, r1) > LOW_RANK_MAX or \
+            x_off0 + r0 > proj.shape[-1] or (w1 is not None and x_off1 + r1 > proj.shape[-1]):
+        raise KernelError("low_rank: contiguous weights of one type, and their inputs inside the projection rows")
+    if out.dtype != torch.float32 or out.stride(-1) != 1 or out.shape[-1] != n0 + n1 or out.shape[0] < n_tokens:
+        raise KernelError("low_rank: out must be float32 [T, n0 + n1]")
+    rc = _lib().rb_low_rank(_ptr(proj), dtype_code(proj.dtype), n_in, in_stride, row_stride, x_off0, r0, _ptr(w0), n0, x_off1, r1,
+                            _ptr(w1), n1, dtype_code(w0.dtype), n_tokens, _ptr(out), out.stride(0), _stream())
+    _check(rc, "low_rank")

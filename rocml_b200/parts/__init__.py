@@ -7,19 +7,22 @@ from .base import (
     register_mixer, register_norm, register_position, registered,
 )
 from .linear import Linear
-from .norm import RMSNorm
-from .position import NoPosition, RotaryNeox, RotaryPairs, SinusoidPosition
+from .norm import LayerNorm, RMSNorm
+from .position import LearnedPosition, NoPosition, RotaryNeox, RotaryPairs, SinusoidPosition
 from .attention import Attention
 from .mlp import GatedMLP
 from .latent_attention import LatentAttention
 from .routed_mlp import RoutedMLP
 from .linear_attention import LinearAttention
 from .state_space import StateSpace
-from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichNormBlock
+from .gated_delta import GatedDelta
+from .side_by_side import SideBySide
+from .block import OutputNormBlock, ParallelBlock, PostNormBlock, PreNormBlock, SandwichNormBlock
 
 __all__ = [
     "BuildEnv", "DeferredNorm", "ResidualSink", "FeedForward", "Mixer", "Norm", "Part", "PositionEncoding", "build_block",
     "build_feed_forward", "build_mixer", "build_norm", "build_position", "register_arrangement",
     "register_feed_forward", "register_mixer", "register_norm", "register_position", "registered",
-    "Linear", "RMSNorm", "NoPosition", "RotaryNeox", "Attention", "GatedMLP", "PreNormBlock", "LatentAttention", "RoutedMLP", "SandwichNormBlock", "SinusoidPosition", "RotaryPairs", "LinearAttention", "ParallelBlock", "StateSpace", "PostNormBlock",
+    "Linear", "RMSNorm", "NoPosition", "RotaryNeox", "Attention", "GatedMLP", "PreNormBlock", "LatentAttention", "RoutedMLP", "SandwichNormBlock", "SinusoidPosition", "RotaryPairs", "LinearAttention", "ParallelBlock", "StateSpace", "PostNormBlock", "LayerNorm",
+    "LearnedPosition", "GatedDelta", "SideBySide", "OutputNormBlock",
 ]

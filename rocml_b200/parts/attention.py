@@ -13,7 +13,9 @@ instead of a window (``chunk``), a sigmoid gate per head on the attention's resu
 layer's input (``gated``; "per_value": a gate for every value of every head), and, through the
 position encoding, rotation by neighbouring pairs.  Beside a window, the first ``keep_first`` positions
 may stay visible to every later query; the softmax's denominator may have one more term exp(``sink``)
-that brings no value; queries and keys may be divided by their root mean square after the position
+that brings no value (one number, or "per_head": a tensor with a number for every query head); queries may be multiplied by a
+temperature that grows with their position (``q_temperature`` {coef, every}: 1 + coef ln(floor((p + 1) / every) + 1), after
+norm and position encoding); queries and keys may be divided by their root mean square after the position
 encoding (``qk_unit_norm``); biases may be given for some of the projections only; and the values that
 a layer caches may be blended with those of an earlier layer of the same step (``value_mix``).
 Three more parameters form one path of their own (``_forward_wide``): ``qk_norm`` "whole" (queries and keys are each
@@ -50,7 +52,8 @@ PROMPT_FUSED_MIN_TOKENS = 4096
 # Tensor-name stems by role, unless the spec's ``names`` says otherwise (the defaults are those of
 # Hugging Face's Qwen3 checkpoints: rocml/src/weights/layer.rs:47-58 lists the same tensors under GGUF names).
 TENSOR_NAMES = {"q": "q_proj", "k": "k_proj", "v": "v_proj", "o": "o_proj", "q_norm": "q_norm", "k_norm": "k_norm",
-                "gate": "gate_proj", "value_mix": "value_mix", "talk": "head_mix", "temperature": "head_temperature"}
+                "gate": "gate_proj", "value_mix": "value_mix", "talk": "head_mix", "temperature": "head_temperature",
+                "sink": "sink"}
 
 VALUE_MIX_SOURCE = "attention.value_mix_source"    # where a step keeps the source layer's values (StepBatch.scratch)
 
@@ -88,7 +91,12 @@ class Attention(Mixer):
         self.window = p.get("window")
         self.chunk = p.get("chunk")
         self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
-        self.sink = None if p.get("sink") is None else float(p["sink"])
+        self.sink_per_head = p.get("sink") == "per_head"
+        self.sink = None if p.get("sink") is None or self.sink_per_head else float(p["sink"])    # per head: a tensor, once loaded
+        temp = dict(p.get("q_temperature") or ())
+        self.q_temp = (float(temp["coef"]), float(temp["every"])) if temp else None
+        if self.q_temp is not None and not self.q_temp[1] > 0:
+            raise ConfigError(f"attention: q_temperature.every must be positive, found {self.q_temp[1]}")
         self.value_mix = p.get("value_mix")
         if self.value_mix not in (None, "source", "mix"):
             raise ConfigError(f"attention: value_mix is 'source' or 'mix', found {self.value_mix!r}")
@@ -96,10 +104,10 @@ class Attention(Mixer):
             raise ConfigError("attention: keep_first counts positions and cannot be negative")
         if self.window and self.chunk:
             raise ConfigError("attention: a layer has a window or blocks of positions, not both")
-        if self.wide and (self.gated or self.keep_first or self.sink is not None or self.qk_unit_norm or self.value_mix or
+        if self.wide and (self.gated or self.keep_first or p.get("sink") is not None or self.q_temp or self.qk_unit_norm or self.value_mix or
                           (self.qk_norm and not self.qk_norm_whole) or p.get("shares_cache")):
             raise ConfigError("attention: a norm over whole projections, head temperatures and mixed heads do not combine with "
-                              "gates, kept first keys, a sink, unit norms, blended values, per-head norms or a shared cache")
+                              "gates, kept first keys, a sink, query temperatures, unit norms, blended values, per-head norms or a shared cache")
         if self.talking_heads and self.nkv * self.nq * self.hdp > 65535 * 16:
             raise ConfigError("attention: too many heads to mix")
         if (self.window is not None and int(self.window) < 1) or (self.chunk is not None and int(self.chunk) < 1):
@@ -110,7 +118,7 @@ class Attention(Mixer):
         # the plain layout: equal head sizes that the kernels take as they are, rotate-half pairs, no gate
         self.plain = not self.wide and self.vd == self.hd == self.hdp and not self.gated and \
             not (self.position.inv_freq is not None and getattr(self.position, "interleaved", False)) and \
-            not (self.keep_first or self.sink is not None or self.qk_unit_norm or self.value_mix)
+            not (self.keep_first or self.sink is not None or self.sink_per_head or self.q_temp or self.qk_unit_norm or self.value_mix)
         if not self.plain and self.shares_cache:
             raise ConfigError("attention: a layer that reads another layer's cache must have the plain layout")
         qd, kvd = self.nq * self.hd, self.nkv * self.hd
@@ -133,6 +141,8 @@ class Attention(Mixer):
                 stems, outs = stems + [n["gate"]], outs + [self.nq * self.vd if self.gate_per_value else self.nq]
             self.qkv = Linear(stems, outs, hidden, in_bias, env)
         self.o = Linear([n["o"]], [hidden], self.nq * self.vd, o_bias, env)
+        # for an arrangement of mixers that share their input and output products (side_by_side)
+        self.in_stems, self.in_outs, self.out_width = list(self.qkv.names), list(self.qkv.outs), self.nq * self.vd
         self.q_norm_w: Optional[torch.Tensor] = None
         self.k_norm_w: Optional[torch.Tensor] = None
         self.v_lambda: Optional[torch.Tensor] = None     # float32 [1] on the device: the share of the source layer's values
@@ -149,7 +159,11 @@ class Attention(Mixer):
         return -int(self.chunk) if self.chunk else 0
 
     def declare(self, prefix: str) -> List[TensorDecl]:
-        out = self.qkv.declare(prefix) + self.o.declare(prefix)
+        return self.qkv.declare(prefix) + self.o.declare(prefix) + self.declare_inner(prefix)
+
+    def declare_inner(self, prefix: str) -> List[TensorDecl]:
+        """The tensors beside the input and the output product."""
+        out = []
         if self.qk_norm_whole:
             out.append(TensorDecl(f"{prefix}{self.names['q_norm']}.weight", (self.nq * self.hd,), "norm"))
             out.append(TensorDecl(f"{prefix}{self.names['k_norm']}.weight", (self.nkv * self.hd,), "norm"))
@@ -163,6 +177,8 @@ class Attention(Mixer):
             out.append(TensorDecl(f"{prefix}{self.names['temperature']}.weight", (self.nq,), "norm"))
         if self.value_mix == "mix":
             out.append(TensorDecl(f"{prefix}{self.names['value_mix']}.weight", (), "fraction"))
+        if self.sink_per_head:
+            out.append(TensorDecl(f"{prefix}{self.names['sink']}.weight", (self.nq,), "bias"))
         return out
 
     def ignorable(self, prefix: str) -> List[str]:
@@ -174,6 +190,11 @@ class Attention(Mixer):
         if not self.plain:
             self.qkv.pad_rows(8)     # a stack with a few gate rows is rarely a multiple of 8 wide
         self.o.load(tensors, prefix)
+        self.load_inner(tensors, prefix)
+
+    def load_inner(self, tensors: Dict[str, torch.Tensor], prefix: str) -> None:
+        if self.sink_per_head:
+            self.sink = tensors[f"{prefix}{self.names['sink']}.weight"].float().contiguous()
         if self.talking_heads:
             self.talk = tensors[f"{prefix}{self.names['talk']}.weight"].float().contiguous()
         if self.head_temperature:
@@ -199,12 +220,22 @@ class Attention(Mixer):
         return n_tokens * (self.qkv.n * max(esz, 4 * parts if parts > 1 else esz) + 3 * self.nq * self.hdp * esz
                            + self.hidden * 4 * parts + self.nq * 4 * (self.hdp + 2) * (parts if parts > 1 else 0))
 
-    def cost(self, q_lens, kv_lens):
-        from ..profile import cost as C
-        T = sum(q_lens)
+    def inner_bytes(self) -> int:
+        return 0
+
+    def inner_workspace(self, n_tokens: int) -> int:
         esz = 4 if self.env.mode == "float32" else 2
-        parts = [self.qkv.cost(T), self.o.cost(T),
-                 C.attention(q_lens, kv_lens, self.nq, self.nkv, self.hdp, esz, self._span() or None)]
+        parts = 8 if n_tokens <= 128 else 0
+        return n_tokens * (2 * self.nq * self.hdp * esz + self.nq * 4 * (self.hdp + 2) * parts)
+
+    def inner_cost(self, q_lens, kv_lens):
+        from ..profile import cost as C
+        esz = 4 if self.env.mode == "float32" else 2
+        return C.attention(q_lens, kv_lens, self.nq, self.nkv, self.hdp, esz, self._span() or None)
+
+    def cost(self, q_lens, kv_lens):
+        T = sum(q_lens)
+        parts = [self.qkv.cost(T), self.o.cost(T), self.inner_cost(q_lens, kv_lens)]
         return sum(p[0] for p in parts), sum(p[1] for p in parts)
 
     can_sink = True        # forward() accepts sink=ResidualSink (see parts.base)
@@ -263,11 +294,21 @@ class Attention(Mixer):
         queries and keys, writes keys and values (padded) to their pages and takes the sigmoid of the gate
         columns; the attention runs at the padded head size; one kernel multiplies each head by its gate and
         drops the padding."""
-        T = batch.n_tokens
-        dev, act = self.env.device, self.env.act_dtype
         if isinstance(xn, DeferredNorm):
             xn = xn.materialize()
-        proj = self.qkv.forward_auto(xn, T)
+        proj = self.qkv.forward_auto(xn, batch.n_tokens)
+        return self._project_out(self._padded_rows(proj, batch, view, window, writes), batch.n_tokens, sink, add_into)
+
+    def mix_rows(self, proj, batch, view, out=None):
+        """The rows that the output product reads, from the layer's projection rows ([T, sum(in_outs)], or float32 partial sums
+        [S, T, ..]).  ``out`` [T, out_width] (any row stride) receives them if given."""
+        if self.wide:
+            raise ConfigError("attention: a norm over whole projections and mixed heads do not stand beside another mixer")
+        return self._padded_rows(proj, batch, view, self._span(), view.writes and not self.shares_cache, out)
+
+    def _padded_rows(self, proj, batch, view, window, writes, rows=None):
+        T = batch.n_tokens
+        dev, act = self.env.device, self.env.act_dtype
         # values blended across layers: the source layer leaves its own for the step's later layers
         v_out = v_first = None
         if self.value_mix == "source":
@@ -286,9 +327,9 @@ class Attention(Mixer):
         # one token a sequence, heads of 128 on both sides: the attention kernel makes the heads from the projection's
         # partial sums itself (norm, partial rotation, division by the root mean square, blended values, the cache write)
         if batch.is_decode and writes and self.hd == self.vd == self.hdp and (raw_gate is not None or not self.gated):
-            attn = torch.empty((T, self.nq * self.hd), dtype=act, device=dev)
+            attn = rows if rows is not None else torch.empty((T, self.nq * self.hd), dtype=act, device=dev)
             if self._decode_fused(proj, attn, batch, view, window, writes, v_first=v_first, v_keep=v_out, gate=raw_gate):
-                return self._project_out(attn, T, sink, add_into)
+                return attn
         q = torch.empty((T, self.nq * self.hdp), dtype=act, device=dev)
         gates = torch.empty((T, self.nq), dtype=torch.float32, device=dev) if self.gated and not self.gate_per_value else None
         with scope(op="rotate_cache"):
@@ -298,12 +339,13 @@ class Attention(Mixer):
                 view.block_table, view.k, view.v, write_kv=writes, cos_sin=self.position.cos_sin(batch),
                 v_head_dim=self.vd, padded_head_dim=self.hdp, interleaved=getattr(self.position, "interleaved", False),
                 gates=gates, post_norm=self.qk_unit_norm, v_first=v_first, v_lambda=self.v_lambda if v_first is not None else None,
-                v_out=v_out)
-        attn = torch.empty((T, self.nq * self.hdp), dtype=act, device=dev)
+                v_out=v_out, q_temp=self.q_temp)
+        last = (self.gated and raw_gate is None) or self.hdp != self.vd         # a kernel that gates or narrows follows for sure
+        attn = rows if rows is not None and not last else torch.empty((T, self.nq * self.hdp), dtype=act, device=dev)
         gated_inside = paged_attention(q, attn, batch, view.k, view.v, view.block_table, self.nq, self.nkv, self.hdp, self.scale,
                                        window, keep=self.keep_first, sink=self.sink, gate=raw_gate)
         if (self.gated and not gated_inside) or self.hdp != self.vd:
-            narrow = torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
+            narrow = rows if rows is not None else torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
             raw = None
             if self.gate_per_value:          # the gate's columns of the projection rows, as they are: the kernel takes the sigmoid
                 off = self.nq * self.hd + self.nkv * (self.hd + self.vd)
@@ -311,7 +353,7 @@ class Attention(Mixer):
             with scope(op="head_gate"):
                 kernels.head_gate(attn, narrow, gates, self.nq, self.hdp, self.vd, T, raw=raw, per_value=self.gate_per_value)
             attn = narrow
-        return self._project_out(attn, T, sink, add_into)
+        return attn
 
     def _forward_wide(self, xn, batch, view, window, sink, add_into):
         """A norm over the whole q and k projections, a temperature per head, the heads' weights mixed after the softmax.
@@ -391,6 +433,8 @@ class Attention(Mixer):
         rot = self.position.rot_dim if self.position.inv_freq is not None else 0
         if rot % 8 or getattr(self.position, "interleaved", False) or (writes and self.nq // self.nkv > 16):
             return False
+        if gate is None:            # the heads alone (the rows may be part of wider ones)
+            proj = proj[..., :(self.nq + (2 * self.nkv if writes else 0)) * self.hd]
         n_pages = max(1, (batch.max_kv_len + DECODE_CHUNK - 1) // DECODE_CHUNK)
         groups = self.nkv * ((self.nq // self.nkv + 15) // 16)
         n_blocks, ppb = kernels.decode_split(batch.n_seqs, groups, n_pages, out.device)
@@ -409,7 +453,7 @@ class Attention(Mixer):
             self.position.cos_sin(batch) if rot else None, writes, self.scale, window, n_blocks, acc, ml, ppb,
             rowscale=rowscale, row_width=row_width, keep=self.keep_first, sink=self.sink, rot_dim=rot,
             post_norm=self.qk_unit_norm, v_first=v_first, v_lambda=self.v_lambda if v_first is not None else None,
-            v_keep=v_keep, gate=gate)
+            v_keep=v_keep, gate=gate, q_temp=self.q_temp)
 
     def attend(self, q, out, batch, view, window):
         """Softmax attention of the step's queries over the cache (see ``paged_attention``)."""

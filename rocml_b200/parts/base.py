@@ -83,11 +83,14 @@ class RoutedRows:
     weights: torch.Tensor     # [T, top] float32
     top: int
     n_tokens: int
+    self_weight: Optional[torch.Tensor] = None     # [T] float32: what the identity experts multiply the token's input by
+    self_x: Optional[torch.Tensor] = None          # [T, H]: that input
 
     def materialize(self) -> torch.Tensor:
         from .. import kernels
         out = torch.empty((1, self.n_tokens, self.rows.shape[1]), dtype=torch.float32, device=self.rows.device)
-        kernels.moe_combine(self.rows, self.row_of, self.weights, self.n_tokens, self.top, out[0])
+        kernels.moe_combine(self.rows, self.row_of, self.weights, self.n_tokens, self.top, out[0], self_weight=self.self_weight,
+                            self_x=self.self_x)
         return out
 
 
@@ -95,6 +98,23 @@ class NormedRows(DeferredNorm):
     """What a block leaves for the block after it when it has already run that block's first norm: ``x`` are
     the finished rows of ``norm`` (nothing is deferred; the residual holds every delta).  Only a block that
     knows this type is handed one; any other norm treats it as 'nothing pending'."""
+
+    def materialize(self) -> torch.Tensor:
+        return self.x
+
+
+@dataclass
+class ScaledDelta:
+    """A mixer's result times a constant that the consumer applies: handed, instead of a delta, to an arrangement that
+    asked for it (``forward(..., scale_later=True)`` of a mixer with ``scales_later``)."""
+
+    delta: torch.Tensor       # [S, T, H] float32
+    factor: float
+
+
+class StreamRows(DeferredNorm):
+    """What a block leaves for a block after it whose sublayers read the stream itself: ``x`` are the stream's rows in the
+    activations' type (the residual holds every delta; ``norm`` is None).  To any norm it means 'nothing pending'."""
 
     def materialize(self) -> torch.Tensor:
         return self.x

@@ -9,8 +9,8 @@ import torch
 from ..config.specs import LayerSpec
 from ..profile import scope
 from ..weights.decl import TensorDecl
-from .base import (BuildEnv, DeferredNorm, NormedRows, ResidualSink, RoutedRows, ShiftedRows, build_feed_forward, build_mixer,
-                   build_norm, register_arrangement)
+from .base import (BuildEnv, DeferredNorm, NormedRows, ResidualSink, RoutedRows, ScaledDelta, ShiftedRows, StreamRows,
+                   build_feed_forward, build_mixer, build_norm, register_arrangement)
 
 
 # From this many tokens in a step a part is offered to add into the residual itself (the products of
@@ -522,6 +522,138 @@ class PostNormBlock:
                 kernels.postln(resid, delta, self.ff_gain, self._w2, self.alpha, self.ff_norm.eps, None, batch.slot_of_token, T,
                                next_mu=n_mu, next_kept=n_kept, next_out=n_out)
         return ShiftedRows(n_out, next_block) if n_out is not None else None
+
+
+@register_arrangement("output_norm")
+class OutputNormBlock:
+    """x += m * norm1(mixer(x)); x += m * norm2(ff(x)): a norm on each sublayer's result only, the sublayers read the stream
+    itself, m is a constant (parameter ``multiplier``, default 1).
+
+    One kernel does a sublayer's sum, norm and addition (``kernels.out_norm``): the result's partial sums in their order (or a routed
+    feed-forward's weighted sum over a token's experts, with what its identity experts give), a constant on the result, the
+    norm, the multiplier and the addition in 32-bit, the stream in place, and the new row in the activations' type for the
+    product that reads it next, in this block or (``StreamRows``) the one after it.  Nothing is left pending.  A layer without a
+    feed-forward has only the first half."""
+
+    chains = True              # forward() accepts next_block
+
+    def __init__(self, spec: LayerSpec, hidden: int, env: BuildEnv, mixer_spec=None):
+        from ..errors import ConfigError
+        p = spec.arrangement_params
+        unknown = sorted(set(p) - {"multiplier"})
+        if unknown:
+            raise ConfigError(f"output_norm: unknown parameters {unknown}")
+        self.spec = spec
+        self.prefix = spec.prefix
+        self.env = env
+        self.hidden = hidden
+        self.mult = float(p.get("multiplier", 1.0))
+        self.norm1 = build_norm(spec.mixer_norm, hidden, env)
+        self.mixer = build_mixer(mixer_spec or spec.mixer, hidden, env)
+        self.ff = self.norm2 = None
+        if spec.feed_forward is not None:
+            self.norm2 = build_norm(spec.ff_norm, hidden, env)
+            self.ff = build_feed_forward(spec.feed_forward, hidden, env)
+        for s in (spec.mixer_norm, spec.ff_norm):
+            if s.kind not in ("rmsnorm", "layernorm"):
+                raise ConfigError("output_norm is built for RMS norms and layer norms")
+        self._weights = {}
+
+    def _parts(self):
+        p, s = self.prefix, self.spec
+        out = [(self.norm1, f"{p}.{s.mixer_norm_name}"), (self.mixer, f"{p}.{s.mixer_name}")]
+        if self.ff is not None:
+            out += [(self.norm2, f"{p}.{s.ff_norm_name}"), (self.ff, f"{p}.{s.ff_name}")]
+        return out
+
+    def declare(self) -> List[TensorDecl]:
+        return [d for part, name in self._parts() for d in part.declare(name)]
+
+    def ignorable(self) -> List[str]:
+        out = [n for part, name in self._parts() for n in getattr(part, "ignorable", lambda prefix: [])(name)]
+        if self.ff is None:        # a layer without a feed-forward may still carry the second half's norm
+            out += [f"{self.prefix}.{self.spec.ff_norm_name}.{what}" for what in ("weight", "bias")]
+        return out
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        for part, name in self._parts():
+            part.load(tensors, name)
+        for n in (self.norm1, self.norm2):
+            if n is not None:
+                bias = getattr(n, "bias", None)
+                self._weights[n] = (n.weight.float().contiguous(), None if bias is None else bias.float().contiguous())
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(part.graph_safe for part, _ in self._parts())
+
+    def weight_bytes(self) -> int:
+        return sum(part.weight_bytes() for part, _ in self._parts())
+
+    def workspace_bytes(self, n_tokens: int) -> int:
+        rows = n_tokens * self.hidden * (4 if self.env.mode == "float32" else 2)
+        return 2 * rows + max(self.mixer.workspace_bytes(n_tokens), self.ff.workspace_bytes(n_tokens) if self.ff is not None else 0)
+
+    def cost(self, q_lens, kv_lens):
+        parts = [part.cost(q_lens, kv_lens) for part, _ in self._parts()]
+        return sum(p[0] for p in parts), sum(p[1] for p in parts)
+
+    def _join(self, resid, delta, norm, out, T):
+        """resid += m * norm(delta); ``out`` receives the new rows."""
+        from .. import kernels
+        w, b = self._weights[norm]
+        layer = b is not None or norm_is_layer(norm)
+        if isinstance(delta, RoutedRows):
+            # identity experts give the token's input, which is the stream's row itself
+            kernels.out_norm(resid, delta.rows, w, b, norm.eps, self.mult, layer, out, row_of=delta.row_of, weights=delta.weights,
+                             top=delta.top, self_weight=delta.self_weight, self_x=resid if delta.self_weight is not None else None, n_rows=T)
+            return
+        factor = 1.0
+        if isinstance(delta, ScaledDelta):
+            delta, factor = delta.delta, delta.factor
+        kernels.out_norm(resid, _as_partial_sums(delta, T), w, b, norm.eps, self.mult, layer, out, scale=factor, n_rows=T)
+
+    def forward(self, resid, pending, batch, view, next_block=None):
+        from .. import kernels
+        T = batch.n_tokens
+        act = self.env.act_dtype
+        same = act == torch.float32                    # in 32-bit mode the products read the stream as it is
+        if isinstance(pending, StreamRows):
+            x = pending.x
+        else:
+            if pending is not None and not isinstance(pending, DeferredNorm):
+                for d in (pending if isinstance(pending, (tuple, list)) else (pending,)):
+                    if d is not None:
+                        kernels.residual_inject(resid, _as_partial_sums(d, T))
+            x = resid
+            if not same:
+                x = torch.empty((T, self.hidden), dtype=act, device=resid.device)
+                with scope(op="stream_rows"):
+                    kernels.cast(resid[:T], x)
+        if getattr(self.mixer, "scales_later", False):
+            delta = self.mixer.forward(x, batch, view, scale_later=True)
+        else:
+            delta = self.mixer.forward(x, batch, view)
+        rows = resid if same else torch.empty((T, self.hidden), dtype=act, device=resid.device)
+        handed = isinstance(next_block, OutputNormBlock) and next_block.env.act_dtype == act
+        with scope(op="mixer_out_norm"):
+            self._join(resid, delta, self.norm1, None if same or (self.ff is None and not handed) else rows, T)
+        if self.ff is not None:
+            if getattr(self.ff, "sums_later", False):
+                delta = self.ff.forward(rows, batch, sum_later=True)
+            else:
+                delta = self.ff.forward(rows, batch)
+            if not same and handed:
+                rows = torch.empty((T, self.hidden), dtype=act, device=resid.device)
+            with scope(op="ff_out_norm"):
+                self._join(resid, delta, self.norm2, rows if handed and not same else None, T)
+        return StreamRows(rows, None, 0.0, self.hidden, None, resid) if handed else None
+
+
+def norm_is_layer(norm) -> bool:
+    """Whether a norm subtracts the mean."""
+    from .norm import LayerNorm
+    return isinstance(norm, LayerNorm)
 
 
 def _as_partial_sums(delta, n_rows: int):

@@ -1,4 +1,4 @@
-"""RMSNorm, fused with the residual addition that precedes it."""
+"""Norms over the last axis (RMS norm, layer norm), fused with the residual addition that precedes them."""
 from __future__ import annotations
 
 from typing import Dict, List, Optional
@@ -73,3 +73,44 @@ class RMSNorm(Norm):
         kernels.add_rmsnorm(resid, delta, self.weight, self.eps, out, n_rows=n, write_back=delta is not None,
                             weight2=other.weight, out2=out2)
         return out, out2
+
+
+@register_norm("layernorm")
+class LayerNorm(Norm):
+    """(x - mean) / sqrt(variance + eps) * w + b, the variance being the mean of the squared deviations; statistics,
+    weight and bias in 32-bit."""
+
+    graph_safe = True
+
+    def __init__(self, spec: NormSpec, size: int, env: BuildEnv):
+        self.eps = float(spec.eps)
+        self.size = size
+        self.env = env
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def declare(self, prefix: str) -> List[TensorDecl]:
+        return [TensorDecl(f"{prefix}.weight", (self.size,), "norm"), TensorDecl(f"{prefix}.bias", (self.size,), "bias")]
+
+    def load(self, tensors: Dict[str, torch.Tensor], prefix: str) -> None:
+        self.weight = tensors[f"{prefix}.weight"].float().contiguous()
+        self.bias = tensors[f"{prefix}.bias"].float().contiguous()
+
+    def weight_bytes(self) -> int:
+        return 8 * self.size
+
+    def workspace_bytes(self, n_tokens: int) -> int:
+        return n_tokens * self.size * (4 if self.env.mode == "float32" else 2)
+
+    def forward(self, resid, delta, n_rows: Optional[int] = None, rows=None, write_back=True):
+        if isinstance(delta, DeferredNorm):
+            delta = None                # the part before has added its result into the residual already
+        if isinstance(delta, (tuple, list)):
+            for d in delta[:-1]:        # a pair of results: all but the last join in a kernel of their own
+                kernels.residual_inject(resid, d)
+            delta = delta[-1]
+        n = (rows.numel() if rows is not None else resid.shape[0]) if n_rows is None else n_rows
+        out = torch.empty((n, self.size), dtype=self.env.act_dtype, device=resid.device)
+        kernels.add_layernorm(resid, delta, self.weight, self.bias, self.eps, out, rows=rows, n_rows=n,
+                              write_back=write_back and delta is not None)
+        return out

@@ -9,6 +9,7 @@ import torch
 
 from ..config.specs import PositionSpec
 from ..errors import ConfigError
+from ..weights.decl import TensorDecl
 from .base import BuildEnv, PositionEncoding, register_position
 
 
@@ -144,6 +145,33 @@ class SinusoidPosition(PositionEncoding):
         i = torch.arange((head_dim + 1) // 2, dtype=torch.float64)
         inv = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / head_dim)
         self.inv_freq = inv.to(torch.float32).to(env.device)
+
+    def cos_sin(self, batch):
+        return None
+
+
+@register_position("learned")
+class LearnedPosition(PositionEncoding):
+    """A table of position vectors, of which row p is added to the embedding output of a token at position p (a model's
+    ``input_position``, not a rotation inside a mixer).  Parameter ``rows``: how many positions the table has.  ``head_dim``
+    here is the model's width."""
+
+    graph_safe = True
+
+    def __init__(self, spec: PositionSpec, head_dim: int, env: BuildEnv):
+        self.rows = int(spec.params.get("rows") or 0)
+        if self.rows < 1:
+            raise ConfigError(f"a table of positions needs at least one row, found {self.rows}")
+        self.width = head_dim
+        self.rot_dim = 0
+        self.inv_freq = None
+        self.table = None
+
+    def declare(self, prefix: str):
+        return [TensorDecl(f"{prefix}.weight", (self.rows, self.width), "matrix")]
+
+    def load(self, tensors, prefix: str) -> None:
+        self.table = tensors[f"{prefix}.weight"]
 
     def cos_sin(self, batch):
         return None

@@ -9,6 +9,9 @@ g * sigmoid(alpha * g) * (u + 1).  ``choice_bias`` adds a per-expert vector to t
 only; the weights are the scores themselves, divided by their sum over the chosen (+ ``renormalize_eps``) if
 ``renormalize`` says so.  ``groups`` > 1: the experts form that many equal groups of neighbours, a group's
 score is the sum of its two largest scores, and only experts of the ``keep_groups`` best groups can be chosen.
+``score`` "softmax": s = softmax(z) over all experts.  ``identity`` (a count): that many more experts stand behind the others in
+the router and the choice; they have no tensors and no rows, their output is h itself: a token's chosen identity weights
+are summed, and the kernel that sums the choices adds that sum times h.
 ``shared`` (an intermediate size): one more expert of the same form that every token uses, its result multiplied
 by sigmoid(w_sg . h) (one number a token) when ``shared_gate`` says so; the gate's row rides along with the
 router's rows in the 32-bit router product, and the shared result joins in the kernel that sums the choices.
@@ -54,9 +57,11 @@ class RoutedMLP(FeedForward):
         self.experts = int(p["experts"])
         self.top = int(p["top"])
         self.inter = int(p["intermediate"])
-        if not 0 < self.top <= self.experts or self.experts > 512 or self.inter <= 0:
-            raise ConfigError(f"routed_mlp: {self.top} of {self.experts} experts of {self.inter} is not supported "
-                              "(1 to 512 experts, at least one and at most all of them a token)")
+        self.identity = int(p.get("identity") or 0)             # experts without tensors, whose output is their input
+        self.places = self.experts + self.identity              # what the router scores
+        if not 0 < self.top <= self.places or self.experts < 1 or self.identity < 0 or self.places > 512 or self.inter <= 0:
+            raise ConfigError(f"routed_mlp: {self.top} of {self.experts} experts of {self.inter} and {self.identity} identity experts "
+                              "is not supported (1 to 512 in all, at least one and at most all of them a token)")
         self.act = p.get("activation", "silu")
         if self.act not in kernels.GATED_ACTS:
             raise ConfigError(f"routed_mlp: activation {self.act!r} is not built (known: {sorted(kernels.GATED_ACTS)})")
@@ -64,16 +69,17 @@ class RoutedMLP(FeedForward):
         self.alpha = float(p.get("alpha", 1.0))
         if self.act == "clamped_swish" and not self.limit > 0:
             raise ConfigError("routed_mlp: clamped_swish needs a positive limit")
-        if p.get("score", "sigmoid") != "sigmoid":
-            raise ConfigError(f"routed_mlp: score {p.get('score')!r} is not built (only 'sigmoid')")
+        self.score = p.get("score", "sigmoid")
+        if self.score not in kernels.ROUTER_SCORES:
+            raise ConfigError(f"routed_mlp: score {self.score!r} is not built (known: {sorted(kernels.ROUTER_SCORES)})")
         self.renormalize = bool(p.get("renormalize", False))
         self.renormalize_eps = float(p.get("renormalize_eps", 0.0))
         self.groups = int(p.get("groups") or 1)
         self.keep_groups = int(p.get("keep_groups") or self.groups)
-        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep_groups <= self.groups or \
-                self.keep_groups * (self.experts // self.groups) < self.top:
+        if self.groups < 1 or self.places % self.groups or not 1 <= self.keep_groups <= self.groups or \
+                self.keep_groups * (self.places // self.groups) < self.top:
             raise ConfigError(f"routed_mlp: {self.groups} groups of which {self.keep_groups} stay do not fit "
-                              f"{self.experts} experts with {self.top} chosen")
+                              f"{self.places} experts with {self.top} chosen")
         self.has_bias = bool(p.get("choice_bias", False))
         self.shared_inter = int(p.get("shared") or 0)
         self.shared_gated = bool(p.get("shared_gate", False)) and self.shared_inter > 0
@@ -101,9 +107,9 @@ class RoutedMLP(FeedForward):
         return f"{prefix}{self.names['expert'].format(e=e)}{self.names[role]}.weight"
 
     def declare(self, prefix: str) -> List[TensorDecl]:
-        out = [TensorDecl(f"{prefix}{self.names['router']}.weight", (self.experts, self.hidden), "matrix")]
+        out = [TensorDecl(f"{prefix}{self.names['router']}.weight", (self.places, self.hidden), "matrix")]
         if self.has_bias:
-            out.append(TensorDecl(f"{prefix}{self.names['choice_bias']}.weight", (self.experts,), "bias"))
+            out.append(TensorDecl(f"{prefix}{self.names['choice_bias']}.weight", (self.places,), "bias"))
         if self.shared is not None:
             out += self.shared.declare(prefix + self.names["shared"])
         if self.shared_gated:
@@ -138,11 +144,11 @@ class RoutedMLP(FeedForward):
         """What a step reads at most: the router and the experts that can be chosen."""
         esz = 4 if self.env.mode == "float32" else 2
         shared = self.shared.weight_bytes() if self.shared is not None else 0
-        return self.experts * self.hidden * 4 + self.experts * 3 * self.inter * self.hidden * esz + shared
+        return self.places * self.hidden * 4 + self.experts * 3 * self.inter * self.hidden * esz + shared
 
     def _expected_experts(self, n_tokens: int) -> float:
         """The experts ``n_tokens`` tokens touch when each picks ``top`` of them at random."""
-        return self.experts * (1.0 - (1.0 - self.top / self.experts) ** n_tokens)
+        return self.experts * (1.0 - (1.0 - self.top / self.places) ** n_tokens)
 
     def _tensor_tiles(self, n_tokens: int) -> bool:
         """Whether this step's products take the tcgen05 kernel: bfloat16, enough rows, sizes it addresses."""
@@ -164,7 +170,7 @@ class RoutedMLP(FeedForward):
         esz = 4 if self.env.mode == "float32" else 2
         rows = self._max_tiles(n_tokens) * self._tile(n_tokens)
         shared = self.shared.workspace_bytes(n_tokens) if self.shared is not None else 0
-        return rows * (self.hidden * (esz + 4) + self.inter * 3 * esz) + n_tokens * (self.hidden * 4 + self.experts * 4) + shared
+        return rows * (self.hidden * (esz + 4) + self.inter * 3 * esz) + n_tokens * (self.hidden * 4 + self.places * 4) + shared
 
     def cost(self, q_lens, kv_lens):
         T = sum(q_lens)
@@ -172,8 +178,8 @@ class RoutedMLP(FeedForward):
         # which experts a step reads depends on its tokens; counted here: the experts T tokens touch when each
         # picks ``top`` of them at random (all of them for a prompt, a part of them for a few tokens)
         used = self._expected_experts(T)
-        nbytes = self.experts * self.hidden * 4 + int(used * 3 * self.inter * self.hidden * esz)
-        flops = 2 * T * self.experts * self.hidden + 2 * T * self.top * 3 * self.inter * self.hidden
+        nbytes = self.places * self.hidden * 4 + int(used * 3 * self.inter * self.hidden * esz)
+        flops = 2 * T * self.places * self.hidden + int(2 * T * self.top * self.experts / self.places * 3 * self.inter * self.hidden)
         if self.shared is not None:
             sb, sf = self.shared.cost(q_lens, kv_lens)
             nbytes, flops = nbytes + sb, flops + sf
@@ -184,7 +190,7 @@ class RoutedMLP(FeedForward):
     def forward(self, xn, batch, sum_later=False):
         T = batch.n_tokens
         dev, act = self.env.device, self.env.act_dtype
-        E, top = self.experts, self.top
+        E, top = self.places, self.top
         tile = self._tile(T)
         max_tiles = self._max_tiles(T)
         rows = max_tiles * tile
@@ -195,19 +201,20 @@ class RoutedMLP(FeedForward):
         place = torch.empty((T, top), dtype=torch.int32, device=dev)
         weights = torch.empty((T, top), dtype=torch.float32, device=dev)
         counts = torch.zeros((E,), dtype=torch.int32, device=dev)
-        starts = torch.empty((E + 1,), dtype=torch.int32, device=dev)
+        starts = torch.empty((self.experts + 1,), dtype=torch.int32, device=dev)
+        self_weight = torch.empty((T,), dtype=torch.float32, device=dev) if self.identity else None
         tile_group = torch.empty((max_tiles,), dtype=torch.int32, device=dev)
         row_of = torch.empty((T, top), dtype=torch.int32, device=dev)
         with scope(op="route"):
             kernels.moe_route(z, self.choice_bias, batch.slot_of_token, T, top, ids, weights, place, counts,
                               n_groups=self.groups, keep_groups=self.keep_groups, renormalize=self.renormalize,
-                              norm_eps=self.renormalize_eps)
-            kernels.moe_plan(counts, tile, starts, tile_group)
+                              norm_eps=self.renormalize_eps, score=self.score, identity=self.identity, self_weight=self_weight)
+            kernels.moe_plan(counts[:self.experts], tile, starts, tile_group)
             xs = torch.empty((rows, self.hidden), dtype=act, device=dev)
             kernels.moe_gather(xn, ids, place, starts, T, top, xs, row_of)
         y = torch.empty((rows, self.inter), dtype=act, device=dev)
         fused = False
-        told = {"used": self._expected_experts(T), "rows_used": T * top}     # for a profiler's accounts only
+        told = {"used": self._expected_experts(T), "rows_used": T * top * self.experts // E}     # for a profiler's accounts only
         if tile == TENSOR_TILE:
             with scope(op="experts_gate_up"):
                 fused = kernels.tile_matmul_tc5(xs, self.gate_up, y, tile_group, self.act, self.limit, self.alpha, **told)
@@ -225,7 +232,7 @@ class RoutedMLP(FeedForward):
         with scope(op="experts_down"):
             if not (tile == TENSOR_TILE and kernels.tile_matmul_tc5(y, self.down, out_rows, tile_group, **told)):
                 kernels.tile_matmul(y, self.down, out_rows, tile_group, tile, **told)
-        routed = RoutedRows(out_rows, row_of, weights, top, T)
+        routed = RoutedRows(out_rows, row_of, weights, top, T, self_weight, xn if self.identity else None)
         if self.shared is not None:
             # the expert every token uses: its partial sums join where the choices are summed
             with scope(op="shared_expert"):
@@ -233,7 +240,8 @@ class RoutedMLP(FeedForward):
             out = torch.empty((1, T, self.hidden), dtype=torch.float32, device=dev)
             with scope(op="experts_sum"):
                 kernels.moe_combine(out_rows, row_of, weights, T, top, out[0], extra=extra,
-                                    extra_gate=z[:, E] if self.shared_gated else None)
+                                    extra_gate=z[:, E] if self.shared_gated else None, self_weight=routed.self_weight,
+                                    self_x=routed.self_x)
             return out
         if sum_later:
             return routed

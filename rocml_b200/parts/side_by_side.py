@@ -1,0 +1,122 @@
+"""Two mixers side by side: both read the same input, result = left_scale * left + right_scale * right.
+
+The two share one input product (their column blocks lie behind one another) and one output product: the rows that
+each mixer's output product would read lie side by side in one row, and the output weight is [Wo_left | Wo_right],
+so that the sum over the inner size adds the two results.  The constants: right_scale / left_scale rides on the right
+mixer's last 32-bit factor (``result_factor``), left_scale on the whole result, which a consumer may apply itself
+(``ScaledDelta``); no weight is rounded again.
+
+A mixer can stand on a side when it shows its input product's column blocks (``in_stems``, ``in_outs``), makes the output
+product's rows from such columns (``mix_rows``, ``out_width``) and names its other tensors and accounts (``declare_inner``,
+``load_inner``, ``inner_bytes``, ``inner_workspace``, ``inner_cost``); the right one needs ``result_factor`` as well.  What
+the two keep per sequence becomes one bundle: the left one's requirement, and the right one's fixed-size states under the
+names ``right_<name>``."""
+from __future__ import annotations
+
+from typing import Dict, List
+
+import torch
+
+from .. import kernels
+from ..cache.requirements import BundleRequirement, StateRequirement
+from ..cache.sequence_cache import CacheView
+from ..config.specs import MixerSpec
+from ..errors import ConfigError
+from ..profile import scope
+from ..weights.decl import TensorDecl
+from .base import BuildEnv, DeferredNorm, Mixer, ScaledDelta, build_mixer, register_mixer
+from .linear import Linear
+
+SIDES = ("left", "right")
+
+
+@register_mixer("side_by_side")
+class SideBySide(Mixer):
+    scales_later = True         # forward() accepts scale_later=True and may then return a ScaledDelta
+
+    def __init__(self, spec: MixerSpec, hidden: int, env: BuildEnv):
+        p = spec.params
+        self.env = env
+        self.hidden = hidden
+        self.prefixes = {s: dict(p.get("prefixes") or ()).get(s, f"{s}.") for s in SIDES}
+        self.scales = (float(p.get("left_scale", 1.0)), float(p.get("right_scale", 1.0)))
+        self.left = build_mixer(p["left"], hidden, env)
+        self.right = build_mixer(p["right"], hidden, env)
+        for side, m in zip(SIDES, (self.left, self.right)):
+            if not hasattr(m, "mix_rows") or (side == "right" and not hasattr(m, "result_factor")):
+                raise ConfigError(f"side_by_side: the {side} mixer cannot stand on that side")
+        states = self.right.cache_requirement()
+        main = states.main if isinstance(states, BundleRequirement) else states
+        if not isinstance(main, StateRequirement):
+            raise ConfigError("side_by_side: the right mixer must keep states of fixed size")
+        # left_scale multiplies the whole result, the right side's share of it is right_scale / left_scale
+        left, right = self.scales
+        self.factor = left if left != 0.0 else 1.0
+        self.right.result_factor = right / left if left != 0.0 else right
+        self.split = sum(self.left.in_outs)
+        stems = [f"{self.prefixes[s]}{n}" for s, m in zip(SIDES, (self.left, self.right)) for n in m.in_stems]
+        self.proj = Linear(stems, list(self.left.in_outs) + list(self.right.in_outs), hidden, False, env)
+        self.o = Linear(["o"], [hidden], self.left.out_width + self.right.out_width, False, env)
+        self.o.label = "o"
+
+    @property
+    def graph_safe(self) -> bool:
+        return self.left.graph_safe and self.right.graph_safe
+
+    def cache_requirement(self):
+        req = self.right.cache_requirement()
+        main, extras = (req.main, dict(req.extras)) if isinstance(req, BundleRequirement) else (req, {})
+        return BundleRequirement.of(self.left.cache_requirement(), right_state=main, **{f"right_{k}": v for k, v in extras.items()})
+
+    def declare(self, prefix: str) -> List[TensorDecl]:
+        out = self.proj.declare(prefix)
+        for s, m in zip(SIDES, (self.left, self.right)):
+            out += m.o.declare(prefix + self.prefixes[s]) + m.declare_inner(prefix + self.prefixes[s])
+        return out
+
+    def load(self, tensors: Dict[str, torch.Tensor], prefix: str) -> None:
+        self.proj.load(tensors, prefix)
+        self.proj.pad_rows(8)
+        outs = []
+        for s, m in zip(SIDES, (self.left, self.right)):
+            m.load_inner(tensors, prefix + self.prefixes[s])
+            outs.append(tensors[f"{prefix}{self.prefixes[s]}{m.o.names[0]}.weight"])
+        if self.scales[0] == 0.0:
+            outs[0] = torch.zeros_like(outs[0])
+        if outs[0].dtype != outs[1].dtype:
+            outs = [w.float() for w in outs]
+        self.o.weight = torch.cat(outs, dim=1).contiguous()
+
+    def weight_bytes(self) -> int:
+        return self.proj.weight_bytes() + self.o.weight_bytes() + self.left.inner_bytes() + self.right.inner_bytes()
+
+    def workspace_bytes(self, n_tokens: int) -> int:
+        esz = 4 if self.env.mode == "float32" else 2
+        parts = 8 if n_tokens <= 128 else 1
+        return n_tokens * (self.proj.n * max(esz, 4 * parts if parts > 1 else esz) + self.hidden * 4 * parts + self.o.k * esz) + \
+            self.left.inner_workspace(n_tokens) + self.right.inner_workspace(n_tokens)
+
+    def cost(self, q_lens, kv_lens):
+        T = sum(q_lens)
+        parts = [self.proj.cost(T), self.o.cost(T), self.left.inner_cost(q_lens, kv_lens), self.right.inner_cost(q_lens, kv_lens)]
+        return sum(p[0] for p in parts), sum(p[1] for p in parts)
+
+    def forward(self, xn, batch, view, scale_later=False):
+        T = batch.n_tokens
+        if isinstance(xn, DeferredNorm):
+            xn = xn.materialize()
+        proj = self.proj.forward_auto(xn, T)
+        rows = torch.empty((T, self.o.k), dtype=self.env.act_dtype, device=self.env.device)
+        state = view.extras["right_state"]
+        right_view = CacheView("state", state.group, state.index, view.writes,
+                               {n[len("right_"):]: v for n, v in view.extras.items() if n.startswith("right_") and n != "right_state"})
+        self.left.mix_rows(proj[..., :self.split], batch, view, rows[:, :self.left.out_width])
+        self.right.mix_rows(proj[..., self.split:], batch, right_view, rows[:, self.left.out_width:])
+        delta = self.o.forward_delta(rows, T)
+        if self.factor == 1.0:
+            return delta
+        if scale_later:
+            return ScaledDelta(delta, self.factor)
+        with scope(op="scale"):
+            kernels.scale_(delta, self.factor)
+        return delta

@@ -57,6 +57,13 @@ def decay_scan(tokens: int, seqs: int, heads: int, dim: int, vdim: int, n_in: in
     return nbytes, 5 * tokens * heads * dim * vdim
 
 
+def delta_scan(tokens: int, seqs: int, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool) -> Cost:
+    """The gated delta rule per (sequence, head): the tokens' 32-bit q, k, v, decays and step sizes in, every sequence's
+    32-bit state in and back, 32-bit results out; per token and state entry a decay, two products and an update."""
+    per_token = 2 * kv_heads * dim + heads * (2 * vdim + (dim if per_channel else 1) + 1)
+    return 4 * tokens * per_token + 8 * seqs * heads * dim * vdim, 7 * tokens * heads * dim * vdim
+
+
 def rope_table(rows: int, half: int) -> Cost:
     return rows * (4 + half * 8) + half * 4, rows * half * 40
 
