@@ -16,8 +16,8 @@
 //                each pair, and keeps its part of the state in registers from the step's first token to its last, so the
 //                state is read and written once a step whatever the number of tokens.  A block has eight warps (or fewer, for
 //                few columns); the tokens' q, k, g and v arrive in shared memory by cp.async, a batch of tokens ahead.
-//                The order of a token's operations depends neither on how the prompt was cut nor on the batch: one
-//                token a step gives the bits of the whole prompt.
+//                The order of a token's operations depends neither on how the prompt was cut nor on the batch.
+//   delta_scan_chunks   the same for prompts, four tokens at a time: the sums over the rows of four tokens meet in one exchange.
 //   low_rank     a narrow product through few inner values for few tokens (a decode step's W2 (W1 h)), 32-bit FMA.
 #include "common.cuh"
 #include "api.h"
@@ -115,7 +115,9 @@ __device__ __forceinline__ void keep_inputs(const PrepArgs& a, const IT* in, flo
 template <typename IT, typename ZT, int VEC>
 __global__ void __launch_bounds__(128)
 delta_prep_kernel(const IT* __restrict__ in, const ZT* __restrict__ z, const PrepArgs a) {
-    pdl_trigger();
+    // (no early signal to the kernel after this one: the recurrence's few blocks, placed while thousands of these wait for
+    // their predecessor, would crowd on the multiprocessors with room left; decode steps gain from it)
+    if (blockDim.x == 32) pdl_trigger();
     pdl_wait();
     const int b = blockIdx.z, slot = a.seq_slot[b];
     if (slot < 0) return;
@@ -386,17 +388,280 @@ delta_scan_kernel(const ScanArgs a) {
     }
 }
 
+// Warps a block: few (columns) while the grid would not fill the device otherwise, eight beyond.
+int scan_warps(int n_seqs, int n_heads, int vdim) {
+    int warps = 8;
+    const long long heads = (long long)n_seqs * n_heads;
+    while (warps > 1 && (heads * ((vdim + warps * WCOLS - 1) / (warps * WCOLS)) < 148 || (warps - 1) * WCOLS >= vdim)) warps >>= 1;
+    return warps < 4 && vdim > 2 * WCOLS ? 4 : warps;
+}
+
 template <int R4, bool CH, int TB>
 int launch_scan(const ScanArgs& a, int n_seqs, cudaStream_t s) {
-    // columns a block takes: few (16) while the grid would not fill the device otherwise, 32 beyond
-    int warps = 8;
-    const long long heads = (long long)n_seqs * a.heads;
-    while (warps > 1 && (heads * ((a.vdim + warps * WCOLS - 1) / (warps * WCOLS)) < 148 || (warps - 1) * WCOLS >= a.vdim)) warps >>= 1;
-    if (warps < 4 && a.vdim > 2 * WCOLS) warps = a.vdim > 8 ? 4 : 2;
-    const int cols = warps * WCOLS;
+    const int warps = scan_warps(n_seqs, a.heads, a.vdim), cols = warps * WCOLS;
     const size_t smem = ((size_t)2 * TB * ((CH ? 3 : 2) * 64 * R4 + cols + 4) + (size_t)TB * cols) * sizeof(float);
     if (smem > 200 * 1024) return RB_ERR_BAD_SIZE;
     auto k = delta_scan_kernel<R4, CH, TB>;
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    RB_LAUNCH((k), dim3((a.vdim + cols - 1) / cols, a.heads, n_seqs), dim3(warps * 32), smem, s, a);
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+// ---- prompts: four tokens at a time -------------------------------------------------------------------------------
+// With S the state before a chunk of four tokens, G_t = g_1 .. g_t the decays up to token t inside it and G_(t,s) = g_(s+1) .. g_t:
+//   a_t = (G_t k_t)^T S + sum_{s < t} (k_t . G_(t,s) k_s) w_s,   w_t = beta_t (v_t - a_t)
+//   o_t = (G_t q_t)^T S + sum_{s <= t} (q_t . G_(t,s) k_s) w_s,   S' = G_4 S + sum_s (G_(4,s) k_s) w_s^T
+// so the columns' lanes exchange their sums once for four tokens instead of once a token, and no decay multiplies the state
+// but the chunk's.  Every G is a product of decays (no quotient), so nothing overflows.  delta_chunk forms the vectors G_t q_t,
+// G_t k_t, G_(4,s) k_s, the decay G_4 and the two triangles of products, once for all columns.
+constexpr int CH_T = 4;
+constexpr int CH_SCAL = 36;            // a chunk's numbers: [4][4] of k . k, [4][4] of q . k, four step sizes
+
+// One warp a (chunk, head).  vecs [T][heads][3][dimp], decay and numbers at the row of the chunk's first token.
+__global__ void __launch_bounds__(128)
+delta_chunk_kernel(const float* __restrict__ u, int ld_u, int uq, int uk, int ug, int ub, int heads, int kv_heads, int dim, int dimp,
+                   int per_channel, const int* __restrict__ seq_slot, const int* __restrict__ cu_q, float* __restrict__ vecs,
+                   float* __restrict__ decay, float* __restrict__ numbers) {
+    pdl_wait();                        // no early signal: see delta_prep_kernel
+    const int b = blockIdx.z;
+    if (seq_slot[b] < 0) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = cu_q[b] + (blockIdx.x * 4 + warp) * CH_T, t_end = cu_q[b + 1];
+    if (t0 >= t_end) return;
+    const int n = min(CH_T, t_end - t0), h = blockIdx.y, kvh = h / (heads / kv_heads);
+    float kk[16], qk[16];              // [t][s], s <= t used
+#pragma unroll
+    for (int i = 0; i < 16; ++i) kk[i] = qk[i] = 0.f;
+    for (int i = lane; i < dimp; i += 32) {
+        float g[4], k[4], q[4];
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            const float* row = u + (size_t)(t0 + t) * ld_u;
+            const bool in = t < n && i < dim;
+            q[t] = in ? row[uq + kvh * dim + i] : 0.f;
+            k[t] = in ? row[uk + kvh * dim + i] : 0.f;
+            g[t] = in ? row[ug + (per_channel ? h * dim + i : h)] : 1.f;
+        }
+        float up = 1.f;                // G_t
+        float part[4];                 // G_(t,s) k_s as t grows
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            up *= g[t];
+#pragma unroll
+            for (int s = 0; s < t; ++s) part[s] *= g[t];
+            part[t] = k[t];
+#pragma unroll
+            for (int s = 0; s <= t; ++s) {
+                kk[t * 4 + s] = fmaf(k[t], part[s], kk[t * 4 + s]);
+                qk[t * 4 + s] = fmaf(q[t], part[s], qk[t * 4 + s]);
+            }
+            if (t < n) {
+                float* dst = vecs + ((size_t)(t0 + t) * heads + h) * 3 * dimp + i;
+                dst[0] = up * q[t];
+                dst[dimp] = up * k[t];
+            }
+        }
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+            if (t < n) vecs[((size_t)(t0 + t) * heads + h) * 3 * dimp + 2 * dimp + i] = part[t];
+        decay[((size_t)t0 * heads + h) * dimp + i] = up;
+    }
+    // thirty-two sums over thirty-two lanes, each lane ending with one: kk 0..15, qk 16..31
+    float x[32];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) { x[i] = kk[i]; x[16 + i] = qk[i]; }
+#pragma unroll
+    for (int m = 16; m >= 1; m >>= 1) {
+        const bool upper = (lane & m) != 0;
+#pragma unroll
+        for (int i = 0; i < m; ++i) {
+            const float send = upper ? x[i] : x[i + m], keep = upper ? x[i + m] : x[i];
+            x[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+        }
+    }
+    float* num = numbers + ((size_t)t0 * heads + h) * CH_SCAL;
+    const int t = (lane >> 2) & 3, s = lane & 3;
+    num[lane] = lane < 16 ? (s < t ? x[0] : 0.f) : (s <= t ? x[0] : 0.f);
+    if (lane < 4) num[32 + lane] = lane < n ? u[(size_t)(t0 + lane) * ld_u + ub + h] : 0.f;
+}
+
+struct ChunkArgs {
+    const float *u, *vecs, *decay, *numbers;
+    int ld_u, uv, heads, dim, vdim, dimp;
+    float* state;                     // [slots][heads][vdim][dim]
+    const int *seq_slot, *cu_q;
+    float* out;
+    int ld_out, vec;                  // vec: v's columns start on 16 bytes
+};
+
+// The recurrence over chunks: lanes, columns and staging as delta_scan_kernel.  R4: groups of four rows a lane holds (dimp = 64 R4).
+template <int R4, int TB>
+__global__ void __launch_bounds__(256)
+delta_scan_chunks_kernel(const ChunkArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int DP = 64 * R4, NCH = TB / CH_T;
+    const int warps = blockDim.x >> 5, cols = warps * WCOLS;
+    const int tok = 3 * DP + cols, chk = DP + CH_SCAL;              // a staged token; a staged chunk's decay and numbers
+    const int buf_floats = TB * tok + NCH * chk;
+    float* outs = sm + 2 * buf_floats;                              // [TB][cols]
+    const int b = blockIdx.z, h = blockIdx.y, j0 = blockIdx.x * cols;
+    const int slot = a.seq_slot[b];
+    if (slot < 0) return;
+    const int t_begin = a.cu_q[b], t_end = a.cu_q[b + 1];
+    if (t_end <= t_begin) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane & 15, half = lane >> 4;
+    const int jl = warp * WCOLS + half * 2;
+    float S[2][R4][4];
+    float* st = a.state + ((size_t)slot * a.heads + h) * a.vdim * a.dim;
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int r = 0; r < R4; ++r)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = (r * RL + l) * 4 + e, j = j0 + jl + c;
+                S[c][r][e] = i < a.dim && j < a.vdim ? st[(size_t)j * a.dim + i] : 0.f;
+            }
+    const int nv = min(cols, a.vdim - j0);
+    for (int i = threadIdx.x; i < 2 * buf_floats; i += blockDim.x) sm[i] = 0.f;      // columns beyond vdim stay zero
+    __syncthreads();
+    pdl_wait();
+    auto stage = [&](int t0, int buf) {
+        const int nb = min(TB, t_end - t0);
+        float* base = sm + buf * buf_floats;
+        constexpr int V4 = 3 * DP / 4;
+        for (int i = threadIdx.x; i < nb * V4; i += blockDim.x) {
+            const int tt = i / V4, x = i - tt * V4;
+            cp_async16(base + tt * tok + 4 * x, a.vecs + ((size_t)(t0 + tt) * a.heads + h) * 3 * DP + 4 * x);
+        }
+        const int v4 = a.vec ? nv >> 2 : nv;
+        for (int i = threadIdx.x; i < nb * v4; i += blockDim.x) {
+            const int tt = i / v4, x = i - tt * v4;
+            const float* src = a.u + (size_t)(t0 + tt) * a.ld_u + a.uv + (size_t)h * a.vdim + j0;
+            if (a.vec) cp_async16(base + tt * tok + 3 * DP + 4 * x, src + 4 * x);
+            else cp_async4(base + tt * tok + 3 * DP + x, src + x);
+        }
+        const int nc = (nb + CH_T - 1) / CH_T;
+        constexpr int C4 = (DP + CH_SCAL) / 4;
+        for (int i = threadIdx.x; i < nc * C4; i += blockDim.x) {
+            const int cc = i / C4, x = i - cc * C4;
+            const size_t at = (size_t)(t0 + cc * CH_T) * a.heads + h;
+            cp_async16(base + TB * tok + cc * chk + 4 * x, x < DP / 4 ? a.decay + at * DP + 4 * x : a.numbers + at * CH_SCAL + 4 * (x - DP / 4));
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage(t_begin, 0);
+    int buf = 0;
+    for (int t0 = t_begin; t0 < t_end; t0 += TB, buf ^= 1) {
+        const int nb = min(TB, t_end - t0), nc = (nb + CH_T - 1) / CH_T;
+        if (t0 + TB < t_end) {
+            stage(t0 + TB, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        float* base = sm + buf * buf_floats;
+        for (int i = nb * tok + threadIdx.x; i < nc * CH_T * tok; i += blockDim.x) base[i] = 0.f;    // a last chunk's missing tokens
+        __syncthreads();
+        for (int cc = 0; cc < nc; ++cc) {
+            const float* x = base + cc * CH_T * tok;
+            const float* dec = base + TB * tok + cc * chk;
+            const float* num = dec + DP;
+            float y[16];                 // [k | q][column][token]
+#pragma unroll
+            for (int i = 0; i < 16; ++i) y[i] = 0.f;
+#pragma unroll
+            for (int r = 0; r < R4; ++r) {
+                const int i = (r * RL + l) * 4;
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    float q[4], k[4];
+                    load4(x + t * tok + i, q);
+                    load4(x + t * tok + DP + i, k);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        y[t] = fmaf(k[e], S[0][r][e], y[t]);
+                        y[4 + t] = fmaf(k[e], S[1][r][e], y[4 + t]);
+                        y[8 + t] = fmaf(q[e], S[0][r][e], y[8 + t]);
+                        y[12 + t] = fmaf(q[e], S[1][r][e], y[12 + t]);
+                    }
+                }
+            }
+            // sixteen sums over sixteen lanes: lane l ends with the l-th
+#pragma unroll
+            for (int m = 8; m >= 1; m >>= 1) {
+                const bool upper = (l & m) != 0;
+#pragma unroll
+                for (int i = 0; i < m; ++i) {
+                    const float send = upper ? y[i] : y[i + m], keep = upper ? y[i + m] : y[i];
+                    y[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+                }
+            }
+            float w[2][4];
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const float beta = num[32 + t];
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    float at = __shfl_sync(0xffffffffu, y[0], (lane & 16) | (c * 4 + t));
+#pragma unroll
+                    for (int s = 0; s < t; ++s) at = fmaf(num[t * 4 + s], w[c][s], at);
+                    w[c][t] = beta * (x[t * tok + 3 * DP + jl + c] - at);
+                }
+            }
+            if (l >= 8) {
+                const int t = l & 3, c = (l >> 2) & 1;
+                float d[4];
+                load4(num + 16 + t * 4, d);
+                float o = y[0];
+#pragma unroll
+                for (int s = 0; s < 4; ++s) o = fmaf(d[s], c ? w[1][s] : w[0][s], o);
+                outs[(cc * CH_T + t) * cols + jl + c] = o;
+            }
+#pragma unroll
+            for (int r = 0; r < R4; ++r) {
+                const int i = (r * RL + l) * 4;
+                float f[4];
+                load4(dec + i, f);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) { S[0][r][e] *= f[e]; S[1][r][e] *= f[e]; }
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    float k[4];
+                    load4(x + t * tok + 2 * DP + i, k);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        S[0][r][e] = fmaf(k[e], w[0][t], S[0][r][e]);
+                        S[1][r][e] = fmaf(k[e], w[1][t], S[1][r][e]);
+                    }
+                }
+            }
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < nb * cols; i += blockDim.x) {
+            const int tt = i / cols, j = i - tt * cols;
+            if (j < nv) a.out[(size_t)(t0 + tt) * a.ld_out + (size_t)h * a.vdim + j0 + j] = outs[i];
+        }
+    }
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int r = 0; r < R4; ++r)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = (r * RL + l) * 4 + e, j = j0 + jl + c;
+                if (i < a.dim && j < a.vdim) st[(size_t)j * a.dim + i] = S[c][r][e];
+            }
+}
+
+template <int R4, int TB>
+int launch_chunks(const ChunkArgs& a, int n_seqs, cudaStream_t s) {
+    const int warps = scan_warps(n_seqs, a.heads, a.vdim), cols = warps * WCOLS;
+    const size_t smem = ((size_t)2 * (TB * (3 * 64 * R4 + cols) + TB / CH_T * (64 * R4 + CH_SCAL)) + (size_t)TB * cols) * sizeof(float);
+    if (smem > 200 * 1024) return RB_ERR_BAD_SIZE;
+    auto k = delta_scan_chunks_kernel<R4, TB>;
     cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     RB_LAUNCH((k), dim3((a.vdim + cols - 1) / cols, a.heads, n_seqs), dim3(warps * 32), smem, s, a);
@@ -533,4 +798,27 @@ extern "C" int rb_low_rank(const void* in, int in_dtype, int n_in, long long in_
 #undef RB_LR
     RB_LAUNCH_CHECK();
     return RB_OK;
+}
+
+// The same for prompts, four tokens at a time: vecs float32 [T][heads][3][dimp], decay float32 [T][heads][dimp], numbers float32
+// [T][heads][36] are work space, dimp = dim rounded up to 64 (128, 256).  RB_ERR_BAD_SIZE for dim > 256.
+extern "C" int rb_delta_scan_chunks(const float* u, int ld_u, int uq, int uk, int uv, int ug, int ub, int ud, int heads, int kv_heads,
+                                    int dim, int vdim, int per_channel, float* state, const int* seq_slot, const int* cu_q, int n_seqs,
+                                    int max_q_len, float* vecs, float* decay, float* numbers, int dimp, float* out, int ld_out,
+                                    void* stream) {
+    (void)ud;
+    if (n_seqs <= 0 || max_q_len <= 0) return RB_OK;
+    if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || n_seqs > 65535 || heads > 65535 || dim > dimp ||
+        (dimp != 64 && dimp != 128 && dimp != 256))
+        return RB_ERR_BAD_SIZE;
+    if (((uintptr_t)vecs | (uintptr_t)decay | (uintptr_t)numbers) & 15) return RB_ERR_BAD_ALIGN;
+    cudaStream_t s = (cudaStream_t)stream;
+    RB_LAUNCH((delta_chunk_kernel), dim3((max_q_len + 4 * CH_T - 1) / (4 * CH_T), heads, n_seqs), dim3(128), 0, s, u, ld_u, uq, uk, ug, ub,
+              heads, kv_heads, dim, dimp, per_channel, seq_slot, cu_q, vecs, decay, numbers);
+    RB_LAUNCH_CHECK();
+    ChunkArgs a{u, vecs, decay, numbers, ld_u, uv, heads, dim, vdim, dimp, state, seq_slot, cu_q, out, ld_out, 0};
+    a.vec = ((vdim | ld_u | uv) & 3) == 0 && ((uintptr_t)u & 15) == 0;
+    if (dimp == 64) return launch_chunks<1, 16>(a, n_seqs, s);
+    if (dimp == 128) return launch_chunks<2, 16>(a, n_seqs, s);
+    return launch_chunks<4, 8>(a, n_seqs, s);
 }

@@ -200,6 +200,8 @@ def _lib():
         lib.rb_delta_prep.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _ll, _i, _vp,
                                       _vp, _i, _f, _f, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]
         lib.rb_delta_scan.argtypes = [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp]
+        lib.rb_delta_scan_chunks.argtypes = [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _vp, _i,
+                                             _vp, _i, _vp]
         lib.rb_low_rank.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _vp, _i, _i, _i, _vp, _i, _i, _i, _vp, _i, _vp]
         lib.rb_gemm_tcgen05_set_wait.argtypes = [_ll, _i]
         lib.rb_gemm_tcgen05_set_wait.restype = None
@@ -1859,6 +1861,36 @@ def delta_scan(u: torch.Tensor, n_tokens: int, rows: DeltaRows, heads: int, kv_h
     rc = _lib().rb_delta_scan(_ptr(u), u.stride(0), *rows.offsets, heads, kv_heads, dim, vdim, 1 if per_channel else 0, _ptr(state),
                               _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, _ptr(out), out.stride(0), _stream())
     _check(rc, "delta_scan")
+
+
+DELTA_CHUNK_NUMBERS = 36       # CH_SCAL of csrc/gated_delta.cu
+
+
+def delta_padded_dim(dim: int) -> Optional[int]:
+    """The rows a head's vectors are padded to in delta_scan_chunks (None: it does not take the size)."""
+    return next((d for d in (64, 128, 256) if dim <= d), None)
+
+
+@_profiled(lambda a, facts: _cost.delta_scan(a["n_tokens"], a["n_seqs"], a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["per_channel"]))
+def delta_scan_chunks(u: torch.Tensor, n_tokens: int, rows: DeltaRows, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool,
+                      state: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, n_seqs: int, max_q_len: int, out: torch.Tensor,
+                      vecs: torch.Tensor, decay: torch.Tensor, numbers: torch.Tensor):
+    """``delta_scan`` for prompts, four tokens at a time (results differ by rounding only).  Work space, float32: ``vecs``
+    [T, heads, 3, dimp], ``decay`` [T, heads, dimp], ``numbers`` [T, heads, 36] with dimp = ``delta_padded_dim``."""
+    dimp = delta_padded_dim(dim)
+    if dimp is None or u.dtype != torch.float32 or u.stride(-1) != 1 or u.shape[-1] < rows.width or u.shape[0] < n_tokens:
+        raise KernelError("delta_scan_chunks: u must be float32 [T, rows.width], heads of at most 256")
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (heads, vdim, dim):
+        raise KernelError("delta_scan_chunks: state must be contiguous float32 [slots, heads, vdim, dim]")
+    if out.dtype != torch.float32 or out.stride(-1) != 1 or out.shape[-1] != heads * vdim or out.shape[0] < n_tokens:
+        raise KernelError("delta_scan_chunks: out must be float32 [T, heads * vdim]")
+    for t, n in ((vecs, heads * 3 * dimp), (decay, heads * dimp), (numbers, heads * DELTA_CHUNK_NUMBERS)):
+        if t.dtype != torch.float32 or not t.is_contiguous() or t.numel() < n_tokens * n:
+            raise KernelError("delta_scan_chunks: the work space is too small")
+    rc = _lib().rb_delta_scan_chunks(_ptr(u), u.stride(0), *rows.offsets, heads, kv_heads, dim, vdim, 1 if per_channel else 0, _ptr(state),
+                                     _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, max_q_len, _ptr(vecs), _ptr(decay),
+                                     _ptr(numbers), dimp, _ptr(out), out.stride(0), _stream())
+    _check(rc, "delta_scan_chunks")
 
 
 @_profiled(lambda a, facts: (a["w0"].numel() * _esz(a["w0"]) + (a["w1"].numel() * _esz(a["w1"]) if a["w1"] is not None else 0)

@@ -12,8 +12,8 @@ What a sequence keeps, whatever its length: the state (stored [heads, v_head_dim
 memory) and the convolution's last conv_taps - 1 inputs, both 32-bit.  One stacked product makes every column block from the
 layer's input (of a narrow product W2 (W1 h) the inner values are among them; the outer product is a tensor-core product for
 prompts and a small kernel for few tokens); one kernel prepares the recurrence's inputs in 32-bit; one kernel carries the
-step's tokens through the recurrence with the state in registers, the same for prompts, pieces and single tokens; one
-kernel normalises and gates.  The inner ranks of narrow products are sizes of the tensors, given as ``decay_rank`` and
+step's tokens through the recurrence with the state in registers (token after token for single tokens and short pieces; four at
+a time for prompts, from vectors that one more kernel prepares); one kernel normalises and gates.  The inner ranks of narrow products are sizes of the tensors, given as ``decay_rank`` and
 ``gate_rank``.
 """
 from __future__ import annotations
@@ -32,6 +32,8 @@ from .base import BuildEnv, DeferredNorm, Mixer, register_mixer
 from .linear import Linear
 
 UNIT_EPS = 1e-6                # under the root of a unit vector's length
+
+CHUNKS_MIN_TOKENS = 16         # a step whose longest sequence brings more tokens runs the recurrence four tokens at a time
 
 LOW_RANK_MAX_TOKENS = 64       # up to it the outer half of a narrow product is the small kernel for few tokens
 
@@ -154,7 +156,8 @@ class GatedDelta(Mixer):
     def inner_workspace(self, n_tokens: int) -> int:
         esz = 4 if self.env.mode == "float32" else 2
         narrow = (self.heads * self.hd if self.per_channel else 0) + (self.inner if self.narrow_gate else 0)
-        return n_tokens * (4 * (self.rows.width + self.inner + narrow) + self.inner * esz)
+        work = self.heads * (4 * (kernels.delta_padded_dim(self.hd) or 0) + kernels.DELTA_CHUNK_NUMBERS) if n_tokens > CHUNKS_MIN_TOKENS else 0
+        return n_tokens * (4 * (self.rows.width + self.inner + narrow + work) + self.inner * esz)
 
     def workspace_bytes(self, n_tokens: int) -> int:
         esz = 4 if self.env.mode == "float32" else 2
@@ -182,7 +185,7 @@ class GatedDelta(Mixer):
         dev, act = self.env.device, self.env.act_dtype
         off = self.off
         # the outer halves of the narrow products
-        z, gate, gate_off = proj[..., off.get("decay", 0):], proj, off.get("gate", 0)
+        z, gate, gate_off, gate_inner = proj[..., off.get("decay", 0):], proj, off.get("gate", 0), None
         if self.per_channel or self.narrow_gate:
             a, b = self.decay_out, self.gate_out
             if T <= LOW_RANK_MAX_TOKENS and max(self.decay_rank, self.gate_rank) <= kernels.LOW_RANK_MAX:
@@ -200,9 +203,7 @@ class GatedDelta(Mixer):
                 if a is not None:
                     z = torch.empty((T, a.n), dtype=torch.float32, device=dev)
                     a.forward(inner[:, off["decay_in"]:off["decay_in"] + self.decay_rank], z, T)
-                if b is not None:
-                    gate, gate_off = torch.empty((T, b.n), dtype=act, device=dev), 0
-                    b.forward(inner[:, off["gate_in"]:off["gate_in"] + self.gate_rank], gate, T)
+                gate_inner = inner
         u = torch.empty((T, self.rows.width), dtype=torch.float32, device=dev)
         kept = view.extras["conv"].state if self.taps > 1 else None
         with scope(op="delta_prep"):
@@ -211,8 +212,17 @@ class GatedDelta(Mixer):
                                batch.seq_slot, batch.cu_q, batch.n_seqs, batch.max_q_len, u, self.rows)
         o = torch.empty((T, self.inner), dtype=torch.float32, device=dev)
         with scope(op="delta_scan"):
-            kernels.delta_scan(u, T, self.rows, self.heads, self.kv, self.hd, self.vd, self.per_channel, view.state, batch.seq_slot,
-                               batch.cu_q, batch.n_seqs, o)
+            sizes = (self.rows, self.heads, self.kv, self.hd, self.vd, self.per_channel, view.state, batch.seq_slot, batch.cu_q, batch.n_seqs)
+            dimp = kernels.delta_padded_dim(self.hd)
+            if batch.max_q_len > CHUNKS_MIN_TOKENS and dimp is not None:
+                vecs, decay, numbers = (torch.empty((T, self.heads, w), dtype=torch.float32, device=dev)
+                                        for w in (3 * dimp, dimp, kernels.DELTA_CHUNK_NUMBERS))
+                kernels.delta_scan_chunks(u, T, *sizes, batch.max_q_len, o, vecs, decay, numbers)
+            else:
+                kernels.delta_scan(u, T, *sizes, o)
+        if gate_inner is not None and self.narrow_gate:
+            gate, gate_off = torch.empty((T, self.inner), dtype=act, device=dev), 0
+            self.gate_out.forward(gate_inner[:, off["gate_in"]:off["gate_in"] + self.gate_rank], gate, T)
         if out is None:
             out = torch.empty((T, self.inner), dtype=act, device=dev)
         with scope(op="norm_gate"):
