@@ -405,3 +405,105 @@ def write_tibenex(folder, cfg_dict, seed, std=0.06, slow_decay=False):
         w[k] = t.to(torch.bfloat16)
     save_file(w, path)
     return folder
+
+
+# ---- Ravelorn: norms on the sublayers' results; the gated delta rule alone (a decay per key channel) and beside attention with
+# a sink per head (a decay per head); softmax-scored experts with identity experts --------------------------------------------
+def _rdelta(heads, kv_heads, dim, vdim, conv, ranks=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}
+    if ranks is not None:
+        m["decay_rank"], m["gate_rank"] = ranks
+    return m
+
+
+def _rleft(heads, kv_heads, dim, vdim, scale, q_temp):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "q_temp": {"coef": q_temp[0], "every": q_temp[1]}}
+
+
+def _rmoe(experts, identity, top, ff):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": identity, "top": top}}
+
+
+def _rpar(left, right, left_scale, right_scale, mlp):
+    return {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": left_scale, "right_scale": right_scale}, "mlp": mlp}
+
+
+def _rchan(mixer, mlp):
+    return {"type": "channel_delta", "mixer": mixer, "mlp": mlp}
+
+
+# RA: several heads on a query/key head everywhere, value sizes narrower and wider, a layer without feed-forward, a temperature
+# that steps every few positions
+RAVELORN_A = {
+    "architecture": "Ravelorn", "vocab": 211, "width": 64, "max_positions": 640, "norm": {"eps": 1e-6}, "residual_mult": 0.6,
+    "logit_softcap": 5.0,
+    "layers": [_rpar(_rleft(4, 2, 16, 16, 0.9, (0.5, 20)), _rdelta(4, 2, 8, 12, 3), 0.7, 1.3, _rmoe(5, 2, 3, 24)),
+               _rchan(_rdelta(4, 2, 12, 20, 4, (10, 6)), None),
+               _rchan(_rdelta(2, 1, 16, 8, 2, (24, 16)), _rmoe(4, 1, 2, 48)),
+               _rpar(_rleft(6, 1, 24, 12, 0.4, (0.2, 33)), _rdelta(3, 3, 20, 16, 5), -0.5, 0.4, None)],
+}
+# RB: head sizes that the bfloat16 attention kernels take, heads of the delta rule that fill its registers, inner sizes that
+# differ, eight query heads a key/value head, a part that spans two groups of rows
+RAVELORN_B = {
+    "architecture": "Ravelorn", "vocab": 333, "width": 128, "max_positions": 1024, "norm": {"eps": 1e-5}, "residual_mult": 0.45,
+    "logit_softcap": 30.0,
+    "layers": [_rpar(_rleft(8, 1, 64, 64, 0.3, (0.3, 64)), _rdelta(6, 3, 64, 64, 4), 1.0, 0.8, _rmoe(6, 1, 3, 64)),
+               _rchan(_rdelta(2, 1, 128, 128, 4, (32, 40)), _rmoe(6, 3, 2, 96)),
+               _rpar(_rleft(4, 2, 128, 128, 0.2, (0.6, 100)), _rdelta(2, 2, 96, 72, 4), 0.4, 0.9, _rmoe(8, 0, 4, 32)),
+               _rchan(_rdelta(3, 3, 136, 64, 3, (16, 8)), _rmoe(3, 1, 1, 32))],
+}
+# RC: sizes that are multiples of four or of nothing, a convolution of one tap and one of more taps than a short step has tokens,
+# one head, all experts chosen, more identity experts than others, scales of one, a cap that bends every logit
+RAVELORN_C = {
+    "architecture": "Ravelorn", "vocab": 97, "width": 72, "max_positions": 560, "norm": {"eps": 3e-5}, "residual_mult": 1.0,
+    "logit_softcap": 1.5,
+    "layers": [_rpar(_rleft(3, 3, 20, 28, 1.0, (1.0, 1)), _rdelta(1, 1, 5, 7, 1), 1.0, 1.0, _rmoe(2, 3, 5, 28)),
+               _rchan(_rdelta(3, 3, 36, 4, 6, (9, 5)), _rmoe(7, 0, 1, 20)),
+               _rchan(_rdelta(5, 5, 10, 30, 9, (7, 12)), None)],
+}
+RAVELORN = {"RA": RAVELORN_A, "RB": RAVELORN_B, "RC": RAVELORN_C}
+
+
+def write_ravelorn(folder, cfg_dict, seed, std=0.08, fixed_routes=True, slow_decay=False):
+    """A Ravelorn model folder with random weights.  ``fixed_routes``: the corrections lie so far apart that every token makes
+    the same choices (the weights still follow the tokens); otherwise the routers' rows are large, which spreads the scores.
+    Sinks of the scores' size; decays that remember tens of tokens (``slow_decay``: hundreds).  The narrow products' inner
+    sizes are left to the tensors' shapes."""
+    from safetensors.torch import load_file, save_file
+    write_model(folder, cfg_dict, seed)
+    path = os.path.join(folder, "model.safetensors")
+    w = load_file(path)
+    g = torch.Generator().manual_seed(seed)
+    for k in sorted(w):
+        t = w[k].float()
+        if k.endswith(".correction"):
+            t = torch.randperm(t.shape[0], generator=g).float() * 1.5 if fixed_routes else torch.rand(t.shape, generator=g) * 0.1
+        elif k.endswith(".router"):
+            t = t * (1.5 * std / 0.02)
+        elif k.endswith(".conv"):
+            t = t * 20.0
+        elif k in ("embed", "pos"):
+            t = t * 40.0
+        elif t.dim() == 2:
+            t = t * (std / 0.02)
+        elif k.endswith(".A_log"):
+            t = (t - 1.0) * 5.0 - (5.5 if slow_decay else 2.0)
+        elif k.endswith(".dt_bias"):
+            t = (t - 1.0) * 5.0 - 0.5
+        elif k.endswith(".sink"):
+            t = t * 50.0
+        elif k.endswith(".norm") and ".mix" in k:
+            t = 1.0 + 3.0 * (t - 1.0)
+        elif k.endswith((".norm1.b", ".norm2.b", "final.norm.b")):
+            t = t * 10.0
+        w[k] = t.to(torch.bfloat16)
+    save_file(w, path)
+    cfg_path = os.path.join(folder, "config.json")
+    with open(cfg_path) as f:
+        cfg = json.load(f)
+    for L in cfg["layers"]:
+        for name in ("decay_rank", "gate_rank"):
+            L["mixer"].pop(name, None)
+    with open(cfg_path, "w") as f:
+        json.dump(cfg, f)
+    return folder
