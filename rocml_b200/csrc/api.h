@@ -283,7 +283,7 @@ int rb_delta_scan(const float* u, int ld_u, int uq, int uk, int uv, int ug, int 
                   int ld_out, void* stream);
 int rb_delta_scan_chunks(const float* u, int ld_u, int uq, int uk, int uv, int ug, int ub, int ud, int heads, int kv_heads, int dim,
                          int vdim, int per_channel, float* state, const int* seq_slot, const int* cu_q, int n_seqs, int max_q_len,
-                         float* vecs, float* decay, float* numbers, int dimp, float* out, int ld_out, void* stream);
+                         int T, float* vecs, float* firsts, int n_chunks, int dimp, float* out, int ld_out, void* stream);
 // out[t, n] = sum_r w_i[n, r] * x_i[t, r] for up to two matrices w_i [n_i, rank_i] and column blocks x_off_i of the rows (n_in
 // partial sums added first); results side by side, float32.
 int rb_low_rank(const void* in, int in_dtype, int n_in, long long in_stride, int row_stride, int x_off0, int rank0,

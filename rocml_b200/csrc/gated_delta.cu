@@ -194,6 +194,120 @@ delta_prep_kernel(const IT* __restrict__ in, const ZT* __restrict__ z, const Pre
     }
 }
 
+// The same for prompts with at most four taps and heads of at most 128 (a lane holds four channels): a warp takes eight tokens in a
+// row, asks for all their rows at once and slides the convolution's window over them in registers.
+constexpr int ROWS_W = PREP_TOK / 4;       // tokens a warp (four warps a block)
+
+template <int TAPS, typename IT>
+__device__ __forceinline__ void conv_rows(const PrepArgs& a, const IT* in, const float* mine, int t0, int n, int t_begin, int col, int c,
+                                          float (&y)[ROWS_W][4]) {
+    float x[ROWS_W + TAPS - 1][4], w[TAPS][4];
+#pragma unroll
+    for (int i = 0; i < ROWS_W + TAPS - 1; ++i) {
+        const int r = t0 - (TAPS - 1) + i;
+        x[i][0] = x[i][1] = x[i][2] = x[i][3] = 0.f;
+        if (i >= n + TAPS - 1) continue;
+        if (r >= t_begin) load4(in + (size_t)r * a.row_stride + col, x[i]);
+        else if (TAPS > 1) load4(mine + (size_t)(TAPS - 1 + (r - t_begin)) * a.channels + c, x[i]);
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load4(a.conv_w + (size_t)j * a.channels + c, w[j]);
+#pragma unroll
+    for (int i = 0; i < ROWS_W; ++i)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j][u], x[i + j][u], acc);
+            y[i][u] = silu(acc);
+        }
+}
+
+template <typename IT, typename ZT, int TAPS>
+__global__ void __launch_bounds__(128)
+delta_prep_rows_kernel(const IT* __restrict__ in, const ZT* __restrict__ z, const PrepArgs a) {
+    pdl_wait();                        // no early signal: see delta_prep_kernel
+    const int b = blockIdx.z, slot = a.seq_slot[b];
+    if (slot < 0) return;
+    const int t_begin = a.cu_q[b], t_end = a.cu_q[b + 1];
+    const int tb = t_begin + blockIdx.y * PREP_TOK;
+    if (tb >= t_end) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = tb + warp * ROWS_W, n = min(ROWS_W, t_end - t0);
+    float* mine = TAPS > 1 ? a.kept + (size_t)slot * (TAPS - 1) * a.channels : nullptr;
+    const int kd = a.kv_heads * a.dim, i0 = lane * 4;
+    const bool keys = (int)blockIdx.x < a.kv_heads;
+    const int h = keys ? blockIdx.x : blockIdx.x - a.kv_heads;
+    if (n > 0 && keys) {
+        const int c = h * a.dim + i0;
+        const bool on = i0 < a.dim;
+        float q[ROWS_W][4] = {}, k[ROWS_W][4] = {};
+        if (on) {
+            conv_rows<TAPS>(a, in, mine, t0, n, t_begin, a.q_off + c, c, q);
+            conv_rows<TAPS>(a, in, mine, t0, n, t_begin, a.k_off + c, kd + c, k);
+        }
+#pragma unroll
+        for (int t = 0; t < ROWS_W; ++t) {
+            float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+            for (int u = 0; u < 4; ++u) { qq = fmaf(q[t][u], q[t][u], qq); kk = fmaf(k[t][u], k[t][u], kk); qk = fmaf(q[t][u], k[t][u], qk); }
+            const float fq = a.q_scale / sqrtf(warp_sum(qq) + a.unit_eps), fk = 1.f / sqrtf(warp_sum(kk) + a.unit_eps);
+            qk = warp_sum(qk);
+            if (t >= n) continue;
+            float* row = a.u + (size_t)(t0 + t) * a.ld_u;
+            if (on) {
+#pragma unroll
+                for (int u = 0; u < 4; ++u) { q[t][u] *= fq; k[t][u] *= fk; }
+                store4(row + a.uq + c, q[t]);
+                store4(row + a.uk + c, k[t]);
+            }
+            if (lane == 0) row[a.ud + h] = qk * fq * fk;
+        }
+    } else if (n > 0) {
+        const float rate = expf(a.a_log[h]);
+        if (i0 < a.vdim) {
+            const int c = h * a.vdim + i0;
+            float v[ROWS_W][4];
+            conv_rows<TAPS>(a, in, mine, t0, n, t_begin, a.v_off + c, 2 * kd + c, v);
+#pragma unroll
+            for (int t = 0; t < ROWS_W; ++t)
+                if (t < n) store4(a.u + (size_t)(t0 + t) * a.ld_u + a.uv + c, v[t]);
+        }
+        if (a.per_channel) {
+            if (i0 < a.dim) {
+                float g[ROWS_W][4], bias[4];
+#pragma unroll
+                for (int t = 0; t < ROWS_W; ++t)
+                    if (t < n) load4(z + (size_t)(t0 + t) * a.z_row_stride + (size_t)h * a.dim + i0, g[t]);
+                load4(a.dt_bias + (size_t)h * a.dim + i0, bias);
+#pragma unroll
+                for (int t = 0; t < ROWS_W; ++t) {
+                    if (t >= n) continue;
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) g[t][u] = expf(-rate * softplus_f32(g[t][u] + bias[u]));
+                    store4(a.u + (size_t)(t0 + t) * a.ld_u + a.ug + (size_t)h * a.dim + i0, g[t]);
+                }
+            }
+        } else if (lane >= 16 && lane - 16 < n) {
+            const int t = t0 + lane - 16;
+            a.u[(size_t)t * a.ld_u + a.ug + h] = expf(-rate * softplus_f32(to_f32(z[(size_t)t * a.z_row_stride + h]) + a.dt_bias[h]));
+        }
+        if (lane < n) {
+            const int t = t0 + lane;
+            a.u[(size_t)t * a.ld_u + a.ub + h] = sigmoid_f32(to_f32(in[(size_t)t * a.row_stride + a.b_off + h]));
+        }
+    }
+    if (blockIdx.y == 0 && TAPS > 1) {
+        __syncthreads();
+        if (keys) {
+            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.q_off + h * a.dim, h * a.dim, a.dim);
+            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.k_off + h * a.dim, kd + h * a.dim, a.dim);
+        } else {
+            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.v_off + h * a.vdim, 2 * kd + h * a.vdim, a.vdim);
+        }
+    }
+}
+
 // ---- the recurrence ---------------------------------------------------------------------------------------------
 constexpr int RL = 16;                // lanes that share a column's rows
 constexpr int WCOLS = 4;              // columns a warp owns: two for each half of the warp
@@ -419,11 +533,12 @@ int launch_scan(const ScanArgs& a, int n_seqs, cudaStream_t s) {
 constexpr int CH_T = 4;
 constexpr int CH_SCAL = 36;            // a chunk's numbers: [4][4] of k . k, [4][4] of q . k, four step sizes
 
-// One warp a (chunk, head).  vecs [T][heads][3][dimp], decay and numbers at the row of the chunk's first token.
+// One warp a (chunk, head).  vecs [heads][T][3][dimp]; firsts [heads][n_chunks][dimp + 36], a chunk's decay and numbers.  The
+// chunks of sequence b are numbered from cu_q[b] / 4 + b, so that no two sequences share a number.
 __global__ void __launch_bounds__(128)
 delta_chunk_kernel(const float* __restrict__ u, int ld_u, int uq, int uk, int ug, int ub, int heads, int kv_heads, int dim, int dimp,
-                   int per_channel, const int* __restrict__ seq_slot, const int* __restrict__ cu_q, float* __restrict__ vecs,
-                   float* __restrict__ decay, float* __restrict__ numbers) {
+                   int per_channel, const int* __restrict__ seq_slot, const int* __restrict__ cu_q, int T, int n_chunks,
+                   float* __restrict__ vecs, float* __restrict__ firsts) {
     pdl_wait();                        // no early signal: see delta_prep_kernel
     const int b = blockIdx.z;
     if (seq_slot[b] < 0) return;
@@ -431,6 +546,8 @@ delta_chunk_kernel(const float* __restrict__ u, int ld_u, int uq, int uk, int ug
     const int t0 = cu_q[b] + (blockIdx.x * 4 + warp) * CH_T, t_end = cu_q[b + 1];
     if (t0 >= t_end) return;
     const int n = min(CH_T, t_end - t0), h = blockIdx.y, kvh = h / (heads / kv_heads);
+    const int chunk = cu_q[b] / CH_T + b + blockIdx.x * 4 + warp;
+    float* first = firsts + ((size_t)h * n_chunks + chunk) * (dimp + CH_SCAL);
     float kk[16], qk[16];              // [t][s], s <= t used
 #pragma unroll
     for (int i = 0; i < 16; ++i) kk[i] = qk[i] = 0.f;
@@ -458,15 +575,15 @@ delta_chunk_kernel(const float* __restrict__ u, int ld_u, int uq, int uk, int ug
                 qk[t * 4 + s] = fmaf(q[t], part[s], qk[t * 4 + s]);
             }
             if (t < n) {
-                float* dst = vecs + ((size_t)(t0 + t) * heads + h) * 3 * dimp + i;
+                float* dst = vecs + ((size_t)h * T + t0 + t) * 3 * dimp + i;
                 dst[0] = up * q[t];
                 dst[dimp] = up * k[t];
             }
         }
 #pragma unroll
         for (int t = 0; t < 4; ++t)
-            if (t < n) vecs[((size_t)(t0 + t) * heads + h) * 3 * dimp + 2 * dimp + i] = part[t];
-        decay[((size_t)t0 * heads + h) * dimp + i] = up;
+            if (t < n) vecs[((size_t)h * T + t0 + t) * 3 * dimp + 2 * dimp + i] = part[t];
+        first[i] = up;
     }
     // thirty-two sums over thirty-two lanes, each lane ending with one: kk 0..15, qk 16..31
     float x[32];
@@ -481,114 +598,176 @@ delta_chunk_kernel(const float* __restrict__ u, int ld_u, int uq, int uk, int ug
             x[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
         }
     }
-    float* num = numbers + ((size_t)t0 * heads + h) * CH_SCAL;
+    float* num = first + dimp;
     const int t = (lane >> 2) & 3, s = lane & 3;
     num[lane] = lane < 16 ? (s < t ? x[0] : 0.f) : (s <= t ? x[0] : 0.f);
     if (lane < 4) num[32 + lane] = lane < n ? u[(size_t)(t0 + lane) * ld_u + ub + h] : 0.f;
 }
 
 struct ChunkArgs {
-    const float *u, *vecs, *decay, *numbers;
-    int ld_u, uv, heads, dim, vdim, dimp;
+    const float *u, *vecs, *firsts;
+    int T, n_chunks, ld_u, uv, heads, dim, vdim, dimp;
     float* state;                     // [slots][heads][vdim][dim]
     const int *seq_slot, *cu_q;
     float* out;
     int ld_out, vec;                  // vec: v's columns start on 16 bytes
 };
 
-// The recurrence over chunks: lanes, columns and staging as delta_scan_kernel.  R4: groups of four rows a lane holds (dimp = 64 R4).
+// Two 32-bit numbers a register pair: one instruction for two multiply-adds.
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ void load22(const float* p, uint64_t* x) {
+    const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
+    x[0] = v.x;
+    x[1] = v.y;
+}
+
+// The recurrence over chunks: lanes and columns as in delta_scan_kernel (R4: groups of four rows a lane holds, dimp = 64 R4),
+// four warps of columns a block, and a fifth warp that brings the next TB tokens and takes the last ones' results away, so
+// that the warps of columns meet it once for TB tokens and do nothing else.
+constexpr int CH_WARPS = 4;
+
 template <int R4, int TB>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__((CH_WARPS + 1) * 32, R4 > 2 ? 1 : (TB <= 8 ? 4 : 3))
 delta_scan_chunks_kernel(const ChunkArgs a) {
     extern __shared__ __align__(16) float sm[];
-    constexpr int DP = 64 * R4, NCH = TB / CH_T;
-    const int warps = blockDim.x >> 5, cols = warps * WCOLS;
-    const int tok = 3 * DP + cols, chk = DP + CH_SCAL;              // a staged token; a staged chunk's decay and numbers
-    const int buf_floats = TB * tok + NCH * chk;
-    float* outs = sm + 2 * buf_floats;                              // [TB][cols]
+    constexpr int DP = 64 * R4, NCH = TB / CH_T, cols = CH_WARPS * WCOLS;
+    constexpr int TOK = 3 * DP, CHK = DP + CH_SCAL;                 // a staged token's vectors; a staged chunk's decay and numbers
+    constexpr int BUF = TB * (TOK + cols) + NCH * CHK;              // [TB][TOK] | [NCH][CHK] | [TB][cols] (v)
+    float* outs = sm + 2 * BUF;                                     // [2][TB][cols]
     const int b = blockIdx.z, h = blockIdx.y, j0 = blockIdx.x * cols;
     const int slot = a.seq_slot[b];
     if (slot < 0) return;
     const int t_begin = a.cu_q[b], t_end = a.cu_q[b + 1];
     if (t_end <= t_begin) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane & 15, half = lane >> 4;
-    const int jl = warp * WCOLS + half * 2;
-    float S[2][R4][4];
+    const int jl = (warp & (CH_WARPS - 1)) * WCOLS + half * 2;
+    const int nv = min(cols, a.vdim - j0);
+    const int batches = (t_end - t_begin + TB - 1) / TB;
     float* st = a.state + ((size_t)slot * a.heads + h) * a.vdim * a.dim;
+    for (int i = threadIdx.x; i < 2 * BUF; i += blockDim.x) sm[i] = 0.f;            // columns beyond vdim stay zero
+    __syncthreads();
+    pdl_wait();
+
+    if (warp == CH_WARPS) {
+        auto stage = [&](int it) {
+            const int t0 = t_begin + it * TB, nb = min(TB, t_end - t0), nc = (nb + CH_T - 1) / CH_T;
+            float* base = sm + (it & 1) * BUF;
+            const float* vec = a.vecs + ((size_t)h * a.T + t0) * TOK;
+            for (int i = lane; i < nb * (TOK / 4); i += 32) cp_async16(base + 4 * i, vec + 4 * i);
+            const float* fst = a.firsts + ((size_t)h * a.n_chunks + t_begin / CH_T + b + it * NCH) * CHK;
+            for (int i = lane; i < nc * (CHK / 4); i += 32) cp_async16(base + TB * TOK + 4 * i, fst + 4 * i);
+            float* vs = base + TB * TOK + NCH * CHK;
+            const float* src = a.u + (size_t)t0 * a.ld_u + a.uv + (size_t)h * a.vdim + j0;
+            if (a.vec) {
+                for (int i = lane; i < nb * (cols / 4); i += 32) {
+                    const int tt = i / (cols / 4), x = 4 * (i % (cols / 4));
+                    if (x < nv) cp_async16(vs + tt * cols + x, src + (size_t)tt * a.ld_u + x);
+                }
+            } else {
+                for (int i = lane; i < nb * cols; i += 32) {
+                    const int tt = i / cols, x = i % cols;
+                    if (x < nv) cp_async4(vs + tt * cols + x, src + (size_t)tt * a.ld_u + x);
+                }
+            }
+            // a last chunk's missing tokens: nothing is added, nothing read
+            for (int i = nb * TOK + lane; i < nc * CH_T * TOK; i += 32) base[i] = 0.f;
+            for (int i = nb * cols + lane; i < nc * CH_T * cols; i += 32) vs[i] = 0.f;
+            asm volatile("cp.async.commit_group;" ::: "memory");
+        };
+        auto take = [&](int it) {
+            const int t0 = t_begin + it * TB, nb = min(TB, t_end - t0);
+            const float* src = outs + (it & 1) * TB * cols;
+            float* dst = a.out + (size_t)t0 * a.ld_out + (size_t)h * a.vdim + j0;
+            for (int i = lane; i < nb * cols; i += 32) {
+                const int tt = i / cols, x = i % cols;
+                if (x < nv) dst[(size_t)tt * a.ld_out + x] = src[i];
+            }
+        };
+        stage(0);
+        for (int it = 0; it < batches; ++it) {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+            __syncthreads();                            // batch `it` is there; the warps of columns are done with the one before
+            if (it + 1 < batches) stage(it + 1);
+            if (it > 0) take(it - 1);
+        }
+        __syncthreads();
+        take(batches - 1);
+        return;
+    }
+
+    uint64_t S[2][R4][2];                               // rows in pairs
 #pragma unroll
     for (int c = 0; c < 2; ++c)
 #pragma unroll
-        for (int r = 0; r < R4; ++r)
+        for (int r = 0; r < R4; ++r) {
+            float x[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int i = (r * RL + l) * 4 + e, j = j0 + jl + c;
-                S[c][r][e] = i < a.dim && j < a.vdim ? st[(size_t)j * a.dim + i] : 0.f;
+                x[e] = i < a.dim && j < a.vdim ? st[(size_t)j * a.dim + i] : 0.f;
             }
-    const int nv = min(cols, a.vdim - j0);
-    for (int i = threadIdx.x; i < 2 * buf_floats; i += blockDim.x) sm[i] = 0.f;      // columns beyond vdim stay zero
-    __syncthreads();
-    pdl_wait();
-    auto stage = [&](int t0, int buf) {
-        const int nb = min(TB, t_end - t0);
-        float* base = sm + buf * buf_floats;
-        constexpr int V4 = 3 * DP / 4;
-        for (int i = threadIdx.x; i < nb * V4; i += blockDim.x) {
-            const int tt = i / V4, x = i - tt * V4;
-            cp_async16(base + tt * tok + 4 * x, a.vecs + ((size_t)(t0 + tt) * a.heads + h) * 3 * DP + 4 * x);
+            S[c][r][0] = pack2(x[0], x[1]);
+            S[c][r][1] = pack2(x[2], x[3]);
         }
-        const int v4 = a.vec ? nv >> 2 : nv;
-        for (int i = threadIdx.x; i < nb * v4; i += blockDim.x) {
-            const int tt = i / v4, x = i - tt * v4;
-            const float* src = a.u + (size_t)(t0 + tt) * a.ld_u + a.uv + (size_t)h * a.vdim + j0;
-            if (a.vec) cp_async16(base + tt * tok + 3 * DP + 4 * x, src + 4 * x);
-            else cp_async4(base + tt * tok + 3 * DP + x, src + x);
-        }
-        const int nc = (nb + CH_T - 1) / CH_T;
-        constexpr int C4 = (DP + CH_SCAL) / 4;
-        for (int i = threadIdx.x; i < nc * C4; i += blockDim.x) {
-            const int cc = i / C4, x = i - cc * C4;
-            const size_t at = (size_t)(t0 + cc * CH_T) * a.heads + h;
-            cp_async16(base + TB * tok + cc * chk + 4 * x, x < DP / 4 ? a.decay + at * DP + 4 * x : a.numbers + at * CH_SCAL + 4 * (x - DP / 4));
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    stage(t_begin, 0);
-    int buf = 0;
-    for (int t0 = t_begin; t0 < t_end; t0 += TB, buf ^= 1) {
-        const int nb = min(TB, t_end - t0), nc = (nb + CH_T - 1) / CH_T;
-        if (t0 + TB < t_end) {
-            stage(t0 + TB, buf ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        float* base = sm + buf * buf_floats;
-        for (int i = nb * tok + threadIdx.x; i < nc * CH_T * tok; i += blockDim.x) base[i] = 0.f;    // a last chunk's missing tokens
+    for (int it = 0; it < batches; ++it) {
+        const int nc = (min(TB, t_end - t_begin - it * TB) + CH_T - 1) / CH_T;
+        const float* base = sm + (it & 1) * BUF;
+        const float* vs = base + TB * TOK + NCH * CHK;
+        float* res = outs + (it & 1) * TB * cols;
         __syncthreads();
         for (int cc = 0; cc < nc; ++cc) {
-            const float* x = base + cc * CH_T * tok;
-            const float* dec = base + TB * tok + cc * chk;
+            const float* x = base + cc * CH_T * TOK;
+            const float* dec = base + TB * TOK + cc * CHK;
             const float* num = dec + DP;
             float y[16];                 // [k | q][column][token]
 #pragma unroll
-            for (int i = 0; i < 16; ++i) y[i] = 0.f;
+            for (int t = 0; t < 4; ++t) {
+                uint64_t yk0 = 0, yk1 = 0, yq0 = 0, yq1 = 0;
 #pragma unroll
-            for (int r = 0; r < R4; ++r) {
-                const int i = (r * RL + l) * 4;
+                for (int r = 0; r < R4; ++r) {
+                    uint64_t q[2], k[2];
+                    load22(x + t * TOK + (r * RL + l) * 4, q);
+                    load22(x + t * TOK + DP + (r * RL + l) * 4, k);
 #pragma unroll
-                for (int t = 0; t < 4; ++t) {
-                    float q[4], k[4];
-                    load4(x + t * tok + i, q);
-                    load4(x + t * tok + DP + i, k);
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        y[t] = fmaf(k[e], S[0][r][e], y[t]);
-                        y[4 + t] = fmaf(k[e], S[1][r][e], y[4 + t]);
-                        y[8 + t] = fmaf(q[e], S[0][r][e], y[8 + t]);
-                        y[12 + t] = fmaf(q[e], S[1][r][e], y[12 + t]);
+                    for (int e = 0; e < 2; ++e) {
+                        yk0 = fma2(k[e], S[0][r][e], yk0);
+                        yk1 = fma2(k[e], S[1][r][e], yk1);
+                        yq0 = fma2(q[e], S[0][r][e], yq0);
+                        yq1 = fma2(q[e], S[1][r][e], yq1);
                     }
                 }
+                float lo, hi;
+                unpack2(yk0, lo, hi); y[t] = lo + hi;
+                unpack2(yk1, lo, hi); y[4 + t] = lo + hi;
+                unpack2(yq0, lo, hi); y[8 + t] = lo + hi;
+                unpack2(yq1, lo, hi); y[12 + t] = lo + hi;
             }
+            // what the corrections need is asked for before the sums are exchanged
+            float tri[4][4], beta[4], v[2][4], d[4];
+            load4(num + 32, beta);
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                load4(num + 4 * t, tri[t]);
+                const float2 vv = *reinterpret_cast<const float2*>(vs + (cc * CH_T + t) * cols + jl);
+                v[0][t] = vv.x;
+                v[1][t] = vv.y;
+            }
+            load4(num + 16 + (l & 3) * 4, d);
             // sixteen sums over sixteen lanes: lane l ends with the l-th
 #pragma unroll
             for (int m = 8; m >= 1; m >>= 1) {
@@ -601,70 +780,73 @@ delta_scan_chunks_kernel(const ChunkArgs a) {
             }
             float w[2][4];
 #pragma unroll
-            for (int t = 0; t < 4; ++t) {
-                const float beta = num[32 + t];
+            for (int c = 0; c < 2; ++c)
 #pragma unroll
-                for (int c = 0; c < 2; ++c) {
-                    float at = __shfl_sync(0xffffffffu, y[0], (lane & 16) | (c * 4 + t));
-#pragma unroll
-                    for (int s = 0; s < t; ++s) at = fmaf(num[t * 4 + s], w[c][s], at);
-                    w[c][t] = beta * (x[t * tok + 3 * DP + jl + c] - at);
-                }
-            }
-            if (l >= 8) {
-                const int t = l & 3, c = (l >> 2) & 1;
-                float d[4];
-                load4(num + 16 + t * 4, d);
-                float o = y[0];
-#pragma unroll
-                for (int s = 0; s < 4; ++s) o = fmaf(d[s], c ? w[1][s] : w[0][s], o);
-                outs[(cc * CH_T + t) * cols + jl + c] = o;
-            }
+                for (int t = 0; t < 4; ++t) w[c][t] = __shfl_sync(0xffffffffu, y[0], (lane & 16) | (c * 4 + t));
 #pragma unroll
             for (int r = 0; r < R4; ++r) {
-                const int i = (r * RL + l) * 4;
-                float f[4];
-                load4(dec + i, f);
+                uint64_t f[2];
+                load22(dec + (r * RL + l) * 4, f);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) { S[0][r][e] *= f[e]; S[1][r][e] *= f[e]; }
+                for (int e = 0; e < 2; ++e) { S[0][r][e] = mul2(S[0][r][e], f[e]); S[1][r][e] = mul2(S[1][r][e], f[e]); }
+            }
 #pragma unroll
-                for (int t = 0; t < 4; ++t) {
-                    float k[4];
-                    load4(x + t * tok + 2 * DP + i, k);
+            for (int t = 0; t < 4; ++t)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        S[0][r][e] = fmaf(k[e], w[0][t], S[0][r][e]);
-                        S[1][r][e] = fmaf(k[e], w[1][t], S[1][r][e]);
+                for (int c = 0; c < 2; ++c) {
+                    float at = w[c][t];
+#pragma unroll
+                    for (int s = 0; s < t; ++s) at = fmaf(tri[t][s], w[c][s], at);
+                    w[c][t] = beta[t] * (v[c][t] - at);
+                }
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const uint64_t w0 = pack2(w[0][t], w[0][t]), w1 = pack2(w[1][t], w[1][t]);
+#pragma unroll
+                for (int r = 0; r < R4; ++r) {
+                    uint64_t ks[2];
+                    load22(x + t * TOK + 2 * DP + (r * RL + l) * 4, ks);
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        S[0][r][e] = fma2(ks[e], w0, S[0][r][e]);
+                        S[1][r][e] = fma2(ks[e], w1, S[1][r][e]);
                     }
                 }
             }
-        }
-        __syncthreads();
-        for (int i = threadIdx.x; i < nb * cols; i += blockDim.x) {
-            const int tt = i / cols, j = i - tt * cols;
-            if (j < nv) a.out[(size_t)(t0 + tt) * a.ld_out + (size_t)h * a.vdim + j0 + j] = outs[i];
+            if (l >= 8) {
+                const int c = (l >> 2) & 1;
+                float o = y[0];
+#pragma unroll
+                for (int s = 0; s < 4; ++s) o = fmaf(d[s], c ? w[1][s] : w[0][s], o);
+                res[(cc * CH_T + (l & 3)) * cols + jl + c] = o;
+            }
         }
     }
+    __syncthreads();
 #pragma unroll
     for (int c = 0; c < 2; ++c)
 #pragma unroll
-        for (int r = 0; r < R4; ++r)
+        for (int r = 0; r < R4; ++r) {
+            float x[4];
+            unpack2(S[c][r][0], x[0], x[1]);
+            unpack2(S[c][r][1], x[2], x[3]);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int i = (r * RL + l) * 4 + e, j = j0 + jl + c;
-                if (i < a.dim && j < a.vdim) st[(size_t)j * a.dim + i] = S[c][r][e];
+                if (i < a.dim && j < a.vdim) st[(size_t)j * a.dim + i] = x[e];
             }
+        }
 }
 
 template <int R4, int TB>
 int launch_chunks(const ChunkArgs& a, int n_seqs, cudaStream_t s) {
-    const int warps = scan_warps(n_seqs, a.heads, a.vdim), cols = warps * WCOLS;
-    const size_t smem = ((size_t)2 * (TB * (3 * 64 * R4 + cols) + TB / CH_T * (64 * R4 + CH_SCAL)) + (size_t)TB * cols) * sizeof(float);
+    const int cols = CH_WARPS * WCOLS;
+    const size_t smem = ((size_t)2 * (TB * (3 * 64 * R4 + cols) + TB / CH_T * (64 * R4 + CH_SCAL)) + (size_t)2 * TB * cols) * sizeof(float);
     if (smem > 200 * 1024) return RB_ERR_BAD_SIZE;
     auto k = delta_scan_chunks_kernel<R4, TB>;
     cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    RB_LAUNCH((k), dim3((a.vdim + cols - 1) / cols, a.heads, n_seqs), dim3(warps * 32), smem, s, a);
+    RB_LAUNCH((k), dim3((a.vdim + cols - 1) / cols, a.heads, n_seqs), dim3((CH_WARPS + 1) * 32), smem, s, a);
     RB_LAUNCH_CHECK();
     return RB_OK;
 }
@@ -743,9 +925,13 @@ extern "C" int rb_delta_prep(const void* in, int in_dtype, int n_in, long long i
                                        ((uintptr_t)dt_bias & 15) == 0));
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
+    const bool rows = vec && n_in == 1 && z_n_in == 1 && max_q_len > 1 && taps <= 4 && dim <= 128 && vdim <= 128;
 #define RB_DP(IT, ZT)                                                                                          \
     do {                                                                                                       \
-        if (vec) RB_LAUNCH((delta_prep_kernel<IT, ZT, 4>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a); \
+        if (rows && taps == 4) RB_LAUNCH((delta_prep_rows_kernel<IT, ZT, 4>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a);      \
+        else if (rows && taps == 3) RB_LAUNCH((delta_prep_rows_kernel<IT, ZT, 3>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a); \
+        else if (rows && taps == 2) RB_LAUNCH((delta_prep_rows_kernel<IT, ZT, 2>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a); \
+        else if (vec) RB_LAUNCH((delta_prep_kernel<IT, ZT, 4>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a); \
         else RB_LAUNCH((delta_prep_kernel<IT, ZT, 1>), grid, block, 0, s, (const IT*)in, (const ZT*)z, a);     \
     } while (0)
     if (in_dtype == RB_F32 && z_dtype == RB_F32) RB_DP(float, float);
@@ -800,25 +986,28 @@ extern "C" int rb_low_rank(const void* in, int in_dtype, int n_in, long long in_
     return RB_OK;
 }
 
-// The same for prompts, four tokens at a time: vecs float32 [T][heads][3][dimp], decay float32 [T][heads][dimp], numbers float32
-// [T][heads][36] are work space, dimp = dim rounded up to 64 (128, 256).  RB_ERR_BAD_SIZE for dim > 256.
+// The same for prompts, four tokens at a time: vecs float32 [heads][T][3][dimp] and firsts float32 [heads][n_chunks][dimp + 36] are
+// work space, n_chunks >= T / 4 + n_seqs, dimp = dim rounded up to 64 (128, 256).  RB_ERR_BAD_SIZE for dim > 256.
 extern "C" int rb_delta_scan_chunks(const float* u, int ld_u, int uq, int uk, int uv, int ug, int ub, int ud, int heads, int kv_heads,
                                     int dim, int vdim, int per_channel, float* state, const int* seq_slot, const int* cu_q, int n_seqs,
-                                    int max_q_len, float* vecs, float* decay, float* numbers, int dimp, float* out, int ld_out,
+                                    int max_q_len, int T, float* vecs, float* firsts, int n_chunks, int dimp, float* out, int ld_out,
                                     void* stream) {
     (void)ud;
     if (n_seqs <= 0 || max_q_len <= 0) return RB_OK;
     if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 || n_seqs > 65535 || heads > 65535 || dim > dimp ||
         (dimp != 64 && dimp != 128 && dimp != 256))
         return RB_ERR_BAD_SIZE;
-    if (((uintptr_t)vecs | (uintptr_t)decay | (uintptr_t)numbers) & 15) return RB_ERR_BAD_ALIGN;
+    if (T <= 0 || n_chunks < T / CH_T + n_seqs) return RB_ERR_BAD_SIZE;
+    if (((uintptr_t)vecs | (uintptr_t)firsts) & 15) return RB_ERR_BAD_ALIGN;
     cudaStream_t s = (cudaStream_t)stream;
     RB_LAUNCH((delta_chunk_kernel), dim3((max_q_len + 4 * CH_T - 1) / (4 * CH_T), heads, n_seqs), dim3(128), 0, s, u, ld_u, uq, uk, ug, ub,
-              heads, kv_heads, dim, dimp, per_channel, seq_slot, cu_q, vecs, decay, numbers);
+              heads, kv_heads, dim, dimp, per_channel, seq_slot, cu_q, T, n_chunks, vecs, firsts);
     RB_LAUNCH_CHECK();
-    ChunkArgs a{u, vecs, decay, numbers, ld_u, uv, heads, dim, vdim, dimp, state, seq_slot, cu_q, out, ld_out, 0};
+    ChunkArgs a{u, vecs, firsts, T, n_chunks, ld_u, uv, heads, dim, vdim, dimp, state, seq_slot, cu_q, out, ld_out, 0};
     a.vec = ((vdim | ld_u | uv) & 3) == 0 && ((uintptr_t)u & 15) == 0;
-    if (dimp == 64) return launch_chunks<1, 16>(a, n_seqs, s);
-    if (dimp == 128) return launch_chunks<2, 16>(a, n_seqs, s);
+    // more blocks than three a multiprocessor: a shorter batch of tokens, so that four fit
+    const bool many = (long long)n_seqs * heads * ((vdim + 15) / 16) > 3 * 148;
+    if (dimp == 64) return many ? launch_chunks<1, 8>(a, n_seqs, s) : launch_chunks<1, 16>(a, n_seqs, s);
+    if (dimp == 128) return many ? launch_chunks<2, 8>(a, n_seqs, s) : launch_chunks<2, 16>(a, n_seqs, s);
     return launch_chunks<4, 8>(a, n_seqs, s);
 }

@@ -200,7 +200,7 @@ def _lib():
         lib.rb_delta_prep.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _ll, _i, _vp,
                                       _vp, _i, _f, _f, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]
         lib.rb_delta_scan.argtypes = [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp]
-        lib.rb_delta_scan_chunks.argtypes = [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _vp, _i,
+        lib.rb_delta_scan_chunks.argtypes = [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _i, _i,
                                              _vp, _i, _vp]
         lib.rb_low_rank.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _vp, _i, _i, _i, _vp, _i, _i, _i, _vp, _i, _vp]
         lib.rb_gemm_tcgen05_set_wait.argtypes = [_ll, _i]
@@ -1874,9 +1874,9 @@ def delta_padded_dim(dim: int) -> Optional[int]:
 @_profiled(lambda a, facts: _cost.delta_scan(a["n_tokens"], a["n_seqs"], a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["per_channel"]))
 def delta_scan_chunks(u: torch.Tensor, n_tokens: int, rows: DeltaRows, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool,
                       state: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, n_seqs: int, max_q_len: int, out: torch.Tensor,
-                      vecs: torch.Tensor, decay: torch.Tensor, numbers: torch.Tensor):
+                      vecs: torch.Tensor, firsts: torch.Tensor):
     """``delta_scan`` for prompts, four tokens at a time (results differ by rounding only).  Work space, float32: ``vecs``
-    [T, heads, 3, dimp], ``decay`` [T, heads, dimp], ``numbers`` [T, heads, 36] with dimp = ``delta_padded_dim``."""
+    [heads, T, 3, dimp] and ``firsts`` [heads, T // 4 + n_seqs, dimp + 36] with dimp = ``delta_padded_dim``."""
     dimp = delta_padded_dim(dim)
     if dimp is None or u.dtype != torch.float32 or u.stride(-1) != 1 or u.shape[-1] < rows.width or u.shape[0] < n_tokens:
         raise KernelError("delta_scan_chunks: u must be float32 [T, rows.width], heads of at most 256")
@@ -1884,12 +1884,13 @@ def delta_scan_chunks(u: torch.Tensor, n_tokens: int, rows: DeltaRows, heads: in
         raise KernelError("delta_scan_chunks: state must be contiguous float32 [slots, heads, vdim, dim]")
     if out.dtype != torch.float32 or out.stride(-1) != 1 or out.shape[-1] != heads * vdim or out.shape[0] < n_tokens:
         raise KernelError("delta_scan_chunks: out must be float32 [T, heads * vdim]")
-    for t, n in ((vecs, heads * 3 * dimp), (decay, heads * dimp), (numbers, heads * DELTA_CHUNK_NUMBERS)):
-        if t.dtype != torch.float32 or not t.is_contiguous() or t.numel() < n_tokens * n:
+    chunks = n_tokens // 4 + n_seqs
+    for t, shape in ((vecs, (heads, n_tokens, 3, dimp)), (firsts, (heads, chunks, dimp + DELTA_CHUNK_NUMBERS))):
+        if t.dtype != torch.float32 or not t.is_contiguous() or tuple(t.shape) != shape:
             raise KernelError("delta_scan_chunks: the work space is too small")
     rc = _lib().rb_delta_scan_chunks(_ptr(u), u.stride(0), *rows.offsets, heads, kv_heads, dim, vdim, 1 if per_channel else 0, _ptr(state),
-                                     _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, max_q_len, _ptr(vecs), _ptr(decay),
-                                     _ptr(numbers), dimp, _ptr(out), out.stride(0), _stream())
+                                     _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, max_q_len, n_tokens, _ptr(vecs),
+                                     _ptr(firsts), chunks, dimp, _ptr(out), out.stride(0), _stream())
     _check(rc, "delta_scan_chunks")
 
 

@@ -215,9 +215,9 @@ class GatedDelta(Mixer):
             sizes = (self.rows, self.heads, self.kv, self.hd, self.vd, self.per_channel, view.state, batch.seq_slot, batch.cu_q, batch.n_seqs)
             dimp = kernels.delta_padded_dim(self.hd)
             if batch.max_q_len > CHUNKS_MIN_TOKENS and dimp is not None:
-                vecs, decay, numbers = (torch.empty((T, self.heads, w), dtype=torch.float32, device=dev)
-                                        for w in (3 * dimp, dimp, kernels.DELTA_CHUNK_NUMBERS))
-                kernels.delta_scan_chunks(u, T, *sizes, batch.max_q_len, o, vecs, decay, numbers)
+                vecs = torch.empty((self.heads, T, 3, dimp), dtype=torch.float32, device=dev)
+                firsts = torch.empty((self.heads, T // 4 + batch.n_seqs, dimp + kernels.DELTA_CHUNK_NUMBERS), dtype=torch.float32, device=dev)
+                kernels.delta_scan_chunks(u, T, *sizes, batch.max_q_len, o, vecs, firsts)
             else:
                 kernels.delta_scan(u, T, *sizes, o)
         if gate_inner is not None and self.narrow_gate:

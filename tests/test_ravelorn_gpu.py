@@ -201,7 +201,8 @@ def test_gated_delta_rule(sizes, per_channel, chunks):
         out = torch.full((T, inner), float("nan"), device=DEV)
         if chunks and max(lens) > 1:
             dimp = kernels.delta_padded_dim(dim)
-            work = [torch.full((T, heads, n), float("nan"), device=DEV) for n in (3 * dimp, dimp, kernels.DELTA_CHUNK_NUMBERS)]
+            work = [torch.full(shape, float("nan"), device=DEV)
+                    for shape in ((heads, T, 3, dimp), (heads, T // 4 + 3, dimp + kernels.DELTA_CHUNK_NUMBERS))]
             kernels.delta_scan_chunks(u, T, layout, heads, kv, dim, vdim, per_channel, state, seq, cu, 3, max(lens), out, *work)
         else:
             kernels.delta_scan(u, T, layout, heads, kv, dim, vdim, per_channel, state, seq, cu, 3, out)
