@@ -71,6 +71,11 @@ int rb_moe_route(const float* z, int ldz, const void* bias, int bias_dtype, cons
 int rb_moe_plan(const int* counts, int E, int tile_rows, int max_tiles, int* starts, int* tile_group, void* stream);
 int rb_moe_gather(const void* x, int dtype, int H, const int* ids, const int* place, const int* starts, int T, int top,
                   void* rows, int* row_of, void* stream);
+// The three in one launch for at most 16 tokens and 256 choices.
+int rb_moe_route_few(const float* z, int ldz, const float* bias, const int* slot_of_token, int T, int E, int top, int n_groups,
+                     int keep_groups, int renormalize, float norm_eps, int score, int identity, int tile_rows, int max_tiles,
+                     const void* x, int dtype, int H, void* rows, int* row_of, float* weights, float* self_weight, int* tile_group,
+                     void* stream);
 // extra (optional): [n_extra][T, H] partial sums added to every token's row, times sigmoid(extra_gate[t * ld]) when
 // extra_gate is given; self_weight (optional): plus self_weight[t] * self_x[t].
 int rb_moe_combine(const float* y, long long ldy, const int* row_of, const float* weights, int T, int top, float* out,

@@ -14,6 +14,7 @@
 //   plan     one block: every expert's rows start at a multiple of `tile_rows`; tile i of the row buffer
 //            belongs to expert tile_group[i] (-1: unused).
 //   gather   a token's normalised row is copied to each of its `top` places; row_of[t, j] names the place.
+//   route_few  route, plan and gather in one launch for a decode step's few tokens.
 //   combine  out[t] = sum_j weight[t, j] * y[row_of[t, j]] in 32-bit, j ascending; optionally plus
 //            sigmoid(extra_gate[t]) * (sum of the partial sums extra[s][t]): an expert that every token uses; and plus
 //            self_weight[t] * self_x[t]: what the identity experts give.
@@ -125,29 +126,17 @@ int launch_router(const void* x, long long ldx, const float* w, float* z, int ld
     return RB_OK;
 }
 
-template <typename BT>
-__global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bias, const int* __restrict__ slot_of_token,
-                 int T, int E, int top, int* __restrict__ ids, float* __restrict__ weights, int* __restrict__ place,
-                 int* __restrict__ counts, int n_groups, int keep_groups, int renormalize, float norm_eps, int score, int identity,
-                 float* __restrict__ self_weight) {
-    pdl_trigger();
-    pdl_wait();
-    extern __shared__ float route_s[];           // [warps][E + n_groups] when groups are cut, else unused
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    const int lane = threadIdx.x & 31;
-    if (t >= T) return;
-    if (slot_of_token[t] < 0) {
-        for (int j = lane; j < top; j += 32) { ids[(size_t)t * top + j] = -1; weights[(size_t)t * top + j] = 0.f; place[(size_t)t * top + j] = 0; }
-        if (lane == 0 && self_weight) self_weight[t] = 0.f;
-        return;
-    }
+// One warp scores one token's experts (z: its row of logits) and names the `top` it chooses, in order: pick(j, expert, score).
+// cs: E + n_groups floats of the warp's own when groups are cut.  Returns the chosen scores' sum.
+template <typename BT, typename F>
+__device__ __forceinline__ float choose_experts(const float* z, const BT* bias, int E, int top, int n_groups, int keep_groups, int score,
+                                                float* cs, int lane, F pick) {
     float s[MAX_EPL], c[MAX_EPL];
     float top_z = -INFINITY;
 #pragma unroll
     for (int i = 0; i < MAX_EPL; ++i) {
         const int e = lane + i * 32;
-        s[i] = e < E ? z[(size_t)t * ldz + e] : -INFINITY;
+        s[i] = e < E ? z[e] : -INFINITY;
         top_z = fmaxf(top_z, s[i]);
     }
     if (score == 1) {          // softmax over all of them
@@ -172,8 +161,7 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bi
     }
     if (n_groups > 1 && keep_groups < n_groups) {
         // the groups' cut: scores to shared memory, a lane scores whole groups, the best groups are marked
-        float* cs = route_s + (size_t)(threadIdx.x >> 5) * (E + n_groups);
-        float* gs = cs + E;
+            float* gs = cs + E;
         const int per = E / n_groups;
 #pragma unroll
         for (int i = 0; i < MAX_EPL; ++i)
@@ -209,8 +197,7 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bi
             if (e < E && gs[e / per] != -INFINITY) c[i] = -INFINITY;       // its group was not kept
         }
     }
-    float picked_sum = 0.f, self_sum = 0.f;
-    const int real = E - identity;           // the experts that have rows
+    float picked_sum = 0.f;
     for (int j = 0; j < top; ++j) {
         float best = -INFINITY, best_s = 0.f;
         int best_e = 0x7fffffff;
@@ -231,19 +218,136 @@ moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bi
             if (lane + i * 32 == best_e) c[i] = -INFINITY;
         if (best_e >= E) best_e = E - 1;      // scores that compare with nothing (NaN): stay inside the tables
         picked_sum += best_s;
-        if (best_e >= real) self_sum += best_s;
-        if (lane == 0) {
-            ids[(size_t)t * top + j] = best_e < real ? best_e : -1;
-            weights[(size_t)t * top + j] = best_s;
-            place[(size_t)t * top + j] = best_e < real ? atomicAdd(&counts[best_e], 1) : 0;
-        }
+        pick(j, best_e, best_s);
     }
+    return picked_sum;
+}
+
+template <typename BT>
+__global__ void __launch_bounds__(128)
+moe_route_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bias, const int* __restrict__ slot_of_token,
+                 int T, int E, int top, int* __restrict__ ids, float* __restrict__ weights, int* __restrict__ place,
+                 int* __restrict__ counts, int n_groups, int keep_groups, int renormalize, float norm_eps, int score, int identity,
+                 float* __restrict__ self_weight) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ float route_s[];           // [warps][E + n_groups] when groups are cut, else unused
+    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (t >= T) return;
+    if (slot_of_token[t] < 0) {
+        for (int j = lane; j < top; j += 32) { ids[(size_t)t * top + j] = -1; weights[(size_t)t * top + j] = 0.f; place[(size_t)t * top + j] = 0; }
+        if (lane == 0 && self_weight) self_weight[t] = 0.f;
+        return;
+    }
+    float self_sum = 0.f;
+    const int real = E - identity;           // the experts that have rows
+    const float picked_sum = choose_experts(
+        z + (size_t)t * ldz, bias, E, top, n_groups, keep_groups, score, route_s + (size_t)(threadIdx.x >> 5) * (E + n_groups), lane,
+        [&](int j, int e, float s) {
+            if (e >= real) self_sum += s;
+            if (lane == 0) {
+                ids[(size_t)t * top + j] = e < real ? e : -1;
+                weights[(size_t)t * top + j] = s;
+                place[(size_t)t * top + j] = e < real ? atomicAdd(&counts[e], 1) : 0;
+            }
+        });
     if (renormalize && lane == 0) {
         const float d = picked_sum + norm_eps;
         for (int j = 0; j < top; ++j) weights[(size_t)t * top + j] /= d;
         self_sum /= d;
     }
     if (self_weight && lane == 0) self_weight[t] = self_sum;
+}
+
+// route, plan and gather in one launch for few tokens: a block a (token, choice).  Every block chooses for all tokens (a warp a token
+// at a time; a few dozen scores), so that it knows every choice without asking another block; its row's place is the number
+// of earlier choices of the same expert, the expert's first row follows from the counts.  Block 0 writes what all share.
+constexpr int FEW_TOKENS = 16, FEW_CHOICES = 256;
+
+template <typename BT, typename AT>
+__global__ void __launch_bounds__(256)
+moe_route_few_kernel(const float* __restrict__ z, int ldz, const BT* __restrict__ bias, const int* __restrict__ slot_of_token, int T, int E,
+                     int top, int n_groups, int keep_groups, int renormalize, float norm_eps, int score, int identity, int tile_rows,
+                     int max_tiles, const AT* __restrict__ x, int H, AT* __restrict__ rows, int* __restrict__ row_of,
+                     float* __restrict__ weights, float* __restrict__ self_weight, int* __restrict__ tile_group) {
+    pdl_wait();
+    extern __shared__ float few_s[];             // [8][E + n_groups] when groups are cut
+    __shared__ int s_ids[FEW_CHOICES], s_first[512 + 1];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, me = blockIdx.x, real = E - identity;
+    for (int t = warp; t < T; t += 8) {
+        if (slot_of_token[t] < 0) {
+            for (int j = lane; j < top; j += 32) {
+                s_ids[t * top + j] = -1;
+                if (me == 0) { row_of[t * top + j] = -1; weights[t * top + j] = 0.f; }
+            }
+            if (me == 0 && lane == 0 && self_weight) self_weight[t] = 0.f;
+            continue;
+        }
+        float own = 0.f;
+        const float sum = choose_experts(z + (size_t)t * ldz, bias, E, top, n_groups, keep_groups, score,
+                                         few_s + (size_t)warp * (E + n_groups), lane, [&](int j, int e, float s) {
+            if (e >= real) own += s;
+            if (lane == 0) {
+                s_ids[t * top + j] = e < real ? e : -1;
+                if (me == 0) weights[t * top + j] = s;
+            }
+        });
+        if (me == 0 && lane == 0) {
+            const float d = renormalize ? sum + norm_eps : 1.f;
+            if (renormalize)
+                for (int j = 0; j < top; ++j) weights[t * top + j] /= d;
+            if (self_weight) self_weight[t] = renormalize ? own / d : own;
+        }
+    }
+    __syncthreads();
+    const int n = T * top;
+    for (int e = threadIdx.x; e < real; e += 256) {
+        int count = 0;
+        for (int i = 0; i < n; ++i) count += s_ids[i] == e;
+        s_first[e + 1] = (count + tile_rows - 1) / tile_rows;        // the expert's tiles
+    }
+    __syncthreads();
+    if (warp == 0) {                             // where every expert's tiles start: a warp's running sum, 32 experts at a time
+        int base = 0;
+        for (int e0 = 0; e0 < real; e0 += 32) {
+            int v = e0 + lane < real ? s_first[e0 + lane + 1] : 0;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, v, o);
+                if (lane >= o) v += up;
+            }
+            __syncwarp();
+            if (e0 + lane < real) s_first[e0 + lane + 1] = base + v;
+            base += __shfl_sync(0xffffffffu, v, 31);
+        }
+        if (lane == 0) s_first[0] = 0;
+    }
+    __syncthreads();
+    if (me == 0) {
+        for (int i = threadIdx.x; i < max_tiles; i += 256)
+            if (i >= s_first[real]) tile_group[i] = -1;
+        for (int e = threadIdx.x; e < real; e += 256)
+            for (int i = s_first[e]; i < s_first[e + 1] && i < max_tiles; ++i) tile_group[i] = e;
+    }
+    const int e = s_ids[me];
+    if (e < 0) {
+        if (threadIdx.x == 0) row_of[me] = -1;
+        return;
+    }
+    int place = 0;
+    for (int i = lane; i < me; i += 32) place += s_ids[i] == e;
+    place = __reduce_add_sync(0xffffffffu, place);
+    const int dst_row = s_first[e] * tile_rows + place;
+    if (threadIdx.x == 0) row_of[me] = dst_row;
+    const AT* src = x + (size_t)(me / top) * H;
+    AT* dst = rows + (size_t)dst_row * H;
+    if ((H * sizeof(AT)) % 16 == 0 && (((uintptr_t)x | (uintptr_t)rows) & 15) == 0) {
+        const int n16 = (int)(H * sizeof(AT) / 16);
+        for (int i = threadIdx.x; i < n16; i += 256) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+    } else {
+        for (int i = threadIdx.x; i < H; i += 256) dst[i] = src[i];
+    }
 }
 
 __global__ void __launch_bounds__(256)
@@ -401,6 +505,34 @@ extern "C" int rb_moe_combine(const float* y, long long ldy, const int* row_of, 
     else if (self_dtype == RB_BF16)
         RB_LAUNCH((moe_combine_kernel<__nv_bfloat16>), dim3(T), dim3(256), 0, (cudaStream_t)stream, y, ldy, row_of, weights, top,
                   out, H, extra, n_extra, extra_stride, extra_gate, extra_gate_ld, self_weight, (const __nv_bfloat16*)self_x);
+    else
+        return RB_ERR_BAD_DTYPE;
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+// moe_route, moe_plan and moe_gather in one launch for at most 16 tokens and 256 choices (RB_ERR_BAD_SIZE beyond).
+extern "C" int rb_moe_route_few(const float* z, int ldz, const float* bias, const int* slot_of_token, int T, int E, int top, int n_groups,
+                                int keep_groups, int renormalize, float norm_eps, int score, int identity, int tile_rows, int max_tiles,
+                                const void* x, int dtype, int H, void* rows, int* row_of, float* weights, float* self_weight,
+                                int* tile_group, void* stream) {
+    if (T <= 0) return RB_OK;
+    if (E <= 0 || E > 32 * MAX_EPL || top <= 0 || top > E || T > FEW_TOKENS || T * top > FEW_CHOICES || tile_rows <= 0 || max_tiles <= 0)
+        return RB_ERR_BAD_SIZE;
+    if (identity < 0 || identity >= E || (identity > 0 && !self_weight) || score < 0 || score > 1) return RB_ERR_BAD_SIZE;
+    if (n_groups < 1) n_groups = 1;
+    if (keep_groups < 1 || keep_groups > n_groups) keep_groups = n_groups;
+    if (E % n_groups || (long long)keep_groups * (E / n_groups) < top) return RB_ERR_BAD_SIZE;
+    const size_t smem = (n_groups > 1 && keep_groups < n_groups) ? (size_t)8 * (E + n_groups) * sizeof(float) : 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == RB_BF16)
+        RB_LAUNCH((moe_route_few_kernel<float, __nv_bfloat16>), dim3(T * top), dim3(256), smem, s, z, ldz, bias, slot_of_token, T, E, top,
+                  n_groups, keep_groups, renormalize, norm_eps, score, identity, tile_rows, max_tiles, (const __nv_bfloat16*)x, H,
+                  (__nv_bfloat16*)rows, row_of, weights, self_weight, tile_group);
+    else if (dtype == RB_F32)
+        RB_LAUNCH((moe_route_few_kernel<float, float>), dim3(T * top), dim3(256), smem, s, z, ldz, bias, slot_of_token, T, E, top, n_groups,
+                  keep_groups, renormalize, norm_eps, score, identity, tile_rows, max_tiles, (const float*)x, H, (float*)rows, row_of, weights,
+                  self_weight, tile_group);
     else
         return RB_ERR_BAD_DTYPE;
     RB_LAUNCH_CHECK();

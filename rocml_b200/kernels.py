@@ -194,6 +194,8 @@ def _lib():
         lib.rb_wide_norm_rope_cache.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _vp, _vp, _i, _i, _vp,
                                                 _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _vp]
         lib.rb_talk_mix.argtypes = [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp]
+        lib.rb_moe_route_few.argtypes = [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _vp,
+                                         _vp, _vp]
         lib.rb_softcap.argtypes = [_vp, _ll, _f, _f, _vp]
         lib.rb_add_layernorm.argtypes = [_vp, _vp, _i, _ll, _vp, _vp, _vp, _i, _vp, _i, _i, _f, _i, _vp]
         lib.rb_out_norm.argtypes = [_vp, _vp, _i, _ll, _f, _vp, _vp, _i, _vp, _vp, _i, _i, _vp, _vp, _f, _f, _vp, _i, _i, _i, _vp]
@@ -1215,6 +1217,37 @@ def moe_route(z: torch.Tensor, bias: Optional[torch.Tensor], slot_of_token: torc
                              _ptr(place), _ptr(counts), int(n_groups), int(keep_groups), 1 if renormalize else 0,
                              float(norm_eps), ROUTER_SCORES[score], int(identity), _ptr(self_weight), _stream())
     _check(rc, "moe_route")
+
+
+ROUTE_FEW_TOKENS, ROUTE_FEW_CHOICES = 16, 256
+
+
+@_profiled(lambda a, facts: (a["n_tokens"] * (a["n_experts"] * 4 + a["x"].shape[1] * _esz(a["x"]) * (1 + a["top"]) + a["top"] * 8),
+                             a["n_tokens"] * a["n_experts"] * 8))
+def moe_route_few(z: torch.Tensor, bias: Optional[torch.Tensor], slot_of_token: torch.Tensor, n_tokens: int, n_experts: int, top: int,
+                  x: torch.Tensor, rows: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, tile_rows: int, tile_group: torch.Tensor,
+                  n_groups: int = 1, keep_groups: int = 1, renormalize: bool = False, norm_eps: float = 0.0, score: str = "sigmoid",
+                  identity: int = 0, self_weight: Optional[torch.Tensor] = None):
+    """``moe_route``, ``moe_plan`` and ``moe_gather`` in one launch for at most 16 tokens and 256 choices (``n_experts``: all that the
+    router scores, the identity experts included); an expert's rows stand in the order of the choices."""
+    E = n_experts
+    if n_tokens > ROUTE_FEW_TOKENS or n_tokens * top > ROUTE_FEW_CHOICES or z.dtype != torch.float32 or z.stride(1) != 1 or z.shape[1] < E:
+        raise KernelError("moe_route_few: at most 16 tokens and 256 choices, router logits float32 [T, >= E]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != E):
+        raise KernelError("moe_route_few: the choice bias must be float32 [E]")
+    if x.dtype != rows.dtype or not x.is_contiguous() or not rows.is_contiguous() or x.shape[1] != rows.shape[1] or \
+            rows.shape[0] < tile_group.numel() * tile_rows:
+        raise KernelError("moe_route_few: x and rows must be contiguous, of one type and width, with room for every tile")
+    for t, dt in ((row_of, torch.int32), (weights, torch.float32)):
+        if t.dtype != dt or not t.is_contiguous() or t.numel() < n_tokens * top:
+            raise KernelError("moe_route_few: row_of (int32) and weights (float32) must be contiguous [T, top]")
+    if score not in ROUTER_SCORES or (identity and (self_weight is None or self_weight.dtype != torch.float32 or self_weight.numel() < n_tokens)):
+        raise KernelError("moe_route_few: a known score, and float32 self_weight [T] with identity experts")
+    rc = _lib().rb_moe_route_few(_ptr(z), z.stride(0), _ptr(bias), _i32(slot_of_token, "slot_of_token"), n_tokens, E, top, int(n_groups),
+                                 int(keep_groups), 1 if renormalize else 0, float(norm_eps), ROUTER_SCORES[score], int(identity),
+                                 int(tile_rows), tile_group.numel(), _ptr(x), dtype_code(x.dtype), x.shape[1], _ptr(rows), _ptr(row_of),
+                                 _ptr(weights), _ptr(self_weight), _ptr(tile_group), _stream())
+    _check(rc, "moe_route_few")
 
 
 @_profiled(lambda a, facts: ((a["counts"].numel() * 2 + a["tile_group"].numel()) * 4, 0))

@@ -18,7 +18,7 @@ router's rows in the 32-bit router product, and the shared result joins in the k
 
 How a step runs, without the host ever learning who chose what (so a decode step is one CUDA graph):
 the router's product, one kernel that scores, chooses and counts, one that lays every expert's rows out
-from a multiple of the row tile, one that copies each token's row to its places, two products over
+from a multiple of the row tile, one that copies each token's row to its places (the three are one for up to 16 tokens), two products over
 tiles of those rows (every tile names its expert's weight), the activation between them, and a
 weighted sum back into token order.  The row tile is 16 for few tokens and 64 beyond (mma.sync, or FMA in
 32-bit); from a thousand token-choices in bfloat16 it is 128 and the two products are the persistent tcgen05
@@ -197,21 +197,24 @@ class RoutedMLP(FeedForward):
         z = torch.empty((T, self.router.shape[0]), dtype=torch.float32, device=dev)    # E scores (+ the shared expert's gate)
         with scope(op="router"):
             kernels.router_logits(xn, self.router, z, T)
-        ids = torch.empty((T, top), dtype=torch.int32, device=dev)
-        place = torch.empty((T, top), dtype=torch.int32, device=dev)
         weights = torch.empty((T, top), dtype=torch.float32, device=dev)
-        counts = torch.zeros((E,), dtype=torch.int32, device=dev)
-        starts = torch.empty((self.experts + 1,), dtype=torch.int32, device=dev)
-        self_weight = torch.empty((T,), dtype=torch.float32, device=dev) if self.identity else None
         tile_group = torch.empty((max_tiles,), dtype=torch.int32, device=dev)
         row_of = torch.empty((T, top), dtype=torch.int32, device=dev)
+        self_weight = torch.empty((T,), dtype=torch.float32, device=dev) if self.identity else None
+        xs = torch.empty((rows, self.hidden), dtype=act, device=dev)
+        how = dict(n_groups=self.groups, keep_groups=self.keep_groups, renormalize=self.renormalize, norm_eps=self.renormalize_eps,
+                   score=self.score, identity=self.identity, self_weight=self_weight)
         with scope(op="route"):
-            kernels.moe_route(z, self.choice_bias, batch.slot_of_token, T, top, ids, weights, place, counts,
-                              n_groups=self.groups, keep_groups=self.keep_groups, renormalize=self.renormalize,
-                              norm_eps=self.renormalize_eps, score=self.score, identity=self.identity, self_weight=self_weight)
-            kernels.moe_plan(counts[:self.experts], tile, starts, tile_group)
-            xs = torch.empty((rows, self.hidden), dtype=act, device=dev)
-            kernels.moe_gather(xn, ids, place, starts, T, top, xs, row_of)
+            if T <= kernels.ROUTE_FEW_TOKENS and T * top <= kernels.ROUTE_FEW_CHOICES:
+                kernels.moe_route_few(z, self.choice_bias, batch.slot_of_token, T, E, top, xn, xs, row_of, weights, tile, tile_group, **how)
+            else:
+                ids = torch.empty((T, top), dtype=torch.int32, device=dev)
+                place = torch.empty((T, top), dtype=torch.int32, device=dev)
+                counts = torch.zeros((E,), dtype=torch.int32, device=dev)
+                starts = torch.empty((self.experts + 1,), dtype=torch.int32, device=dev)
+                kernels.moe_route(z, self.choice_bias, batch.slot_of_token, T, top, ids, weights, place, counts, **how)
+                kernels.moe_plan(counts[:self.experts], tile, starts, tile_group)
+                kernels.moe_gather(xn, ids, place, starts, T, top, xs, row_of)
         y = torch.empty((rows, self.inter), dtype=act, device=dev)
         fused = False
         told = {"used": self._expected_experts(T), "rows_used": T * top * self.experts // E}     # for a profiler's accounts only

@@ -284,6 +284,24 @@ def test_softmax_scores_correction_and_identity_experts(E, identity, top):
     assert close(weights[live], torch.gather(s, 1, want)[live], 1e-5)
     real_ids = want[live][want[live] < real]
     assert counts.tolist() == [int((real_ids == e).sum()) if e < real else 0 for e in range(E)]
+    # one launch for few tokens: the same choices, rows in whole tiles of their expert, the tokens' rows copied
+    n = 13
+    x = torch.randn(n, H).to(torch.bfloat16)
+    tiles = n * top // 4 + min(real, n * top) + 1
+    xs, row_of, group = torch.zeros((tiles * 4, H), dtype=torch.bfloat16, device=DEV), torch.full((n, top), -9, dtype=torch.int32, device=DEV), torch.full((tiles,), -9, dtype=torch.int32, device=DEV)
+    w2, own2 = torch.zeros((n, top), device=DEV), torch.zeros(n, device=DEV)
+    kernels.moe_route_few(z.to(DEV), corr.to(DEV), slot.to(DEV), n, E, top, x.to(DEV), xs, row_of, w2, 4, group, score="softmax",
+                          identity=identity, self_weight=own2)
+    assert torch.equal(w2, weights[:n]) and torch.equal(own2, own[:n])
+    used = set()
+    for t in range(n):
+        for j in range(top):
+            e, row = int(ids[t, j]), int(row_of[t, j])
+            assert (row < 0) == (e < 0)
+            if e >= 0:
+                assert int(group[row // 4]) == e and row not in used and torch.equal(xs[row].cpu(), x[t])
+                used.add(row)
+    assert sorted(set(group.tolist())) == sorted({-1} | {e for e in ids[:n].flatten().tolist() if e >= 0})
     rows = torch.randn(20, H)
     row_of = torch.randint(-1, 20, (T, top), dtype=torch.int32)
     x = torch.randn(T, H).to(torch.bfloat16)
