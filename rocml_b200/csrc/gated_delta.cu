@@ -28,18 +28,30 @@ namespace {
 template <typename IT>
 __device__ __forceinline__ float sum_in(const IT* p, int n_in, size_t in_stride) {
     float v = 0.f;
-    for (int s = 0; s < n_in; ++s) v += to_f32(p[(size_t)s * in_stride]);
+    for (int s = 0; s < n_in; s += 4) {                 // four partial sums in flight, added in order
+        float y[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = s + j < n_in ? to_f32(p[(size_t)(s + j) * in_stride]) : 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v += y[j];
+    }
     return v;
 }
 template <int VEC, typename IT>
 __device__ __forceinline__ void sum_vec(const IT* p, int n_in, size_t in_stride, float* x) {
     if constexpr (VEC == 4) {
         x[0] = x[1] = x[2] = x[3] = 0.f;
-        for (int s = 0; s < n_in; ++s) {
-            float y[4];
-            load4(p + (size_t)s * in_stride, y);
+        for (int s = 0; s < n_in; s += 4) {             // four partial sums in flight, added in order
+            float y[4][4];
 #pragma unroll
-            for (int u = 0; u < 4; ++u) x[u] += y[u];
+            for (int j = 0; j < 4; ++j) {
+                if (s + j < n_in) load4(p + (size_t)(s + j) * in_stride, y[j]);
+                else y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) x[u] += y[j][u];
         }
     } else {
         x[0] = sum_in(p, n_in, in_stride);
@@ -99,16 +111,23 @@ __device__ __forceinline__ void conv_silu(const PrepArgs& a, const IT* in, const
 
 // The slot's new rows for channels [c0, c0 + n): the last taps - 1 of (old rows, the step's rows).  A channel is one thread's,
 // which reads every row before it overwrites it (a row comes from the same or a later place).
-template <typename IT>
+template <int VEC, typename IT>
 __device__ __forceinline__ void keep_inputs(const PrepArgs& a, const IT* in, float* mine, int t_begin, int len, int col0, int c0,
                                             int n) {
     const int back = a.taps - 1;
-    for (int i = threadIdx.x; i < n; i += blockDim.x)
-        for (int j = 0; j < back; ++j) {
-            const int at = len + j;
-            mine[(size_t)j * a.channels + c0 + i] =
-                at < back ? mine[(size_t)at * a.channels + c0 + i]
-                          : sum_in(in + (size_t)(t_begin + at - back) * a.row_stride + col0 + i, a.n_in, a.in_stride);
+    for (int i = threadIdx.x * VEC; i < n; i += blockDim.x * VEC)
+        for (int j0 = 0; j0 < back; j0 += 4) {          // four rows in flight; a later group's rows are not written before they are read
+            float x[4][VEC];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int at = len + j0 + j;
+                if (j0 + j >= back) continue;
+                if (at < back) load_vec<VEC>(mine + (size_t)at * a.channels + c0 + i, x[j]);
+                else sum_vec<VEC>(in + (size_t)(t_begin + at - back) * a.row_stride + col0 + i, a.n_in, a.in_stride, x[j]);
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (j0 + j < back) store_vec<VEC>(mine + (size_t)(j0 + j) * a.channels + c0 + i, x[j]);
         }
 }
 
@@ -159,8 +178,8 @@ delta_prep_kernel(const IT* __restrict__ in, const ZT* __restrict__ z, const Pre
         }
         if (blockIdx.y == 0 && a.taps > 1) {
             __syncthreads();
-            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.q_off + c, c, a.dim);
-            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.k_off + c, kd + c, a.dim);
+            keep_inputs<VEC>(a, in, mine, t_begin, t_end - t_begin, a.q_off + c, c, a.dim);
+            keep_inputs<VEC>(a, in, mine, t_begin, t_end - t_begin, a.k_off + c, kd + c, a.dim);
         }
         return;
     }
@@ -190,7 +209,7 @@ delta_prep_kernel(const IT* __restrict__ in, const ZT* __restrict__ z, const Pre
     }
     if (blockIdx.y == 0 && a.taps > 1) {
         __syncthreads();
-        keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.v_off + c, 2 * kd + c, a.vdim);
+        keep_inputs<VEC>(a, in, mine, t_begin, t_end - t_begin, a.v_off + c, 2 * kd + c, a.vdim);
     }
 }
 
@@ -300,10 +319,10 @@ delta_prep_rows_kernel(const IT* __restrict__ in, const ZT* __restrict__ z, cons
     if (blockIdx.y == 0 && TAPS > 1) {
         __syncthreads();
         if (keys) {
-            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.q_off + h * a.dim, h * a.dim, a.dim);
-            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.k_off + h * a.dim, kd + h * a.dim, a.dim);
+            keep_inputs<4>(a, in, mine, t_begin, t_end - t_begin, a.q_off + h * a.dim, h * a.dim, a.dim);
+            keep_inputs<4>(a, in, mine, t_begin, t_end - t_begin, a.k_off + h * a.dim, kd + h * a.dim, a.dim);
         } else {
-            keep_inputs(a, in, mine, t_begin, t_end - t_begin, a.v_off + h * a.vdim, 2 * kd + h * a.vdim, a.vdim);
+            keep_inputs<4>(a, in, mine, t_begin, t_end - t_begin, a.v_off + h * a.vdim, 2 * kd + h * a.vdim, a.vdim);
         }
     }
 }
@@ -858,47 +877,69 @@ struct LowRank {
     int x0, rank0, n0, x1, rank1, n1;
 };
 
+// A block takes 64 rows of one matrix for eight tokens, four lanes a row: a lane multiplies eight neighbouring weights in turn
+// with the tokens' inner values (shared memory, eight tokens a value, laid out so that the four lanes meet no bank twice).
+constexpr int LR_ROWS = 64;
+__device__ __forceinline__ int lr_at(int r) { return (r >> 3) * 72 + (r & 7) * LR_TOK; }
+
 template <typename IT, typename WT>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(4 * LR_ROWS)
 low_rank_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, int row_stride, const LowRank p, int T,
                 float* __restrict__ out, int ld_out) {
     pdl_trigger();
-    pdl_wait();
-    extern __shared__ __align__(16) float xs[];        // [rank][LR_TOK]
-    const int blocks0 = (p.n0 + 127) / 128;
+    extern __shared__ __align__(16) float xs[];        // [rank][LR_TOK], see lr_at
+    const int blocks0 = (p.n0 + LR_ROWS - 1) / LR_ROWS;
     const bool second = (int)blockIdx.x >= blocks0;
     const int rank = second ? p.rank1 : p.rank0, n = second ? p.n1 : p.n0, x_off = second ? p.x1 : p.x0;
     const WT* w = static_cast<const WT*>(second ? p.w1 : p.w0);
-    const int row = ((int)blockIdx.x - (second ? blocks0 : 0)) * 128 + threadIdx.x;
+    const int row = ((int)blockIdx.x - (second ? blocks0 : 0)) * LR_ROWS + (threadIdx.x >> 2), sub = threadIdx.x & 3;
     const int t0 = blockIdx.y * LR_TOK;
-    for (int i = threadIdx.x; i < rank * LR_TOK; i += 128) {
+    const bool vec = (rank & 7) == 0 && ((uintptr_t)w & (4 * sizeof(WT) - 1)) == 0;
+    const WT* wr = w + (size_t)(row < n ? row : 0) * rank;
+    // the weights do not depend on the kernel before this one: a lane's first sixteen are asked for before the wait
+    float first[2][8];
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+        if (vec && (c * 4 + sub) * 8 < rank) { load4(wr + (c * 4 + sub) * 8, first[c]); load4(wr + (c * 4 + sub) * 8 + 4, first[c] + 4); }
+    pdl_wait();
+    for (int i = threadIdx.x; i < rank * LR_TOK; i += 4 * LR_ROWS) {
         const int tt = i / rank, r = i - tt * rank;
-        xs[r * LR_TOK + tt] = t0 + tt < T ? sum_in(in + (size_t)(t0 + tt) * row_stride + x_off + r, n_in, in_stride) : 0.f;
+        xs[lr_at(r) + tt] = t0 + tt < T ? sum_in(in + (size_t)(t0 + tt) * row_stride + x_off + r, n_in, in_stride) : 0.f;
     }
     __syncthreads();
-    if (row >= n) return;
     float acc[LR_TOK] = {};
-    const WT* wr = w + (size_t)row * rank;
     auto add = [&](float wv, int r) {
-        const float4 lo = *reinterpret_cast<const float4*>(xs + r * LR_TOK), hi = *reinterpret_cast<const float4*>(xs + r * LR_TOK + 4);
+        const float* x = xs + lr_at(r);
+        const float4 lo = *reinterpret_cast<const float4*>(x), hi = *reinterpret_cast<const float4*>(x + 4);
         acc[0] = fmaf(wv, lo.x, acc[0]); acc[1] = fmaf(wv, lo.y, acc[1]); acc[2] = fmaf(wv, lo.z, acc[2]); acc[3] = fmaf(wv, lo.w, acc[3]);
         acc[4] = fmaf(wv, hi.x, acc[4]); acc[5] = fmaf(wv, hi.y, acc[5]); acc[6] = fmaf(wv, hi.z, acc[6]); acc[7] = fmaf(wv, hi.w, acc[7]);
     };
-    int r = 0;
-    if ((rank & 3) == 0 && ((uintptr_t)w & (4 * sizeof(WT) - 1)) == 0) {
-        for (; r + 16 <= rank; r += 16) {               // sixteen weights in flight
-            float wv[16];
+    if (vec) {
 #pragma unroll
-            for (int u = 0; u < 4; ++u) load4(wr + r + 4 * u, wv + 4 * u);
+        for (int c = 0; c < 2; ++c)
+            if ((c * 4 + sub) * 8 < rank)
 #pragma unroll
-            for (int u = 0; u < 16; ++u) add(wv[u], r + u);
+                for (int u = 0; u < 8; ++u) add(first[c][u], (c * 4 + sub) * 8 + u);
+        for (int r = (8 + sub) * 8; r < rank; r += 32) {
+            float wv[8];
+            load4(wr + r, wv);
+            load4(wr + r + 4, wv + 4);
+#pragma unroll
+            for (int u = 0; u < 8; ++u) add(wv[u], r + u);
         }
+    } else {
+        for (int r = sub; r < rank; r += 4) add(to_f32(wr[r]), r);
     }
-    for (; r < rank; ++r) add(to_f32(wr[r]), r);
+#pragma unroll
+    for (int tt = 0; tt < LR_TOK; ++tt) {
+        acc[tt] += __shfl_xor_sync(0xffffffffu, acc[tt], 1);
+        acc[tt] += __shfl_xor_sync(0xffffffffu, acc[tt], 2);
+    }
+    if (row >= n) return;
     float* o = out + (size_t)t0 * ld_out + (second ? p.n0 : 0) + row;
 #pragma unroll
     for (int tt = 0; tt < LR_TOK; ++tt)
-        if (t0 + tt < T) o[(size_t)tt * ld_out] = acc[tt];
+        if ((tt & 3) == sub && t0 + tt < T) o[(size_t)tt * ld_out] = acc[tt];
 }
 }  // namespace
 
@@ -968,14 +1009,14 @@ extern "C" int rb_low_rank(const void* in, int in_dtype, int n_in, long long in_
     if (T <= 0) return RB_OK;
     if (rank0 <= 0 || n0 <= 0 || n_in < 1 || n1 < 0 || (n1 > 0 && rank1 <= 0)) return RB_ERR_BAD_SIZE;
     const int rank = n1 > 0 && rank1 > rank0 ? rank1 : rank0;
-    const size_t smem = (size_t)rank * LR_TOK * sizeof(float);
+    const size_t smem = (size_t)((rank + 7) / 8) * 72 * sizeof(float);
     if (smem > 48 * 1024) return RB_ERR_BAD_SIZE;
     const LowRank p{w0, w1, x_off0, rank0, n0, x_off1, rank1, n1};
-    const dim3 grid((n0 + 127) / 128 + (n1 + 127) / 128, (T + LR_TOK - 1) / LR_TOK);
+    const dim3 grid((n0 + LR_ROWS - 1) / LR_ROWS + (n1 + LR_ROWS - 1) / LR_ROWS, (T + LR_TOK - 1) / LR_TOK);
     if (grid.y > 65535) return RB_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
-#define RB_LR(IT, WT) RB_LAUNCH((low_rank_kernel<IT, WT>), grid, dim3(128), smem, s, (const IT*)in, n_in, (size_t)in_stride, row_stride, p, T, out, ld_out)
+#define RB_LR(IT, WT) RB_LAUNCH((low_rank_kernel<IT, WT>), grid, dim3(4 * LR_ROWS), smem, s, (const IT*)in, n_in, (size_t)in_stride, row_stride, p, T, out, ld_out)
     if (in_dtype == RB_F32 && w_dtype == RB_BF16) RB_LR(float, bf);
     else if (in_dtype == RB_F32 && w_dtype == RB_F32) RB_LR(float, float);
     else if (in_dtype == RB_BF16 && w_dtype == RB_BF16) RB_LR(bf, bf);

@@ -271,7 +271,7 @@ moe_route_few_kernel(const float* __restrict__ z, int ldz, const BT* __restrict_
                      int top, int n_groups, int keep_groups, int renormalize, float norm_eps, int score, int identity, int tile_rows,
                      int max_tiles, const AT* __restrict__ x, int H, AT* __restrict__ rows, int* __restrict__ row_of,
                      float* __restrict__ weights, float* __restrict__ self_weight, int* __restrict__ tile_group) {
-    pdl_wait();
+    pdl_wait();                                  // no early signal: see grouped_mma_kernel
     extern __shared__ float few_s[];             // [8][E + n_groups] when groups are cut
     __shared__ int s_ids[FEW_CHOICES], s_first[512 + 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, me = blockIdx.x, real = E - identity;
@@ -429,7 +429,8 @@ extern "C" int rb_router_logits(const void* x, int x_dtype, long long ldx, const
     // tokens a block: as many as fit 96 KB of shared memory, at most 8
     const int fit = (int)((96 * 1024) / ((size_t)K * sizeof(float)));
     if (fit < 1) return RB_ERR_BAD_SIZE;
-    const int tt = fit >= 8 ? 8 : (fit >= 4 ? 4 : (fit >= 2 ? 2 : 1));
+    // (a decode step's few tokens: two a block, so that more than a handful of blocks share the work)
+    const int tt = T <= 16 ? (fit >= 2 ? 2 : 1) : (fit >= 8 ? 8 : (fit >= 4 ? 4 : (fit >= 2 ? 2 : 1)));
 #define RB_RL(XT)                                                                         \
     switch (tt) {                                                                         \
         case 8: return launch_router<XT, 8>(x, ldx, w, z, ldz, T, E, K, s);               \

@@ -1831,7 +1831,7 @@ def out_norm(resid: torch.Tensor, delta: torch.Tensor, weight: torch.Tensor, bia
 
 DELTA_MAX_TAPS = 32       # PREP_MAX_TAPS of csrc/gated_delta.cu
 DELTA_MAX_DIM = 512       # rows of a head's state that fit the registers of delta_scan
-LOW_RANK_MAX = 1536       # inner values of low_rank
+LOW_RANK_MAX = 1360       # inner values of low_rank
 
 
 class DeltaRows:
