@@ -1,7 +1,7 @@
 """What a mixer asks of the cache."""
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Optional, Tuple
 
 import torch
@@ -35,6 +35,17 @@ class KVRequirement:
         if self.chunk is not None:
             return length - length % self.chunk
         return 0
+
+    def covering(self, other: "KVRequirement") -> "KVRequirement":
+        """What the cache must keep when a layer that asks ``other`` reads it too: every key that either can read."""
+        if (self.n_kv_heads, self.head_dim, self.shared_values) != (other.n_kv_heads, other.head_dim, other.shared_values):
+            raise ValueError(f"a layer with {other.n_kv_heads} key/value heads of {other.head_dim} cannot read a cache of "
+                             f"{self.n_kv_heads} heads of {self.head_dim}")
+        if (self.window, self.chunk, self.keep_first) == (other.window, other.chunk, other.keep_first):
+            return self
+        if self.window is not None and other.window is not None:
+            return replace(self, window=max(self.window, other.window), keep_first=max(self.keep_first, other.keep_first))
+        return replace(self, window=None, chunk=None, keep_first=0)          # masks of other kinds: everything stays
 
     @property
     def releases(self) -> bool:

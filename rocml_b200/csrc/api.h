@@ -103,7 +103,7 @@ int rb_decay_scan_blocks(const void* in, int in_dtype, int n_in, long long in_st
 // rows; gate_act 0: none, 1: silu, 2: sigmoid.
 int rb_group_norm_gate(const float* o, int ld_o, const void* proj, int proj_dtype, int n_in, long long in_stride,
                        int row_stride, int g_off, const void* w, int w_dtype, float eps, int groups, int W, int gate_act,
-                       void* out, int out_dtype, int ld_out, const int* slot_of_token, int T, void* stream);
+                       void* out, int out_dtype, int ld_out, const int* slot_of_token, int T, const float* den, void* stream);
 
 // Many small products in one launch, by head or by tiles of sorted rows (grouped_matmul.cu).
 int rb_grouped_matmul(const void* x, int x_dtype, long long ldx, int x_col_stride, const void* w, int w_dtype,
@@ -121,7 +121,7 @@ int rb_qk_norm_rope_cache(const void* in, int in_dtype, int n_in, long long in_s
                           const int* positions, const int* slot_of_token, const int* block_table, int max_pages,
                           void* k_cache, void* v_cache, int write_kv, const void* cos_sin, int vd, int hdp,
                           int interleaved, int n_gate, float* gate_out, int post_norm, const float* v_first,
-                          const float* v_lambda, float* v_out, float temp_coef, float temp_every, void* stream);
+                          const float* v_lambda, float* v_out, float temp_coef, float temp_every, int maps, void* stream);
 
 int rb_rope_table(const int* positions, const float* inv_freq, int T, int half, float mag, void* out, void* stream);
 
@@ -164,23 +164,23 @@ int rb_gemm_tcgen05_add(const void* x, const void* w, const float* bias, float* 
 int rb_attention_generic(const void* q, int q_stride, void* out, int o_stride, int dtype, const void* k_cache,
                          const void* v_cache, const int* block_table, int max_pages, const int* seq_slot,
                          const int* cu_q, const int* kv_len, int B, int max_q_len, int nq, int nkv, int hd,
-                         float scale, int window, int keep, float sink, const float* sinks, int chunk, int n_chunks, float* part_acc,
+                         float scale, int window, int keep, float sink, const float* sinks, float softcap, int chunk, int n_chunks, float* part_acc,
                          float* part_ml, int cross, void* stream);
 
 int rb_attention_prefill(const void* q, int q_stride, void* out, int o_stride, const void* k_cache,
                          const void* v_cache, const int* block_table, int max_pages, const int* seq_slot,
                          const int* cu_q, const int* kv_len, int B, int max_q_len, int nq, int nkv, int hd, float scale,
-                         int window, int keep, float sink, const float* sinks, void* stream);
+                         int window, int keep, float sink, const float* sinks, float softcap, void* stream);
 
 int rb_attention_prefill_tc5(const void* q, int q_stride, int T, void* out, int o_stride, const void* k_cache,
                              const void* v_cache, int n_pages, const int* block_table, int max_pages,
                              const int* seq_slot, const int* cu_q, const int* kv_len, int B, int max_q_len, int nq,
-                             int nkv, int hd, float scale, int window, int keep, float sink, const float* sinks, int heads_first, int* status,
+                             int nkv, int hd, float scale, int window, int keep, float sink, const float* sinks, float softcap, int heads_first, int* status,
                              const void* gate, long long gate_row_stride, int cross, void* stream);
 
 int rb_attention_decode(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                         const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
-                        const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window, int keep, float sink, const float* sinks,
+                        const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window, int keep, float sink, const float* sinks, float softcap,
                         int n_chunks, int pages_per_block, float* part_acc, float* part_ml, int* counters, void* out,
                         int o_stride, const void* gate, int gate_f32, int gate_n_in, long long gate_in_stride,
                         long long gate_row_stride, int cross, void* stream);
@@ -191,7 +191,7 @@ int rb_attention_decode_fused(const float* proj, int n_in, long long in_stride, 
                               int row_width, void* k_cache, void* v_cache, const int* block_table, int max_pages, const int* seq_slot,
                               const int* cu_q, const int* kv_len, int B, int nq, int nkv, int hd, float scale,
                               int window, int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
-                              int* counters, void* out, int o_stride, int keep, float sink, const float* sinks, float temp_coef,
+                              int* counters, void* out, int o_stride, int keep, float sink, const float* sinks, float softcap, float temp_coef,
                               float temp_every, int rot_dim, int post_norm,
                               const float* v_first, const float* v_lambda, float* v_keep, const void* gate, int gate_f32,
                               int gate_n_in, long long gate_in_stride, long long gate_row_stride, void* stream);
@@ -303,6 +303,41 @@ int rb_wide_norm_rope_cache(const void* in, int in_dtype, int n_in, long long in
                             const int* block_table, int max_pages, int T, void* stream);
 int rb_talk_mix(const void* o, int o_stride, const float* mix, void* out, int out_stride, int nq, int nkv, int hdp, int vd,
                 int dtype, const int* slot_of_token, int T, void* stream);
+int rb_diff_heads(const void* o, int o_stride, float lambda, float eps, float factor, void* out, int out_stride, int heads, int hdp,
+                  int vd, int dtype, const int* slot_of_token, int T, void* stream);
+
+// An activation on its own (elementwise.cu), and the norm of a sublayer with two results (outnorm.cu).
+int rb_unary_act(const void* in, int in_dtype, int n_in, long long in_stride, void* out, int out_dtype, long long n, int kind,
+                 void* stream);
+int rb_pair_norm(const float* da, int na, long long sa, const float* db, int nb, long long sb, const float* wa, const float* wb,
+                 float eps_in, float factor, float* out_v, float* resid, const float* w, float eps, float mult, void* out,
+                 int out_dtype, int n_rows, int H, void* stream);
+
+// A matrix memory with exponential gates (mlstm.cu).
+int rb_mlstm_gates(const float* gates, int n_in, long long in_stride, int row_stride, int i_off, int f_off, float cap, int heads,
+                   float* m_state, const int* seq_slot, const int* cu_q, const int* positions, int n_seqs, int max_q_len, int T,
+                   float* log_keep, float* log_add, float* em, void* stream);
+int rb_mlstm_step(const void* x, int x_dtype, int n_in, long long in_stride, int row_stride, int q_off, int k_off, int v_off,
+                  const float* gates, int g_n_in, long long g_in_stride, int g_row_stride, int i_off, int f_off, float cap,
+                  float q_scale, float eps, int heads, int dim, int vdim, float* S_state, float* n_state, float* m_state,
+                  const int* seq_slot, const int* cu_q, const int* positions, int n_seqs, float* out, int ld_out, float* den,
+                  void* stream);
+int rb_mlstm_blocks(const void* x, int x_dtype, int n_in, long long in_stride, int row_stride, int q_off, int k_off, int v_off,
+                    float q_scale, float eps, int heads, int dim, int vdim, const float* log_keep, const float* log_add,
+                    const float* em, int T, float* S_state, float* n_state, const int* seq_slot, const int* cu_q, int n_seqs,
+                    int blocks, float* work, float* work_n, float* block_decay, float* scores, float* out, int ld_out,
+                    float* den, void* stream);
+
+// A real-gated linear recurrent unit (rglru.cu).
+int rb_rglru_gates(const float* u, int ld_u, const void* ra, const void* ri, int w_dtype, const float* ra_b, const float* ri_b,
+                   const float* rate, int blocks, int part, int T, float* a, float* x, void* stream);
+int rb_rglru_scan(const float* a, const float* x, int width, const void* y, int y_dtype, int n_in, long long in_stride,
+                  int row_stride, float factor, float* state, const int* seq_slot, const int* cu_q, int n_seqs, void* out,
+                  int out_dtype, int ld_out, void* stream);
+int rb_rglru_step(const float* u, int ld_u, const void* ra, const void* ri, int w_dtype, const float* ra_b, const float* ri_b,
+                  const float* rate, int blocks, int part, int T, const void* y, int y_dtype, int n_in, long long in_stride,
+                  int row_stride, float factor, float* state, const int* slot_of_token, void* out, int out_dtype, int ld_out,
+                  void* stream);
 
 #ifdef __cplusplus
 }

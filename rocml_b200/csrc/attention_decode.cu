@@ -100,6 +100,7 @@ struct Projections {
     // temp_coef != 0: the query of a token at position p is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1),
     // after everything else that happens to it
     float temp_coef, temp_every;
+    float softcap;            // > 0: scores become softcap * tanh(score / softcap)
 };
 
 // One head of 128 values, 4 per lane: the sum of the partial sums, then (what != 2) RMSNorm with `w`
@@ -412,6 +413,9 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             ldmatrix_x4(tile_addr<HD>(qs_base, lane & 7, ks * 2 + (lane >> 3)), qb[ks][0], qb[ks][1], qb[ks + 1][0], qb[ks + 1][1]);
     }
     const float sl2 = scale * LOG2E;
+    const bool capping = pj.softcap > 0.f;
+    const SoftCap capped = soft_cap(scale, pj.softcap);
+    auto scored = [&](float dot) { return capping ? capped(dot) : dot * sl2; };
 
     auto attend_page = [&](int pg, int buf) {
         const int j0 = pg * CHUNK + warp * WK;
@@ -435,13 +439,13 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             const int key0 = j0 + gq, key1 = key0 + 8;
             if (whole) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) st[e] = (st[e] + st2[e]) * sl2;
+                for (int e = 0; e < 4; ++e) st[e] = scored(st[e] + st2[e]);
             } else {
                 const bool ok0 = (key0 >= win_lo || key0 < keep) && key0 <= hi, ok1 = (key1 >= win_lo || key1 < keep) && key1 <= hi;
-                st[0] = ok0 ? (st[0] + st2[0]) * sl2 : -INFINITY;
-                st[1] = ok0 ? (st[1] + st2[1]) * sl2 : -INFINITY;
-                st[2] = ok1 ? (st[2] + st2[2]) * sl2 : -INFINITY;
-                st[3] = ok1 ? (st[3] + st2[3]) * sl2 : -INFINITY;
+                st[0] = ok0 ? scored(st[0] + st2[0]) : -INFINITY;
+                st[1] = ok0 ? scored(st[1] + st2[1]) : -INFINITY;
+                st[2] = ok1 ? scored(st[2] + st2[2]) : -INFINITY;
+                st[3] = ok1 ? scored(st[3] + st2[3]) : -INFINITY;
             }
             float mx[2] = {fmaxf(st[0], st[2]), fmaxf(st[1], st[3])};
             float alpha[2];
@@ -505,7 +509,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
 #pragma unroll
             for (int j = 0; j < WK / 8; ++j) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) s[j][e] *= sl2;
+                for (int e = 0; e < 4; ++e) s[j][e] = scored(s[j][e]);
                 mx[0] = fmaxf(mx[0], fmaxf(s[j][0], s[j][1]));
                 mx[1] = fmaxf(mx[1], fmaxf(s[j][2], s[j][3]));
             }
@@ -516,7 +520,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                 for (int e = 0; e < 4; ++e) {
                     const int key = j0 + j * 8 + tq * 2 + (e & 1);
                     const bool ok = (key >= win_lo || key < keep) && key <= hi;
-                    s[j][e] = ok ? s[j][e] * sl2 : -INFINITY;
+                    s[j][e] = ok ? scored(s[j][e]) : -INFINITY;
                 }
                 mx[0] = fmaxf(mx[0], fmaxf(s[j][0], s[j][1]));
                 mx[1] = fmaxf(mx[1], fmaxf(s[j][2], s[j][3]));
@@ -850,13 +854,14 @@ static int decode_entry(const void* q, int q_stride, const void* k_cache, const 
 extern "C" int rb_attention_decode(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                                    const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                                    const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window,
-                                   int keep, float sink, const float* sinks, int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
+                                   int keep, float sink, const float* sinks, float softcap, int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
                                    int* counters, void* out, int o_stride, const void* gate, int gate_f32, int gate_n_in,
                                    long long gate_in_stride, long long gate_row_stride, int cross, void* stream) {
     Projections none = {};
     if (cross < 0 || (cross > 1 && (nkv != cross * cross || gate != nullptr))) return RB_ERR_BAD_SIZE;
     none.cross = cross;
     none.sinks = sinks;
+    none.softcap = softcap;
     if (gate != nullptr) {      // nq * hd columns of the projection rows: the result times their sigmoid
         if (gate_n_in < 1) return RB_ERR_BAD_SIZE;
         none.gate = GateCols{gate, gate_f32, gate_n_in, gate_in_stride, gate_row_stride};
@@ -884,7 +889,7 @@ extern "C" int rb_attention_decode_fused(const float* proj, int n_in, long long 
                                          const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                                          const int* kv_len, int B, int nq, int nkv, int hd, float scale, int window,
                                          int n_chunks, int pages_per_block, float* part_acc, float* part_ml,
-                                         int* counters, void* out, int o_stride, int keep, float sink, const float* sinks,
+                                         int* counters, void* out, int o_stride, int keep, float sink, const float* sinks, float softcap,
                                          float temp_coef, float temp_every, int rot_dim, int post_norm, const float* v_first, const float* v_lambda, float* v_keep,
                                          const void* gate, int gate_f32, int gate_n_in, long long gate_in_stride,
                                          long long gate_row_stride, void* stream) {
@@ -907,6 +912,7 @@ extern "C" int rb_attention_decode_fused(const float* proj, int n_in, long long 
     pj.row_eps = row_eps; pj.row_inv_width = row_width > 0 ? 1.f / (float)row_width : 0.f;
     if (row_sumsq != nullptr && (row_groups < 1 || row_width < 1)) return RB_ERR_BAD_SIZE;
     pj.rot_dim = rot_dim; pj.post_norm = post_norm;
+    pj.softcap = softcap;
     pj.sinks = sinks; pj.temp_coef = temp_coef; pj.temp_every = temp_every;
     pj.v_first = v_first; pj.v_lambda = v_lambda; pj.v_keep = v_keep;
     if (gate != nullptr) pj.gate = GateCols{gate, gate_f32, gate_n_in, gate_in_stride, gate_row_stride};
@@ -978,6 +984,6 @@ extern "C" int rb_attention_decode_static(const void* q, int q_stride, const voi
     cudaError_t e = cudaMemsetAsync(sc->counters, 0, n_counters * sizeof(int), (cudaStream_t)stream);
     if (e != cudaSuccess) return (int)e;
     return rb_attention_decode(q, q_stride, k_cache, v_cache, block_table, max_pages, seq_slot, cu_q, kv_len, n_seqs,
-                               nq, nkv, hd, scale, window, 0, RB_NO_SINK, nullptr, n_chunks, 1, sc->acc, sc->ml, sc->counters, out, o_stride,
+                               nq, nkv, hd, scale, window, 0, RB_NO_SINK, nullptr, 0.f, n_chunks, 1, sc->acc, sc->ml, sc->counters, out, o_stride,
                                nullptr, 0, 0, 0, 0, 0, stream);
 }

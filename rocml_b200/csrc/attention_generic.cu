@@ -5,7 +5,8 @@
 // positions lo..pos with pos the token's absolute position (causal, inclusive:
 // rocml-kernels/kernels/attn_prefill.hip:57-60,121) and lo = max(0, pos - window + 1) when the
 // layer has a window (a negative `window` means blocks of that many positions: rb::span_lo).  Query head h reads key/value head h / g (attn_decode.hip:108); the
-// score is (q . k) * scale, scale applied after the dot (attn_decode.hip:158); softmax is an
+// score is (q . k) * scale, scale applied after the dot (attn_decode.hip:158), then, with a soft cap,
+// cap * tanh(score / cap); softmax is an
 // online max/sum in 32-bit with expf (attn_decode.hip:160-170); o = sum p v / l
 // (attn_prefill.hip:201-203).
 //
@@ -47,7 +48,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
                          const int* __restrict__ block_table, int max_pages,
                          const int* __restrict__ seq_slot, const int* __restrict__ cu_q,
                          const int* __restrict__ kv_len, int nq, int nkv, int hd, float scale, int window,
-                         int keep, float sink, const float* __restrict__ sinks, int chunk, int n_chunks, float* __restrict__ part_acc,
+                         int keep, float sink, const float* __restrict__ sinks, float softcap, int chunk, int n_chunks, float* __restrict__ part_acc,
                          float* __restrict__ part_ml, int cross) {
     pdl_trigger();
     pdl_wait();
@@ -214,7 +215,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
 #pragma unroll
             for (int i = 0; i < NR; ++i) {
                 const bool valid = row_ok[i] && j <= row_pos[i] && (j >= row_lo[i] || j < keep) && j <= hi && j >= lo;
-                const float sv = s[i] * scale;
+                const float sv = softcap > 0.f ? softcap * tanhf(s[i] * scale / softcap) : s[i] * scale;
                 const float tmax = warp_max(valid ? sv : NEG_BIG);
                 const float m_new = fmaxf(m[i], tmax);
                 const float alpha = expf(m[i] - m_new);
@@ -335,7 +336,7 @@ template <typename T>
 int launch_attn(const void* q, int q_stride, void* out, int o_stride, const void* k_cache, const void* v_cache,
                 const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                 const int* kv_len, int B, int max_q_len, int nq, int nkv, int hd, float scale, int window,
-                int keep, float sink, const float* sinks, int chunk, int n_chunks, float* part_acc, float* part_ml, int cross, cudaStream_t s) {
+                int keep, float sink, const float* sinks, float softcap, int chunk, int n_chunks, float* part_acc, float* part_ml, int cross, cudaStream_t s) {
     const int g = nq / nkv;
     const int HG = g < ROWS ? g : ROWS;
     const int QB = ROWS / HG;
@@ -351,7 +352,7 @@ int launch_attn(const void* q, int q_stride, void* out, int o_stride, const void
     dim3 grid((unsigned)gx, nkv * head_chunks, B);
     RB_LAUNCH((k), dim3(grid), dim3(128), smem, s, (const T*)q, q_stride, (T*)out, o_stride, (const T*)k_cache, (const T*)v_cache,
                               block_table, max_pages, seq_slot, cu_q, kv_len, nq, nkv, hd, scale, window,
-                              keep, sink, sinks, chunk, n_chunks, part_acc, part_ml, cross);
+                              keep, sink, sinks, softcap, chunk, n_chunks, part_acc, part_ml, cross);
     RB_LAUNCH_CHECK();
     return RB_OK;
 }
@@ -361,7 +362,7 @@ extern "C" int rb_attention_generic(const void* q, int q_stride, void* out, int 
                                     const void* k_cache, const void* v_cache, const int* block_table,
                                     int max_pages, const int* seq_slot, const int* cu_q, const int* kv_len,
                                     int B, int max_q_len, int nq, int nkv, int hd, float scale, int window,
-                                    int keep, float sink, const float* sinks, int chunk, int n_chunks, float* part_acc,
+                                    int keep, float sink, const float* sinks, float softcap, int chunk, int n_chunks, float* part_acc,
                                     float* part_ml, int cross, void* stream) {
     if (B <= 0 || max_q_len <= 0) return RB_OK;
     if (keep < 0 || (keep > 0 && window < 0)) return RB_ERR_BAD_SIZE;
@@ -373,10 +374,10 @@ extern "C" int rb_attention_generic(const void* q, int q_stride, void* out, int 
     if (dtype == RB_BF16)
         return launch_attn<__nv_bfloat16>(q, q_stride, out, o_stride, k_cache, v_cache, block_table, max_pages,
                                           seq_slot, cu_q, kv_len, B, max_q_len, nq, nkv, hd, scale, window,
-                                          keep, sink, sinks, chunk, n_chunks, part_acc, part_ml, cross, s);
+                                          keep, sink, sinks, softcap, chunk, n_chunks, part_acc, part_ml, cross, s);
     if (dtype == RB_F32)
         return launch_attn<float>(q, q_stride, out, o_stride, k_cache, v_cache, block_table, max_pages, seq_slot,
-                                  cu_q, kv_len, B, max_q_len, nq, nkv, hd, scale, window, keep, sink, sinks, chunk, n_chunks,
+                                  cu_q, kv_len, B, max_q_len, nq, nkv, hd, scale, window, keep, sink, sinks, softcap, chunk, n_chunks,
                                   part_acc, part_ml, cross, s);
     return RB_ERR_BAD_DTYPE;
 }

@@ -37,7 +37,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                          const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_table,
                          int max_pages, const int* __restrict__ seq_slot, const int* __restrict__ cu_q,
                          const int* __restrict__ kv_len, int nq, int nkv, float scale, int window, int keep,
-                         float sink, const float* __restrict__ sinks) {
+                         float sink, const float* __restrict__ sinks, float softcap) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(128) uint8_t smem_raw[];
@@ -88,6 +88,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
     float m_run[2] = {NEG_BIG, NEG_BIG}, l_run[2] = {0.f, 0.f};
     const int row_pos[2] = {pos0 + m0 + warp * 16 + g, pos0 + m0 + warp * 16 + g + 8};
     const float sl2 = scale * LOG2E;
+    const SoftCap capped = soft_cap(scale, softcap);
     const uint32_t qs_base = smem_addr(Qs);
 
     for (int j = 0; j < n_tiles; ++j) {
@@ -130,7 +131,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                 const int key = kt * BN + j * 8 + t * 2 + (e & 1);
                 const int r = e >> 1;
                 const bool ok = key <= row_pos[r] && (key >= span_lo(row_pos[r], window) || key < keep);
-                s[j][e] = ok ? s[j][e] * sl2 : -INFINITY;
+                s[j][e] = ok ? (softcap > 0.f ? capped(s[j][e]) : s[j][e] * sl2) : -INFINITY;
                 mx[r] = fmaxf(mx[r], s[j][e]);
             }
         }
@@ -215,7 +216,7 @@ template <int HD>
 int launch(const void* q, int q_stride, void* out, int o_stride, const void* k_cache, const void* v_cache,
            const int* block_table, int max_pages, const int* seq_slot, const int* cu_q, const int* kv_len, int B,
            int max_q_len, int nq, int nkv, float scale, int window, int keep, float sink, const float* sinks,
-           cudaStream_t s) {
+           float softcap, cudaStream_t s) {
     const size_t smem = (size_t)(BM + 4 * BN) * HD * sizeof(__nv_bfloat16);
     auto k = attention_prefill_kernel<HD>;
     static bool attr_done = false;
@@ -228,21 +229,21 @@ int launch(const void* q, int q_stride, void* out, int o_stride, const void* k_c
     if (grid.y > 65535 || grid.z > 65535) return RB_ERR_BAD_SIZE;
     RB_LAUNCH((k), grid, dim3(NWARPS * 32), smem, s, (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out,
               o_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_table, max_pages,
-              seq_slot, cu_q, kv_len, nq, nkv, scale, window, keep, sink, sinks);
+              seq_slot, cu_q, kv_len, nq, nkv, scale, window, keep, sink, sinks, softcap);
     return RB_OK;
 }
 }  // namespace
 
 // q rows [T, >= nq*hd] bfloat16 -> out rows; keys and values from the pages.  keep: beside a window the keys at
 // positions below it stay visible; sink: a score whose exponential joins every row's denominator (RB_NO_SINK: none); sinks:
-// one such score a query head instead.  Returns
+// one such score a query head instead; softcap > 0: scores become softcap * tanh(score / softcap).  Returns
 // RB_ERR_BAD_SIZE for head sizes other than 64, 128, 256 and RB_ERR_BAD_ALIGN for rows or pointers
 // off a 16-byte boundary (the caller then uses the plain kernel).
 extern "C" int rb_attention_prefill(const void* q, int q_stride, void* out, int o_stride, const void* k_cache,
                                     const void* v_cache, const int* block_table, int max_pages,
                                     const int* seq_slot, const int* cu_q, const int* kv_len, int B, int max_q_len,
                                     int nq, int nkv, int hd, float scale, int window, int keep, float sink,
-                                    const float* sinks, void* stream) {
+                                    const float* sinks, float softcap, void* stream) {
     if (B <= 0 || max_q_len <= 0) return RB_OK;
     if (nkv <= 0 || nq % nkv || keep < 0) return RB_ERR_BAD_SIZE;
     if (window <= 0) keep = 0;                            // kept first keys stand beside a window only
@@ -251,7 +252,7 @@ extern "C" int rb_attention_prefill(const void* q, int q_stride, void* out, int 
         return RB_ERR_BAD_ALIGN;
     cudaStream_t s = (cudaStream_t)stream;
 #define RB_AP(HD) return launch<HD>(q, q_stride, out, o_stride, k_cache, v_cache, block_table, max_pages, seq_slot, \
-                                    cu_q, kv_len, B, max_q_len, nq, nkv, scale, window, keep, sink, sinks, s)
+                                    cu_q, kv_len, B, max_q_len, nq, nkv, scale, window, keep, sink, sinks, softcap, s)
     if (hd == 128) RB_AP(128);
     if (hd == 64) RB_AP(64);
     if (hd == 256) RB_AP(256);

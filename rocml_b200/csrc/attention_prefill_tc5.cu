@@ -109,7 +109,9 @@ struct Barriers {
     uint32_t tmem_slot, abort_flag;
 };
 
-template <int HD>
+// CAP: scores go through a soft cap (SoftCap of common.cuh) as they leave tensor memory; the softmax then works on them as
+// they are.
+template <int HD, bool CAP>
 __global__ void __launch_bounds__(192, Sizes<HD>::BLOCKS_PER_SM)
 attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, int o_stride,
@@ -117,7 +119,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                              const int* __restrict__ cu_q, const int* __restrict__ kv_len, int nq, int nkv,
                              float scale, int window, int keep, float sink, const float* __restrict__ sinks, int heads_first, int strict_order,
                              int* __restrict__ status, const __nv_bfloat16* __restrict__ gate, long long gate_row_stride,
-                             int cross) {
+                             int cross, float softcap) {
     using Z = Sizes<HD>;
     constexpr int HALVES = Z::HALVES, Q_BYTES = Z::Q_BYTES, KV_TILE = Z::KV_TILE, Q_HALF = Z::Q_HALF, KV_HALF = Z::KV_HALF;
     constexpr int TILE_BYTES = Z::TILE_BYTES, SMEM_BYTES = Z::SMEM_BYTES, TMEM_COLS = Z::TMEM_COLS;
@@ -279,7 +281,8 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const int r = quarter * 32 + lane;
         const int row_pos = pos0 + m0 + r;
         const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
-        const float sl2 = scale * LOG2E;
+        const float sl2 = CAP ? 1.f : scale * LOG2E;
+        const rb::SoftCap capped = rb::soft_cap(scale, softcap);
         float m_used = NEG_BIG, l_sum = 0.f;
         bool alive = true;
         for (int j = 0; j < n_tiles; ++j) {
@@ -295,6 +298,10 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
             // positive, so the maximum is taken first (three inputs an instruction) and the scale is
             // folded into the exponent's multiply-add, p = 2^(s * scale * log2 e - m), with the bare
             // special-function instruction for 2^x.
+            if (CAP) {
+#pragma unroll
+                for (int i = 0; i < BNK; ++i) sv[i] = capped(sv[i]);
+            }
             // a tile that every row of this warp sees whole needs no mask
             const int warp_first_pos = pos0 + m0 + quarter * 32;
             if (!(key0 + BNK - 1 <= warp_first_pos && (key0 >= rb::span_lo(warp_first_pos + 31, window) || key0 + BNK <= keep))) {
@@ -486,11 +493,11 @@ int make_map(const void* ptr, long long rows, long long cols, long long ld, int 
     cache[key] = *out;
     return RB_OK;
 }
-template <int HD>
+template <int HD, bool CAP>
 int launch_tc5(const void* q, int q_stride, int T, void* out, int o_stride, const void* k_cache, const void* v_cache,
                int n_pages, const int* block_table, int max_pages, const int* seq_slot, const int* cu_q,
                const int* kv_len, int B, int max_q_len, int nq, int nkv, float scale, int window, int keep, float sink,
-               const float* sinks, int heads_first, int* status, const void* gate, long long gate_row_stride, int cross, cudaStream_t stream) {
+               const float* sinks, float softcap, int heads_first, int* status, const void* gate, long long gate_row_stride, int cross, cudaStream_t stream) {
     // RB_PREFILL_STRICT_ORDER=0: see `strict_order` in the kernel's MMA thread
     static const int strict_order = [] { const char* e = getenv("RB_PREFILL_STRICT_ORDER"); return (e && e[0] == '0') ? 0 : 1; }();
     CUtensorMap mq, mk, mv;
@@ -499,7 +506,7 @@ int launch_tc5(const void* q, int q_stride, int T, void* out, int o_stride, cons
     const long long cache_rows = (long long)n_pages * (cross > 1 ? cross : nkv) * RB_PAGE;
     if ((rc = make_map(k_cache, cache_rows, HD, HD, BNK, &mk)) != RB_OK) return rc;
     if ((rc = make_map(v_cache, cache_rows, HD, HD, BNK, &mv)) != RB_OK) return rc;
-    auto k = attention_prefill_tc5_kernel<HD>;
+    auto k = attention_prefill_tc5_kernel<HD, CAP>;
     static bool attr_done = false;
     if (!attr_done) {
         cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, Sizes<HD>::SMEM_BYTES);
@@ -511,7 +518,7 @@ int launch_tc5(const void* q, int q_stride, int T, void* out, int o_stride, cons
     if (grid.y > 65535 || grid.z > 65535) return RB_ERR_BAD_SIZE;
     RB_LAUNCH((k), grid, dim3(192), Sizes<HD>::SMEM_BYTES, stream, mq, mk, mv, (__nv_bfloat16*)out, o_stride,
               block_table, max_pages, seq_slot, cu_q, kv_len, nq, nkv, scale, window, keep, sink, sinks, heads_first, strict_order,
-              status, (const __nv_bfloat16*)gate, gate_row_stride, cross);
+              status, (const __nv_bfloat16*)gate, gate_row_stride, cross, softcap);
     return RB_OK;
 }
 }  // namespace
@@ -522,13 +529,14 @@ int launch_tc5(const void* q, int q_stride, int T, void* out, int o_stride, cons
 // sinks: one such score a query head instead.  Head sizes 64, 128 and 256;
 // RB_ERR_BAD_SIZE / RB_ERR_BAD_ALIGN otherwise (the caller then uses the mma.sync kernel).  gate: nq * hd bfloat16 columns of
 // the tokens' projection rows (gate_row_stride elements apart), or null: the result is multiplied by their sigmoid.
+// softcap > 0: scores become softcap * tanh(score / softcap).
 // cross (n > 1, the caches' own number of heads): every query head's weights on the values of every stored head; nkv = n * n
 // counts (key head, value head) pairs, nq = n * query heads the results, q holds nq / n heads.
 extern "C" int rb_attention_prefill_tc5(const void* q, int q_stride, int T, void* out, int o_stride,
                                         const void* k_cache, const void* v_cache, int n_pages,
                                         const int* block_table, int max_pages, const int* seq_slot,
                                         const int* cu_q, const int* kv_len, int B, int max_q_len, int nq, int nkv,
-                                        int hd, float scale, int window, int keep, float sink, const float* sinks, int heads_first,
+                                        int hd, float scale, int window, int keep, float sink, const float* sinks, float softcap, int heads_first,
                                         int* status, const void* gate, long long gate_row_stride, int cross, void* stream) {
     if (B <= 0 || max_q_len <= 0 || T <= 0) return RB_OK;
     if (cross < 0 || (cross > 1 && (nkv != cross * cross || gate))) return RB_ERR_BAD_SIZE;
@@ -539,9 +547,14 @@ extern "C" int rb_attention_prefill_tc5(const void* q, int q_stride, int T, void
         (q_stride % 8) || (o_stride % 8))
         return RB_ERR_BAD_ALIGN;
 #define RB_TC5_ARGS q, q_stride, T, out, o_stride, k_cache, v_cache, n_pages, block_table, max_pages, seq_slot, cu_q, kv_len, \
-                    B, max_q_len, nq, nkv, scale, window, keep, sink, sinks, heads_first, status, gate, gate_row_stride, cross, (cudaStream_t)stream
-    if (hd == 64) return launch_tc5<64>(RB_TC5_ARGS);
-    if (hd == 128) return launch_tc5<128>(RB_TC5_ARGS);
-    return launch_tc5<256>(RB_TC5_ARGS);
+                    B, max_q_len, nq, nkv, scale, window, keep, sink, sinks, softcap, heads_first, status, gate, gate_row_stride, cross, (cudaStream_t)stream
+    if (softcap > 0.f) {
+        if (hd == 64) return launch_tc5<64, true>(RB_TC5_ARGS);
+        if (hd == 128) return launch_tc5<128, true>(RB_TC5_ARGS);
+        return launch_tc5<256, true>(RB_TC5_ARGS);
+    }
+    if (hd == 64) return launch_tc5<64, false>(RB_TC5_ARGS);
+    if (hd == 128) return launch_tc5<128, false>(RB_TC5_ARGS);
+    return launch_tc5<256, false>(RB_TC5_ARGS);
 #undef RB_TC5_ARGS
 }

@@ -108,6 +108,24 @@ __device__ __forceinline__ float add_sink(float m, float& l, float sink) {
     return a;
 }
 
+// A soft cap on a score, s <- cap * tanh(s / cap), before the mask and the softmax.  With t = e^(2 s / cap) it is
+// cap - 2 cap / (t + 1): two special-function instructions, whose absolute error (about 1e-7 of the cap) is what enters the
+// exponent; saturates to +-cap where t leaves the range.  In base 2: the raw dot product times `k`, result times log2 e.
+struct SoftCap {
+    float k;        // 2 * scale / cap * log2 e (0: no cap)
+    float cap2;     // cap * log2 e
+    float m2cap2;   // -2 * cap2
+    __device__ __forceinline__ float operator()(float dot) const {
+        float t;
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(t) : "f"(dot * k));
+        return fmaf(m2cap2, __fdividef(1.f, t + 1.f), cap2);
+    }
+};
+__device__ __forceinline__ SoftCap soft_cap(float scale, float cap) {
+    constexpr float log2e = 1.4426950408889634f;
+    return cap > 0.f ? SoftCap{2.f * scale / cap * log2e, cap * log2e, -2.f * cap * log2e} : SoftCap{0.f, 0.f, 0.f};
+}
+
 // Columns of the step's projection rows that gate an attention kernel's result value by value, so that no kernel
 // of its own has to: out[t][c] *= sigmoid(sum over the partial sums of raw[s][t][c]), formed in 32-bit.
 struct GateCols {
@@ -143,6 +161,8 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
 __device__ __forceinline__ float gelu_tanh(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+// gelu as it is: z / 2 * (1 + erf(z / sqrt(2)))
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.7071067811865476f)); }
 __device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
 
 // Four neighbouring elements at once (the pointer on 4 elements' alignment).

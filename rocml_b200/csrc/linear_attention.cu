@@ -15,7 +15,7 @@
 //                 order of p.  One token a sequence (a decode step) is the same kernel with one token.
 //                 The order of a token's operations does not depend on how the prompt was cut or on the batch.
 //   group_norm_gate   what follows the recurrence: o divided by its root mean square over each of G groups of
-//                 columns (G = heads: per head; G = 1: all heads together), times an optional weight vector, times
+//                 columns (G = heads: per head; G = 1: all heads together), each first divided by den[token][group] if given, times an optional weight vector, times
 //                 act(gate) with the gate another column block of the projection; written in the activations' type
 //                 for the output product.
 #include "common.cuh"
@@ -459,7 +459,7 @@ template <typename IT, typename AT, typename WT>
 __global__ void __launch_bounds__(256)
 group_norm_gate_kernel(const float* __restrict__ o, int ld_o, const IT* __restrict__ proj, int n_in, size_t in_stride,
                        int row_stride, int g_off, const WT* __restrict__ w, float eps, int groups, int W, int gate_act,
-                       AT* __restrict__ out, int ld_out, const int* __restrict__ slot_of_token) {
+                       AT* __restrict__ out, int ld_out, const int* __restrict__ slot_of_token, const float* __restrict__ den) {
     pdl_trigger();
     pdl_wait();
     __shared__ float scratch[33];
@@ -484,7 +484,9 @@ group_norm_gate_kernel(const float* __restrict__ o, int ld_o, const IT* __restri
                 ss += x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3];
             }
             ss = groups == 1 ? block_sum(ss, scratch) : warp_sum(ss);
-            const float inv = rsqrtf(ss / (float)gw + eps);
+            // a divisor of the group's values, (o / d) / rms(o / d): both factors at once
+            const float rd = den ? 1.f / den[(size_t)t * groups + gi] : 1.f;
+            const float inv = rsqrtf(ss * rd * rd / (float)gw + eps) * rd;
             for (int i = me * 4; i < gw; i += n_me * 4) {
                 const int c = gi * gw + i;
                 float x[4], z[4] = {0.f, 0.f, 0.f, 0.f}, ww[4] = {1.f, 1.f, 1.f, 1.f};
@@ -507,7 +509,8 @@ group_norm_gate_kernel(const float* __restrict__ o, int ld_o, const IT* __restri
         float ss = 0.f;
         for (int i = threadIdx.x; i < W; i += blockDim.x) { const float x = row[i]; ss += x * x; }
         ss = block_sum(ss, scratch);
-        const float inv = rsqrtf(ss / (float)W + eps);
+        const float rd = den ? 1.f / den[t] : 1.f;
+        const float inv = rsqrtf(ss * rd * rd / (float)W + eps) * rd;
         for (int i = threadIdx.x; i < W; i += blockDim.x) {
             float x = row[i] * inv;
             if (w) x *= to_f32(w[i]);
@@ -521,7 +524,8 @@ group_norm_gate_kernel(const float* __restrict__ o, int ld_o, const IT* __restri
         float ss = 0.f;
         for (int i = lane; i < gw; i += 32) { const float x = row[gi * gw + i]; ss += x * x; }
         ss = warp_sum(ss);
-        const float inv = rsqrtf(ss / (float)gw + eps);
+        const float rd = den ? 1.f / den[(size_t)t * groups + gi] : 1.f;
+        const float inv = rsqrtf(ss * rd * rd / (float)gw + eps) * rd;
         for (int i = lane; i < gw; i += 32) {
             const int c = gi * gw + i;
             float x = row[c] * inv;
@@ -582,14 +586,14 @@ extern "C" int rb_decay_scan(const void* in, int in_dtype, int n_in, long long i
 extern "C" int rb_group_norm_gate(const float* o, int ld_o, const void* proj, int proj_dtype, int n_in, long long in_stride,
                                   int row_stride, int g_off, const void* w, int w_dtype, float eps, int groups, int W,
                                   int gate_act, void* out, int out_dtype, int ld_out, const int* slot_of_token, int T,
-                                  void* stream) {
+                                  const float* den, void* stream) {
     if (T <= 0) return RB_OK;
     if (groups <= 0 || W <= 0 || W % groups || n_in < 1) return RB_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
 #define RB_GNG(IT, AT, WT)                                                                                               \
     RB_LAUNCH((group_norm_gate_kernel<IT, AT, WT>), dim3(T), dim3(256), 0, s, o, ld_o, (const IT*)proj, n_in,            \
-              (size_t)in_stride, row_stride, g_off, (const WT*)w, eps, groups, W, gate_act, (AT*)out, ld_out, slot_of_token)
+              (size_t)in_stride, row_stride, g_off, (const WT*)w, eps, groups, W, gate_act, (AT*)out, ld_out, slot_of_token, den)
     const bool wf = !w || w_dtype == RB_F32;
     if (proj_dtype == RB_BF16 && out_dtype == RB_BF16 && !wf) RB_GNG(bf, bf, bf);
     else if (proj_dtype == RB_BF16 && out_dtype == RB_BF16) RB_GNG(bf, bf, float);

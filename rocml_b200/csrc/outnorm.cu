@@ -7,6 +7,8 @@
 //                  layer norm or an RMS norm with a weight and an optional bias.  The new row is also written in the type
 //                  of the product that reads it next, because the sublayers of such a layer read the stream itself.
 //
+//   pair_norm      the same for a sublayer with two results that are normalised apart and added: d = factor * (rms(a) * wa + rms(b) * wb).
+//
 // One block a row, the row in shared memory between the passes (mean, squared deviations, result), 16-byte accesses
 // where width and addresses allow.  All arithmetic is 32-bit; partial sums are added in their order, so a row's result
 // depends on nothing else in the batch.
@@ -97,6 +99,75 @@ struct Routed {
     int top;
     const float* self_weight;      // may be null
 };
+
+// Two results of one sublayer, each normalised on its own: v = factor * (rms(a) * wa + rms(b) * wb), a and b sums of partial sums.
+// Without `w` v is the result (out_v float32 [T, H]); with it resid[row] += mult * rms(v) * w, and `out` receives the new row.
+template <typename OT>
+__global__ void __launch_bounds__(1024)
+pair_norm_kernel(const float* __restrict__ da, int na, size_t sa, const float* __restrict__ db, int nb, size_t sb,
+                 const float* __restrict__ wa, const float* __restrict__ wb, float eps_in, float factor, float* __restrict__ out_v,
+                 float* __restrict__ resid, const float* __restrict__ w, float eps, float mult, OT* __restrict__ out, int H, int vec) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float row[];       // 2 rows of H floats (padded to 4) + 2 * 33
+    const int ldr = (H + 3) & ~3;
+    float* row_b = row + ldr;
+    float* red = row_b + ldr;
+    const int t = blockIdx.x;
+    float s0 = 0.f, s1 = 0.f;
+    for (int part = 0; part < 2; ++part) {
+        const float* d = (part ? db : da) + (size_t)t * H;
+        const int nd = part ? nb : na;
+        const size_t st = part ? sb : sa;
+        float* dst = part ? row_b : row;
+        float ss = 0.f;
+        if (vec) {
+            for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int s = 0; s < nd; s += 4) {          // four partial sums in flight, added in order
+                    float p[4][4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        if (s + j < nd) load4(d + (size_t)(s + j) * st + i, p[j]);
+                        else p[j][0] = p[j][1] = p[j][2] = p[j][3] = 0.f;
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+#pragma unroll
+                        for (int u = 0; u < 4; ++u) v[u] += p[j][u];
+                }
+                ss += v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+                store4(dst + i, v);
+            }
+        } else {
+            for (int i = threadIdx.x; i < H; i += blockDim.x) {
+                float v = 0.f;
+                for (int s = 0; s < nd; ++s) v += d[(size_t)s * st + i];
+                ss = fmaf(v, v, ss);
+                dst[i] = v;
+            }
+        }
+        if (part) s1 = ss; else s0 = ss;
+    }
+    s0 = block_sum(s0, red);
+    s1 = block_sum(s1, red + 33);
+    const float ia = rsqrtf(s0 / (float)H + eps_in) * factor, ib = rsqrtf(s1 / (float)H + eps_in) * factor;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = row[i] * ia * wa[i] + row_b[i] * ib * wb[i];
+        row[i] = v;
+        ss = fmaf(v, v, ss);
+        if (!w) out_v[(size_t)t * H + i] = v;
+    }
+    if (!w) return;
+    const float inv = rsqrtf(block_sum(ss, red) / (float)H + eps) * mult;
+    float* x = resid + (size_t)t * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = fmaf(row[i] * inv, w[i], x[i]);
+        x[i] = v;
+        if (out) out[(size_t)t * H + i] = from_f32<OT>(v);
+    }
+}
 
 template <typename OT, typename XT>
 __global__ void __launch_bounds__(1024)
@@ -269,6 +340,33 @@ extern "C" int rb_out_norm(float* resid, const float* delta, int n_delta, long l
     else if (!out || out_dtype == RB_F32) { if (xf) RB_ON(float, float); else RB_ON(float, __nv_bfloat16); }
     else return RB_ERR_BAD_DTYPE;
 #undef RB_ON
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+extern "C" int rb_pair_norm(const float* da, int na, long long sa, const float* db, int nb, long long sb, const float* wa, const float* wb,
+                            float eps_in, float factor, float* out_v, float* resid, const float* w, float eps, float mult, void* out,
+                            int out_dtype, int n_rows, int H, void* stream) {
+    if (n_rows <= 0) return RB_OK;
+    if (H <= 0 || !da || !db || na < 1 || nb < 1 || !wa || !wb || (w ? !resid : !out_v)) return RB_ERR_BAD_SIZE;
+    const size_t smem = (size_t)(2 * ((H + 3) & ~3) + 66) * sizeof(float);
+    if (smem > 200 * 1024) return RB_ERR_BAD_SIZE;
+    const int vec = (H & 3) == 0 && (((uintptr_t)da | (uintptr_t)db) & 15) == 0 && ((sa | sb) & 3) == 0;
+    int threads = (H + 31) & ~31;
+    const int most = n_rows > 256 ? 256 : 1024;
+    threads = threads < 64 ? 64 : (threads > most ? most : threads);
+#define RB_PN(OT)                                                                                                                  \
+    do {                                                                                                                           \
+        auto k = pair_norm_kernel<OT>;                                                                                             \
+        cudaError_t e = allow_smem(k, smem);                                                                                       \
+        if (e != cudaSuccess) return (int)e;                                                                                       \
+        RB_LAUNCH((k), dim3(n_rows), dim3(threads), smem, (cudaStream_t)stream, da, na, (size_t)sa, db, nb, (size_t)sb, wa, wb,    \
+                  eps_in, factor, out_v, resid, w, eps, mult, (OT*)out, H, vec);                                                   \
+    } while (0)
+    if (!out || out_dtype == RB_F32) RB_PN(float);
+    else if (out_dtype == RB_BF16) RB_PN(__nv_bfloat16);
+    else return RB_ERR_BAD_DTYPE;
+#undef RB_PN
     RB_LAUNCH_CHECK();
     return RB_OK;
 }

@@ -19,7 +19,9 @@
 // general kernel: `post_norm`, queries and keys divided by their root mean square over the head after the rotation
 // (no weight); `v_out`, the value heads as they came from the projection, 32-bit [T, nkv * vd], for later layers;
 // `v_first` and `v_lambda`, such rows of an earlier layer and a factor on the device: what is stored is
-// (1 - lambda) v + lambda v_first; `temp_coef` != 0: queries times 1 + temp_coef ln(floor((pos + 1) / temp_every) + 1).  The table of cosines and sines may carry a common factor (the position
+// (1 - lambda) v + lambda v_first; `temp_coef` != 0: queries times 1 + temp_coef ln(floor((pos + 1) / temp_every) + 1); `maps` > 1: a head has that many queries and
+// keys of `hd` entries, [map 0 | map 1 ..], normalised and turned each on its own; a stored key head holds its maps side by side, and a
+// query becomes one row a map with its entries in that map's place and zeros in the others', so that each row scores its own map.  The table of cosines and sines may carry a common factor (the position
 // encoding's magnitude); the kernel's own sincosf path has none.
 #include "common.cuh"
 #include "api.h"
@@ -41,14 +43,15 @@ __global__ void qk_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, s
                                           const float2* __restrict__ cs_table, int vd, int hdp, int interleaved,
                                           int n_gate, float* __restrict__ gate_out, int post_norm,
                                           const float* __restrict__ v_first, const float* __restrict__ v_lambda,
-                                          float* __restrict__ v_out, float temp_coef, float temp_every) {
+                                          float* __restrict__ v_out, float temp_coef, float temp_every, int maps) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float smem[];
     const int warps_per_block = blockDim.x >> 5;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* buf = smem + (size_t)warp * hdp;
-    const int kv_heads = write_kv ? 2 * nkv : 0;
+    const int n_keys = nkv * maps;                 // key heads in the row: `maps` of them share a stored head
+    const int kv_heads = write_kv ? n_keys + nkv : 0;
     const int heads_total = nq + kv_heads + (n_gate > 0 ? 1 : 0);
     const long long item = (long long)blockIdx.x * warps_per_block + warp;
     if (item >= (long long)T * heads_total) return;
@@ -60,7 +63,7 @@ __global__ void qk_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, s
 
     if (h >= nq + kv_heads) {
         // the gates: the row's last n_gate columns, sigmoid in 32-bit
-        const IT* g = in + (size_t)t * row_stride + (size_t)nq * hd + (write_kv ? (size_t)nkv * (hd + vd) : 0);
+        const IT* g = in + (size_t)t * row_stride + (size_t)nq * hd + (write_kv ? (size_t)n_keys * hd + (size_t)nkv * vd : 0);
         for (int i = lane; i < n_gate; i += 32) {
             float v = 0.f;
             for (int s = 0; s < n_in; ++s) v += to_f32(g[(size_t)s * in_stride + i]);
@@ -70,9 +73,11 @@ __global__ void qk_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, s
     }
     int kind, head;  // 0 q, 1 k, 2 v
     if (h < nq) { kind = 0; head = h; }
-    else if (h < nq + nkv) { kind = 1; head = h - nq; }
-    else { kind = 2; head = h - nq - nkv; }
-    const IT* src = in + (size_t)t * row_stride + (kind == 2 ? (size_t)(nq + nkv) * hd + (size_t)head * vd : (size_t)h * hd);
+    else if (h < nq + n_keys) { kind = 1; head = h - nq; }
+    else { kind = 2; head = h - nq - n_keys; }
+    const IT* src = in + (size_t)t * row_stride + (kind == 2 ? (size_t)(nq + n_keys) * hd + (size_t)head * vd : (size_t)h * hd);
+    const int map = kind == 2 ? 0 : head % maps, off = map * hd;      // where this map's entries lie inside the head
+    if (kind == 1) head /= maps;
     if (kind == 2) hd = vd;     // from here on: the width of this head in the row
 
     AT* dst = nullptr;
@@ -84,7 +89,13 @@ __global__ void qk_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, s
         if (page >= 0) dst = (kind == 1 ? k_cache : v_cache) + (((size_t)page * nkv + head) * RB_PAGE + (pos % RB_PAGE)) * hdp;
         else if (kind == 1 || !v_out) return;
     }
-    if (dst) for (int i = hd + lane; i < hdp; i += 32) dst[i] = from_f32<AT>(0.f);
+    if (dst) {
+        // zeros around a query's own map; behind a stored head's last map; behind the values
+        const int z0 = kind == 0 || map == maps - 1 || kind == 2 ? off + hd : hdp;
+        for (int i = z0 + lane; i < hdp; i += 32) dst[i] = from_f32<AT>(0.f);
+        if (kind == 0) for (int i = lane; i < off; i += 32) dst[i] = from_f32<AT>(0.f);
+        dst += off;
+    }
 
     float ss = 0.f;
     if (n_in > 1 && sizeof(IT) == 4 && (hd & 3) == 0 && (in_stride & 3) == 0 && (row_stride & 3) == 0 &&
@@ -349,13 +360,13 @@ static int launch_qk(const void* in, int n_in, long long in_stride, int row_stri
                      const float* inv_freq, int rot_dim, const int* positions, const int* slot_of_token,
                      const int* block_table, int max_pages, void* k_cache, void* v_cache, int write_kv,
                      const float2* cs_table, int vd, int hdp, int interleaved, int n_gate, float* gate_out, int post_norm,
-                     const float* v_first, const float* v_lambda, float* v_out, float temp_coef, float temp_every, cudaStream_t s) {
+                     const float* v_first, const float* v_lambda, float* v_out, float temp_coef, float temp_every, int maps, cudaStream_t s) {
     const int warps = 4;
-    const long long items = (long long)T * (nq + (write_kv ? 2 * nkv : 0) + (n_gate > 0 ? 1 : 0));
+    const long long items = (long long)T * (nq + (write_kv ? nkv * (maps + 1) : 0) + (n_gate > 0 ? 1 : 0));
     const long long blocks = (items + warps - 1) / warps;
     if (blocks > 0x7fffffffLL) return RB_ERR_BAD_SIZE;
     const size_t esz = sizeof(IT);
-    if (hd == 128 && vd == 128 && hdp == 128 && n_gate == 0 && !(inv_freq && interleaved) &&
+    if (maps == 1 && hd == 128 && vd == 128 && hdp == 128 && n_gate == 0 && !(inv_freq && interleaved) &&
         (!inv_freq || rot_dim % 8 == 0) && (((uintptr_t)in | (uintptr_t)q_out | (uintptr_t)k_cache |
                                                           (uintptr_t)v_cache | (uintptr_t)qw | (uintptr_t)kw |
                                                           (uintptr_t)cs_table | (uintptr_t)v_first | (uintptr_t)v_out) & 15) == 0 &&
@@ -378,7 +389,7 @@ static int launch_qk(const void* in, int n_in, long long in_stride, int row_stri
               n_in, (size_t)in_stride, row_stride, (AT*)q_out, q_stride, T, nq, nkv, hd, (const WT*)qw,
               (const WT*)kw, eps, inv_freq, rot_dim, positions, slot_of_token, block_table, max_pages,
               (AT*)k_cache, (AT*)v_cache, write_kv, cs_table, vd, hdp, interleaved, n_gate, gate_out, post_norm,
-              v_first, v_lambda, v_out, temp_coef, temp_every);
+              v_first, v_lambda, v_out, temp_coef, temp_every, maps);
     return RB_OK;
 }
 
@@ -389,19 +400,20 @@ extern "C" int rb_qk_norm_rope_cache(const void* in, int in_dtype, int n_in, lon
                                      const int* slot_of_token, const int* block_table, int max_pages,
                                      void* k_cache, void* v_cache, int write_kv, const void* cos_sin, int vd, int hdp,
                                      int interleaved, int n_gate, float* gate_out, int post_norm, const float* v_first,
-                                     const float* v_lambda, float* v_out, float temp_coef, float temp_every, void* stream) {
+                                     const float* v_lambda, float* v_out, float temp_coef, float temp_every, int maps, void* stream) {
     if (T <= 0) return RB_OK;
     if (temp_coef != 0.f && !(temp_every > 0.f)) return RB_ERR_BAD_SIZE;
     if (vd <= 0) vd = hd;
-    if (hdp <= 0) hdp = hd > vd ? hd : vd;
-    if (hd <= 0 || n_in < 1 || hdp < hd || hdp < vd || (inv_freq && (rot_dim <= 0 || rot_dim % 2 || rot_dim > hd)) ||
+    if (maps < 1 || (maps > 1 && nq % maps)) return RB_ERR_BAD_SIZE;
+    if (hdp <= 0) hdp = hd * maps > vd ? hd * maps : vd;
+    if (hd <= 0 || n_in < 1 || hdp < hd * maps || hdp < vd || (inv_freq && (rot_dim <= 0 || rot_dim % 2 || rot_dim > hd)) ||
         n_gate < 0 || (n_gate > 0 && !gate_out) || (v_first && !v_lambda) || ((v_first || v_out) && !write_kv))
         return RB_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
 #define RB_QK_ARGS in, n_in, in_stride, row_stride, q_out, q_stride, T, nq, nkv, hd, q_norm_w, k_norm_w, eps, \
                    inv_freq, rot_dim, positions, slot_of_token, block_table, max_pages, k_cache, v_cache, write_kv, \
-                   (const float2*)cos_sin, vd, hdp, interleaved, n_gate, gate_out, post_norm, v_first, v_lambda, v_out, temp_coef, temp_every, s
+                   (const float2*)cos_sin, vd, hdp, interleaved, n_gate, gate_out, post_norm, v_first, v_lambda, v_out, temp_coef, temp_every, maps, s
     if (in_dtype == RB_BF16 && act_dtype == RB_BF16 && w_dtype == RB_BF16) return launch_qk<bf, bf, bf>(RB_QK_ARGS);
     if (in_dtype == RB_BF16 && act_dtype == RB_BF16 && w_dtype == RB_F32) return launch_qk<bf, bf, float>(RB_QK_ARGS);
     if (in_dtype == RB_F32 && act_dtype == RB_BF16 && w_dtype == RB_BF16) return launch_qk<float, bf, bf>(RB_QK_ARGS);

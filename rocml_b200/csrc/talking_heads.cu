@@ -1,5 +1,5 @@
-// Attention whose heads' weights are mixed after the softmax, and whose queries and keys are normalised over the
-// whole projection.
+// Attention whose heads' weights are mixed after the softmax, whose queries and keys are normalised over the
+// whole projection, or whose heads take the difference of two maps.
 //
 // With a'_h = sum_g M[h][g] a_g and head h reading the values of its own key/value head m(h), the result is
 // o_h = sum_g M[h][g] (sum_j a_g(i, j) v_m(h)(j)): every query head's weights applied to the values of every stored
@@ -13,6 +13,8 @@
 //                 the token's place in the paged cache, padded alike.  32-bit until the stores.  One block a token.
 //   talk_mix      out[t][h][:] = sum_g M[h][g] * o[t][pair (g, m(h))][:], 32-bit sums, padding dropped.  Prompts: a block a
 //                 token with the token's pair results in shared memory; few tokens: a thread four values, straight from memory.
+//   diff_heads    out[t][h][:] = rms(o[t][2h][:] - lambda o[t][2h + 1][:]) * factor over the head's values (no weight): two maps
+//                 of a head over the same values; padding dropped.  A warp a (token, head), 32-bit.
 #include "common.cuh"
 #include "api.h"
 
@@ -208,6 +210,50 @@ __global__ void talk_mix_kernel(const AT* __restrict__ o, int o_stride, const fl
     }
     out[(size_t)t * out_stride + (size_t)h * vd + d] = from_f32<AT>(acc);
 }
+constexpr int DIFF_MAX_WIDTH = 512;
+template <typename AT>
+__global__ void __launch_bounds__(256)
+diff_heads_kernel(const AT* __restrict__ o, int o_stride, float lambda, float eps, float factor, AT* __restrict__ out, int out_stride,
+                  int heads, int hdp, int vd, const int* __restrict__ slot_of_token, int T) {
+    pdl_trigger();
+    pdl_wait();
+    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (item >= (long long)T * heads) return;
+    const int t = (int)(item / heads), h = (int)(item - (long long)t * heads);
+    if (slot_of_token[t] < 0) return;
+    const AT* a = o + (size_t)t * o_stride + (size_t)(2 * h) * hdp;
+    const AT* b = a + hdp;
+    AT* dst = out + (size_t)t * out_stride + (size_t)h * vd;
+    constexpr int G = DIFF_MAX_WIDTH / 128;
+    float ss = 0.f;
+    if ((vd & 3) == 0 && (hdp & 3) == 0 && (o_stride & 3) == 0 && (out_stride & 3) == 0 &&
+        (((uintptr_t)o | (uintptr_t)out) & (4 * sizeof(AT) - 1)) == 0) {
+        float v[G][4], w[G][4];
+#pragma unroll
+        for (int g = 0; g < G; ++g) {
+            const int i = (g * 32 + lane) * 4;
+            if (i < vd) { load4(a + i, v[g]); load4(b + i, w[g]); }
+            else { v[g][0] = v[g][1] = v[g][2] = v[g][3] = 0.f; w[g][0] = w[g][1] = w[g][2] = w[g][3] = 0.f; }
+        }
+#pragma unroll
+        for (int g = 0; g < G; ++g)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) { v[g][u] = fmaf(-lambda, w[g][u], v[g][u]); ss = fmaf(v[g][u], v[g][u], ss); }
+        const float inv = rsqrtf(warp_sum(ss) / (float)vd + eps) * factor;
+#pragma unroll
+        for (int g = 0; g < G; ++g) {
+            const int i = (g * 32 + lane) * 4;
+#pragma unroll
+            for (int u = 0; u < 4; ++u) v[g][u] *= inv;
+            if (i < vd) store4(dst + i, v[g]);
+        }
+        return;
+    }
+    for (int i = lane; i < vd; i += 32) { const float v = fmaf(-lambda, to_f32(b[i]), to_f32(a[i])); ss = fmaf(v, v, ss); }
+    const float inv = rsqrtf(warp_sum(ss) / (float)vd + eps) * factor;
+    for (int i = lane; i < vd; i += 32) dst[i] = from_f32<AT>(fmaf(-lambda, to_f32(b[i]), to_f32(a[i])) * inv);
+}
 }  // namespace
 
 extern "C" int rb_wide_norm_rope_cache(const void* in, int in_dtype, int n_in, long long in_stride, int row_stride, int nq,
@@ -294,6 +340,23 @@ extern "C" int rb_talk_mix(const void* o, int o_stride, const float* mix, void* 
                   out_stride, nq, nkv, hdp, vd, slot_of_token, T);
     else
         return RB_ERR_BAD_DTYPE;
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+extern "C" int rb_diff_heads(const void* o, int o_stride, float lambda, float eps, float factor, void* out, int out_stride, int heads, int hdp,
+                             int vd, int dtype, const int* slot_of_token, int T, void* stream) {
+    if (T <= 0) return RB_OK;
+    if (heads <= 0 || vd <= 0 || hdp < vd || vd > DIFF_MAX_WIDTH) return RB_ERR_BAD_SIZE;
+    const long long blocks = ((long long)T * heads + 7) / 8;
+    if (blocks > 0x7fffffffLL) return RB_ERR_BAD_SIZE;
+#define RB_DH(AT)                                                                                                                  \
+    RB_LAUNCH((diff_heads_kernel<AT>), dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, (const AT*)o, o_stride, lambda, \
+              eps, factor, (AT*)out, out_stride, heads, hdp, vd, slot_of_token, T)
+    if (dtype == RB_BF16) RB_DH(__nv_bfloat16);
+    else if (dtype == RB_F32) RB_DH(float);
+    else return RB_ERR_BAD_DTYPE;
+#undef RB_DH
     RB_LAUNCH_CHECK();
     return RB_OK;
 }

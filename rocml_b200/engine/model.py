@@ -12,6 +12,7 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import kernels
+from ..cache.requirements import BundleRequirement, KVRequirement
 from ..profile import scope
 from ..config.specs import MixerSpec, ModelSpec
 from ..errors import ConfigError
@@ -136,8 +137,21 @@ class Model:
 
     def cache_requirements(self):
         # an arrangement that keeps something of its own a sequence (the row of the token before) answers for its layer
-        return [getattr(self.blocks[e.layer], "cache_requirement", self.blocks[e.layer].mixer.cache_requirement)()
-                for e in self.spec.schedule]
+        out = [getattr(self.blocks[e.layer], "cache_requirement", self.blocks[e.layer].mixer.cache_requirement)()
+               for e in self.spec.schedule]
+        # a run that reads another's keys may see further back than the one that keeps them: the keeper's cache serves both
+        for i, src in enumerate(self.reads_cache_of()):
+            if src is None:
+                continue
+            keeper, reader = out[src], out[i]
+            mine = keeper.main if isinstance(keeper, BundleRequirement) else keeper
+            if isinstance(mine, KVRequirement) and isinstance(reader, KVRequirement):
+                try:
+                    mine = mine.covering(reader)
+                except ValueError as e:
+                    raise ConfigError(f"schedule entry {i}: {e}") from None
+                out[src] = BundleRequirement(mine, keeper.extras) if isinstance(keeper, BundleRequirement) else mine
+        return out
 
     def reads_cache_of(self):
         return [e.reads_cache_of for e in self.spec.schedule]

@@ -131,23 +131,23 @@ def _lib():
         lib.rb_cast.argtypes = [_vp, _i, _vp, _i, _ll, _vp]
         lib.rb_qk_norm_rope_cache.argtypes = [_vp, _i, _i, _ll, _i, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _f,
                                               _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _i, _i, _vp, _i, _vp,
-                                              _vp, _vp, _f, _f, _vp]
+                                              _vp, _vp, _f, _f, _i, _vp]
         lib.rb_rope_table.argtypes = [_vp, _vp, _i, _i, _f, _vp, _vp]
         lib.rb_gemm_generic.argtypes = [_vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _ll, _ll, _i, _ll, _vp]
         lib.rb_attention_generic.argtypes = [_vp, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i,
-                                             _i, _i, _i, _f, _i, _i, _f, _vp, _i, _i, _vp, _vp, _i, _vp]
+                                             _i, _i, _i, _f, _i, _i, _f, _vp, _f, _i, _i, _vp, _vp, _i, _vp]
         lib.rb_attention_merge.argtypes = [_vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp]
         lib.rb_argmax.argtypes = [_vp, _ll, _i, _i, _vp, _vp, _vp, _i, _vp]
         lib.rb_attention_prefill.argtypes = [_vp, _i, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i,
-                                             _f, _i, _i, _f, _vp, _vp]
+                                             _f, _i, _i, _f, _vp, _f, _vp]
         lib.rb_attention_prefill_tc5.argtypes = [_vp, _i, _i, _vp, _i, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i,
-                                                 _i, _i, _i, _f, _i, _i, _f, _vp, _i, _vp, _vp, _ll, _i, _vp]
-        lib.rb_attention_decode.argtypes = [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _f, _vp, _i,
+                                                 _i, _i, _i, _f, _i, _i, _f, _vp, _f, _i, _vp, _vp, _ll, _i, _vp]
+        lib.rb_attention_decode.argtypes = [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _f, _vp, _f, _i,
                                             _i, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _ll, _ll, _i, _vp]
         lib.rb_attention_decode_fused.argtypes = [_vp, _i, _ll, _i, _vp, _vp, _i, _f, _vp, _i, _vp, _i, _ll, _f, _i,
                                                   _vp, _vp, _vp, _i, _vp, _vp,
                                                   _vp, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _vp, _vp, _vp, _i,
-                                                  _i, _f, _vp, _f, _f, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _ll, _ll, _vp]
+                                                  _i, _f, _vp, _f, _f, _f, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _ll, _ll, _vp]
         lib.rb_sample.argtypes = [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp]
         lib.rb_gemm_tcgen05.argtypes = [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _ll, _ll, _i, _ll, _i, _i, _vp, _vp]
         lib.rb_gemm_tcgen05_add.argtypes = [_vp, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _i, _vp, _vp]
@@ -179,7 +179,7 @@ def _lib():
         lib.rb_decay_scan_blocks.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _i,
                                              _i, _vp, _vp, _i, _vp]
         lib.rb_group_norm_gate.argtypes = [_vp, _i, _vp, _i, _i, _ll, _i, _i, _vp, _i, _f, _i, _i, _i, _vp, _i, _i, _vp,
-                                           _i, _vp]
+                                           _i, _vp, _vp]
         lib.rb_postln.argtypes = [_vp, _vp, _i, _ll, _vp, _vp, _f, _f, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp]
         lib.rb_token_shift.argtypes = [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _vp]
         lib.rb_causal_conv.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _vp]
@@ -196,6 +196,18 @@ def _lib():
         lib.rb_talk_mix.argtypes = [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp]
         lib.rb_moe_route_few.argtypes = [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _vp,
                                          _vp, _vp]
+        lib.rb_diff_heads.argtypes = [_vp, _i, _f, _f, _f, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp]
+        lib.rb_unary_act.argtypes = [_vp, _i, _i, _ll, _vp, _i, _ll, _i, _vp]
+        lib.rb_pair_norm.argtypes = [_vp, _i, _ll, _vp, _i, _ll, _vp, _vp, _f, _f, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _i, _vp]
+        lib.rb_mlstm_gates.argtypes = [_vp, _i, _ll, _i, _i, _i, _f, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp]
+        lib.rb_mlstm_step.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _vp, _i, _ll, _i, _i, _i, _f, _f, _f, _i, _i, _i, _vp, _vp,
+                                      _vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _vp]
+        lib.rb_mlstm_blocks.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp,
+                                        _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp]
+        lib.rb_rglru_gates.argtypes = [_vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp]
+        lib.rb_rglru_scan.argtypes = [_vp, _vp, _i, _vp, _i, _i, _ll, _i, _f, _vp, _vp, _vp, _i, _vp, _i, _i, _vp]
+        lib.rb_rglru_step.argtypes = [_vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _ll, _i, _f, _vp, _vp, _vp, _i,
+                                      _i, _vp]
         lib.rb_softcap.argtypes = [_vp, _ll, _f, _f, _vp]
         lib.rb_add_layernorm.argtypes = [_vp, _vp, _i, _ll, _vp, _vp, _vp, _i, _vp, _i, _i, _f, _i, _vp]
         lib.rb_out_norm.argtypes = [_vp, _vp, _i, _ll, _f, _vp, _vp, _i, _vp, _vp, _i, _i, _vp, _vp, _f, _f, _vp, _i, _i, _i, _vp]
@@ -326,7 +338,7 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_out: torch.Tensor, n_tokens: int, n
                        padded_head_dim: Optional[int] = None, interleaved: bool = False,
                        gates: Optional[torch.Tensor] = None, post_norm: bool = False,
                        v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None,
-                       v_out: Optional[torch.Tensor] = None, q_temp=None):
+                       v_out: Optional[torch.Tensor] = None, q_temp=None, maps: int = 1):
     """``cos_sin`` (from rope_table, float32 [T, rot_dim / 2, 2]) replaces the kernel's own sincosf.
     proj [T, nq*hd (+ nkv*hd + nkv*vd) (+ gates)] (or [S, T, ...] partial sums): q normalised and rotated into
     q_out (rows of nq*hdp, any row stride; it may be ``proj`` itself when nothing is padded); k (normalised,
@@ -337,11 +349,13 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_out: torch.Tensor, n_tokens: int, n
     mean square over the head (eps inside the root, no weight) after the rotation.  ``v_out`` (float32 [T, nkv * vd])
     receives the value heads as projected; ``v_first`` (such rows of an earlier layer) and ``v_lambda`` (float32,
     one number on the device): the cache receives (1 - lambda) v + lambda v_first.  ``q_temp`` (coef, every): queries are
-    multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p, after everything else."""
+    multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p, after everything else.  ``maps`` > 1: ``nq`` counts the
+    queries of all maps, nq = maps * heads, head by head; a stored key head is ``maps`` keys of hd side by side (hdp >= maps * hd), a
+    query's row has its entries in its own map's place and zeros in the others'."""
     vd = hd if v_head_dim is None else int(v_head_dim)
-    hdp = max(hd, vd) if padded_head_dim is None else int(padded_head_dim)
+    hdp = max(hd * maps, vd) if padded_head_dim is None else int(padded_head_dim)
     n_gate = 0 if gates is None else gates.shape[-1]
-    width = nq * hd + (nkv * (hd + vd) if write_kv else 0)
+    width = nq * hd + (nkv * (maps * hd + vd) if write_kv else 0)
     n_in, in_stride, row_stride = _partials(proj, "qk_norm_rope_cache")
     if proj.shape[-1] < width + n_gate:
         raise KernelError(f"qk_norm_rope_cache: projections must be at least {width + n_gate} wide")
@@ -377,7 +391,7 @@ def qk_norm_rope_cache(proj: torch.Tensor, q_out: torch.Tensor, n_tokens: int, n
         rot_dim, _i32(positions, "positions"), _i32(slot_of_token, "slot_of_token"),
         None if block_table is None else _i32(block_table, "block_table"), max_pages, _ptr(k_cache), _ptr(v_cache),
         1 if write_kv else 0, _ptr(cos_sin), vd, hdp, 1 if interleaved else 0, n_gate, _ptr(gates),
-        1 if post_norm else 0, _ptr(v_first), _ptr(v_lambda), _ptr(v_out), *_temperature(q_temp), _stream())
+        1 if post_norm else 0, _ptr(v_first), _ptr(v_lambda), _ptr(v_out), *_temperature(q_temp), int(maps), _stream())
     _check(rc, "qk_norm_rope_cache")
 
 
@@ -429,10 +443,11 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                       block_table: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                       n_seqs: int, max_q_len: int, nq: int, nkv: int, hd: int, scale: float, window: int = 0,
                       chunk: int = 0, n_chunks: int = 1, part_acc: Optional[torch.Tensor] = None,
-                      part_ml: Optional[torch.Tensor] = None, keep: int = 0, sink=None, cross: int = 0):
+                      part_ml: Optional[torch.Tensor] = None, keep: int = 0, sink=None, cross: int = 0, softcap: float = 0.0):
     """q rows [T, >= nq*hd] (row stride free) -> out rows [T, >= nq*hd]; keys and values from the pages.
     ``keep``: the keys at positions below it stay visible beside the window; ``sink``: a score that adds
-    exp(sink) to every row's denominator and brings no value (None: no such term; a float32 tensor [nq]: one a query head).  ``cross`` (n > 1, the cache's
+    exp(sink) to every row's denominator and brings no value (None: no such term; a float32 tensor [nq]: one a query head).
+    ``softcap`` > 0: scores become softcap * tanh(score / softcap).  ``cross`` (n > 1, the cache's
     own number of key/value heads): every query head's weights are applied to the values of EVERY stored head;
     ``nkv`` = n * n then counts (key head, value head) pairs, ``nq`` = n * query heads the results, pair
     (a, m) at a * n + m with the results of key head a's queries in their order, and q holds nq / n heads."""
@@ -445,7 +460,7 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), dtype_code(q.dtype), _ptr(k_cache), _ptr(v_cache),
         _i32(block_table, "block_table"), block_table.shape[1], _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"),
         _i32(kv_len, "kv_len"), n_seqs, max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), *_sink(sink, nq),
-        int(chunk), int(n_chunks), _ptr(part_acc), _ptr(part_ml), int(cross), _stream())
+        float(softcap), int(chunk), int(n_chunks), _ptr(part_acc), _ptr(part_ml), int(cross), _stream())
     _check(rc, "attention_generic")
 
 
@@ -489,7 +504,7 @@ def attention_prefill_tc5(q: torch.Tensor, n_tokens: int, out: torch.Tensor, k_c
                           block_table: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                           n_seqs: int, max_q_len: int, nq: int, nkv: int, hd: int, scale: float, window: int = 0,
                           max_kv_len: Optional[int] = None, keep: int = 0, sink=None,
-                          gate: Optional[torch.Tensor] = None, cross: int = 0) -> bool:
+                          gate: Optional[torch.Tensor] = None, cross: int = 0, softcap: float = 0.0) -> bool:
     """bfloat16 flash attention with tcgen05 (accumulators in tensor memory, TMA loads), head sizes 64, 128 and 256.
     ``cross`` (n > 1, the cache's own number of key/value heads): as in ``attention_generic``.
     ``keep``: beside a window the keys at positions below it stay visible; ``sink``: a score whose exponential
@@ -512,7 +527,7 @@ def attention_prefill_tc5(q: torch.Tensor, n_tokens: int, out: torch.Tensor, k_c
         _ptr(q), q.stride(0), n_tokens, _ptr(out), out.stride(0), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0],
         _i32(block_table, "block_table"), block_table.shape[1], _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"),
         _i32(kv_len, "kv_len"), n_seqs, max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), *_sink(sink, nq),
-        1 if prefill_heads_first(n_seqs, nkv, hd, max_q_len if max_kv_len is None else max_kv_len, window) else 0,
+        float(softcap), 1 if prefill_heads_first(n_seqs, nkv, hd, max_q_len if max_kv_len is None else max_kv_len, window) else 0,
         _ptr(status_word(q.device)), _ptr(gate), gate.stride(0) if gate is not None else 0, int(cross), _stream())
     if rc in (10001, 10003):
         return False
@@ -524,7 +539,7 @@ def attention_prefill_tc5(q: torch.Tensor, n_tokens: int, out: torch.Tensor, k_c
 def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       block_table: torch.Tensor, seq_slot: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                       n_seqs: int, max_q_len: int, nq: int, nkv: int, hd: int, scale: float, window: int = 0,
-                      keep: int = 0, sink=None) -> bool:
+                      keep: int = 0, sink=None, softcap: float = 0.0) -> bool:
     """bfloat16 flash attention on the tensor cores for any number of query tokens per sequence.
     ``keep``: beside a window the keys at positions below it stay visible; ``sink``: a score whose exponential
     joins every row's denominator.
@@ -537,7 +552,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     rc = _lib().rb_attention_prefill(
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_cache), _ptr(v_cache), _i32(block_table, "block_table"),
         block_table.shape[1], _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), _i32(kv_len, "kv_len"), n_seqs,
-        max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), *_sink(sink, nq), _stream())
+        max_q_len, nq, nkv, hd, float(scale), int(window), int(keep), *_sink(sink, nq), float(softcap), _stream())
     if rc in (10001, 10003):
         return False
     _check(rc, "attention_prefill")
@@ -607,7 +622,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
                      n_seqs: int, nq: int, nkv: int, hd: int, scale: float, window: int, n_chunks: int,
                      part_acc: Optional[torch.Tensor], part_ml: Optional[torch.Tensor],
                      pages_per_block: int = 1, keep: int = 0, sink=None,
-                     gate: Optional[torch.Tensor] = None, cross: int = 0) -> bool:
+                     gate: Optional[torch.Tensor] = None, cross: int = 0, softcap: float = 0.0) -> bool:
     """``cross`` (n > 1, the cache's own number of key/value heads): as in ``attention_generic``.  ``keep``: the keys at positions below it stay visible beside the window (not with ``pages_per_block`` 0);
     ``sink``: a score whose exponential joins every row's denominator.  ``gate``: [T, nq * hd] or [S, T, nq * hd]
     (partial sums, added in order) columns of the projection rows, bfloat16 or float32, unit stride along a row: the
@@ -636,7 +651,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
     rc = _lib().rb_attention_decode(
         _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _i32(block_table, "block_table"), block_table.shape[1],
         _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), _i32(kv_len, "kv_len"), n_seqs, nq, nkv, hd, float(scale),
-        int(window), int(keep), *_sink(sink, nq), int(n_chunks), int(pages_per_block), _ptr(part_acc), _ptr(part_ml),
+        int(window), int(keep), *_sink(sink, nq), float(softcap), int(n_chunks), int(pages_per_block), _ptr(part_acc), _ptr(part_ml),
         _ptr(decode_counters(q.device)), _ptr(out),
         out.stride(0), _ptr(gate), 1 if gate is not None and gate.dtype == torch.float32 else 0, g_n, g_in, g_row, int(cross),
         _stream())
@@ -656,7 +671,7 @@ def attention_decode_fused(proj: torch.Tensor, out: torch.Tensor, k_cache: torch
                            pages_per_block: int = 1, rowscale=None, row_width: int = 0, keep: int = 0,
                            sink=None, rot_dim: int = 0, post_norm: bool = False,
                            v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None,
-                           v_keep: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, q_temp=None) -> bool:
+                           v_keep: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, q_temp=None, softcap: float = 0.0) -> bool:
     """attention_decode for head size 128 that takes the step's projections as the matrix product left
     them: ``proj`` float32 [S, T, (nq + 2 nkv) * 128] partial sums (or [T, ...]; only the nq query heads
     when ``write_kv`` is off).  The kernel adds them, applies the per-head norm and the rotation
@@ -710,7 +725,7 @@ def attention_decode_fused(proj: torch.Tensor, out: torch.Tensor, k_cache: torch
         _ptr(k_cache), _ptr(v_cache), _i32(block_table, "block_table"), block_table.shape[1],
         _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), _i32(kv_len, "kv_len"), n_seqs, nq, nkv, hd, float(scale),
         int(window), int(n_chunks), int(pages_per_block), _ptr(part_acc), _ptr(part_ml),
-        _ptr(decode_counters(out.device)), _ptr(out), out.stride(0), int(keep), *_sink(sink, nq), *_temperature(q_temp), rot, 1 if post_norm else 0,
+        _ptr(decode_counters(out.device)), _ptr(out), out.stride(0), int(keep), *_sink(sink, nq), float(softcap), *_temperature(q_temp), rot, 1 if post_norm else 0,
         _ptr(v_first), _ptr(v_lambda), _ptr(v_keep), _ptr(gate), 1 if gate is not None and gate.dtype == torch.float32 else 0,
         g_n, g_in, g_row, _stream())
     if rc in (10001, 10003):
@@ -1379,11 +1394,15 @@ def decay_scan_blocks(proj: torch.Tensor, n_tokens: int, q_off: int, k_off: int,
 @_profiled(lambda a, facts: (a["n_tokens"] * a["o"].shape[1] * (4 + _esz(a["proj"]) * _n_in(a["proj"]) + _esz(a["out"])),
                              a["n_tokens"] * a["o"].shape[1] * 8))
 def group_norm_gate(o: torch.Tensor, proj: torch.Tensor, g_off: int, weight: Optional[torch.Tensor], eps: float, groups: int,
-                    gate_act: str, out: torch.Tensor, slot_of_token: torch.Tensor, n_tokens: int):
+                    gate_act: str, out: torch.Tensor, slot_of_token: torch.Tensor, n_tokens: int, divisor: Optional[torch.Tensor] = None):
     """out [T, W] = o / rms(o over each of ``groups`` equal column groups, eps inside the root) (* weight [W]) *
     act(gate), the gate being columns g_off .. g_off + W of ``proj`` (partial sums added first); ``gate_act`` "none",
-    "silu" or "sigmoid".  o float32; out in the activations' type."""
+    "silu" or "sigmoid".  o float32; out in the activations' type.  ``divisor`` float32 [T, groups]: o's groups are divided by it
+    before the norm."""
     W = o.shape[1]
+    if divisor is not None and (divisor.dtype != torch.float32 or not divisor.is_contiguous() or divisor.shape[-1] != groups or
+                                divisor.shape[0] < n_tokens):
+        raise KernelError("group_norm_gate: the divisor must be contiguous float32 [T, groups]")
     n_in, in_stride, row_stride = _partials(proj, "group_norm_gate")
     if o.dtype != torch.float32 or o.stride(1) != 1 or out.stride(1) != 1 or out.shape[1] != W or g_off + W > proj.shape[-1]:
         raise KernelError("group_norm_gate: o must be float32 [T, W], out [T, W], the gate inside the projection rows")
@@ -1392,7 +1411,7 @@ def group_norm_gate(o: torch.Tensor, proj: torch.Tensor, g_off: int, weight: Opt
     rc = _lib().rb_group_norm_gate(_ptr(o), o.stride(0), _ptr(proj), dtype_code(proj.dtype), n_in, in_stride, row_stride,
                                    g_off, _ptr(weight), dtype_code(weight.dtype) if weight is not None else F32, float(eps),
                                    groups, W, UNIT_ACTS[gate_act], _ptr(out), dtype_code(out.dtype), out.stride(0),
-                                   _i32(slot_of_token, "slot_of_token"), n_tokens, _stream())
+                                   _i32(slot_of_token, "slot_of_token"), n_tokens, _ptr(divisor), _stream())
     _check(rc, "group_norm_gate")
 
 
@@ -1945,3 +1964,199 @@ def low_rank(proj: torch.Tensor, n_tokens: int, x_off0: int, w0: torch.Tensor, x
     rc = _lib().rb_low_rank(_ptr(proj), dtype_code(proj.dtype), n_in, in_stride, row_stride, x_off0, r0, _ptr(w0), n0, x_off1, r1,
                             _ptr(w1), n1, dtype_code(w0.dtype), n_tokens, _ptr(out), out.stride(0), _stream())
     _check(rc, "low_rank")
+
+
+# ---- the difference of two maps, an activation on its own, the norm of two results --------------------------------------------
+
+@_profiled(lambda a, facts: (a["n_tokens"] * a["heads"] * 3 * a["vd"] * _esz(a["o"]), 5 * a["n_tokens"] * a["heads"] * a["vd"]))
+def diff_heads(o: torch.Tensor, lam: float, eps: float, factor: float, out: torch.Tensor, heads: int, hdp: int, vd: int,
+               slot_of_token: torch.Tensor, n_tokens: int):
+    """out[t, h, :vd] = rms(o[t, 2h, :vd] - lam * o[t, 2h + 1, :vd]) * factor (eps inside the root, no weight); ``o`` holds
+    2 * heads results of ``hdp`` entries a token."""
+    if o.dtype != out.dtype or o.stride(-1) != 1 or out.stride(-1) != 1 or o.shape[-1] < 2 * heads * hdp or out.shape[-1] < heads * vd:
+        raise KernelError("diff_heads: shapes or types do not fit")
+    rc = _lib().rb_diff_heads(_ptr(o), o.stride(0), float(lam), float(eps), float(factor), _ptr(out), out.stride(0), heads, hdp, vd,
+                              dtype_code(o.dtype), _i32(slot_of_token, "slot_of_token"), n_tokens, _stream())
+    _check(rc, "diff_heads")
+
+
+PLAIN_ACTS = {"gelu": 0, "gelu_tanh": 1, "silu": 2}
+
+
+@_profiled(lambda a, facts: (a["x"].numel() * _esz(a["x"]) + a["out"].numel() * _esz(a["out"]), a["out"].numel() * 10))
+def unary_act(x: torch.Tensor, out: torch.Tensor, kind: str):
+    """out [T, I] = act(x), x [T, I] or [S, T, I] partial sums that are added first; kinds "gelu" (with erf), "gelu_tanh", "silu"."""
+    n_in, in_stride, row_stride = _partials(x, "unary_act")
+    if tuple(out.shape) != tuple(x.shape[-2:]) or row_stride != x.shape[-1] or not out.is_contiguous():
+        raise KernelError("unary_act: shapes do not fit")
+    rc = _lib().rb_unary_act(_ptr(x), dtype_code(x.dtype), n_in, in_stride, _ptr(out), dtype_code(out.dtype), out.numel(),
+                             PLAIN_ACTS[kind], _stream())
+    _check(rc, "unary_act")
+
+
+def _partial_rows(d: torch.Tensor, n: int, H: int, what: str):
+    if d.dtype != torch.float32 or d.dim() != 3 or d.shape[1] < n or d.shape[2] != H or d.stride(2) != 1 or d.stride(1) != H:
+        raise KernelError(f"{what}: results must be float32 [S, >= T, H] with dense rows")
+    return _ptr(d), d.shape[0], d.stride(0)
+
+
+@_profiled(lambda a, facts: (a["n_rows"] * a["a"].shape[2] * 4 * (a["a"].shape[0] + a["b"].shape[0] + 2)
+                             + (a["n_rows"] * a["a"].shape[2] * _esz(a["out"]) if a["out"] is not None else 0), 10 * a["n_rows"] * a["a"].shape[2]))
+def pair_norm(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, eps_in: float, factor: float, n_rows: int,
+              out_v: Optional[torch.Tensor] = None, resid: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None,
+              eps: float = 0.0, mult: float = 1.0, out: Optional[torch.Tensor] = None):
+    """v = factor * (rms(a) * wa + rms(b) * wb) for two results a and b (float32 [S, >= T, H] partial sums; eps_in inside the
+    roots).  ``out_v`` float32 [T, H] receives v; or ``resid`` float32 [T, H] += mult * rms(v) * ``weight`` in place and ``out`` [T, H]
+    (optional) receives the new rows in its own type."""
+    H = a.shape[2]
+    pa, pb = _partial_rows(a, n_rows, H, "pair_norm"), _partial_rows(b, n_rows, H, "pair_norm")
+    for t, name in ((out_v, "out_v"), (resid, "resid")):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.shape[-1] != H or t.numel() < n_rows * H):
+            raise KernelError(f"pair_norm: {name} must be contiguous float32 [T, H]")
+    if (weight is None) == (out_v is None) or (weight is None) != (resid is None):
+        raise KernelError("pair_norm: give out_v, or resid with weight")
+    if out is not None and (not out.is_contiguous() or out.shape[-1] != H or out.numel() < n_rows * H):
+        raise KernelError("pair_norm: out must be contiguous [T, H]")
+    rc = _lib().rb_pair_norm(*pa, *pb, _f32vec(wa, H, "pair_norm: wa"), _f32vec(wb, H, "pair_norm: wb"), float(eps_in), float(factor),
+                             _ptr(out_v), _ptr(resid), _f32vec(weight, H, "pair_norm: weight"), float(eps), float(mult), _ptr(out),
+                             dtype_code(out.dtype) if out is not None else F32, n_rows, H, _stream())
+    _check(rc, "pair_norm")
+
+
+# ---- a matrix memory with exponential gates (mLSTM) ------------------------------------------------------------------------------
+
+MLSTM_BLOCK = 64        # tokens a block of mlstm_blocks
+
+
+def _mlstm_states(S, n, m, heads, dim, vdim, what):
+    for t, shape, name in ((S, (heads, dim, vdim), "S"), (n, (heads, dim), "n"), (m, (heads, 2), "m")):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or tuple(t.shape[1:]) != shape):
+            raise KernelError(f"{what}: the state {name} must be contiguous float32 [slots, {', '.join(map(str, shape))}]")
+
+
+def _gate_cols(gates, i_off, f_off, heads, what):
+    if gates.dtype != torch.float32 or max(i_off, f_off) + heads > gates.shape[-1]:
+        raise KernelError(f"{what}: gates must be float32 and hold {heads} columns from i_off and f_off")
+    return (_ptr(gates),) + _partials(gates, what)
+
+
+@_profiled(lambda a, facts: (a["n_tokens"] * a["heads"] * 4 * (2 * _n_in(a["gates"]) + 3), 30 * a["n_tokens"] * a["heads"]))
+def mlstm_gates(gates: torch.Tensor, n_tokens: int, i_off: int, f_off: int, cap: float, heads: int, m_state: torch.Tensor,
+                seq_slot: torch.Tensor, cu_q: torch.Tensor, positions: torch.Tensor, n_seqs: int, max_q_len: int,
+                log_keep: torch.Tensor, log_add: torch.Tensor, em: torch.Tensor):
+    """The log gates of a step's tokens from columns of ``gates`` (float32 [T, N] or [S, T, N] partial sums): log_keep, log_add and
+    em = e^(-m), float32 [heads, T] each; ``m_state`` float32 [slots, heads, 2] moves on."""
+    _mlstm_states(None, None, m_state, heads, 1, 1, "mlstm_gates")
+    for t in (log_keep, log_add, em):
+        if t.dtype != torch.float32 or not t.is_contiguous() or tuple(t.shape) != (heads, n_tokens):
+            raise KernelError("mlstm_gates: results must be contiguous float32 [heads, T]")
+    rc = _lib().rb_mlstm_gates(*_gate_cols(gates, i_off, f_off, heads, "mlstm_gates"), i_off, f_off, float(cap), heads, _ptr(m_state),
+                               _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), _i32(positions, "positions"), n_seqs, max_q_len,
+                               n_tokens, _ptr(log_keep), _ptr(log_add), _ptr(em), _stream())
+    _check(rc, "mlstm_gates")
+
+
+def _mlstm_cols(proj, q_off, k_off, v_off, heads, dim, vdim, out, den, n_tokens, what):
+    if max(q_off, k_off) + heads * dim > proj.shape[-1] or v_off + heads * vdim > proj.shape[-1]:
+        raise KernelError(f"{what}: the projection rows are too narrow")
+    if out.dtype != torch.float32 or out.stride(-1) != 1 or out.shape[-1] != heads * vdim or out.shape[0] < n_tokens:
+        raise KernelError(f"{what}: out must be float32 [T, heads * vdim]")
+    if den.dtype != torch.float32 or not den.is_contiguous() or den.shape[-1] != heads or den.shape[0] < n_tokens:
+        raise KernelError(f"{what}: den must be contiguous float32 [T, heads]")
+    return (_ptr(proj), dtype_code(proj.dtype)) + _partials(proj, what)
+
+
+@_profiled(lambda a, facts: _cost.mlstm(a["n_seqs"], a["n_seqs"], a["heads"], a["dim"], a["vdim"], _esz(a["proj"]) * _n_in(a["proj"])))
+def mlstm_step(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, i_off: int, f_off: int, cap: float,
+               q_scale: float, eps: float, heads: int, dim: int, vdim: int, S: torch.Tensor, n: torch.Tensor, m: torch.Tensor,
+               seq_slot: torch.Tensor, cu_q: torch.Tensor, positions: torch.Tensor, n_seqs: int, out: torch.Tensor, den: torch.Tensor):
+    """One token a sequence: the states S [slots, heads, dim, vdim], n [slots, heads, dim] and m [slots, heads, 2] (float32) take the
+    token's k v^T, k and gates; ``out`` float32 [T, heads * vdim] = S^T q and ``den`` float32 [T, heads] = max(|n . q|, e^(-m)) + eps."""
+    _mlstm_states(S, n, m, heads, dim, vdim, "mlstm_step")
+    cols = _mlstm_cols(proj, q_off, k_off, v_off, heads, dim, vdim, out, den, n_seqs, "mlstm_step")
+    rc = _lib().rb_mlstm_step(*cols, q_off, k_off, v_off, *_gate_cols(gates, i_off, f_off, heads, "mlstm_step"), i_off, f_off, float(cap),
+                              float(q_scale), float(eps), heads, dim, vdim, _ptr(S), _ptr(n), _ptr(m), _i32(seq_slot, "seq_slot"),
+                              _i32(cu_q, "cu_q"), _i32(positions, "positions"), n_seqs, _ptr(out), out.stride(0), _ptr(den), _stream())
+    _check(rc, "mlstm_step")
+
+
+@_profiled(lambda a, facts: _cost.mlstm(a["n_tokens"], a["n_seqs"], a["heads"], a["dim"], a["vdim"], _esz(a["proj"]) * _n_in(a["proj"])))
+def mlstm_blocks(proj: torch.Tensor, n_tokens: int, q_off: int, k_off: int, v_off: int, q_scale: float, eps: float, heads: int, dim: int,
+                 vdim: int, log_keep: torch.Tensor, log_add: torch.Tensor, em: torch.Tensor, S: torch.Tensor, n: torch.Tensor,
+                 seq_slot: torch.Tensor, cu_q: torch.Tensor, n_seqs: int, out: torch.Tensor, den: torch.Tensor):
+    """The same for prompts, from the gates of ``mlstm_gates``, by blocks of 64 tokens side by side."""
+    _mlstm_states(S, n, None, heads, dim, vdim, "mlstm_blocks")
+    cols = _mlstm_cols(proj, q_off, k_off, v_off, heads, dim, vdim, out, den, n_tokens, "mlstm_blocks")
+    blocks = n_tokens // MLSTM_BLOCK + n_seqs
+    work = torch.empty(blocks * heads * (dim * vdim + dim + 1 + MLSTM_BLOCK * MLSTM_BLOCK), dtype=torch.float32, device=proj.device)
+    sizes = [blocks * heads * MLSTM_BLOCK * MLSTM_BLOCK, blocks * heads * dim * vdim, blocks * heads * dim, blocks * heads]
+    scores, sums, sums_n, decay = torch.split(work, sizes)
+    rc = _lib().rb_mlstm_blocks(*cols, q_off, k_off, v_off, float(q_scale), float(eps), heads, dim, vdim, _ptr(log_keep), _ptr(log_add),
+                                _ptr(em), n_tokens, _ptr(S), _ptr(n), _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, blocks,
+                                _ptr(sums), _ptr(sums_n), _ptr(decay), _ptr(scores), _ptr(out), out.stride(0), _ptr(den), _stream())
+    _check(rc, "mlstm_blocks")
+
+
+# ---- a real-gated linear recurrent unit --------------------------------------------------------------------------------------------
+
+def _rglru_weights(u, ra, ri, ra_b, ri_b, rate, what):
+    blocks, part, _ = ra.shape
+    width = blocks * part
+    if tuple(ra.shape) != (blocks, part, part) or ri.shape != ra.shape or ri.dtype != ra.dtype or not ra.is_contiguous() or not ri.is_contiguous():
+        raise KernelError(f"{what}: the gates' weights must be two contiguous [blocks, part, part] tensors of one type")
+    if u.dtype != torch.float32 or u.stride(-1) != 1 or u.shape[-1] != width:
+        raise KernelError(f"{what}: u must be float32 [T, blocks * part]")
+    return (_ptr(u), u.stride(0), _ptr(ra), _ptr(ri), dtype_code(ra.dtype), _f32vec(ra_b, width, f"{what}: ra_b"),
+            _f32vec(ri_b, width, f"{what}: ri_b"), _f32vec(rate, width, f"{what}: rate"), blocks, part)
+
+
+def _branch(y, width, what):
+    if y.shape[-1] < width:
+        raise KernelError(f"{what}: the other branch's columns must be at least {width} wide")
+    return (_ptr(y), dtype_code(y.dtype)) + _partials(y, what)
+
+
+@_profiled(lambda a, facts: (a["n_tokens"] * a["u"].shape[1] * 12 + 2 * a["ra"].numel() * _esz(a["ra"]),
+                             4 * a["n_tokens"] * a["u"].shape[1] * a["ra"].shape[1]))
+def rglru_gates(u: torch.Tensor, n_tokens: int, ra: torch.Tensor, ri: torch.Tensor, ra_b: torch.Tensor, ri_b: torch.Tensor,
+                rate: torch.Tensor, a: torch.Tensor, x: torch.Tensor):
+    """Decay ``a`` = e^(rate * r) and input ``x`` = sqrt(1 - a^2) i u of every token and channel (float32 [T, width]), r and i the
+    sigmoids of the block products of ``u`` (float32 [T, width]) with ``ra`` and ``ri`` [blocks, part, part] plus their biases."""
+    args = _rglru_weights(u, ra, ri, ra_b, ri_b, rate, "rglru_gates")
+    for t in (a, x):
+        if t.dtype != torch.float32 or not t.is_contiguous() or t.shape[-1] != u.shape[-1] or t.shape[0] < n_tokens:
+            raise KernelError("rglru_gates: results must be contiguous float32 [T, width]")
+    _check(_lib().rb_rglru_gates(*args, n_tokens, _ptr(a), _ptr(x), _stream()), "rglru_gates")
+
+
+@_profiled(lambda a, facts: (a["n_tokens"] * a["a"].shape[1] * (8 + _esz(a["y"]) * _n_in(a["y"]) + _esz(a["out"])) + 8 * a["n_seqs"] * a["a"].shape[1],
+                             14 * a["n_tokens"] * a["a"].shape[1]))
+def rglru_scan(a: torch.Tensor, x: torch.Tensor, n_tokens: int, y: torch.Tensor, factor: float, state: torch.Tensor, seq_slot: torch.Tensor,
+               cu_q: torch.Tensor, n_seqs: int, out: torch.Tensor):
+    """S = a S + x along every sequence from ``state`` (float32 [slots, width], which receives the last one); ``out`` [T, width]
+    (any row stride) = S * gelu_tanh(y) * factor, y columns of the projection rows ([T, ..] or partial sums [S, T, ..])."""
+    width = a.shape[-1]
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (width,):
+        raise KernelError("rglru_scan: state must be contiguous float32 [slots, width]")
+    if out.stride(-1) != 1 or out.shape[-1] < width:
+        raise KernelError("rglru_scan: out must be [T, width]")
+    rc = _lib().rb_rglru_scan(_ptr(a), _ptr(x), width, *_branch(y, width, "rglru_scan"), float(factor), _ptr(state),
+                              _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, _ptr(out), dtype_code(out.dtype), out.stride(0),
+                              _stream())
+    _check(rc, "rglru_scan")
+
+
+@_profiled(lambda a, facts: (a["n_tokens"] * a["u"].shape[1] * (12 + _esz(a["y"]) * _n_in(a["y"]) + _esz(a["out"])) + 2 * a["ra"].numel() * _esz(a["ra"]),
+                             4 * a["n_tokens"] * a["u"].shape[1] * a["ra"].shape[1]))
+def rglru_step(u: torch.Tensor, n_tokens: int, ra: torch.Tensor, ri: torch.Tensor, ra_b: torch.Tensor, ri_b: torch.Tensor,
+               rate: torch.Tensor, y: torch.Tensor, factor: float, state: torch.Tensor, slot_of_token: torch.Tensor, out: torch.Tensor):
+    """One token a sequence: ``rglru_gates`` and ``rglru_scan`` in one kernel."""
+    args = _rglru_weights(u, ra, ri, ra_b, ri_b, rate, "rglru_step")
+    width = u.shape[-1]
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (width,):
+        raise KernelError("rglru_step: state must be contiguous float32 [slots, width]")
+    if out.stride(-1) != 1 or out.shape[-1] < width:
+        raise KernelError("rglru_step: out must be [T, width]")
+    rc = _lib().rb_rglru_step(*args, n_tokens, *_branch(y, width, "rglru_step"), float(factor), _ptr(state),
+                              _i32(slot_of_token, "slot_of_token"), _ptr(out), dtype_code(out.dtype), out.stride(0), _stream())
+    _check(rc, "rglru_step")

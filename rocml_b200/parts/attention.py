@@ -18,9 +18,16 @@ temperature that grows with their position (``q_temperature`` {coef, every}: 1 +
 norm and position encoding); queries and keys may be divided by their root mean square after the position
 encoding (``qk_unit_norm``); biases may be given for some of the projections only; and the values that
 a layer caches may be blended with those of an earlier layer of the same step (``value_mix``).
-Three more parameters form one path of their own (``_forward_wide``): ``qk_norm`` "whole" (queries and keys are each
+``softcap``: scores become softcap * tanh(score / softcap) before the softmax.  ``difference`` (a number d: differential attention):
+q and k hold two maps a head, [map 1 | map 2], each normalised and turned on its own; the head's result is rms(a1 - lambda a2) (1 - d)
+with a1 and a2 the two maps' attentions over the head's one set of values and lambda = e^(lq1 . lk1) - e^(lq2 . lk2) + d, one number
+a layer.  A stored key head is its two keys side by side and a query becomes two rows, each with zeros in the other map's place, so
+that the attention is the same grouped-query attention with twice the query heads.
+A layer that reads another layer's cache (``shares_cache``) projects queries only, whatever its own window.
+Four more parameters form one path of their own (``_wide_rows``): ``qk_norm`` "whole" (queries and keys are each
 normalised over ALL their heads together, with a weight vector of that width, before the position encoding),
-``head_temperature`` (query head n's scores are multiplied by a number of the layer, folded into the query) and
+``conv_taps`` (a short causal convolution over time on every channel of q, k and v, right after the projection; its last inputs are
+kept per sequence), ``head_temperature`` (query head n's scores are multiplied by a number of the layer, folded into the query) and
 ``talking_heads`` (after the softmax the heads' weights are mixed by a matrix of the layer, a'_n = sum_g M[n, g] a_g,
 and head n applies a'_n to the values of its own key/value head).
 Heads of unequal or odd sizes are written into the cache padded with zeros to one width that the
@@ -35,7 +42,7 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import kernels
-from ..cache.requirements import KVRequirement
+from ..cache.requirements import BundleRequirement, KVRequirement, StateRequirement
 from ..config.specs import MixerSpec, tensor_names
 from ..errors import ConfigError
 from ..profile import scope
@@ -53,7 +60,8 @@ PROMPT_FUSED_MIN_TOKENS = 4096
 # Hugging Face's Qwen3 checkpoints: rocml/src/weights/layer.rs:47-58 lists the same tensors under GGUF names).
 TENSOR_NAMES = {"q": "q_proj", "k": "k_proj", "v": "v_proj", "o": "o_proj", "q_norm": "q_norm", "k_norm": "k_norm",
                 "gate": "gate_proj", "value_mix": "value_mix", "talk": "head_mix", "temperature": "head_temperature",
-                "sink": "sink"}
+                "sink": "sink", "q_conv": "q_conv", "k_conv": "k_conv", "v_conv": "v_conv",
+                "lq1": "lambda_q1", "lk1": "lambda_k1", "lq2": "lambda_q2", "lk2": "lambda_k2"}
 
 VALUE_MIX_SOURCE = "attention.value_mix_source"    # where a step keeps the source layer's values (StepBatch.scratch)
 
@@ -76,16 +84,25 @@ class Attention(Mixer):
         self.vd = int(p.get("v_head_dim") or self.hd)
         self.gated = bool(p.get("gated", False))
         self.gate_per_value = p.get("gated") == "per_value"
-        self.hdp = -(-max(self.hd, self.vd) // 16) * 16         # the width of every head in the cache
+        self.difference = None if p.get("difference") is None else float(p["difference"])
+        self.maps = 1 if self.difference is None else 2         # queries and keys a head holds side by side
+        self.hdp = -(-max(self.maps * self.hd, self.vd) // 16) * 16         # the width of every head in the cache
+        self.nqm = self.nq * self.maps                          # query rows of the attention
+        self.softcap = float(p.get("softcap") or 0.0)
+        if self.softcap < 0:
+            raise ConfigError(f"attention: softcap must be positive, found {self.softcap}")
         if min(self.hd, self.vd) <= 0 or self.hdp > 512:
-            raise ConfigError(f"head sizes {self.hd} (keys) and {self.vd} (values) are not supported: 1 to 512")
+            raise ConfigError(f"head sizes {self.hd}{' x 2' if self.maps > 1 else ''} (keys) and {self.vd} (values) are not supported: 1 to 512")
         bias = p.get("bias", False)
         self.bias = bool(bias)
         self.qk_norm = bool(p.get("qk_norm", False))
         self.qk_norm_whole = p.get("qk_norm") == "whole"
         self.head_temperature = bool(p.get("head_temperature", False))
         self.talking_heads = bool(p.get("talking_heads", False))
-        self.wide = self.qk_norm_whole or self.head_temperature or self.talking_heads
+        self.conv_taps = int(p.get("conv_taps") or 0)            # 0: no convolution
+        if not 0 <= self.conv_taps <= kernels.CONV_MAX_TAPS:
+            raise ConfigError(f"attention: a convolution of {self.conv_taps} taps is not built (at most {kernels.CONV_MAX_TAPS})")
+        self.wide = self.qk_norm_whole or self.head_temperature or self.talking_heads or self.conv_taps > 0
         self.qk_norm_eps = float(p.get("qk_norm_eps", 1e-6))
         self.qk_unit_norm = bool(p.get("qk_unit_norm", False))
         self.window = p.get("window")
@@ -104,10 +121,14 @@ class Attention(Mixer):
             raise ConfigError("attention: keep_first counts positions and cannot be negative")
         if self.window and self.chunk:
             raise ConfigError("attention: a layer has a window or blocks of positions, not both")
-        if self.wide and (self.gated or self.keep_first or p.get("sink") is not None or self.q_temp or self.qk_unit_norm or self.value_mix or
+        if self.wide and ((self.gated and (self.talking_heads or not self.gate_per_value)) or self.keep_first or p.get("sink") is not None or
+                          self.q_temp or self.qk_unit_norm or self.value_mix or self.maps > 1 or self.softcap or
                           (self.qk_norm and not self.qk_norm_whole) or p.get("shares_cache")):
-            raise ConfigError("attention: a norm over whole projections, head temperatures and mixed heads do not combine with "
-                              "gates, kept first keys, a sink, query temperatures, unit norms, blended values, per-head norms or a shared cache")
+            raise ConfigError("attention: a norm over whole projections, convolutions, head temperatures and mixed heads do not combine with "
+                              "gates a head, kept first keys, a sink, query temperatures, unit norms, blended values, per-head norms, two maps, "
+                              "a soft cap or a shared cache")
+        if self.maps > 1 and (self.gated or self.value_mix):
+            raise ConfigError("attention: two maps a head do not combine with gates or blended values")
         if self.talking_heads and self.nkv * self.nq * self.hdp > 65535 * 16:
             raise ConfigError("attention: too many heads to mix")
         if (self.window is not None and int(self.window) < 1) or (self.chunk is not None and int(self.chunk) < 1):
@@ -116,12 +137,12 @@ class Attention(Mixer):
         self.shares_cache = bool(p.get("shares_cache", False))  # set by the model for a reading layer
         self.position = build_position(spec.position, self.hd, env)
         # the plain layout: equal head sizes that the kernels take as they are, rotate-half pairs, no gate
-        self.plain = not self.wide and self.vd == self.hd == self.hdp and not self.gated and \
+        self.plain = not self.wide and self.maps == 1 and not self.softcap and self.vd == self.hd == self.hdp and not self.gated and \
             not (self.position.inv_freq is not None and getattr(self.position, "interleaved", False)) and \
             not (self.keep_first or self.sink is not None or self.sink_per_head or self.q_temp or self.qk_unit_norm or self.value_mix)
-        if not self.plain and self.shares_cache:
-            raise ConfigError("attention: a layer that reads another layer's cache must have the plain layout")
-        qd, kvd = self.nq * self.hd, self.nkv * self.hd
+        if self.shares_cache and (self.gated or self.value_mix):
+            raise ConfigError("attention: a layer that reads another layer's cache has no gates and blends no values")
+        qd, kvd = self.nqm * self.hd, self.nkv * self.maps * self.hd
         try:
             self.names = n = tensor_names(p, TENSOR_NAMES)
         except ValueError as e:
@@ -143,6 +164,10 @@ class Attention(Mixer):
         self.o = Linear([n["o"]], [hidden], self.nq * self.vd, o_bias, env)
         # for an arrangement of mixers that share their input and output products (side_by_side)
         self.in_stems, self.in_outs, self.out_width = list(self.qkv.names), list(self.qkv.outs), self.nq * self.vd
+        self.in_biased = list(self.qkv.biased)
+        self.conv_channels = qd + kvd + self.nkv * self.vd        # what the convolution sees: q | k | v
+        self.conv_w: Optional[torch.Tensor] = None       # float32 [channels, taps]
+        self.lam: Optional[float] = None                 # the difference's factor on the second map
         self.q_norm_w: Optional[torch.Tensor] = None
         self.k_norm_w: Optional[torch.Tensor] = None
         self.v_lambda: Optional[torch.Tensor] = None     # float32 [1] on the device: the share of the source layer's values
@@ -150,7 +175,10 @@ class Attention(Mixer):
         self.temperature: Optional[torch.Tensor] = None  # float32 [nq]: a factor on every head's scores
 
     def cache_requirement(self):
-        return KVRequirement(self.nkv, self.hdp, self.window, chunk=self.chunk, keep_first=self.keep_first)
+        req = KVRequirement(self.nkv, self.hdp, self.window, chunk=self.chunk, keep_first=self.keep_first)
+        if self.conv_taps > 1:
+            return BundleRequirement.of(req, conv=StateRequirement((self.conv_taps - 1, self.conv_channels), torch.float32))
+        return req
 
     def _span(self) -> int:
         """The mask as the kernels take it: 0 every earlier key, n the last n keys, -n blocks of n positions."""
@@ -171,6 +199,12 @@ class Attention(Mixer):
             out.append(TensorDecl(f"{prefix}{self.names['q_norm']}.weight", (self.hd,), "norm"))
             if not self.shares_cache:
                 out.append(TensorDecl(f"{prefix}{self.names['k_norm']}.weight", (self.hd,), "norm"))
+        if self.conv_taps:
+            for role, n in zip(("q_conv", "k_conv", "v_conv"), self.in_outs):
+                out.append(TensorDecl(f"{prefix}{self.names[role]}.weight", (n, self.conv_taps), "matrix"))
+        if self.maps > 1:
+            for role in ("lq1", "lk1", "lq2", "lk2"):
+                out.append(TensorDecl(f"{prefix}{self.names[role]}.weight", (self.hd,), "matrix"))
         if self.talking_heads:
             out.append(TensorDecl(f"{prefix}{self.names['talk']}.weight", (self.nq, self.nq), "mixing"))
         if self.head_temperature:
@@ -193,6 +227,11 @@ class Attention(Mixer):
         self.load_inner(tensors, prefix)
 
     def load_inner(self, tensors: Dict[str, torch.Tensor], prefix: str) -> None:
+        if self.conv_taps:
+            self.conv_w = torch.cat([tensors[f"{prefix}{self.names[r]}.weight"].float() for r in ("q_conv", "k_conv", "v_conv")]).contiguous()
+        if self.maps > 1:
+            lq1, lk1, lq2, lk2 = (tensors[f"{prefix}{self.names[r]}.weight"].double() for r in ("lq1", "lk1", "lq2", "lk2"))
+            self.lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + self.difference
         if self.sink_per_head:
             self.sink = tensors[f"{prefix}{self.names['sink']}.weight"].float().contiguous()
         if self.talking_heads:
@@ -217,8 +256,8 @@ class Attention(Mixer):
         """Projections, attention output and the delta (as partial sums: up to 8 of each for few tokens)."""
         esz = 4 if self.env.mode == "float32" else 2
         parts = 8 if n_tokens <= 128 else 1
-        return n_tokens * (self.qkv.n * max(esz, 4 * parts if parts > 1 else esz) + 3 * self.nq * self.hdp * esz
-                           + self.hidden * 4 * parts + self.nq * 4 * (self.hdp + 2) * (parts if parts > 1 else 0))
+        return n_tokens * (self.qkv.n * max(esz, 4 * parts if parts > 1 else esz) + 3 * self.nqm * self.hdp * esz + 4 * (self.conv_channels if self.conv_taps else 0)
+                           + self.hidden * 4 * parts + self.nqm * 4 * (self.hdp + 2) * (parts if parts > 1 else 0))
 
     def inner_bytes(self) -> int:
         return 0
@@ -226,12 +265,12 @@ class Attention(Mixer):
     def inner_workspace(self, n_tokens: int) -> int:
         esz = 4 if self.env.mode == "float32" else 2
         parts = 8 if n_tokens <= 128 else 0
-        return n_tokens * (2 * self.nq * self.hdp * esz + self.nq * 4 * (self.hdp + 2) * parts)
+        return n_tokens * (2 * self.nqm * self.hdp * esz + self.nqm * 4 * (self.hdp + 2) * parts + 4 * (self.conv_channels if self.conv_taps else 0))
 
     def inner_cost(self, q_lens, kv_lens):
         from ..profile import cost as C
         esz = 4 if self.env.mode == "float32" else 2
-        return C.attention(q_lens, kv_lens, self.nq, self.nkv, self.hdp, esz, self._span() or None)
+        return C.attention(q_lens, kv_lens, self.nqm, self.nkv, self.hdp, esz, self._span() or None)
 
     def cost(self, q_lens, kv_lens):
         T = sum(q_lens)
@@ -258,7 +297,9 @@ class Attention(Mixer):
         window = self._span()
         writes = view.writes and not self.shares_cache
         if self.wide:
-            return self._forward_wide(xn, batch, view, window, sink, add_into)
+            if isinstance(xn, DeferredNorm):
+                xn = xn.materialize()
+            return self._project_out(self._wide_rows(self.qkv.forward_auto(xn, T), batch, view, window), T, sink, add_into)
         if not self.plain:
             return self._forward_padded(xn, batch, view, window, writes, sink, add_into)
         attn = torch.empty((T, qd), dtype=act, device=dev)
@@ -303,7 +344,7 @@ class Attention(Mixer):
         """The rows that the output product reads, from the layer's projection rows ([T, sum(in_outs)], or float32 partial sums
         [S, T, ..]).  ``out`` [T, out_width] (any row stride) receives them if given."""
         if self.wide:
-            raise ConfigError("attention: a norm over whole projections and mixed heads do not stand beside another mixer")
+            return self._wide_rows(proj, batch, view, self._span(), out)
         return self._padded_rows(proj, batch, view, self._span(), view.writes and not self.shares_cache, out)
 
     def _padded_rows(self, proj, batch, view, window, writes, rows=None):
@@ -326,24 +367,33 @@ class Attention(Mixer):
             raw_gate = proj[..., off:off + self.nq * self.vd]
         # one token a sequence, heads of 128 on both sides: the attention kernel makes the heads from the projection's
         # partial sums itself (norm, partial rotation, division by the root mean square, blended values, the cache write)
-        if batch.is_decode and writes and self.hd == self.vd == self.hdp and (raw_gate is not None or not self.gated):
+        if batch.is_decode and writes and self.maps == 1 and self.hd == self.vd == self.hdp and (raw_gate is not None or not self.gated):
             attn = rows if rows is not None else torch.empty((T, self.nq * self.hd), dtype=act, device=dev)
             if self._decode_fused(proj, attn, batch, view, window, writes, v_first=v_first, v_keep=v_out, gate=raw_gate):
                 return attn
-        q = torch.empty((T, self.nq * self.hdp), dtype=act, device=dev)
+        q = torch.empty((T, self.nqm * self.hdp), dtype=act, device=dev)
         gates = torch.empty((T, self.nq), dtype=torch.float32, device=dev) if self.gated and not self.gate_per_value else None
         with scope(op="rotate_cache"):
             kernels.qk_norm_rope_cache(
-                proj, q, T, self.nq, self.nkv, self.hd, self.q_norm_w, self.k_norm_w, self.qk_norm_eps,
+                proj, q, T, self.nqm, self.nkv, self.hd, self.q_norm_w, self.k_norm_w, self.qk_norm_eps,
                 self.position.inv_freq, self.position.rot_dim, batch.positions, batch.slot_of_token,
                 view.block_table, view.k, view.v, write_kv=writes, cos_sin=self.position.cos_sin(batch),
                 v_head_dim=self.vd, padded_head_dim=self.hdp, interleaved=getattr(self.position, "interleaved", False),
                 gates=gates, post_norm=self.qk_unit_norm, v_first=v_first, v_lambda=self.v_lambda if v_first is not None else None,
-                v_out=v_out, q_temp=self.q_temp)
+                v_out=v_out, q_temp=self.q_temp, maps=self.maps)
+        if self.maps > 1:
+            both = torch.empty((T, self.nqm * self.hdp), dtype=act, device=dev)
+            paged_attention(q, both, batch, view.k, view.v, view.block_table, self.nqm, self.nkv, self.hdp, self.scale, window,
+                            keep=self.keep_first, sink=self.sink, softcap=self.softcap)
+            attn = rows if rows is not None else torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
+            with scope(op="diff_heads"):
+                kernels.diff_heads(both, self.lam, self.qk_norm_eps, 1.0 - self.difference, attn, self.nq, self.hdp, self.vd,
+                                   batch.slot_of_token, T)
+            return attn
         last = (self.gated and raw_gate is None) or self.hdp != self.vd         # a kernel that gates or narrows follows for sure
         attn = rows if rows is not None and not last else torch.empty((T, self.nq * self.hdp), dtype=act, device=dev)
         gated_inside = paged_attention(q, attn, batch, view.k, view.v, view.block_table, self.nq, self.nkv, self.hdp, self.scale,
-                                       window, keep=self.keep_first, sink=self.sink, gate=raw_gate)
+                                       window, keep=self.keep_first, sink=self.sink, gate=raw_gate, softcap=self.softcap)
         if (self.gated and not gated_inside) or self.hdp != self.vd:
             narrow = rows if rows is not None else torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
             raw = None
@@ -355,8 +405,9 @@ class Attention(Mixer):
             attn = narrow
         return attn
 
-    def _forward_wide(self, xn, batch, view, window, sink, add_into):
-        """A norm over the whole q and k projections, a temperature per head, the heads' weights mixed after the softmax.
+    def _wide_rows(self, proj, batch, view, window, rows=None):
+        """A norm over the whole q and k projections, a convolution ahead of it, a temperature per head, a gate for every value, or the
+        heads' weights mixed after the softmax.
 
         One kernel normalises, rotates, scales and pads the queries and writes keys and values to their pages.  Mixing
         weights and then applying them to values is the same as applying every head's own weights to the values of every
@@ -364,31 +415,40 @@ class Attention(Mixer):
         (key head, value head) pairs (``cross``), and a small kernel forms the sums over g in 32-bit."""
         T = batch.n_tokens
         dev, act = self.env.device, self.env.act_dtype
-        if isinstance(xn, DeferredNorm):
-            xn = xn.materialize()
-        proj = self.qkv.forward_auto(xn, T)
         rot = self.position.rot_dim if self.position.inv_freq is not None else 0
         q = torch.empty((T, self.nq * self.hdp), dtype=act, device=dev)
+        raw = proj[..., self.conv_channels:self.conv_channels + self.nq * self.vd] if self.gated else None
+        if self.conv_taps:
+            u = torch.empty((T, self.conv_channels), dtype=torch.float32, device=dev)
+            with scope(op="causal_conv"):
+                kernels.causal_conv(proj, T, 0, self.conv_channels, self.conv_taps, self.conv_w, None, "none",
+                                    view.extras["conv"].state if self.conv_taps > 1 else None, batch.seq_slot, batch.cu_q,
+                                    batch.n_seqs, batch.max_q_len, u)
+            proj = u
         with scope(op="rotate_cache"):
             kernels.wide_norm_rope_cache(proj, q, T, self.nq, self.nkv, self.hd, self.vd, self.hdp, self.q_norm_w, self.k_norm_w,
                                          self.qk_norm_eps, self.temperature, self.position.cos_sin(batch) if rot else None, rot,
                                          getattr(self.position, "interleaved", False), batch.positions, batch.slot_of_token,
                                          view.block_table, view.k, view.v)
         pairs = self.nkv if self.talking_heads and self.nkv > 1 else 1
-        wide = torch.empty((T, self.nq * pairs * self.hdp), dtype=act, device=dev)
-        paged_attention(q, wide, batch, view.k, view.v, view.block_table, self.nq * pairs, self.nkv * pairs, self.hdp, self.scale,
-                        window, cross=pairs if pairs > 1 else 0)
+        if rows is not None and self.hdp == self.vd and not self.talking_heads:
+            wide = rows
+        else:
+            wide = torch.empty((T, self.nq * pairs * self.hdp), dtype=act, device=dev)
+        inside = raw if self.hdp == self.vd else None           # an attention kernel that takes gate columns multiplies by their sigmoid
+        done = paged_attention(q, wide, batch, view.k, view.v, view.block_table, self.nq * pairs, self.nkv * pairs, self.hdp, self.scale,
+                               window, cross=pairs if pairs > 1 else 0, gate=inside)
         if self.talking_heads:
-            attn = torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
+            attn = rows if rows is not None else torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
             with scope(op="mix_heads"):
                 kernels.talk_mix(wide, self.talk, attn, self.nq, self.nkv, self.hdp, self.vd, batch.slot_of_token, T)
-        elif self.hdp != self.vd:
-            attn = torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
+        elif self.hdp != self.vd or (raw is not None and not done):
+            attn = rows if rows is not None else torch.empty((T, self.nq * self.vd), dtype=act, device=dev)
             with scope(op="head_gate"):
-                kernels.head_gate(wide, attn, None, self.nq, self.hdp, self.vd, T)
+                kernels.head_gate(wide, attn, None, self.nq, self.hdp, self.vd, T, raw=raw, per_value=raw is not None)
         else:
             attn = wide
-        return self._project_out(attn, T, sink, add_into)
+        return attn
 
     def _project_out(self, attn, T, sink, add_into):
         if sink is not None:
@@ -453,7 +513,7 @@ class Attention(Mixer):
             self.position.cos_sin(batch) if rot else None, writes, self.scale, window, n_blocks, acc, ml, ppb,
             rowscale=rowscale, row_width=row_width, keep=self.keep_first, sink=self.sink, rot_dim=rot,
             post_norm=self.qk_unit_norm, v_first=v_first, v_lambda=self.v_lambda if v_first is not None else None,
-            v_keep=v_keep, gate=gate, q_temp=self.q_temp)
+            v_keep=v_keep, gate=gate, q_temp=self.q_temp, softcap=self.softcap)
 
     def attend(self, q, out, batch, view, window):
         """Softmax attention of the step's queries over the cache (see ``paged_attention``)."""
@@ -461,9 +521,9 @@ class Attention(Mixer):
 
 
 def paged_attention(q, out, batch, k_cache, v_cache, block_table, nq, nkv, hd, scale, window, keep=0, sink=None, gate=None,
-                    cross=0) -> bool:
+                    cross=0, softcap=0.0) -> bool:
     """Softmax attention of the step's queries (rows of nq heads of ``hd``) over paged keys and values
-    [pages, nkv, 64, hd], causal, inside ``window`` when it is not 0 (and the first ``keep`` positions beside it);
+    [pages, nkv, 64, hd], causal, inside ``window`` when it is not 0 (and the first ``keep`` positions beside it), scores through ``softcap`` when it is not 0;
     ``sink``: a score whose exponential joins every row's denominator.  One token per sequence:
     keys split in fixed chunks, partial results merged; otherwise whole rows.  Any mixer whose cache is
     such pages calls this (keys and values may be the same tensor).  ``gate``: nq * hd columns of the step's projection
@@ -489,28 +549,29 @@ def paged_attention(q, out, batch, k_cache, v_cache, block_table, nq, nkv, hd, s
             ml = torch.empty((T, nq, parts, 2), dtype=torch.float32, device=q.device)
         fast = kernels.attention_decode(q, out, k_cache, v_cache, block_table, batch.seq_slot, batch.cu_q,
                                         batch.kv_len, batch.n_seqs, nq, nkv, hd, scale,
-                                        window, n_blocks, acc, ml, ppb, keep=keep, sink=sink, gate=gate, cross=cross)
+                                        window, n_blocks, acc, ml, ppb, keep=keep, sink=sink, gate=gate, cross=cross, softcap=softcap)
         n_chunks = n_pages
         if fast:
             return gate is not None
         if n_chunks > 1:
             kernels.attention_generic(q, out, k_cache, v_cache, block_table, batch.seq_slot, batch.cu_q,
                                       batch.kv_len, batch.n_seqs, 1, nq, nkv, hd, scale,
-                                      window, chunk, n_chunks, acc, ml, keep=keep, sink=sink, cross=cross)
+                                      window, chunk, n_chunks, acc, ml, keep=keep, sink=sink, cross=cross, softcap=softcap)
             kernels.attention_merge(acc, ml, out, batch.positions, batch.slot_of_token, T, nq, hd,
                                     chunk, n_chunks, window, keep=keep, sink=sink)
             return False
     tc5_gate = gate if gate is not None and gate.dim() == 2 and gate.dtype == torch.bfloat16 else None
     if kernels.attention_prefill_tc5(q, batch.n_tokens, out, k_cache, v_cache, block_table, batch.seq_slot,
                                      batch.cu_q, batch.kv_len, batch.n_seqs, batch.max_q_len, nq, nkv,
-                                     hd, scale, window, max_kv_len=batch.max_kv_len, keep=keep, sink=sink, gate=tc5_gate, cross=cross):
+                                     hd, scale, window, max_kv_len=batch.max_kv_len, keep=keep, sink=sink, gate=tc5_gate, cross=cross,
+                                     softcap=softcap):
         return tc5_gate is not None
     if cross <= 1 and kernels.attention_prefill(q, out, k_cache, v_cache, block_table, batch.seq_slot, batch.cu_q,
                                  batch.kv_len, batch.n_seqs, batch.max_q_len, nq, nkv, hd,
-                                 scale, window, keep=keep, sink=sink):
+                                 scale, window, keep=keep, sink=sink, softcap=softcap):
         return False
     kernels.attention_generic(q, out, k_cache, v_cache, block_table, batch.seq_slot, batch.cu_q,
                               batch.kv_len, batch.n_seqs, batch.max_q_len, nq, nkv, hd,
-                              scale, window, keep=keep, sink=sink, cross=cross)
+                              scale, window, keep=keep, sink=sink, cross=cross, softcap=softcap)
     return False
 

@@ -112,6 +112,26 @@ class ScaledDelta:
     factor: float
 
 
+@dataclass
+class NormedPair:
+    """Two results of one mixer that are normalised apart and added: factor * (rms(left) * left_w + rms(right) * right_w), eps inside
+    the roots.  Handed, instead of a delta, to an arrangement that asked for it (``forward(..., norm_later=True)`` of a mixer with
+    ``norms_later``) and forms it in the kernel that consumes it; ``materialize`` does it otherwise."""
+
+    left: torch.Tensor        # [S, T, H] float32
+    right: torch.Tensor       # [S', T, H] float32
+    left_w: torch.Tensor      # [H] float32
+    right_w: torch.Tensor
+    eps: float
+    factor: float
+
+    def materialize(self) -> torch.Tensor:
+        from .. import kernels
+        out = torch.empty((1,) + tuple(self.left.shape[1:]), dtype=torch.float32, device=self.left.device)
+        kernels.pair_norm(self.left, self.right, self.left_w, self.right_w, self.eps, self.factor, out.shape[1], out_v=out[0])
+        return out
+
+
 class StreamRows(DeferredNorm):
     """What a block leaves for a block after it whose sublayers read the stream itself: ``x`` are the stream's rows in the
     activations' type (the residual holds every delta; ``norm`` is None).  To any norm it means 'nothing pending'."""

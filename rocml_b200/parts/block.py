@@ -9,7 +9,7 @@ import torch
 from ..config.specs import LayerSpec
 from ..profile import scope
 from ..weights.decl import TensorDecl
-from .base import (BuildEnv, DeferredNorm, NormedRows, ResidualSink, RoutedRows, ScaledDelta, ShiftedRows, StreamRows,
+from .base import (BuildEnv, DeferredNorm, NormedPair, NormedRows, ResidualSink, RoutedRows, ScaledDelta, ShiftedRows, StreamRows,
                    build_feed_forward, build_mixer, build_norm, register_arrangement)
 
 
@@ -608,6 +608,10 @@ class OutputNormBlock:
             kernels.out_norm(resid, delta.rows, w, b, norm.eps, self.mult, layer, out, row_of=delta.row_of, weights=delta.weights,
                              top=delta.top, self_weight=delta.self_weight, self_x=resid if delta.self_weight is not None else None, n_rows=T)
             return
+        if isinstance(delta, NormedPair) and not layer and b is None:
+            kernels.pair_norm(delta.left, delta.right, delta.left_w, delta.right_w, delta.eps, delta.factor, T, resid=resid, weight=w,
+                              eps=norm.eps, mult=self.mult, out=out)
+            return
         factor = 1.0
         if isinstance(delta, ScaledDelta):
             delta, factor = delta.delta, delta.factor
@@ -630,8 +634,9 @@ class OutputNormBlock:
                 x = torch.empty((T, self.hidden), dtype=act, device=resid.device)
                 with scope(op="stream_rows"):
                     kernels.cast(resid[:T], x)
-        if getattr(self.mixer, "scales_later", False):
-            delta = self.mixer.forward(x, batch, view, scale_later=True)
+        later = {k: True for k, can in (("scale_later", "scales_later"), ("norm_later", "norms_later")) if getattr(self.mixer, can, False)}
+        if later:
+            delta = self.mixer.forward(x, batch, view, **later)
         else:
             delta = self.mixer.forward(x, batch, view)
         rows = resid if same else torch.empty((T, self.hidden), dtype=act, device=resid.device)
@@ -658,7 +663,7 @@ def norm_is_layer(norm) -> bool:
 
 def _as_partial_sums(delta, n_rows: int):
     """A sublayer's result in the form the sum's kernel adds: float32 [S, >= rows, H]."""
-    if isinstance(delta, RoutedRows):
+    if isinstance(delta, (RoutedRows, NormedPair)):
         delta = delta.materialize()
     if delta is None or _is_partial_sums(delta, n_rows):
         return delta

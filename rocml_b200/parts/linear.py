@@ -104,6 +104,19 @@ class Linear:
         self.outs.append(pad)
         self.n += pad
 
+    def rows(self, start: int, stop: int, label: str) -> "Linear":
+        """A product with rows start .. stop of the loaded stack alone (the same memory)."""
+        part = Linear([label], [stop - start], self.k, False, self.env)
+        part.label = label
+        part.weight = self.weight[start:stop]
+        part.bias = self.bias[start:stop].contiguous() if self.bias is not None else None
+        part.has_bias = part.bias is not None
+        return part
+
+    def one_piece(self, x: torch.Tensor, m: int) -> bool:
+        """Whether ``forward_auto`` would return one result in the activations' type (not partial sums)."""
+        return not ((self._tensor_core(x) and self._splits(m) > 1) or self._splits_f32(x, m) > 1)
+
     def interleave_pairs(self) -> bool:
         """For a stack of two equally wide projections (gate, up): reorder the rows so that blocks
         of 16 gate rows alternate with the 16 up rows of the same outputs.  The tensor-core
@@ -269,7 +282,7 @@ class Linear:
     def forward_auto(self, x: torch.Tensor, m: int) -> torch.Tensor:
         """The product in whichever form is cheapest for the step: [S, M, N] float32 partial sums
         when few rows stream the weight, else [M, N] in the activations' type."""
-        if (self._tensor_core(x) and self._splits(m) > 1) or self._splits_f32(x, m) > 1:
+        if not self.one_piece(x, m):
             return self.forward_delta(x, m)
         out = torch.empty((m, self.n), dtype=x.dtype, device=x.device)
         return self.forward(x, out, m)

@@ -1,4 +1,4 @@
-"""Gated feed-forward: down(act(gate(x)) * up(x)) (rocml/src/forward/ffn.rs:57-107)."""
+"""Feed-forwards: gated, down(act(gate(x)) * up(x)) (rocml/src/forward/ffn.rs:57-107), and plain, down(act(up(x)))."""
 from __future__ import annotations
 
 from typing import Dict, List
@@ -8,6 +8,7 @@ import torch
 from .. import kernels
 from ..config.specs import FeedForwardSpec, tensor_names
 from ..errors import ConfigError
+from ..profile import scope
 from ..weights.decl import TensorDecl
 from .base import BuildEnv, DeferredNorm, FeedForward, register_feed_forward
 from .linear import GATED_PAIR_MAX_ROWS, Linear
@@ -103,6 +104,65 @@ class GatedMLP(FeedForward):
             deferred = self.down.forward_residual(h, T, sink)
             if deferred is not None:
                 return deferred
+        if add_into is not None and self.down.forward_add(h, T, add_into):
+            return None
+        return self.down.forward_delta(h, T)
+
+
+@register_feed_forward("dense_mlp")
+class DenseMLP(FeedForward):
+    """down(act(up(x))): no gate.  The activation is a parameter: "gelu" (z / 2 * (1 + erf(z / sqrt 2))), "gelu_tanh" or "silu",
+    computed in 32-bit."""
+
+    graph_safe = True
+
+    def __init__(self, spec: FeedForwardSpec, hidden: int, env: BuildEnv):
+        p = spec.params
+        self.env = env
+        self.hidden = hidden
+        self.inter = int(p["intermediate"])
+        self.act = p.get("activation", "gelu")
+        if self.act not in kernels.PLAIN_ACTS:
+            raise ConfigError(f"activation {self.act!r} is not built (known: {', '.join(kernels.PLAIN_ACTS)})")
+        bias = bool(p.get("bias", False))
+        try:
+            n = tensor_names(p, {k: TENSOR_NAMES[k] for k in ("up", "down")})
+        except ValueError as e:
+            raise ConfigError(f"dense_mlp: {e}") from None
+        self.up = Linear([n["up"]], [self.inter], hidden, bias, env)
+        self.down = Linear([n["down"]], [hidden], self.inter, bias, env)
+
+    def declare(self, prefix: str) -> List[TensorDecl]:
+        return self.up.declare(prefix) + self.down.declare(prefix)
+
+    def load(self, tensors: Dict[str, torch.Tensor], prefix: str) -> None:
+        self.up.load(tensors, prefix)
+        self.down.load(tensors, prefix)
+
+    def weight_bytes(self) -> int:
+        return self.up.weight_bytes() + self.down.weight_bytes()
+
+    def workspace_bytes(self, n_tokens: int) -> int:
+        """up, its activation and the delta (as partial sums: up to 8 of each for few tokens)."""
+        esz = 4 if self.env.mode == "float32" else 2
+        parts = 8 if n_tokens <= 128 else 1
+        return n_tokens * (self.inter * (4 * parts if parts > 1 else esz) + self.inter * esz + self.hidden * 4 * parts)
+
+    def cost(self, q_lens, kv_lens):
+        T = sum(q_lens)
+        a, b = self.up.cost(T), self.down.cost(T)
+        return a[0] + b[0], a[1] + b[1]
+
+    can_add_into = True    # forward() accepts add_into=residual (see parts.base)
+
+    def forward(self, xn, batch, add_into=None):
+        T = batch.n_tokens
+        if isinstance(xn, DeferredNorm):
+            xn = xn.materialize()
+        u = self.up.forward_auto(xn, T)            # [T, I] or [S, T, I] partial sums
+        h = torch.empty((T, self.inter), dtype=self.env.act_dtype, device=self.env.device)
+        with scope(op="activation"):
+            kernels.unary_act(u, h, self.act)
         if add_into is not None and self.down.forward_add(h, T, add_into):
             return None
         return self.down.forward_delta(h, T)

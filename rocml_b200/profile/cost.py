@@ -64,6 +64,13 @@ def delta_scan(tokens: int, seqs: int, heads: int, kv_heads: int, dim: int, vdim
     return 4 * tokens * per_token + 8 * seqs * heads * dim * vdim, 7 * tokens * heads * dim * vdim
 
 
+def mlstm(tokens: int, seqs: int, heads: int, dim: int, vdim: int, esz: int) -> Cost:
+    """A matrix memory with exponential gates per (sequence, head): the tokens' q, k, v (``esz`` bytes an element) in, every
+    sequence's 32-bit state in and back, 32-bit results out; per token and state entry a decay, an update and two operations of
+    the result."""
+    return tokens * heads * ((2 * dim + vdim) * esz + vdim * 4) + 8 * seqs * heads * dim * (vdim + 1), 5 * tokens * heads * dim * vdim
+
+
 def rope_table(rows: int, half: int) -> Cost:
     return rows * (4 + half * 8) + half * 4, rows * half * 40
 
