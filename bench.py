@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine at Qwen3-8B layer sizes, random bfloat16 weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl reference]
-    python bench.py --workload 4b-long | 32b | pipilix | zokelorn | safesun | tibenex | ravelorn
+    python bench.py --workload 4b-long | 32b | pipilix | zokelorn | safesun | tibenex | ravelorn | kemizen
 
 A step is one decode step of the default batch (8 sequences, prompts of 1,024 tokens, cache
 sized for a context of 4,096 per sequence).  One JSON line goes to stdout:
@@ -56,7 +56,7 @@ def main():
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration has (0: all)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="leave out batch 1 and 64 and the 32-bit path")
-    ap.add_argument("--workload", default=None, choices=["4b-long", "32b", "pipilix", "zokelorn", "safesun", "tibenex", "ravelorn"],
+    ap.add_argument("--workload", default=None, choices=["4b-long", "32b", "pipilix", "zokelorn", "safesun", "tibenex", "ravelorn", "kemizen"],
                     help="instead of the bench line: a whole generation of that workload through Engine.generate")
     args = ap.parse_args()
 
@@ -70,7 +70,7 @@ def main():
         return 2
 
     from rocml_b200 import measure as M
-    if args.workload in ("pipilix", "zokelorn", "safesun", "tibenex", "ravelorn"):
+    if args.workload in ("pipilix", "zokelorn", "safesun", "tibenex", "ravelorn", "kemizen"):
         print(json.dumps(M.compare(None, args.layers, steps=max(8, min(args.steps, 64)), family=args.workload)))
         return 0
     if args.workload:

@@ -327,11 +327,15 @@ int rb_mlstm_blocks(const void* x, int x_dtype, int n_in, long long in_stride, i
                     const float* em, int T, float* S_state, float* n_state, const int* seq_slot, const int* cu_q, int n_seqs,
                     int blocks, float* work, float* work_n, float* block_decay, float* scores, float* out, int ld_out,
                     float* den, void* stream);
+int rb_mlstm_chain(const void* x, int row_stride, int q_off, int k_off, int v_off, float q_scale, float eps, int heads, int dim,
+                   int vdim, const float* log_keep, const float* log_add, const float* em, int T, float* S_state, float* n_state,
+                   const int* seq_slot, const int* cu_q, int n_seqs, int blocks, void* planes, float* ec, float* wt,
+                   float* block_decay, float* out, int ld_out, float* den, void* stream);
 
-// A real-gated linear recurrent unit (rglru.cu).
+// A real-gated linear recurrent unit (rglru.cu).  ax: (a, x) pairs [T][width].
 int rb_rglru_gates(const float* u, int ld_u, const void* ra, const void* ri, int w_dtype, const float* ra_b, const float* ri_b,
-                   const float* rate, int blocks, int part, int T, float* a, float* x, void* stream);
-int rb_rglru_scan(const float* a, const float* x, int width, const void* y, int y_dtype, int n_in, long long in_stride,
+                   const float* rate, int blocks, int part, int T, float* ax, void* stream);
+int rb_rglru_scan(const float* ax, int width, const void* y, int y_dtype, int n_in, long long in_stride,
                   int row_stride, float factor, float* state, const int* seq_slot, const int* cu_q, int n_seqs, void* out,
                   int out_dtype, int ld_out, void* stream);
 int rb_rglru_step(const float* u, int ld_u, const void* ra, const void* ri, int w_dtype, const float* ra_b, const float* ri_b,

@@ -653,12 +653,13 @@ extern "C" int rb_gated_act(const void* in, int in_dtype, int n_in, long long in
 // in: [S][rows, I] (S partial sums, added first, in order) -> out [rows, I].  kind 0: gelu(z) = z / 2 * (1 + erf(z / sqrt 2));
 // 1: gelu in its tanh form; 2: silu.
 template <typename IT, typename OT>
-__global__ void unary_act_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, OT* __restrict__ out, size_t n, int kind) {
+__global__ void unary_act_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, OT* __restrict__ out, size_t n, int kind, int vec) {
     pdl_trigger();
     pdl_wait();
     for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4; i < n; i += (size_t)gridDim.x * blockDim.x * 4) {
         float v[4] = {0.f, 0.f, 0.f, 0.f};
-        if (i + 4 <= n) {
+        const bool whole = vec && i + 4 <= n;               // 4-element accesses
+        if (whole) {
             for (int s = 0; s < n_in; s += 4) {                 // four partial sums in flight, added in order
                 float p[4][4];
 #pragma unroll
@@ -673,29 +674,28 @@ __global__ void unary_act_kernel(const IT* __restrict__ in, int n_in, size_t in_
             }
         } else {
             for (int s = 0; s < n_in; ++s)
-                for (int u = 0; i + u < n; ++u) v[u] += to_f32(in[(size_t)s * in_stride + i + u]);
+                for (int u = 0; u < 4 && i + u < n; ++u) v[u] += to_f32(in[(size_t)s * in_stride + i + u]);
         }
 #pragma unroll
         for (int u = 0; u < 4; ++u) v[u] = kind == 0 ? gelu_erf(v[u]) : (kind == 1 ? gelu_tanh(v[u]) : silu(v[u]));
-        if (i + 4 <= n) rb::store4(out + i, v);
+        if (whole) rb::store4(out + i, v);
         else
-            for (int u = 0; i + u < n; ++u) out[i + u] = from_f32<OT>(v[u]);
+            for (int u = 0; u < 4 && i + u < n; ++u) out[i + u] = from_f32<OT>(v[u]);
     }
 }
 
-// in and out on four elements' alignment, in_stride a multiple of 4 (or one partial sum).
 extern "C" int rb_unary_act(const void* in, int in_dtype, int n_in, long long in_stride, void* out, int out_dtype, long long n, int kind,
                             void* stream) {
     if (n <= 0) return RB_OK;
     if (n_in < 1 || kind < 0 || kind > 2) return RB_ERR_BAD_SIZE;
     const size_t isz = in_dtype == RB_F32 ? 4 : 2, osz = out_dtype == RB_F32 ? 4 : 2;
-    if (((uintptr_t)in & (4 * isz - 1)) || ((uintptr_t)out & (4 * osz - 1)) || (n_in > 1 && (in_stride & 3))) return RB_ERR_BAD_ALIGN;
+    const int vec = ((uintptr_t)in & (4 * isz - 1)) == 0 && ((uintptr_t)out & (4 * osz - 1)) == 0 && (n_in == 1 || (in_stride & 3) == 0);
     const long long want = (n / 4 + 256) / 256;
     const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
     typedef __nv_bfloat16 bf;
 #define RB_UA(IT, OT)                                                                                                       \
     RB_LAUNCH((unary_act_kernel<IT, OT>), dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const IT*)in, n_in, (size_t)in_stride, \
-              (OT*)out, (size_t)n, kind)
+              (OT*)out, (size_t)n, kind, vec)
     if (in_dtype == RB_BF16 && out_dtype == RB_BF16) RB_UA(bf, bf);
     else if (in_dtype == RB_F32 && out_dtype == RB_BF16) RB_UA(float, bf);
     else if (in_dtype == RB_F32 && out_dtype == RB_F32) RB_UA(float, float);

@@ -712,7 +712,7 @@ constexpr int PAIR_STAGE = 2 * BM * BK * 2;       // A 128 x 64 + B half 128 x 6
 constexpr int PAIR_STAGES = 6;
 constexpr int PAIR_SMEM = PAIR_STAGES * PAIR_STAGE + 1024 + 256;
 
-// EPI: 0 plain, 3 added into `out` (the float32 residual stream) instead of written, 1 SiLU(gate) * up (rows
+// EPI: 0 plain, 4 through an activation of its own (act_kind 0 gelu with erf, 1 gelu in its tanh form, 2 silu), 3 added into `out` (the float32 residual stream) instead of written, 1 SiLU(gate) * up (rows
 // of the weight interleaved by 16), 2 a prompt's q | k | v projection
 // with heads of 128: a tile's 256 columns are two whole heads and an epilogue thread owns a token, so
 // the per-head RMSNorm and the rotation (pairs i, i + 64) are done on the accumulator itself, and
@@ -981,6 +981,18 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
 #pragma unroll
                             for (int i = 0; i < 16; ++i) v[i] += (f0 + i < p.b_rows) ? p.bias[f0 + i] : 0.f;
                         }
+                        if (EPI == 4) {
+                            if (p.act_kind == 0) {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) v[i] = rb::gelu_erf(v[i]);
+                            } else if (p.act_kind == 1) {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) v[i] = rb::gelu_tanh(v[i]);
+                            } else {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) v[i] = rb::silu(v[i]);
+                            }
+                        }
                         if (vec_ok && f0 + 16 <= p.b_rows) {
                             store16(row + f0, v);
                         } else {
@@ -1230,6 +1242,10 @@ static int gemm_entry(const void* x, const void* w, const float* bias, void* out
     if (K <= 0 || splits < 1) return RB_ERR_BAD_SIZE;
     if (K % 8 || ldx % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return RB_ERR_BAD_ALIGN;
     if (splits > 1 && out_dtype != RB_F32) return RB_ERR_BAD_DTYPE;
+    // gated < 0: no gate, the activation -gated - 1 on the product itself (only the kernel of CTA pairs has it)
+    const bool plain_act = gated < 0;
+    const int act = plain_act ? -gated - 1 : 0;
+    if (plain_act) gated = 0;
     if (gated && (splits != 1 || out_dtype != RB_BF16 || N % 32)) return RB_ERR_BAD_SIZE;
     const int kb_total = (K + BK - 1) / BK;
     if (splits > kb_total) return RB_ERR_BAD_SIZE;  // a split would be empty and its partial result unwritten
@@ -1326,11 +1342,17 @@ static int gemm_entry(const void* x, const void* w, const float* bias, void* out
         CUtensorMap mb_half;
         if ((rc = tensor_map(w, N, K, K, BM, &mb_half)) != RB_OK) return rc;
         if (accumulate) return launch_pair<float, 3>(ma, mb_half, out, p, s);
+        if (plain_act) {
+            if (out_dtype != RB_BF16 || act > 2) return RB_ERR_BAD_DTYPE;
+            p.act_kind = act;
+            return launch_pair<__nv_bfloat16, 4>(ma, mb_half, out, p, s);
+        }
         if (out_dtype == RB_BF16)
             return gated ? launch_pair<__nv_bfloat16, 1>(ma, mb_half, out, p, s)
                          : launch_pair<__nv_bfloat16, 0>(ma, mb_half, out, p, s);
         if (out_dtype == RB_F32) return launch_pair<float, 0>(ma, mb_half, out, p, s);
     }
+    if (plain_act) return RB_ERR_BAD_SIZE;
     if (!swap && splits == 1 && (bn == 256 || bn == 128)) {
         // many tokens: the persistent kernel with two accumulators (2 x 256 columns fill tensor memory)
         if (out_dtype == RB_BF16) {

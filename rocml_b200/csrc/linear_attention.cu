@@ -536,6 +536,47 @@ group_norm_gate_kernel(const float* __restrict__ o, int ld_o, const IT* __restri
         }
     }
 }
+// The same for groups of many columns, a block a (token, group): few tokens, or few and wide groups, then fill the device better than
+// a warp a group.  Four columns a thread.
+template <typename IT, typename AT, typename WT>
+__global__ void __launch_bounds__(256)
+group_norm_gate_wide_kernel(const float* __restrict__ o, int ld_o, const IT* __restrict__ proj, int n_in, size_t in_stride, int row_stride,
+                            int g_off, const WT* __restrict__ w, float eps, int groups, int gw, int gate_act, AT* __restrict__ out,
+                            int ld_out, const int* __restrict__ slot_of_token, const float* __restrict__ den) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int t = blockIdx.x, gi = blockIdx.y;
+    if (slot_of_token[t] < 0) return;
+    const float* row = o + (size_t)t * ld_o + (size_t)gi * gw;
+    const IT* g = proj + (size_t)t * row_stride + g_off + (size_t)gi * gw;
+    const int i = threadIdx.x * 4;                       // (the block has a thread for every four columns)
+    float x[4] = {0.f, 0.f, 0.f, 0.f}, z[4] = {0.f, 0.f, 0.f, 0.f}, ww[4] = {1.f, 1.f, 1.f, 1.f};
+    const float rd = den ? 1.f / den[(size_t)t * groups + gi] : 1.f;
+    if (i < gw) {
+        load4(row + i, x);
+        if (w) load4(w + (size_t)gi * gw + i, ww);
+        for (int s = 0; s < n_in; s += 4) {              // four partial sums in flight, added in order
+            float p[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                if (s + j < n_in) load4(g + (size_t)(s + j) * in_stride + i, p[j]);
+                else p[j][0] = p[j][1] = p[j][2] = p[j][3] = 0.f;
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) z[u] += p[j][u];
+        }
+    }
+    const float ss = block_sum(x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3], scratch);
+    if (i >= gw) return;
+    const float inv = rsqrtf(ss * rd * rd / (float)gw + eps) * rd;
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+        x[u] = x[u] * inv * ww[u] * (gate_act == 1 ? silu(z[u]) : (gate_act == 2 ? sigmoid_f32(z[u]) : 1.f));
+    store4(out + (size_t)t * ld_out + (size_t)gi * gw + i, x);
+}
 }  // namespace
 
 // The state tile's width and the parts a column is cut in, from the sizes alone (so that a token's sums are
@@ -591,16 +632,26 @@ extern "C" int rb_group_norm_gate(const float* o, int ld_o, const void* proj, in
     if (groups <= 0 || W <= 0 || W % groups || n_in < 1) return RB_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
+    const int gw = W / groups;
+    const size_t psz = proj_dtype == RB_F32 ? 4 : 2, osz = out_dtype == RB_F32 ? 4 : 2, wsz = w_dtype == RB_F32 ? 4 : 2;
+    const bool wide = groups > 1 && groups <= 65535 && gw >= 128 && gw <= 1024 && ((gw | ld_o | row_stride | g_off | ld_out) & 3) == 0 &&
+                      (in_stride & 3) == 0 && ((uintptr_t)o & 15) == 0 && ((uintptr_t)proj & (4 * psz - 1)) == 0 &&
+                      ((uintptr_t)out & (4 * osz - 1)) == 0 && (!w || ((uintptr_t)w & (4 * wsz - 1)) == 0);
+    const int wide_threads = ((gw / 4) + 31) & ~31;
 #define RB_GNG(IT, AT, WT)                                                                                               \
+    if (wide)                                                                                                            \
+        RB_LAUNCH((group_norm_gate_wide_kernel<IT, AT, WT>), dim3(T, groups), dim3(wide_threads), 0, s, o, ld_o, (const IT*)proj, n_in, \
+                  (size_t)in_stride, row_stride, g_off, (const WT*)w, eps, groups, gw, gate_act, (AT*)out, ld_out, slot_of_token, den);  \
+    else                                                                                                                 \
     RB_LAUNCH((group_norm_gate_kernel<IT, AT, WT>), dim3(T), dim3(256), 0, s, o, ld_o, (const IT*)proj, n_in,            \
               (size_t)in_stride, row_stride, g_off, (const WT*)w, eps, groups, W, gate_act, (AT*)out, ld_out, slot_of_token, den)
     const bool wf = !w || w_dtype == RB_F32;
-    if (proj_dtype == RB_BF16 && out_dtype == RB_BF16 && !wf) RB_GNG(bf, bf, bf);
-    else if (proj_dtype == RB_BF16 && out_dtype == RB_BF16) RB_GNG(bf, bf, float);
-    else if (proj_dtype == RB_F32 && out_dtype == RB_BF16 && !wf) RB_GNG(float, bf, bf);
-    else if (proj_dtype == RB_F32 && out_dtype == RB_BF16) RB_GNG(float, bf, float);
-    else if (proj_dtype == RB_F32 && out_dtype == RB_F32 && wf) RB_GNG(float, float, float);
-    else if (proj_dtype == RB_F32 && out_dtype == RB_F32) RB_GNG(float, float, bf);
+    if (proj_dtype == RB_BF16 && out_dtype == RB_BF16 && !wf) { RB_GNG(bf, bf, bf); }
+    else if (proj_dtype == RB_BF16 && out_dtype == RB_BF16) { RB_GNG(bf, bf, float); }
+    else if (proj_dtype == RB_F32 && out_dtype == RB_BF16 && !wf) { RB_GNG(float, bf, bf); }
+    else if (proj_dtype == RB_F32 && out_dtype == RB_BF16) { RB_GNG(float, bf, float); }
+    else if (proj_dtype == RB_F32 && out_dtype == RB_F32 && wf) { RB_GNG(float, float, float); }
+    else if (proj_dtype == RB_F32 && out_dtype == RB_F32) { RB_GNG(float, float, bf); }
     else return RB_ERR_BAD_DTYPE;
 #undef RB_GNG
     RB_LAUNCH_CHECK();

@@ -23,9 +23,17 @@
 //                 states the blocks start from, along each sequence; every block's results.  c is kept as two floats, so
 //                 that a difference of two large sums is as exact as a small one.
 //
+//   mlstm chain   the same blocks for bfloat16 projections on the tensor cores (mma.sync), without the states in between going
+//                 through memory: a thread block owns 32 of a head's columns and walks the sequence's blocks of tokens with its
+//                 part of the state in registers; one more block a head does n and the divisors.  32-bit numbers enter a product as
+//                 the sum of three bfloat16 numbers (24 bits), their partner there being bfloat16 as it came from the
+//                 projection, so that every product is that of the 32-bit numbers, with 32-bit sums.  A kernel before it forms
+//                 the decayed scores (as three planes) and the decays for all blocks at once.
+//
 // All arithmetic is 32-bit.  q, k, v are columns of the layer's projection, in the activations' type or as 32-bit partial
 // sums that are added first; the gates' columns are 32-bit always.
 #include "common.cuh"
+#include "mma_tiles.cuh"
 #include "api.h"
 
 using namespace rb;
@@ -44,8 +52,14 @@ struct Cols {
     int row_stride;
     __device__ __forceinline__ float operator()(int t, int col) const {
         const IT* x = p + (size_t)t * row_stride + col;
-        float v = 0.f;
-        for (int s = 0; s < n_in; ++s) v += to_f32(x[(size_t)s * in_stride]);
+        float v = to_f32(x[0]);
+        for (int s = 1; s < n_in; s += 4) {                 // four partial sums in flight, added in order
+            float y[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) y[j] = s + j < n_in ? to_f32(x[(size_t)(s + j) * in_stride]) : 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v += y[j];
+        }
         return v;
     }
 };
@@ -456,6 +470,336 @@ mlstm_block_out_kernel(const Cols<IT> x, int q_off, int v_off, float q_scale, fl
         }
     }
 }
+
+// ---- prompts on the tensor cores --------------------------------------------------------------------------------------------
+using namespace mma_tiles;
+typedef __nv_bfloat16 bf16;
+
+// x = hi + mid + lo in bfloat16, two neighbouring numbers packed
+__device__ __forceinline__ void split3(float x, float y, uint32_t (&p)[3]) {
+#pragma unroll
+    for (int i = 0; i < 3; ++i) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+        p[i] = *reinterpret_cast<const uint32_t*>(&h);
+        const float2 f = __bfloat1622float2(h);
+        x -= f.x;
+        y -= f.y;
+    }
+}
+
+struct Rows16 {            // bfloat16 projection rows
+    const bf16* p;
+    long long stride;
+};
+
+constexpr int PLANE = CB * CB;      // one plane of a block's decayed scores
+
+// The decayed scores of a block as three planes [3][t][s], their sums over s, and for every token e^(c_t) * q_scale (`ec`) and
+// e^(c_end - c_t + log add_t) (`wt`), [heads][T]; e^(c_end) per block and head.  A warp owns 16 tokens t.
+template <int DIM>
+__global__ void __launch_bounds__(128)
+mlstm_scores_tc_kernel(const Rows16 x, int q_off, int k_off, float q_scale, int heads, const float* __restrict__ log_keep,
+                       const float* __restrict__ log_add, int T, const int* __restrict__ seq_slot, const int* __restrict__ cu_q, int n_seqs,
+                       bf16* __restrict__ planes, float* __restrict__ ec, float* __restrict__ wt, float* __restrict__ block_decay,
+                       float* __restrict__ den) {
+    pdl_wait();         // (no early signal: the kernel after this one has few blocks that run long)
+    extern __shared__ __align__(128) uint8_t raw_sm[];
+    bf16* Qs = reinterpret_cast<bf16*>(raw_sm);        // [64][DIM]
+    bf16* Ks = Qs + CB * DIM;
+    __shared__ BlockGates g;
+    int t0, m;
+    if (!find_tokens(blockIdx.y, seq_slot, cu_q, n_seqs, &t0, &m)) return;
+    const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    load_tile<DIM>(Qs, x.p + (long long)t0 * x.stride + q_off + h * DIM, x.stride, CB, m, threadIdx.x, 128);
+    load_tile<DIM>(Ks, x.p + (long long)t0 * x.stride + k_off + h * DIM, x.stride, CB, m, threadIdx.x, 128);
+    cp_async_commit();
+    block_gates(g, log_keep + (size_t)h * T, log_add + (size_t)h * T, t0, m);
+    if (threadIdx.x < m) {
+        const int t = threadIdx.x;
+        ec[(size_t)h * T + t0 + t] = expf(g.hi[t] + g.lo[t]) * q_scale;
+        wt[(size_t)h * T + t0 + t] = expf(g.decay(m - 1, t) + g.add[t]);
+    }
+    if (threadIdx.x == 0) block_decay[(size_t)blockIdx.y * heads + h] = expf(g.hi[m - 1] + g.lo[m - 1]);
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    const uint32_t qb = smem_addr(Qs), kb = smem_addr(Ks);
+#pragma unroll 4
+    for (int ks = 0; ks < DIM / 16; ++ks) {
+        uint32_t a[4];
+        ldmatrix_x4(tile_addr<DIM>(qb, warp * 16 + (lane & 15), ks * 2 + (lane >> 4)), a[0], a[1], a[2], a[3]);
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) {
+            if (j * 8 > warp * 16 + 15) continue;                       // keys after this warp's last token
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4(tile_addr<DIM>(kb, j * 8 + (lane & 7) + ((lane >> 4) & 1) * 8, ks * 2 + ((lane >> 3) & 1)), b0, b1, b2, b3);
+            mma_bf16(acc[j], a, b0, b1);
+            mma_bf16(acc[j + 1], a, b2, b3);
+        }
+    }
+    bf16* dst = planes + ((size_t)blockIdx.y * heads + h) * 3 * PLANE;
+    const int r0 = warp * 16 + (lane >> 2);
+    float sum[2] = {0.f, 0.f};
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+        const int s = j * 8 + (lane & 3) * 2;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int t = r0 + 8 * r;
+            float v[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e)
+                v[e] = s + e <= t && t < m ? acc[j][2 * r + e] * q_scale * expf(g.decay(t, s + e) + g.add[s + e]) : 0.f;
+            sum[r] += v[0] + v[1];
+            uint32_t p[3];
+            split3(v[0], v[1], p);
+#pragma unroll
+            for (int i = 0; i < 3; ++i) *reinterpret_cast<uint32_t*>(dst + i * PLANE + t * CB + s) = p[i];
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 1);
+        sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 2);
+        if ((lane & 3) == 0 && r0 + 8 * r < m) den[(size_t)(t0 + r0 + 8 * r) * heads + h] = sum[r];
+    }
+}
+
+constexpr int CHAIN_COLS = 32;      // columns of the state a block owns
+constexpr int RED_LD = 40;          // row length of the partial results (so that a half warp's pairs meet no bank twice)
+
+template <int DIM>
+struct ChainSizes {
+    static constexpr int QK = CB * DIM * 2, V = CB * CHAIN_COLS * 2, P = 3 * PLANE * 2;
+    static constexpr int BUF = 2 * QK + V + P;
+    static constexpr int RED = 4 * CB * RED_LD * 4;
+    static constexpr int SMEM = 2 * BUF + RED + 4 * CB * 4 + 128;
+};
+
+__device__ __forceinline__ uint32_t v_addr(uint32_t base, int row, int chunk) {       // rows of 64 bytes, four 16-byte chunks
+    return base + (uint32_t)(row * 64 + ((chunk ^ ((row >> 1) & 3)) << 4));
+}
+
+// Warps: two groups of 16 columns times four quarters of the head's dimensions.  S^T (columns of S as rows of the tile) lives in
+// the accumulators of its own update, which are at once the B operand of Q S.
+template <int DIM>
+__global__ void __launch_bounds__(256)
+mlstm_chain_kernel(const Rows16 x, int q_off, int k_off, int v_off, float eps, int heads, int vdim, const bf16* __restrict__ planes,
+                   const float* __restrict__ ec, const float* __restrict__ wt, const float* __restrict__ block_decay,
+                   const float* __restrict__ em, int T, float* __restrict__ S_state, float* __restrict__ n_state,
+                   const int* __restrict__ seq_slot, const int* __restrict__ cu_q, float* __restrict__ out, int ld_out,
+                   float* __restrict__ den) {
+    pdl_wait();
+    using Z = ChainSizes<DIM>;
+    extern __shared__ __align__(128) uint8_t raw_sm[];
+    float* red = reinterpret_cast<float*>(raw_sm + 2 * Z::BUF);            // [4][64][RED_LD]
+    float* tok = red + 4 * CB * RED_LD;                                    // [2 buffers][ec 64 | wt 64]
+    const int h = blockIdx.y, b = blockIdx.z;
+    const int slot = seq_slot[b];
+    if (slot < 0) return;
+    const int t_begin = cu_q[b], n_tok = cu_q[b + 1] - t_begin;
+    if (n_tok <= 0) return;
+    int first = 0;
+    for (int i = 0; i < b; ++i) first += seq_slot[i] >= 0 ? (cu_q[i + 1] - cu_q[i] + CB - 1) / CB : 0;
+    const int nb = (n_tok + CB - 1) / CB;
+    const bool n_role = blockIdx.x == gridDim.x - 1;
+    const int p0 = blockIdx.x * CHAIN_COLS;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int grp = warp & 1, dq = warp >> 1;
+
+    auto fetch = [&](int c) {
+        uint8_t* buf = raw_sm + (c & 1) * Z::BUF;
+        const int t0 = t_begin + c * CB, m = min(CB, n_tok - c * CB);
+        const bf16* row = x.p + (long long)t0 * x.stride;
+        load_tile<DIM>(reinterpret_cast<bf16*>(buf), row + q_off + h * DIM, x.stride, CB, m, tid, 256);
+        load_tile<DIM>(reinterpret_cast<bf16*>(buf + Z::QK), row + k_off + h * DIM, x.stride, CB, m, tid, 256);
+        if (!n_role) {
+            uint8_t* vb = buf + 2 * Z::QK;
+            {
+                const int r = tid >> 2, ch = tid & 3;                       // 64 rows of four chunks
+                cp_async16(vb + r * 64 + ((ch ^ ((r >> 1) & 3)) << 4),
+                           row + (r < m ? (long long)r * x.stride : 0) + v_off + h * vdim + p0 + ch * 8, r < m);
+            }
+            const bf16* pl = planes + ((size_t)(first + c) * heads + h) * 3 * PLANE;
+            load_tile<CB>(reinterpret_cast<bf16*>(vb + Z::V), pl, CB, 3 * CB, 3 * CB, tid, 256);
+        }
+        cp_async_commit();
+        if (tid < 2 * CB) {
+            const int t = tid & (CB - 1);
+            tok[(c & 1) * 2 * CB + tid] = t < m ? (tid < CB ? ec : wt)[(size_t)h * T + t0 + t] : 0.f;
+        }
+    };
+
+    if (n_role) {
+        // n and the divisors: a thread a dimension for the sums over tokens, a warp eight tokens for the products with q
+        float* ns = red;
+        float n = tid < DIM ? n_state[((size_t)slot * heads + h) * DIM + tid] : 0.f;
+        fetch(0);
+        for (int c = 0; c < nb; ++c) {
+            if (c + 1 < nb) { fetch(c + 1); cp_async_wait<1>(); }
+            else cp_async_wait<0>();
+            if (tid < DIM) ns[tid] = n;
+            __syncthreads();
+            const uint8_t* Q = raw_sm + (c & 1) * Z::BUF;
+            const uint8_t* K = Q + Z::QK;
+            const float* te = tok + (c & 1) * 2 * CB;
+            const int t0 = t_begin + c * CB, m = min(CB, n_tok - c * CB);
+            for (int r = warp; r < m; r += 8) {
+                float acc = 0.f;
+                for (int d = lane * 8; d < DIM; d += 256) {
+                    const uint4 raw = *reinterpret_cast<const uint4*>(Q + r * DIM * 2 + (((d >> 3) ^ (r & 7)) << 4));
+                    const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        acc = fmaf(__uint_as_float(w[u] << 16), ns[d + 2 * u], acc);
+                        acc = fmaf(__uint_as_float(w[u] & 0xFFFF0000u), ns[d + 2 * u + 1], acc);
+                    }
+                }
+                acc = warp_sum(acc);
+                if (lane == 0) {
+                    float* dp = den + (size_t)(t0 + r) * heads + h;
+                    *dp = fmaxf(fabsf(fmaf(te[r], acc, *dp)), em[(size_t)h * T + t0 + r]) + eps;
+                }
+            }
+            if (tid < DIM) {
+                float sum = 0.f;
+#pragma unroll 8
+                for (int s = 0; s < CB; ++s)
+                    sum = fmaf(te[CB + s], __bfloat162float(*reinterpret_cast<const bf16*>(K + s * DIM * 2 + (((tid >> 3) ^ (s & 7)) << 4) + (tid & 7) * 2)), sum);
+                n = fmaf(block_decay[(size_t)(first + c) * heads + h], n, sum);
+            }
+            __syncthreads();
+        }
+        if (tid < DIM) n_state[((size_t)slot * heads + h) * DIM + tid] = n;
+        return;
+    }
+
+    constexpr int KS = DIM / 64;                 // k steps of 16 dimensions in a warp's quarter
+    constexpr int NT = 2 * KS;                   // tiles of 8 dimensions
+    const int r0 = lane >> 2, c0 = (lane & 3) * 2;
+    float st[NT][4];
+    float* Sg = S_state + (((size_t)slot * heads + h) * DIM + dq * (DIM / 4)) * vdim + p0 + grp * 16;
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) st[j][e] = Sg[(size_t)(j * 8 + c0 + (e & 1)) * vdim + r0 + (e >> 1) * 8];
+    fetch(0);
+    for (int c = 0; c < nb; ++c) {
+        if (c + 1 < nb) { fetch(c + 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        const uint32_t qb = smem_addr(raw_sm + (c & 1) * Z::BUF), kb = qb + Z::QK, vb = kb + Z::QK, pb = vb + Z::V;
+        const float* te = tok + (c & 1) * 2 * CB;
+        const float* tw = te + CB;
+        float o[4][2][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
+        // Q S over this warp's dimensions
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) {
+            uint32_t b0[2][3], b1[2][3];
+            split3(st[2 * ks][0], st[2 * ks][1], b0[0]);
+            split3(st[2 * ks + 1][0], st[2 * ks + 1][1], b1[0]);
+            split3(st[2 * ks][2], st[2 * ks][3], b0[1]);
+            split3(st[2 * ks + 1][2], st[2 * ks + 1][3], b1[1]);
+            uint32_t a[4][4];
+#pragma unroll
+            for (int mt = 0; mt < 4; ++mt)
+                ldmatrix_x4(tile_addr<DIM>(qb, mt * 16 + (lane & 15), (dq * KS + ks) * 2 + (lane >> 4)), a[mt][0], a[mt][1], a[mt][2], a[mt][3]);
+#pragma unroll
+            for (int i = 2; i >= 0; --i)                                   // the small parts first; eight sums side by side
+#pragma unroll
+                for (int mt = 0; mt < 4; ++mt) {
+                    mma_bf16(o[mt][0], a[mt], b0[0][i], b1[0][i]);
+                    mma_bf16(o[mt][1], a[mt], b0[1][i], b1[1][i]);
+                }
+        }
+        // times e^(c_t), plus the block's own tokens: this warp's sixteen
+        uint32_t vv[4];
+        ldmatrix_x4_trans(v_addr(vb, dq * 16 + (lane & 15), grp * 2 + (lane >> 4)), vv[0], vv[1], vv[2], vv[3]);
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt) {
+            const float e0 = te[mt * 16 + r0], e1 = te[mt * 16 + r0 + 8];
+#pragma unroll
+            for (int j = 0; j < 2; ++j) { o[mt][j][0] *= e0; o[mt][j][1] *= e0; o[mt][j][2] *= e1; o[mt][j][3] *= e1; }
+        }
+#pragma unroll
+        for (int i = 2; i >= 0; --i)
+#pragma unroll
+            for (int mt = 0; mt < 4; ++mt) {
+                if (mt < dq) continue;                                     // tokens before this warp's
+                uint32_t a[4];
+                ldmatrix_x4(tile_addr<CB>(pb + i * PLANE * 2, mt * 16 + (lane & 15), dq * 2 + (lane >> 4)), a[0], a[1], a[2], a[3]);
+                mma_bf16(o[mt][0], a, vv[0], vv[1]);
+                mma_bf16(o[mt][1], a, vv[2], vv[3]);
+            }
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt) {
+            float* dst = red + ((size_t)dq * CB + mt * 16 + r0) * RED_LD + grp * 16 + c0;
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                *reinterpret_cast<float2*>(dst + j * 8) = make_float2(o[mt][j][0], o[mt][j][1]);
+                *reinterpret_cast<float2*>(dst + j * 8 + 8 * RED_LD) = make_float2(o[mt][j][2], o[mt][j][3]);
+            }
+        }
+        // the state after the block
+        const float decay = block_decay[(size_t)(first + c) * heads + h];
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) st[j][e] *= decay;
+#pragma unroll
+        for (int kt = 0; kt < 4; ++kt) {
+            uint32_t vr[4], a[3][4];
+            ldmatrix_x4_trans(v_addr(vb, kt * 16 + (lane & 7) + ((lane >> 4) & 1) * 8, grp * 2 + ((lane >> 3) & 1)), vr[0], vr[1], vr[2], vr[3]);
+            const float2 wa = *reinterpret_cast<const float2*>(tw + kt * 16 + c0), wb = *reinterpret_cast<const float2*>(tw + kt * 16 + 8 + c0);
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {
+                const float2 w = r < 2 ? wa : wb;
+                uint32_t p[3];
+                split3(__uint_as_float(vr[r] << 16) * w.x, __uint_as_float(vr[r] & 0xFFFF0000u) * w.y, p);
+#pragma unroll
+                for (int i = 0; i < 3; ++i) a[i][r] = p[i];
+            }
+            uint32_t kk[NT / 2][4];
+#pragma unroll
+            for (int j = 0; j < NT / 2; ++j)
+                ldmatrix_x4_trans(tile_addr<DIM>(kb, kt * 16 + (lane & 15), dq * KS * 2 + 2 * j + (lane >> 4)), kk[j][0], kk[j][1], kk[j][2], kk[j][3]);
+#pragma unroll
+            for (int i = 2; i >= 0; --i)
+#pragma unroll
+                for (int j = 0; j < NT / 2; ++j) {
+                    mma_bf16(st[2 * j], a[i], kk[j][0], kk[j][1]);
+                    mma_bf16(st[2 * j + 1], a[i], kk[j][2], kk[j][3]);
+                }
+        }
+        __syncthreads();                          // every part of the result is there, every tile has been read
+        const int t0 = t_begin + c * CB, m = min(CB, n_tok - c * CB);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int r = (tid >> 3) + 32 * u, col = (tid & 7) * 4;
+            if (r < m) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    float p[4];
+                    load4(red + ((size_t)q * CB + r) * RED_LD + col, p);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) v[e] += p[e];
+                }
+                store4(out + (size_t)(t0 + r) * ld_out + (size_t)h * vdim + p0 + col, v);
+            }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) Sg[(size_t)(j * 8 + c0 + (e & 1)) * vdim + r0 + (e >> 1) * 8] = st[j][e];
+}
 }  // namespace
 
 // gates: float32 partial sums [n_in][T][row_stride]; log_keep, log_add, em: float32 [heads][T].
@@ -523,6 +867,42 @@ extern "C" int rb_mlstm_blocks(const void* x, int x_dtype, int n_in, long long i
     else if (x_dtype == RB_BF16) RB_MB(__nv_bfloat16);
     else return RB_ERR_BAD_DTYPE;
 #undef RB_MB
+    RB_LAUNCH_CHECK();
+    return RB_OK;
+}
+
+// The same for bfloat16 projection rows on the tensor cores: dim 64, 128, 192 or 256, vdim a multiple of 32, every head of q, k and v
+// on a 16-byte boundary.  planes: bfloat16 [blocks][heads][3][64][64]; ec, wt: float32 [heads][T]; block_decay float32 [blocks][heads].
+extern "C" int rb_mlstm_chain(const void* x, int row_stride, int q_off, int k_off, int v_off, float q_scale, float eps, int heads, int dim,
+                              int vdim, const float* log_keep, const float* log_add, const float* em, int T, float* S_state, float* n_state,
+                              const int* seq_slot, const int* cu_q, int n_seqs, int blocks, void* planes, float* ec, float* wt,
+                              float* block_decay, float* out, int ld_out, float* den, void* stream) {
+    if (n_seqs <= 0 || blocks <= 0) return RB_OK;
+    if (heads <= 0 || vdim <= 0 || vdim % CHAIN_COLS || dim % 64 || dim < 64 || dim > 256 || n_seqs > 65535 || heads > 65535 || blocks > 65535)
+        return RB_ERR_BAD_SIZE;
+    if (((uintptr_t)x & 15) || row_stride % 8 || q_off % 8 || k_off % 8 || v_off % 8 || ((uintptr_t)planes & 15) || ((uintptr_t)out & 15) || ld_out % 4)
+        return RB_ERR_BAD_ALIGN;
+    cudaStream_t s = (cudaStream_t)stream;
+    const Rows16 r{(const bf16*)x, row_stride};
+    const dim3 grid(vdim / CHAIN_COLS + 1, heads, n_seqs);
+#define RB_MC(DIM)                                                                                                                  \
+    do {                                                                                                                            \
+        auto k1 = mlstm_scores_tc_kernel<DIM>;                                                                                      \
+        auto k2 = mlstm_chain_kernel<DIM>;                                                                                          \
+        constexpr int sm1 = 2 * CB * DIM * 2, sm2 = ChainSizes<DIM>::SMEM;                                                          \
+        cudaError_t e = cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, sm1);                                 \
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(k2, cudaFuncAttributeMaxDynamicSharedMemorySize, sm2);                       \
+        if (e != cudaSuccess) return (int)e;                                                                                        \
+        RB_LAUNCH((k1), dim3(heads, blocks), dim3(128), sm1, s, r, q_off, k_off, q_scale, heads, log_keep, log_add, T, seq_slot,    \
+                  cu_q, n_seqs, (bf16*)planes, ec, wt, block_decay, den);                                                           \
+        RB_LAUNCH((k2), grid, dim3(256), sm2, s, r, q_off, k_off, v_off, eps, heads, vdim, (const bf16*)planes, ec, wt, block_decay, \
+                  em, T, S_state, n_state, seq_slot, cu_q, out, ld_out, den);                                                       \
+    } while (0)
+    if (dim == 64) RB_MC(64);
+    else if (dim == 128) RB_MC(128);
+    else if (dim == 192) RB_MC(192);
+    else RB_MC(256);
+#undef RB_MC
     RB_LAUNCH_CHECK();
     return RB_OK;
 }

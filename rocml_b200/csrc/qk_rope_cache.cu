@@ -203,7 +203,9 @@ struct RotateExt {
     float temp_coef, temp_every;
 };
 
-template <typename IT, typename AT, typename WT, bool EXT>
+// MAPS 2: a head of 128 is two maps of 64 side by side, each normalised and turned on its own (sixteen lanes each); a query's two
+// maps go to two rows, each with zeros in the other's place.
+template <typename IT, typename AT, typename WT, bool EXT, int MAPS>
 __global__ void __launch_bounds__(128)
 qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, int row_stride,
                                 AT* __restrict__ q_out, int q_stride, int T, int nq, int nkv,
@@ -216,7 +218,8 @@ qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_s
     constexpr int hd = 128;
     // the lanes that hold a rotation pair's first and second member, and how far apart the two sit
     const int pair_lanes = EXT ? max(ext.rot_dim >> 3, 1) : 16;
-    const int cs_lane = EXT ? (int)(threadIdx.x & 31) % pair_lanes : (int)(threadIdx.x & 15);
+    constexpr int ML = 32 / MAPS;                                 // lanes a map
+    const int cs_lane = EXT ? (int)(threadIdx.x & (ML - 1)) % pair_lanes : (int)(threadIdx.x & 15);
     const int half = EXT ? ext.rot_dim >> 1 : 64;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int heads_total = nq + (write_kv ? 2 * nkv : 0);
@@ -225,7 +228,8 @@ qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_s
     // the norms' weights do not depend on the kernel before this one
     float wq[4] = {1.f, 1.f, 1.f, 1.f}, wk[4] = {1.f, 1.f, 1.f, 1.f};
     const bool has_w = q_norm_w != nullptr;
-    if (has_w) { load_w4(q_norm_w, lane, wq); load_w4(k_norm_w, lane, wk); }
+    const int ml = lane & (ML - 1);                               // this lane's place in its map
+    if (has_w) { load_w4(q_norm_w, ml, wq); load_w4(k_norm_w, ml, wk); }
     pdl_wait();
     if (item >= (long long)T * groups) return;
     const int t = (int)(item / groups);
@@ -243,8 +247,8 @@ qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_s
         cs_a = c4[0];
         cs_b = c4[1];
     }
-    const bool turns = !EXT || lane < 2 * pair_lanes;             // this lane's dimensions take part in the rotation
-    const bool pair_first = EXT ? lane < pair_lanes : lane < 16;
+    const bool turns = !EXT || ml < 2 * pair_lanes;             // this lane's dimensions take part in the rotation
+    const bool pair_first = EXT ? ml < pair_lanes : lane < 16;
     const int partner = EXT ? (pair_first ? lane + pair_lanes : (turns ? lane - pair_lanes : lane)) : lane ^ 16;
     const float lam = (EXT && ext.v_first) ? ext.v_lambda[0] : 0.f;
     int page = -2;
@@ -300,7 +304,7 @@ qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_s
         const int kind = h < nq ? 0 : (h < nq + nkv ? 1 : 2);   // 0 q, 1 k, 2 v
         AT* dst;
         if (kind == 0) {
-            dst = q_out + (size_t)t * q_stride + (size_t)h * hd;
+            dst = q_out + (size_t)t * q_stride + (size_t)h * hd * MAPS;
         } else {
             const int head = kind == 1 ? h - nq : h - nq - nkv;
             if (EXT && kind == 2 && ext.v_out)
@@ -317,8 +321,10 @@ qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_s
         float (&x)[4] = v[j];
         if (kind != 2) {
             if (has_w) {
-                const float ss = warp_sum(x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3]);
-                const float inv = rsqrtf(ss / (float)hd + eps);
+                float ss = x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3];
+#pragma unroll
+                for (int o = ML / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+                const float inv = rsqrtf(ss / (float)(hd / MAPS) + eps);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) x[i] = x[i] * inv * (kind == 0 ? wq[i] : wk[i]);
             }
@@ -341,6 +347,13 @@ qk_norm_rope_cache_hd128_kernel(const IT* __restrict__ in, int n_in, size_t in_s
 #pragma unroll
                 for (int i = 0; i < 4; ++i) x[i] *= f;
             }
+        }
+        if (MAPS > 1 && kind == 0) {                             // this map's row has the entries, the other map's zeros
+            const float z[4] = {0.f, 0.f, 0.f, 0.f};
+            const int map = lane / ML;
+            store4(dst + map * hd + lane * 4, x);
+            store4(dst + (1 - map) * hd + lane * 4, z);
+            continue;
         }
         if (sizeof(AT) == 4) {
             *reinterpret_cast<float4*>(dst + lane * 4) = make_float4(x[0], x[1], x[2], x[3]);
@@ -366,20 +379,22 @@ static int launch_qk(const void* in, int n_in, long long in_stride, int row_stri
     const long long blocks = (items + warps - 1) / warps;
     if (blocks > 0x7fffffffLL) return RB_ERR_BAD_SIZE;
     const size_t esz = sizeof(IT);
-    if (maps == 1 && hd == 128 && vd == 128 && hdp == 128 && n_gate == 0 && !(inv_freq && interleaved) &&
+    if (((maps == 1 && hd == 128) || (maps == 2 && hd == 64 && !post_norm)) && vd == 128 && hdp == 128 && n_gate == 0 && !(inv_freq && interleaved) &&
         (!inv_freq || rot_dim % 8 == 0) && (((uintptr_t)in | (uintptr_t)q_out | (uintptr_t)k_cache |
                                                           (uintptr_t)v_cache | (uintptr_t)qw | (uintptr_t)kw |
                                                           (uintptr_t)cs_table | (uintptr_t)v_first | (uintptr_t)v_out) & 15) == 0 &&
         (row_stride * esz) % 16 == 0 && ((size_t)in_stride * esz) % 16 == 0 && (q_stride * sizeof(AT)) % 16 == 0) {
-        const long long groups = (long long)T * ((nq + (write_kv ? 2 * nkv : 0) + HPW - 1) / HPW);
-        const bool ext = post_norm || v_first || v_out || temp_coef != 0.f || (inv_freq && rot_dim != 128);
+        const int heads = nq / maps;
+        const long long groups = (long long)T * ((heads + (write_kv ? 2 * nkv : 0) + HPW - 1) / HPW);
+        const bool ext = post_norm || v_first || v_out || temp_coef != 0.f || (inv_freq && rot_dim != 128) || maps > 1;
         const RotateExt e{inv_freq ? rot_dim : 128, post_norm, v_first, v_lambda, v_out, temp_coef, temp_every};
-#define RB_QK128(EXT)                                                                                                          \
-        RB_LAUNCH((qk_norm_rope_cache_hd128_kernel<IT, AT, WT, EXT>), dim3((int)((groups + 3) / 4)), dim3(128), 0, s, (const IT*)in, \
-                  n_in, (size_t)in_stride, row_stride, (AT*)q_out, q_stride, T, nq, nkv, (const WT*)qw, (const WT*)kw, eps,    \
+#define RB_QK128(EXT, MAPS)                                                                                                    \
+        RB_LAUNCH((qk_norm_rope_cache_hd128_kernel<IT, AT, WT, EXT, MAPS>), dim3((int)((groups + 3) / 4)), dim3(128), 0, s, (const IT*)in, \
+                  n_in, (size_t)in_stride, row_stride, (AT*)q_out, q_stride, T, heads, nkv, (const WT*)qw, (const WT*)kw, eps,    \
                   inv_freq, positions, slot_of_token, block_table, max_pages, (AT*)k_cache, (AT*)v_cache, write_kv, cs_table, e)
-        if (ext) RB_QK128(true);
-        else RB_QK128(false);
+        if (maps == 2) RB_QK128(true, 2);
+        else if (ext) RB_QK128(true, 1);
+        else RB_QK128(false, 1);
 #undef RB_QK128
         return RB_OK;
     }

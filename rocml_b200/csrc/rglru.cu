@@ -7,14 +7,17 @@
 //   out = S * gelu_tanh(y) * factor
 //
 //   rglru_gates   prompts: both block products of a tile of 64 tokens and 64 channels side by side, and from them the decay a
-//                 and the input sqrt(1 - a^2) i u of every token and channel.
-//   rglru_scan    prompts: a block owns 32 channels of a sequence, a warp one run of its tokens.  Each warp first forms its
-//                 run's own sum and product of decays, then every warp knows the state its run starts from, and walks it
+//                 and the input sqrt(1 - a^2) i u of every token and channel, next to each other.  With bfloat16 weights on the tensor
+//                 cores (mma.sync): the 32-bit u enters as the sum of three bfloat16 numbers (24 bits), the sums are 32-bit, so
+//                 the products are those of the 32-bit numbers.  Otherwise FMA.
+//   rglru_scan    prompts: a block owns 16 channels of a sequence, half a warp one run of its tokens.  Each first forms its
+//                 run's own sum and product of decays, then every half warp knows the state its run starts from, and walks it
 //                 again to write the results.
 //   rglru_step    one token a sequence: products, gates, recurrence and result in one kernel.
 //
 // Everything is 32-bit; u comes from the convolution in 32-bit, y is a column block of the projection.
 #include "common.cuh"
+#include "mma_tiles.cuh"
 #include "api.h"
 
 using namespace rb;
@@ -33,7 +36,7 @@ template <typename WT>
 __global__ void __launch_bounds__(256)
 rglru_gates_kernel(const float* __restrict__ u, int ld_u, const WT* __restrict__ ra, const WT* __restrict__ ri,
                    const float* __restrict__ ra_b, const float* __restrict__ ri_b, const float* __restrict__ rate, int part, int tiles,
-                   int T, float* __restrict__ a_out, float* __restrict__ x_out, int width) {
+                   int T, float2* __restrict__ ax, int width) {
     pdl_trigger();
     pdl_wait();
     __shared__ __align__(16) float Us[TK * LD], Rs[TK * LD], Is[TK * LD];
@@ -78,8 +81,102 @@ rglru_gates_kernel(const float* __restrict__ u, int ld_u, const WT* __restrict__
             const int ch = blk * part + c;
             float a, x;
             gate_pair(ar[p][q] + ra_b[ch], ai[p][q] + ri_b[ch], rate[ch], u[(size_t)t * ld_u + ch], &a, &x);
-            a_out[(size_t)t * width + ch] = a;
-            x_out[(size_t)t * width + ch] = x;
+            ax[(size_t)t * width + ch] = make_float2(a, x);
+        }
+    }
+}
+
+// The same on the tensor cores.  A warp owns 16 tokens and 32 channels of both gates; a step of 64 inputs is split into its three
+// planes as it is staged.
+__global__ void __launch_bounds__(256)
+rglru_gates_tc_kernel(const float* __restrict__ u, int ld_u, const __nv_bfloat16* __restrict__ ra, const __nv_bfloat16* __restrict__ ri,
+                      const float* __restrict__ ra_b, const float* __restrict__ ri_b, const float* __restrict__ rate, int part, int tiles,
+                      int T, float2* __restrict__ ax, int width) {
+    using namespace mma_tiles;
+    typedef __nv_bfloat16 bf16;
+    pdl_trigger();
+    pdl_wait();
+    __shared__ __align__(128) bf16 Us[3][64 * 64], Rs[64 * 64], Is[64 * 64];       // rows of 64 inputs, swizzled
+    const int blk = blockIdx.x / tiles, n0 = (blockIdx.x % tiles) * 64, m0 = blockIdx.y * 64;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int mt = warp & 3, nh = warp >> 2;
+    const float* ub = u + (size_t)blk * part;
+    const bf16* rw = ra + (size_t)blk * part * part;
+    const bf16* iw = ri + (size_t)blk * part * part;
+    float ar[4][4], ai[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ar[j][e] = ai[j][e] = 0.f;
+    const uint32_t u0 = smem_addr(Us[0]), rs = smem_addr(Rs), is = smem_addr(Is);
+    for (int k0 = 0; k0 < part; k0 += 64) {
+        __syncthreads();
+#pragma unroll
+        for (int v = 0; v < 2; ++v) {                                    // weights: 64 rows of eight 16-byte chunks each
+            const int idx = tid + v * 256, r = idx >> 3, ch = idx & 7;
+            const bool in = n0 + r < part && k0 + ch * 8 < part;
+            const size_t at = in ? (size_t)(n0 + r) * part + k0 + ch * 8 : 0;
+            cp_async16(reinterpret_cast<uint8_t*>(Rs) + r * 128 + ((ch ^ (r & 7)) << 4), rw + at, in);
+            cp_async16(reinterpret_cast<uint8_t*>(Is) + r * 128 + ((ch ^ (r & 7)) << 4), iw + at, in);
+        }
+        cp_async_commit();
+#pragma unroll
+        for (int v = 0; v < 4; ++v) {                                    // inputs: four numbers a thread and turn
+            const int idx = tid + v * 256, r = idx >> 4, c = (idx & 15) * 4;
+            float f[4] = {0.f, 0.f, 0.f, 0.f};
+            if (m0 + r < T && k0 + c < part) load4(ub + (size_t)(m0 + r) * ld_u + k0 + c, f);
+            const int at = r * 128 + (((c >> 3) ^ (r & 7)) << 4) + (c & 4) * 2;
+#pragma unroll
+            for (int i = 0; i < 3; ++i) {
+                const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+                *reinterpret_cast<uint2*>(reinterpret_cast<uint8_t*>(Us[i]) + at) =
+                    make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+                const float2 fa = __bfloat1622float2(a), fb = __bfloat1622float2(b);
+                f[0] -= fa.x; f[1] -= fa.y; f[2] -= fb.x; f[3] -= fb.y;
+            }
+        }
+        cp_async_wait<0>();
+        __syncthreads();
+        const int steps = min(4, (part - k0 + 15) / 16);
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            if (ks >= steps) break;
+            uint32_t a[3][4];
+#pragma unroll
+            for (int i = 0; i < 3; ++i)
+                ldmatrix_x4(tile_addr<64>(u0 + i * 64 * 64 * 2, mt * 16 + (lane & 15), ks * 2 + (lane >> 4)), a[i][0], a[i][1], a[i][2], a[i][3]);
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int row = nh * 32 + j * 8 + (lane & 7) + ((lane >> 4) & 1) * 8, ch = ks * 2 + ((lane >> 3) & 1);
+                uint32_t r0, r1, r2, r3, i0, i1, i2, i3;
+                ldmatrix_x4(tile_addr<64>(rs, row, ch), r0, r1, r2, r3);
+                ldmatrix_x4(tile_addr<64>(is, row, ch), i0, i1, i2, i3);
+#pragma unroll
+                for (int i = 2; i >= 0; --i) {                            // the small parts first
+                    mma_bf16(ar[j], a[i], r0, r1);
+                    mma_bf16(ar[j + 1], a[i], r2, r3);
+                    mma_bf16(ai[j], a[i], i0, i1);
+                    mma_bf16(ai[j + 1], a[i], i2, i3);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int c = n0 + nh * 32 + j * 8 + (lane & 3) * 2;
+        if (c >= part) continue;                                         // (part is even: both channels of a pair or none)
+        const int ch = blk * part + c;
+        const float2 rb = *reinterpret_cast<const float2*>(ra_b + ch), ib = *reinterpret_cast<const float2*>(ri_b + ch),
+                     rt = *reinterpret_cast<const float2*>(rate + ch);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int t = m0 + mt * 16 + (lane >> 2) + 8 * e;
+            if (t >= T) continue;
+            const float2 uu = *reinterpret_cast<const float2*>(u + (size_t)t * ld_u + ch);
+            float4 o;
+            gate_pair(ar[j][2 * e] + rb.x, ai[j][2 * e] + ib.x, rt.x, uu.x, &o.x, &o.y);
+            gate_pair(ar[j][2 * e + 1] + rb.y, ai[j][2 * e + 1] + ib.y, rt.y, uu.y, &o.z, &o.w);
+            *reinterpret_cast<float4*>(ax + (size_t)t * width + ch) = o;
         }
     }
 }
@@ -91,66 +188,70 @@ struct Branch {            // the other branch's columns of the projection rows:
     size_t in_stride;
     int row_stride;
     __device__ __forceinline__ float operator()(int t, int c) const {
-        float v = 0.f;
-        for (int s = 0; s < n_in; ++s) v += to_f32(p[(size_t)s * in_stride + (size_t)t * row_stride + c]);
+        const YT* x = p + (size_t)t * row_stride + c;
+        float v = to_f32(x[0]);
+        for (int s = 1; s < n_in; s += 4) {                 // four in flight, added in order
+            float y[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) y[j] = s + j < n_in ? to_f32(x[(size_t)(s + j) * in_stride]) : 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v += y[j];
+        }
         return v;
     }
 };
 
-constexpr int SW = 32;             // warps a block: runs of tokens
+constexpr int SCH = 16;            // channels a block
+constexpr int SW = 32;             // runs of tokens: half a warp each (512 threads: several blocks a multiprocessor)
 template <typename YT, typename AT>
-__global__ void __launch_bounds__(SW * 32)
-rglru_scan_kernel(const float* __restrict__ a, const float* __restrict__ x, int width, const Branch<YT> y, float factor,
-                  float* __restrict__ state, const int* __restrict__ seq_slot, const int* __restrict__ cu_q, AT* __restrict__ out, int ld_out) {
-    pdl_trigger();
-    pdl_wait();
-    __shared__ float prod[SW][32], own[SW][32];
+__global__ void __launch_bounds__(SW * SCH)
+rglru_scan_kernel(const float2* __restrict__ ax, int width, const Branch<YT> y, float factor, float* __restrict__ state,
+                  const int* __restrict__ seq_slot, const int* __restrict__ cu_q, AT* __restrict__ out, int ld_out) {
+    pdl_wait();                                     // (no early signal: few blocks that run long)
+    __shared__ float prod[SW][SCH], own[SW][SCH];
     const int b = blockIdx.y;
     const int slot = seq_slot[b];
     if (slot < 0) return;
     const int t0 = cu_q[b], n = cu_q[b + 1] - t0;
     if (n <= 0) return;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int c = blockIdx.x * 32 + lane;
+    const int run = threadIdx.x / SCH, lane = threadIdx.x % SCH;
+    const int c = blockIdx.x * SCH + lane;
     const bool here = c < width;
-    const int run = (n + SW - 1) / SW;
-    const int lo = min(n, warp * run), hi = min(n, lo + run);
-    const float* ap = a + (size_t)t0 * width + c;
-    const float* xp = x + (size_t)t0 * width + c;
+    const int len = (n + SW - 1) / SW;
+    const int lo = min(n, run * len), hi = min(n, lo + len);
+    const float2* p = ax + (size_t)t0 * width + c;
     float* st = state + (size_t)slot * width + c;
-    const float start = here ? *st : 0.f;           // every warp reads it before the barrier, one writes it after
+    const float start = here ? *st : 0.f;           // every run reads it before the barrier, one writes it after
     float P = 1.f, S = 0.f;
-    constexpr int U = 8;
+    constexpr int U = 16;
     if (here) {
         for (int t = lo; t < hi; t += U) {
-            float av[U], xv[U];
+            float2 v[U];
 #pragma unroll
-            for (int j = 0; j < U; ++j) {
-                av[j] = t + j < hi ? ap[(size_t)(t + j) * width] : 1.f;
-                xv[j] = t + j < hi ? xp[(size_t)(t + j) * width] : 0.f;
-            }
+            for (int j = 0; j < U; ++j) v[j] = t + j < hi ? p[(size_t)(t + j) * width] : make_float2(1.f, 0.f);
 #pragma unroll
-            for (int j = 0; j < U; ++j) { S = fmaf(av[j], S, xv[j]); P *= av[j]; }
+            for (int j = 0; j < U; ++j) { S = fmaf(v[j].x, S, v[j].y); P *= v[j].x; }
         }
     }
-    prod[warp][lane] = P;
-    own[warp][lane] = S;
+    prod[run][lane] = P;
+    own[run][lane] = S;
     __syncthreads();
     if (!here || lo >= hi) return;
     S = start;
-    for (int w = 0; w < warp; ++w) S = fmaf(prod[w][lane], S, own[w][lane]);
+    for (int w = 0; w < run; ++w) S = fmaf(prod[w][lane], S, own[w][lane]);
     AT* op = out + (size_t)t0 * ld_out + c;
-    for (int t = lo; t < hi; t += U) {
-        float av[U], xv[U], yv[U];
+    constexpr int U2 = 8;
+    for (int t = lo; t < hi; t += U2) {
+        float2 v[U2];
+        float yv[U2];
 #pragma unroll
-        for (int j = 0; j < U; ++j) {
-            av[j] = t + j < hi ? ap[(size_t)(t + j) * width] : 1.f;
-            xv[j] = t + j < hi ? xp[(size_t)(t + j) * width] : 0.f;
+        for (int j = 0; j < U2; ++j) {
+            v[j] = t + j < hi ? p[(size_t)(t + j) * width] : make_float2(1.f, 0.f);
             yv[j] = t + j < hi ? y(t0 + t + j, c) : 0.f;
         }
 #pragma unroll
-        for (int j = 0; j < U; ++j) {
-            S = fmaf(av[j], S, xv[j]);
+        for (int j = 0; j < U2; ++j) {
+            S = fmaf(v[j].x, S, v[j].y);
             if (t + j < hi) op[(size_t)(t + j) * ld_out] = from_f32<AT>(S * gelu_tanh(yv[j]) * factor);
         }
     }
@@ -176,11 +277,18 @@ rglru_step_kernel(const float* __restrict__ u, int ld_u, const WT* __restrict__ 
         const int t = idx / part, k = idx - t * part;
         us[idx] = t0 + t < T ? u[(size_t)(t0 + t) * ld_u + (size_t)blk * part + k] : 0.f;
     }
+    // what this lane will end up with: its state and its part of the other branch are asked for before the products
+    const int r0 = n0 + warp * 4;
+    const int c = r0 + (lane >> 3), t = t0 + (lane & 7), ch = blk * part + c;
+    const bool mine = c < part && t < T;
+    const int slot = mine ? slot_of_token[t] : -1;
+    float* st = state + (size_t)(slot < 0 ? 0 : slot) * width + (mine ? ch : 0);
+    float before = 0.f, yv = 0.f, zr = 0.f, zi = 0.f, rt = 0.f;
+    if (slot >= 0) { before = *st; yv = y(t, ch); zr = ra_b[ch]; zi = ri_b[ch]; rt = rate[ch]; }
     __syncthreads();
     float v[64];
 #pragma unroll
     for (int j = 0; j < 64; ++j) v[j] = 0.f;
-    const int r0 = n0 + warp * 4;
     for (int k = lane * V; k < part; k += 32 * V) {
         float uv[ST][V];
 #pragma unroll
@@ -213,30 +321,32 @@ rglru_step_kernel(const float* __restrict__ u, int ld_u, const WT* __restrict__ 
                 const float mine = up ? v[j + n] : v[j], other = up ? v[j] : v[j + n];
                 v[j] = mine + __shfl_xor_sync(0xffffffffu, other, o);
             }
-    const int c = r0 + (lane >> 3), t = t0 + (lane & 7);        // what this lane ended up with
-    if (c >= part || t >= T) return;
-    const int slot = slot_of_token[t];
     if (slot < 0) return;
-    const int ch = blk * part + c;
     float a, x;
-    gate_pair(v[0] + ra_b[ch], v[1] + ri_b[ch], rate[ch], us[(lane & 7) * part + c], &a, &x);
-    float* st = state + (size_t)slot * width + ch;
-    const float S = fmaf(a, *st, x);
+    gate_pair(v[0] + zr, v[1] + zi, rt, us[(lane & 7) * part + c], &a, &x);
+    const float S = fmaf(a, before, x);
     *st = S;
-    out[(size_t)t * ld_out + ch] = from_f32<AT>(S * gelu_tanh(y(t, ch)) * factor);
+    out[(size_t)t * ld_out + ch] = from_f32<AT>(S * gelu_tanh(yv) * factor);
 }
 }  // namespace
 
 extern "C" int rb_rglru_gates(const float* u, int ld_u, const void* ra, const void* ri, int w_dtype, const float* ra_b, const float* ri_b,
-                              const float* rate, int blocks, int part, int T, float* a, float* x, void* stream) {
+                              const float* rate, int blocks, int part, int T, float* ax, void* stream) {
     if (T <= 0) return RB_OK;
     if (blocks <= 0 || part <= 0) return RB_ERR_BAD_SIZE;
     const int tiles = (part + TN - 1) / TN;
     const dim3 grid(blocks * tiles, (T + TM - 1) / TM);
     if (grid.y > 65535) return RB_ERR_BAD_SIZE;
+    if (w_dtype == RB_BF16 && part % 8 == 0 && ld_u % 4 == 0 && (((uintptr_t)u | (uintptr_t)ra | (uintptr_t)ri | (uintptr_t)ax) & 15) == 0 &&
+        (((uintptr_t)ra_b | (uintptr_t)ri_b | (uintptr_t)rate) & 7) == 0) {
+        RB_LAUNCH((rglru_gates_tc_kernel), grid, dim3(256), 0, (cudaStream_t)stream, u, ld_u, (const __nv_bfloat16*)ra, (const __nv_bfloat16*)ri,
+                  ra_b, ri_b, rate, part, tiles, T, (float2*)ax, blocks * part);
+        RB_LAUNCH_CHECK();
+        return RB_OK;
+    }
 #define RB_RG(WT)                                                                                                               \
     RB_LAUNCH((rglru_gates_kernel<WT>), grid, dim3(256), 0, (cudaStream_t)stream, u, ld_u, (const WT*)ra, (const WT*)ri, ra_b,  \
-              ri_b, rate, part, tiles, T, a, x, blocks * part)
+              ri_b, rate, part, tiles, T, (float2*)ax, blocks * part)
     if (w_dtype == RB_F32) RB_RG(float);
     else if (w_dtype == RB_BF16) RB_RG(__nv_bfloat16);
     else return RB_ERR_BAD_DTYPE;
@@ -245,15 +355,16 @@ extern "C" int rb_rglru_gates(const float* u, int ld_u, const void* ra, const vo
     return RB_OK;
 }
 
-extern "C" int rb_rglru_scan(const float* a, const float* x, int width, const void* y, int y_dtype, int n_in, long long in_stride,
+extern "C" int rb_rglru_scan(const float* ax, int width, const void* y, int y_dtype, int n_in, long long in_stride,
                              int row_stride, float factor, float* state, const int* seq_slot, const int* cu_q, int n_seqs, void* out,
                              int out_dtype, int ld_out, void* stream) {
     if (n_seqs <= 0) return RB_OK;
     if (width <= 0 || n_in < 1 || n_seqs > 65535) return RB_ERR_BAD_SIZE;
-    const dim3 grid((width + 31) / 32, n_seqs);
+    if ((uintptr_t)ax & 7) return RB_ERR_BAD_ALIGN;
+    const dim3 grid((width + SCH - 1) / SCH, n_seqs);
     typedef __nv_bfloat16 bf;
 #define RB_RS(YT, AT)                                                                                                            \
-    RB_LAUNCH((rglru_scan_kernel<YT, AT>), grid, dim3(SW * 32), 0, (cudaStream_t)stream, a, x, width,                            \
+    RB_LAUNCH((rglru_scan_kernel<YT, AT>), grid, dim3(SW * SCH), 0, (cudaStream_t)stream, (const float2*)ax, width,                            \
               Branch<YT>{(const YT*)y, n_in, (size_t)in_stride, row_stride}, factor, state, seq_slot, cu_q, (AT*)out, ld_out)
     if (y_dtype == RB_BF16 && out_dtype == RB_BF16) RB_RS(bf, bf);
     else if (y_dtype == RB_F32 && out_dtype == RB_BF16) RB_RS(float, bf);

@@ -121,6 +121,91 @@ causal_conv_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, int ro
     }
 }
 
+// The same, four neighbouring channels a thread (channels, strides and addresses allow 4-element accesses).
+template <typename IT>
+__device__ __forceinline__ void sum4(const IT* p, int n_in, size_t in_stride, float (&v)[4]) {
+    v[0] = v[1] = v[2] = v[3] = 0.f;
+    for (int s = 0; s < n_in; s += 4) {                     // four partial sums in flight, added in order
+        float x[4][4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            if (s + j < n_in) load4(p + (size_t)(s + j) * in_stride, x[j]);
+            else x[j][0] = x[j][1] = x[j][2] = x[j][3] = 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) v[u] += x[j][u];
+    }
+}
+
+template <typename IT, int TAPS>
+__global__ void __launch_bounds__(CONV_CH)
+causal_conv4_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, int row_stride, int col0, int channels, const float* __restrict__ w,
+                    const float* __restrict__ bias, int act, float* __restrict__ kept, const int* __restrict__ seq_slot,
+                    const int* __restrict__ cu_q, float* __restrict__ out, int ld_out) {
+    pdl_trigger();
+    pdl_wait();
+    constexpr int BACK = TAPS - 1;
+    const int b = blockIdx.z;
+    const int slot = seq_slot[b];
+    if (slot < 0) return;
+    const int t_begin = cu_q[b], t_end = cu_q[b + 1];
+    const int t0 = t_begin + blockIdx.y * CONV_TOK;
+    if (t0 >= t_end) return;
+    const int c = (blockIdx.x * CONV_CH + threadIdx.x) * 4;
+    if (c >= channels) return;
+    float* mine = kept + (size_t)slot * BACK * channels + c;       // [BACK][channels]
+    float wt[4][TAPS], win[TAPS][4], bc[4] = {0.f, 0.f, 0.f, 0.f};
+    if (bias) load4(bias + c, bc);
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wt[u][j] = w[(size_t)(c + u) * TAPS + j];
+#pragma unroll
+    for (int j = 0; j < BACK; ++j) {
+        const int t = t0 - BACK + j;                               // the rows before the block's first
+        if (t >= t_begin) sum4(in + (size_t)t * row_stride + col0 + c, n_in, in_stride, win[j + 1]);
+        else load4(mine + (size_t)(BACK + (t - t_begin)) * channels, win[j + 1]);
+    }
+    const int n = min(CONV_TOK, t_end - t0);
+    const IT* src = in + (size_t)t0 * row_stride + col0 + c;
+    for (int tt = 0; tt < n; tt += 4) {
+        float fresh[4][4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+            if (tt + k < n) sum4(src + (size_t)(tt + k) * row_stride, n_in, in_stride, fresh[k]);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            if (tt + k >= n) continue;
+            float acc[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+#pragma unroll
+                for (int j = 0; j < BACK; ++j) win[j][u] = win[j + 1][u];
+                win[BACK][u] = fresh[k][u];
+                acc[u] = bc[u];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc[u] = fmaf(wt[u][j], win[j][u], acc[u]);
+                if (act == 1) acc[u] = silu(acc[u]);
+            }
+            store4(out + (size_t)(t0 + tt + k) * ld_out + c, acc);
+        }
+    }
+    if (blockIdx.y == 0 && BACK > 0) {          // as above: one thread alone reads and rewrites a channel's kept rows
+        const int len = t_end - t_begin;
+        float last[TAPS][4];
+#pragma unroll
+        for (int j = 0; j < BACK; ++j) {
+            const int at = len + j;
+            if (at < BACK) load4(mine + (size_t)at * channels, last[j]);
+            else sum4(in + (size_t)(t_begin + at - BACK) * row_stride + col0 + c, n_in, in_stride, last[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < BACK; ++j) store4(mine + (size_t)j * channels, last[j]);
+    }
+}
+
 constexpr int SCAN_THREADS = 256;
 constexpr int SCAN_TB = 8;
 
@@ -632,6 +717,22 @@ extern "C" int rb_causal_conv(const void* in, int in_dtype, int n_in, long long 
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid((channels + CONV_CH - 1) / CONV_CH, (max_q_len + CONV_TOK - 1) / CONV_TOK, n_seqs);
     if (grid.y > 65535) return RB_ERR_BAD_SIZE;
+    const size_t isz = in_dtype == RB_F32 ? 4 : 2;
+    if ((taps == 2 || taps == 3 || taps == 4) && ((channels | col0 | row_stride | ld_out) & 3) == 0 && (in_stride & 3) == 0 &&
+        ((uintptr_t)in & (4 * isz - 1)) == 0 && (((uintptr_t)kept | (uintptr_t)out | (uintptr_t)bias) & 15) == 0 && kept) {
+        const dim3 grid4((channels / 4 + CONV_CH - 1) / CONV_CH, grid.y, n_seqs);
+#define RB_CONV4(IT, TAPS)                                                                                                     \
+    RB_LAUNCH((causal_conv4_kernel<IT, TAPS>), grid4, dim3(CONV_CH), 0, s, (const IT*)in, n_in, (size_t)in_stride, row_stride, col0, \
+              channels, w, bias, act, kept, seq_slot, cu_q, out, ld_out)
+#define RB_CONV4_T(IT) do { if (taps == 4) RB_CONV4(IT, 4); else if (taps == 3) RB_CONV4(IT, 3); else RB_CONV4(IT, 2); } while (0)
+        if (in_dtype == RB_F32) RB_CONV4_T(float);
+        else if (in_dtype == RB_BF16) RB_CONV4_T(__nv_bfloat16);
+        else return RB_ERR_BAD_DTYPE;
+#undef RB_CONV4_T
+#undef RB_CONV4
+        RB_LAUNCH_CHECK();
+        return RB_OK;
+    }
 #define RB_CONV(IT, TAPS)                                                                                                      \
     RB_LAUNCH((causal_conv_kernel<IT, TAPS>), grid, dim3(CONV_CH), 0, s, (const IT*)in, n_in, (size_t)in_stride, row_stride, col0, \
               channels, taps, w, bias, act, kept, seq_slot, cu_q, out, ld_out)

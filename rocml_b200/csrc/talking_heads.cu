@@ -43,16 +43,16 @@ __device__ __forceinline__ float turned(const float* x, int d, int rot, bool nei
 }
 
 template <typename IT, typename AT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 wide_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, size_t in_stride, int row_stride, int nq, int nkv, int hd,
                             int vd, int hdp, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
                             const float* __restrict__ factor, const float* __restrict__ cos_sin, int rot, int neighbours,
                             AT* __restrict__ q_out, int q_stride, AT* __restrict__ k_cache, AT* __restrict__ v_cache,
                             const int* __restrict__ positions, const int* __restrict__ slot_of_token,
-                            const int* __restrict__ block_table, int max_pages) {
+                            const int* __restrict__ block_table, int max_pages, int vec) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ __align__(16) float buf[];            // (nq + nkv) * hd floats + 33
+    extern __shared__ __align__(16) float buf[];            // (nq + nkv) * hd floats + 64
     const int qw = nq * hd, kw = nkv * hd;
     float* kb = buf + qw;
     float* red = kb + kw;
@@ -60,6 +60,8 @@ wide_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, size_t in_strid
     const int slot = slot_of_token[t];
     if (slot < 0) return;
     const IT* row = in + (size_t)t * row_stride;
+    const int pos = positions[t];
+    const int page = block_table[(size_t)slot * max_pages + pos / RB_PAGE];
     float sq = 0.f, sk = 0.f;
     if (((qw | kw | row_stride) & 3) == 0 && (in_stride & 3) == 0 && ((uintptr_t)in & (4 * sizeof(IT) - 1)) == 0) {
         for (int i = threadIdx.x * 4; i < qw + kw; i += blockDim.x * 4) {      // four values a load; a group of four lies in q or in k
@@ -84,28 +86,80 @@ wide_norm_rope_cache_kernel(const IT* __restrict__ in, int n_in, size_t in_strid
     // both sums of squares in one pass over the block
     sq = warp_sum(sq);
     sk = warp_sum(sk);
-    if ((threadIdx.x & 31) == 0) { red[threadIdx.x >> 5] = sq; red[8 + (threadIdx.x >> 5)] = sk; }
+    if ((threadIdx.x & 31) == 0) { red[threadIdx.x >> 5] = sq; red[32 + (threadIdx.x >> 5)] = sk; }
     __syncthreads();
     sq = sk = 0.f;
-#pragma unroll
-    for (int w = 0; w < 8; ++w) { sq += red[w]; sk += red[8 + w]; }       // 256 threads: eight warps, added in their order
+    for (int w = 0; w < (int)(blockDim.x >> 5); ++w) { sq += red[w]; sk += red[32 + w]; }       // the warps' sums in their order
     const float inv_q = wq ? rsqrtf(sq / (float)qw + eps) : 1.f;
     const float inv_k = wk ? rsqrtf(sk / (float)kw + eps) : 1.f;
-    for (int i = threadIdx.x; i < qw + kw; i += blockDim.x) {
-        if (i < qw) { if (wq) buf[i] *= inv_q * wq[i]; }
-        else if (wk) buf[i] *= inv_k * wk[i - qw];
+    if (!vec) {
+        for (int i = threadIdx.x; i < qw + kw; i += blockDim.x) {
+            if (i < qw) { if (wq) buf[i] *= inv_q * wq[i]; }
+            else if (wk) buf[i] *= inv_k * wk[i - qw];
+        }
+        __syncthreads();
     }
-    __syncthreads();
     const float* cs = cos_sin ? cos_sin + (size_t)t * (rot >> 1) * 2 : nullptr;
     const int r = cs ? rot : 0;
+    if (vec) {
+        // four neighbouring entries a thread: heads as wide as they are stored, pairs half a rotation apart (or no rotation)
+        const int half = r >> 1, q4 = qw >> 2, k4 = kw >> 2, v4 = (nkv * vd) >> 2;
+        for (int g = threadIdx.x; g < q4 + k4 + v4; g += blockDim.x) {
+            float x[4];
+            if (g >= q4 + k4) {                                    // a value: as it came
+                if (page < 0) break;
+                const int i = (g - q4 - k4) * 4, h = i / vd, d = i - h * vd;
+                x[0] = x[1] = x[2] = x[3] = 0.f;
+                for (int s = 0; s < n_in; ++s) {
+                    float p[4];
+                    load4(row + (size_t)s * in_stride + qw + kw + i, p);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) x[u] += p[u];
+                }
+                store4(v_cache + (((size_t)page * nkv + h) * RB_PAGE + (pos % RB_PAGE)) * hdp + d, x);
+                continue;
+            }
+            const int i = g * 4, j = g < q4 ? i : i - qw, h = j / hd, d = j - h * hd;
+            // the norm on the way: this entry's and, below, its partner's
+            const float* w = g < q4 ? wq : wk;
+            const float inv = g < q4 ? inv_q : inv_k;
+            auto normed = [&](int at, float (&e)[4]) {
+                load4(buf + at, e);
+                if (w) {
+                    float f[4];
+                    load4(w + (g < q4 ? at : at - qw), f);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) e[u] *= inv * f[u];
+                }
+            };
+            normed(i, x);
+            if (d < r) {
+                const int p0 = d < half ? d : d - half;
+                float y[4], c0[4], c1[4];
+                normed(i + (d < half ? half : -half), y);
+                load4(cs + 2 * p0, c0);
+                load4(cs + 2 * p0 + 4, c1);
+                const float c[4] = {c0[0], c0[2], c1[0], c1[2]}, sn[4] = {c0[1], c0[3], c1[1], c1[3]};
+#pragma unroll
+                for (int u = 0; u < 4; ++u) x[u] = d < half ? x[u] * c[u] - y[u] * sn[u] : x[u] * c[u] + y[u] * sn[u];
+            }
+            if (g < q4) {
+                const float f = factor ? factor[h] : 1.f;
+#pragma unroll
+                for (int u = 0; u < 4; ++u) x[u] *= f;
+                store4(q_out + (size_t)t * q_stride + i, x);
+            } else if (page >= 0) {
+                store4(k_cache + (((size_t)page * nkv + h) * RB_PAGE + (pos % RB_PAGE)) * hdp + d, x);
+            }
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < nq * hdp; i += blockDim.x) {
         const int h = i / hdp, d = i - h * hdp;
         float v = 0.f;
         if (d < hd) v = turned(buf + h * hd, d, r, neighbours != 0, cs) * (factor ? factor[h] : 1.f);
         q_out[(size_t)t * q_stride + i] = from_f32<AT>(v);
     }
-    const int pos = positions[t];
-    const int page = block_table[(size_t)slot * max_pages + pos / RB_PAGE];
     if (page < 0) return;
     for (int i = threadIdx.x; i < nkv * hdp; i += blockDim.x) {
         const int h = i / hdp, d = i - h * hdp;
@@ -264,8 +318,12 @@ extern "C" int rb_wide_norm_rope_cache(const void* in, int in_dtype, int n_in, l
     if (T <= 0) return RB_OK;
     if (nq <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || hdp < hd || hdp < vd || rot < 0 || (rot & 1) || rot > hd || n_in < 1)
         return RB_ERR_BAD_SIZE;
-    const size_t smem = (size_t)((nq + nkv) * hd + 33) * sizeof(float);
+    const size_t smem = (size_t)((nq + nkv) * hd + 64) * sizeof(float);
     if (smem > 200 * 1024) return RB_ERR_BAD_SIZE;
+    const size_t isz = in_dtype == RB_F32 ? 4 : 2, asz = act_dtype == RB_F32 ? 4 : 2;
+    const int vec = hd == hdp && vd == hdp && (hd & 3) == 0 && (!cos_sin || (!neighbours && rot % 8 == 0)) && ((row_stride | q_stride) & 3) == 0 &&
+                    (in_stride & 3) == 0 && ((uintptr_t)in & (4 * isz - 1)) == 0 && (((uintptr_t)cos_sin | (uintptr_t)wq | (uintptr_t)wk) & 15) == 0 &&
+                    (((uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & (4 * asz - 1)) == 0;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
 #define RB_WN(IT, AT)                                                                                                    \
@@ -275,9 +333,9 @@ extern "C" int rb_wide_norm_rope_cache(const void* in, int in_dtype, int n_in, l
             cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
             if (e != cudaSuccess) return (int)e;                                                                         \
         }                                                                                                                \
-        RB_LAUNCH((k), dim3(T), dim3(256), smem, s, (const IT*)in, n_in, (size_t)in_stride, row_stride, nq, nkv, hd, vd, \
+        RB_LAUNCH((k), dim3(T), dim3(T > 296 ? 256 : 1024), smem, s, (const IT*)in, n_in, (size_t)in_stride, row_stride, nq, nkv, hd, vd, \
                   hdp, wq, wk, eps, factor, cos_sin, rot, neighbours, (AT*)q_out, q_stride, (AT*)k_cache, (AT*)v_cache,  \
-                  positions, slot_of_token, block_table, max_pages);                                                     \
+                  positions, slot_of_token, block_table, max_pages, vec);                                                \
     } while (0)
     if (in_dtype == RB_F32 && act_dtype == RB_BF16) RB_WN(float, bf);
     else if (in_dtype == RB_BF16 && act_dtype == RB_BF16) RB_WN(bf, bf);

@@ -204,8 +204,10 @@ def _lib():
                                       _vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _vp]
         lib.rb_mlstm_blocks.argtypes = [_vp, _i, _i, _ll, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp,
                                         _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp]
-        lib.rb_rglru_gates.argtypes = [_vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp]
-        lib.rb_rglru_scan.argtypes = [_vp, _vp, _i, _vp, _i, _i, _ll, _i, _f, _vp, _vp, _vp, _i, _vp, _i, _i, _vp]
+        lib.rb_rglru_gates.argtypes = [_vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _vp]
+        lib.rb_mlstm_chain.argtypes = [_vp, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _vp, _vp, _vp,
+                                       _vp, _vp, _i, _vp, _vp]
+        lib.rb_rglru_scan.argtypes = [_vp, _i, _vp, _i, _i, _ll, _i, _f, _vp, _vp, _vp, _i, _vp, _i, _i, _vp]
         lib.rb_rglru_step.argtypes = [_vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _ll, _i, _f, _vp, _vp, _vp, _i,
                                       _i, _vp]
         lib.rb_softcap.argtypes = [_vp, _ll, _f, _f, _vp]
@@ -874,6 +876,24 @@ def _row_scale(rowscale, m: int, what: str):
     if sumsq.dtype != torch.float32 or sumsq.dim() != 2 or sumsq.stride(1) != 1 or sumsq.shape[1] < m:
         raise KernelError(f"{what}: the rows' sums of squares must be float32 [groups, >= rows]")
     return _ptr(sumsq), sumsq.shape[0], sumsq.stride(0), float(eps)
+
+
+@_profiled(lambda a, facts: (a["w"].numel() * 2 + _rows(a) * (a["w"].shape[1] + a["w"].shape[0]) * 2, 2 * _rows(a) * a["w"].numel()))
+def gemm_tcgen05_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str, bias: Optional[torch.Tensor] = None,
+                     m: Optional[int] = None) -> bool:
+    """out bfloat16 [M, N] = act(x . w^T (+ bias)) for more than 256 rows and at least 256 features, the activation (see ``unary_act``)
+    in the product's epilogue.  False when the kernel does not take the sizes or the layout (use the two kernels)."""
+    M = x.shape[0] if m is None else m
+    N, K = w.shape
+    if M <= 256 or N < 256 or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or x.stride(1) != 1 or \
+            not w.is_contiguous() or x.shape[1] != K or out.shape[1] != N or out.stride(1) != 1:
+        return False
+    rc = _lib().rb_gemm_tcgen05(_ptr(x), _ptr(w), _f32vec(bias, N, "gemm_tcgen05_act: bias"), _ptr(out), BF16, M, N, K, x.stride(0),
+                                out.stride(0), 1, 0, 0, -1 - PLAIN_ACTS[act], _ptr(status_word(x.device)), _stream())
+    if rc in (10001, 10003):
+        return False
+    _check(rc, "gemm_tcgen05_act")
+    return True
 
 
 @_profiled(lambda a, facts: _cost.gated_linear(_rows(a), a["w"].shape[0], a["w"].shape[1], 2, 2, 2))
@@ -2028,6 +2048,13 @@ def pair_norm(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tens
 MLSTM_BLOCK = 64        # tokens a block of mlstm_blocks
 
 
+def mlstm_chains(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, dim: int, vdim: int) -> bool:
+    """Whether ``mlstm_blocks`` runs on the tensor cores, the state in registers from block to block: bfloat16 rows in one piece, heads
+    of 64, 128, 192 or 256 (values a multiple of 32), every head on a 16-byte boundary."""
+    return (proj.dtype == torch.bfloat16 and proj.dim() == 2 and dim % 64 == 0 and dim <= 256 and vdim % 32 == 0 and
+            (proj.stride(0) | q_off | k_off | v_off) % 8 == 0 and proj.data_ptr() % 16 == 0)
+
+
 def _mlstm_states(S, n, m, heads, dim, vdim, what):
     for t, shape, name in ((S, (heads, dim, vdim), "S"), (n, (heads, dim), "n"), (m, (heads, 2), "m")):
         if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or tuple(t.shape[1:]) != shape):
@@ -2088,6 +2115,16 @@ def mlstm_blocks(proj: torch.Tensor, n_tokens: int, q_off: int, k_off: int, v_of
     _mlstm_states(S, n, None, heads, dim, vdim, "mlstm_blocks")
     cols = _mlstm_cols(proj, q_off, k_off, v_off, heads, dim, vdim, out, den, n_tokens, "mlstm_blocks")
     blocks = n_tokens // MLSTM_BLOCK + n_seqs
+    if mlstm_chains(proj, q_off, k_off, v_off, dim, vdim):
+        planes = torch.empty((blocks, heads, 3, MLSTM_BLOCK, MLSTM_BLOCK), dtype=torch.bfloat16, device=proj.device)
+        ec, wt, decay = torch.split(torch.empty(2 * heads * n_tokens + blocks * heads, dtype=torch.float32, device=proj.device),
+                                    [heads * n_tokens, heads * n_tokens, blocks * heads])
+        rc = _lib().rb_mlstm_chain(_ptr(proj), proj.stride(0), q_off, k_off, v_off, float(q_scale), float(eps), heads, dim, vdim,
+                                   _ptr(log_keep), _ptr(log_add), _ptr(em), n_tokens, _ptr(S), _ptr(n), _i32(seq_slot, "seq_slot"),
+                                   _i32(cu_q, "cu_q"), n_seqs, blocks, _ptr(planes), _ptr(ec), _ptr(wt), _ptr(decay), _ptr(out),
+                                   out.stride(0), _ptr(den), _stream())
+        _check(rc, "mlstm_chain")
+        return
     work = torch.empty(blocks * heads * (dim * vdim + dim + 1 + MLSTM_BLOCK * MLSTM_BLOCK), dtype=torch.float32, device=proj.device)
     sizes = [blocks * heads * MLSTM_BLOCK * MLSTM_BLOCK, blocks * heads * dim * vdim, blocks * heads * dim, blocks * heads]
     scores, sums, sums_n, decay = torch.split(work, sizes)
@@ -2119,28 +2156,29 @@ def _branch(y, width, what):
 @_profiled(lambda a, facts: (a["n_tokens"] * a["u"].shape[1] * 12 + 2 * a["ra"].numel() * _esz(a["ra"]),
                              4 * a["n_tokens"] * a["u"].shape[1] * a["ra"].shape[1]))
 def rglru_gates(u: torch.Tensor, n_tokens: int, ra: torch.Tensor, ri: torch.Tensor, ra_b: torch.Tensor, ri_b: torch.Tensor,
-                rate: torch.Tensor, a: torch.Tensor, x: torch.Tensor):
-    """Decay ``a`` = e^(rate * r) and input ``x`` = sqrt(1 - a^2) i u of every token and channel (float32 [T, width]), r and i the
+                rate: torch.Tensor, ax: torch.Tensor):
+    """``ax`` float32 [T, width, 2]: the decay a = e^(rate * r) and the input sqrt(1 - a^2) i u of every token and channel, r and i the
     sigmoids of the block products of ``u`` (float32 [T, width]) with ``ra`` and ``ri`` [blocks, part, part] plus their biases."""
     args = _rglru_weights(u, ra, ri, ra_b, ri_b, rate, "rglru_gates")
-    for t in (a, x):
-        if t.dtype != torch.float32 or not t.is_contiguous() or t.shape[-1] != u.shape[-1] or t.shape[0] < n_tokens:
-            raise KernelError("rglru_gates: results must be contiguous float32 [T, width]")
-    _check(_lib().rb_rglru_gates(*args, n_tokens, _ptr(a), _ptr(x), _stream()), "rglru_gates")
+    if ax.dtype != torch.float32 or not ax.is_contiguous() or tuple(ax.shape[1:]) != (u.shape[-1], 2) or ax.shape[0] < n_tokens:
+        raise KernelError("rglru_gates: the result must be contiguous float32 [T, width, 2]")
+    _check(_lib().rb_rglru_gates(*args, n_tokens, _ptr(ax), _stream()), "rglru_gates")
 
 
-@_profiled(lambda a, facts: (a["n_tokens"] * a["a"].shape[1] * (8 + _esz(a["y"]) * _n_in(a["y"]) + _esz(a["out"])) + 8 * a["n_seqs"] * a["a"].shape[1],
-                             14 * a["n_tokens"] * a["a"].shape[1]))
-def rglru_scan(a: torch.Tensor, x: torch.Tensor, n_tokens: int, y: torch.Tensor, factor: float, state: torch.Tensor, seq_slot: torch.Tensor,
+@_profiled(lambda a, facts: (a["n_tokens"] * a["ax"].shape[1] * (8 + _esz(a["y"]) * _n_in(a["y"]) + _esz(a["out"])) + 8 * a["n_seqs"] * a["ax"].shape[1],
+                             14 * a["n_tokens"] * a["ax"].shape[1]))
+def rglru_scan(ax: torch.Tensor, n_tokens: int, y: torch.Tensor, factor: float, state: torch.Tensor, seq_slot: torch.Tensor,
                cu_q: torch.Tensor, n_seqs: int, out: torch.Tensor):
-    """S = a S + x along every sequence from ``state`` (float32 [slots, width], which receives the last one); ``out`` [T, width]
+    """S = a S + x, ``ax`` float32 [T, width, 2] the pairs (a, x), along every sequence from ``state`` (float32 [slots, width], which receives the last one); ``out`` [T, width]
     (any row stride) = S * gelu_tanh(y) * factor, y columns of the projection rows ([T, ..] or partial sums [S, T, ..])."""
-    width = a.shape[-1]
+    width = ax.shape[1]
+    if ax.dtype != torch.float32 or not ax.is_contiguous() or ax.shape[0] < n_tokens or ax.shape[2] != 2:
+        raise KernelError("rglru_scan: ax must be contiguous float32 [T, width, 2]")
     if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (width,):
         raise KernelError("rglru_scan: state must be contiguous float32 [slots, width]")
     if out.stride(-1) != 1 or out.shape[-1] < width:
         raise KernelError("rglru_scan: out must be [T, width]")
-    rc = _lib().rb_rglru_scan(_ptr(a), _ptr(x), width, *_branch(y, width, "rglru_scan"), float(factor), _ptr(state),
+    rc = _lib().rb_rglru_scan(_ptr(ax), width, *_branch(y, width, "rglru_scan"), float(factor), _ptr(state),
                               _i32(seq_slot, "seq_slot"), _i32(cu_q, "cu_q"), n_seqs, _ptr(out), dtype_code(out.dtype), out.stride(0),
                               _stream())
     _check(rc, "rglru_scan")

@@ -147,6 +147,14 @@ class Linear:
         return out
 
     @_labelled
+    def forward_act(self, x: torch.Tensor, m: int, act: str) -> Optional[torch.Tensor]:
+        """[M, N] = act(x . W^T (+ bias)) in one kernel, or None when this step's product cannot be done that way."""
+        if not self._tensor_core(x) or self._splits(m) != 1:
+            return None
+        out = torch.empty((m, self.n), dtype=torch.bfloat16, device=x.device)
+        return out if kernels.gemm_tcgen05_act(x, self.weight, out, act, self.bias, m) else None
+
+    @_labelled
     def forward_gated_pair(self, x: torch.Tensor, m: int, rowscale=None) -> Optional[torch.Tensor]:
         """The same for few rows when the sum over K is split in two: the two halves' blocks form a
         cluster and the activation is applied where they meet, so no second kernel waits for partial

@@ -112,7 +112,7 @@ class GatedMLP(FeedForward):
 @register_feed_forward("dense_mlp")
 class DenseMLP(FeedForward):
     """down(act(up(x))): no gate.  The activation is a parameter: "gelu" (z / 2 * (1 + erf(z / sqrt 2))), "gelu_tanh" or "silu",
-    computed in 32-bit."""
+    computed in 32-bit: for prompts of more than 256 tokens in the product's epilogue, otherwise by a kernel of its own."""
 
     graph_safe = True
 
@@ -159,10 +159,12 @@ class DenseMLP(FeedForward):
         T = batch.n_tokens
         if isinstance(xn, DeferredNorm):
             xn = xn.materialize()
-        u = self.up.forward_auto(xn, T)            # [T, I] or [S, T, I] partial sums
-        h = torch.empty((T, self.inter), dtype=self.env.act_dtype, device=self.env.device)
-        with scope(op="activation"):
-            kernels.unary_act(u, h, self.act)
+        h = self.up.forward_act(xn, T, self.act)       # prompts: the activation in the product's epilogue
+        if h is None:
+            u = self.up.forward_auto(xn, T)            # [T, I] or [S, T, I] partial sums
+            h = torch.empty((T, self.inter), dtype=self.env.act_dtype, device=self.env.device)
+            with scope(op="activation"):
+                kernels.unary_act(u, h, self.act)
         if add_into is not None and self.down.forward_add(h, T, add_into):
             return None
         return self.down.forward_delta(h, T)

@@ -9,7 +9,7 @@
 
 What a sequence keeps, whatever its length: S and the convolution's last inputs, both 32-bit.  One stacked product makes both branches;
 one kernel convolves; prompts then take one kernel for the gates and one that scans (runs of tokens side by side), single tokens one
-kernel for everything.  From the projections on everything is 32-bit, the block products too (FMA on 32-bit inputs)."""
+kernel for everything.  From the projections on everything is 32-bit, the block products too."""
 from __future__ import annotations
 
 from typing import Dict, List, Optional
@@ -142,11 +142,11 @@ class RealGatedLRU(Mixer):
             with scope(op="rglru_step"):
                 kernels.rglru_step(u, T, *weights, proj[..., :self.width], self.result_factor, view.state, batch.slot_of_token, out)
             return out
-        a, x = torch.empty_like(u), torch.empty_like(u)
+        ax = torch.empty((T, self.width, 2), dtype=torch.float32, device=dev)
         with scope(op="rglru_gates"):
-            kernels.rglru_gates(u, T, *weights, a, x)
+            kernels.rglru_gates(u, T, *weights, ax)
         with scope(op="rglru_scan"):
-            kernels.rglru_scan(a, x, T, proj[..., :self.width], self.result_factor, view.state, batch.seq_slot, batch.cu_q, batch.n_seqs, out)
+            kernels.rglru_scan(ax, T, proj[..., :self.width], self.result_factor, view.state, batch.seq_slot, batch.cu_q, batch.n_seqs, out)
         return out
 
     def forward(self, xn, batch, view):

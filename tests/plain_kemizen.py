@@ -97,8 +97,9 @@ def weights(scores, positions, size):
     return torch.softmax(scores.masked_fill(~seen[None], float("-inf")), dim=-1)
 
 
-def mlstm_scan(q, k, v, i, f, state=None):
-    """q, k [T, H, dim] (q already scaled), v [T, H, vdim], i and f [T, H] log gates: (o [T, H, vdim], (S, n, m))."""
+def mlstm_scan(q, k, v, i, f, state=None, below=None):
+    """q, k [T, H, dim] (q already scaled), v [T, H, vdim], i and f [T, H] log gates: (o [T, H, vdim], (S, n, m)).  ``below``: a list that
+    receives every token's divisors [H]."""
     T, H, dim = q.shape
     if state is None:
         state = (torch.zeros((H, dim, v.shape[2]), dtype=q.dtype), torch.zeros((H, dim), dtype=q.dtype), torch.zeros(H, dtype=q.dtype))
@@ -110,8 +111,10 @@ def mlstm_scan(q, k, v, i, f, state=None):
         S = keep[:, None, None] * S + add[:, None, None] * k[t][:, :, None] * v[t][:, None, :]
         n = keep[:, None] * n + add[:, None] * k[t]
         m = m2
-        below = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
-        o[t] = torch.einsum("hkv,hk->hv", S, q[t]) / below[:, None]
+        d = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        o[t] = torch.einsum("hkv,hk->hv", S, q[t]) / d[:, None]
+        if below is not None:
+            below.append(d)
     return o, (S, n, m)
 
 

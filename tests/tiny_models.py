@@ -507,3 +507,105 @@ def write_ravelorn(folder, cfg_dict, seed, std=0.08, fixed_routes=True, slow_dec
     with open(cfg_path, "w") as f:
         json.dump(cfg, f)
     return folder
+
+
+# ---- Kemizen: norms on the sublayers' results, weights around zero; a matrix memory, differential attention (with the keys and values of
+# an earlier layer), attention behind convolutions beside a recurrent block; feed-forwards without a gate ---------------------------
+def _kmem(heads, dim, vdim, cap, ff):
+    return {"type": "mlstm", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def _krot(base, dims, scaling=None):
+    r = {"base": base, "dims": dims}
+    if scaling is not None:
+        r["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return r
+
+
+def _kdiff(heads, kv_heads, dim, vdim, scale, diff, rot, ff, size=None, softcap=None, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "diff": diff, "rot": rot}
+    for k, v in (("mask", None if size is None else {"size": size}), ("softcap", softcap), ("kv_from", kv_from)):
+        if v is not None:
+            m[k] = v
+    return {"type": "attention", "mixer": m, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def _kpar(heads, kv_heads, dim, vdim, scale, conv, rot, width, blocks, rconv, ff):
+    return {"type": "parallel", "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "conv": conv, "rot": rot},
+                                          "right": {"width": width, "blocks": blocks, "conv": rconv}},
+            "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+# KA: head sizes that no attention kernel takes as they are, part of a head turning, a reader that sees further back than the layer
+# whose keys it uses and one that sees less far, layers without feed-forward
+_KA_ROT = _krot(10000.0, 8, (4.0, 64, 8.0, 1.0))
+KEMIZEN_A = {
+    "architecture": "Kemizen", "vocab": 211, "width": 64, "embedding": {"scale": 1.5}, "norm": {"eps": 1e-6},
+    "layers": [_kdiff(4, 2, 12, 20, 0.5, 0.3, _KA_ROT, 96, size=50, softcap=3.0),
+               _kmem(3, 12, 20, 4.0, None),
+               _kpar(6, 2, 20, 12, 0.3, 3, _krot(500.0, 12), 48, 3, 4, 40),
+               _kdiff(4, 2, 12, 20, 0.7, 0.5, _KA_ROT, None, size=90, softcap=5.0, kv_from=0),
+               _kmem(2, 8, 8, 15.0, 72),
+               _kdiff(4, 2, 12, 20, 0.4, 0.2, _KA_ROT, 48, size=7, softcap=2.0, kv_from=0)],
+}
+# KB: sizes that the tensor-core kernels take, windows across page borders, eight query rows a key/value head
+_KB_ROT = _krot(1e6, 64, (8.0, 256, 32.0, 1.0))
+KEMIZEN_B = {
+    "architecture": "Kemizen", "vocab": 333, "width": 128, "embedding": {"scale": 0.8}, "norm": {"eps": 1e-5},
+    "layers": [_kmem(2, 64, 96, 15.0, 128),
+               _kdiff(4, 1, 64, 128, 0.125, 0.4, _KB_ROT, 320, size=130, softcap=20.0),
+               _kpar(4, 2, 128, 128, 0.09, 4, _krot(10000.0, 128), 256, 2, 4, 192),
+               _kdiff(4, 1, 64, 128, 0.2, 0.6, _KB_ROT, 64, size=64, softcap=8.0, kv_from=1),
+               _kmem(1, 128, 32, 2.0, None),
+               _kpar(2, 1, 64, 64, 0.2, 2, _krot(300.0, 32), 96, 4, 3, None)],
+}
+# KC: one head and sizes that are multiples of nothing, convolutions of one tap and of more taps than a short step has tokens, a window of
+# one token, no window, no cap, no ramp, a gate cap that lets the exponents grow
+KEMIZEN_C = {
+    "architecture": "Kemizen", "vocab": 97, "width": 72, "embedding": {"scale": 1.0}, "norm": {"eps": 3e-5},
+    "layers": [_kpar(3, 3, 10, 7, 0.6, 1, _krot(50.0, 4), 30, 3, 6, 50),
+               _kdiff(1, 1, 6, 7, 1.0, 0.8, _krot(100.0, 2), 33, size=1),
+               _kdiff(3, 3, 10, 31, 0.4, 0.1, _krot(100.0, 10), 20),
+               _kmem(5, 9, 5, 60.0, 30),
+               _kpar(2, 1, 24, 40, 0.3, 7, _krot(1000.0, 24), 13, 1, 1, None),
+               _kdiff(3, 3, 10, 31, 0.6, 0.5, _krot(100.0, 10), None, size=300, kv_from=2)],
+}
+KEMIZEN = {"KA": KEMIZEN_A, "KB": KEMIZEN_B, "KC": KEMIZEN_C}
+
+
+def write_kemizen(folder, cfg_dict, seed, std=0.08, slow=False):
+    """A Kemizen model folder with random weights: gates of the memory that move over several units and forget over tens of tokens
+    (``slow``: hundreds), channels that decay over tens of tokens (``slow``: thousands), differences whose factor is not the constant alone."""
+    from safetensors.torch import load_file, save_file
+    write_model(folder, cfg_dict, seed)
+    path = os.path.join(folder, "model.safetensors")
+    w = load_file(path)
+    for k in sorted(w):
+        t = w[k].float()
+        if k.endswith(".conv"):
+            t = t * 20.0
+        elif k == "embed":
+            t = t * 40.0
+        elif k.endswith((".mix.i", ".mix.f")):
+            t = t * (2.0 * std / 0.02)
+        elif t.dim() == 2 and not k.endswith((".ra.b", ".ri.b")):
+            t = t * (std / 0.02)
+        elif t.dim() == 3:
+            t = t * (3.0 * std / 0.02)
+        elif k.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
+            t = t * (60.0 / t.numel() ** 0.5)
+        elif k.endswith(".f.b"):
+            t = t * 25.0 + (7.0 if slow else 2.0)
+        elif k.endswith(".i.b"):
+            t = t * 25.0
+        elif k.endswith(".lam"):
+            t = (t - 1.0) * 10.0 - (9.0 if slow else 4.0)
+        elif k.endswith((".norm1", ".norm2", "final.norm")):
+            t = (t - 1.0) * 3.0
+        elif k.endswith((".norm", ".out")):
+            t = 1.0 + 3.0 * (t - 1.0)
+        elif k.endswith(".b"):
+            t = t * 15.0
+        w[k] = t.to(torch.bfloat16)
+    save_file(w, path)
+    return folder
