@@ -51,16 +51,28 @@ struct Cols {
     size_t in_stride;
     int row_stride;
     __device__ __forceinline__ float operator()(int t, int col) const {
-        const IT* x = p + (size_t)t * row_stride + col;
-        float v = to_f32(x[0]);
-        for (int s = 1; s < n_in; s += 4) {                 // four partial sums in flight, added in order
-            float y[4];
+        const int cols[1] = {col};
+        float v[1];
+        many<1>(t, cols, v);
+        return v[0];
+    }
+    // N columns at a time: four partial sums of each in flight, added in order
+    template <int N>
+    __device__ __forceinline__ void many(int t, const int (&col)[N], float (&v)[N]) const {
+        const IT* x = p + (size_t)t * row_stride;
 #pragma unroll
-            for (int j = 0; j < 4; ++j) y[j] = s + j < n_in ? to_f32(x[(size_t)(s + j) * in_stride]) : 0.f;
+        for (int e = 0; e < N; ++e) v[e] = to_f32(x[col[e]]);
+        for (int s = 1; s < n_in; s += 4) {
+            float y[4][N];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) v += y[j];
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int e = 0; e < N; ++e) y[j][e] = s + j < n_in ? to_f32(x[(size_t)(s + j) * in_stride + col[e]]) : 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int e = 0; e < N; ++e) v[e] += y[j][e];
         }
-        return v;
     }
 };
 
@@ -119,14 +131,15 @@ mlstm_gates_kernel(const Cols<float> g, int i_off, int f_off, float cap, int hea
 }
 
 // ---- one token a sequence -------------------------------------------------------------------------------------------
-template <typename IT>
-__global__ void __launch_bounds__(256)
+template <typename IT, int V>
+__global__ void __launch_bounds__(256, 3)
 mlstm_step_kernel(const Cols<IT> x, int q_off, int k_off, int v_off, const Cols<float> g, int i_off, int f_off, float cap,
                   float q_scale, float eps, int heads, int dim, int vdim, float* __restrict__ S_state, float* __restrict__ n_state,
                   float* __restrict__ m_state, const int* __restrict__ seq_slot, const int* __restrict__ cu_q,
                   const int* __restrict__ positions, float* __restrict__ out, int ld_out, float* __restrict__ den) {
     pdl_trigger();
     pdl_wait();
+    constexpr int LPR = 32 / V, RG = 256 / LPR, R = 8;      // threads a row of 32 columns, rows side by side, rows in flight a thread
     extern __shared__ __align__(16) float sm[];
     __shared__ float part[8][32];
     __shared__ float red[33];
@@ -137,28 +150,57 @@ mlstm_step_kernel(const Cols<IT> x, int q_off, int k_off, int v_off, const Cols<
     if (slot < 0) return;
     const int t = cu_q[b];
     if (cu_q[b + 1] <= t) return;
-    const int pos = positions[t];
+    const bool last = blockIdx.x == gridDim.x - 1;          // this block does n, the divisor and m
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int col = (threadIdx.x % LPR) * V, j = blockIdx.x * 32 + col, r0 = threadIdx.x / LPR;
+    const bool mine_cols = !last && j < vdim;               // (V divides vdim)
+    float* S = S_state + (((size_t)slot * heads + h) * dim) * vdim + j;
+    float s[R][V];
+    auto ask = [&](int base) {
+#pragma unroll
+        for (int u = 0; u < R; ++u) {
+            const int c = base + r0 + u * RG;
+            if (c < dim) {
+                if constexpr (V == 4) *reinterpret_cast<float4*>(s[u]) = *reinterpret_cast<const float4*>(S + (size_t)c * vdim);
+                else s[u][0] = S[(size_t)c * vdim];
+            }
+        }
+    };
+    if (mine_cols) ask(0);                                  // the state travels while the gates are formed
+    const int pos = positions[t];
     float* mine = m_state + ((size_t)slot * heads + h) * 2;
-    const float i = capped_gate(g(t, i_off + h), cap), f = log_sigmoid(capped_gate(g(t, f_off + h), cap));
-    const float m0 = mine[(pos + 1) & 1], m1 = fmaxf(f + m0, i);
+    const float m0 = mine[(pos + 1) & 1];
+    const int gate_cols[2] = {i_off + h, f_off + h};
+    float gate[2];
+    g.template many<2>(t, gate_cols, gate);
+    // q, k and v of the first pass together (a column past the end stands for the last one)
+    const int c_first = min((int)threadIdx.x, dim - 1), j_first = mine_cols ? j : 0;
+    int row_cols[2 + V];
+    float row[2 + V];
+    row_cols[0] = q_off + h * dim + c_first; row_cols[1] = k_off + h * dim + c_first;
+#pragma unroll
+    for (int e = 0; e < V; ++e) row_cols[2 + e] = v_off + h * vdim + j_first + e;
+    x.template many<2 + V>(t, row_cols, row);
+    const float i = capped_gate(gate[0], cap), f = log_sigmoid(capped_gate(gate[1], cap));
+    const float m1 = fmaxf(f + m0, i);
     const float keep = expf(f + m0 - m1), add = expf(i - m1);
-    for (int c = threadIdx.x; c < dim; c += 256) {
+    if (threadIdx.x < dim) {
+        qs[threadIdx.x] = row[0] * q_scale;
+        ks[threadIdx.x] = row[1] * add;
+    }
+    for (int c = threadIdx.x + 256; c < dim; c += 256) {
         qs[c] = x(t, q_off + h * dim + c) * q_scale;
         ks[c] = x(t, k_off + h * dim + c) * add;
     }
-    const bool last = blockIdx.x == gridDim.x - 1;          // this block does n, the divisor and m
-    const int j = blockIdx.x * 32 + lane;
-    float v = 0.f;
-    if (!last && j < vdim) v = x(t, v_off + h * vdim + j);
+    const float* v = row + 2;
     __syncthreads();
     if (last) {
         float* n = n_state + ((size_t)slot * heads + h) * dim;
         float acc = 0.f;
         for (int c = threadIdx.x; c < dim; c += 256) {
-            const float s = fmaf(keep, n[c], ks[c]);
-            n[c] = s;
-            acc = fmaf(s, qs[c], acc);
+            const float w = fmaf(keep, n[c], ks[c]);
+            n[c] = w;
+            acc = fmaf(w, qs[c], acc);
         }
         acc = block_sum(acc, red);
         if (threadIdx.x == 0) {
@@ -167,34 +209,40 @@ mlstm_step_kernel(const Cols<IT> x, int q_off, int k_off, int v_off, const Cols<
         }
         return;
     }
-    float* S = S_state + (((size_t)slot * heads + h) * dim) * vdim + j;
-    float acc = 0.f;
-    if (j < vdim) {
-        int c = warp;
-        for (; c + 56 < dim; c += 64) {           // eight rows' loads in flight
-            float s[8];
+    float acc[V] = {};
+    if (mine_cols) {
+        for (int base = 0;;) {
 #pragma unroll
-            for (int u = 0; u < 8; ++u) s[u] = S[(size_t)(c + 8 * u) * vdim];
+            for (int u = 0; u < R; ++u) {
+                const int c = base + r0 + u * RG;
+                if (c < dim) {
 #pragma unroll
-            for (int u = 0; u < 8; ++u) {
-                s[u] = fmaf(ks[c + 8 * u], v, keep * s[u]);
-                S[(size_t)(c + 8 * u) * vdim] = s[u];
-                acc = fmaf(s[u], qs[c + 8 * u], acc);
+                    for (int e = 0; e < V; ++e) {
+                        s[u][e] = fmaf(ks[c], v[e], keep * s[u][e]);
+                        acc[e] = fmaf(s[u][e], qs[c], acc[e]);
+                    }
+                    if constexpr (V == 4) *reinterpret_cast<float4*>(S + (size_t)c * vdim) = *reinterpret_cast<const float4*>(s[u]);
+                    else S[(size_t)c * vdim] = s[u][0];
+                }
             }
-        }
-        for (; c < dim; c += 8) {
-            const float s = fmaf(ks[c], v, keep * S[(size_t)c * vdim]);
-            S[(size_t)c * vdim] = s;
-            acc = fmaf(s, qs[c], acc);
+            base += R * RG;
+            if (base >= dim) break;
+            ask(base);
         }
     }
-    part[warp][lane] = acc;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+#pragma unroll
+        for (int o = LPR; o < 32; o <<= 1) acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], o);
+        if (lane < LPR) part[warp][col + e] = acc[e];
+    }
     __syncthreads();
-    if (warp == 0 && j < vdim) {
+    const int jo = blockIdx.x * 32 + lane;
+    if (warp == 0 && jo < vdim) {
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < 8; ++w) o += part[w][lane];
-        out[(size_t)t * ld_out + (size_t)h * vdim + j] = o;
+        out[(size_t)t * ld_out + (size_t)h * vdim + jo] = o;
     }
 }
 
@@ -626,19 +674,28 @@ mlstm_chain_kernel(const Rows16 x, int q_off, int k_off, int v_off, float eps, i
             load_tile<CB>(reinterpret_cast<bf16*>(vb + Z::V), pl, CB, 3 * CB, 3 * CB, tid, 256);
         }
         cp_async_commit();
-        if (tid < 2 * CB) {
-            const int t = tid & (CB - 1);
-            tok[(c & 1) * 2 * CB + tid] = t < m ? (tid < CB ? ec : wt)[(size_t)h * T + t0 + t] : 0.f;
-        }
     };
+    // a token's two factors and the block's decay travel in registers until the block before them is done
+    float next_tok = 0.f, next_decay = 0.f;
+    auto ask = [&](int c) {
+        const int t = tid & (CB - 1);
+        next_decay = block_decay[(size_t)(first + c) * heads + h];
+        if (tid < 2 * CB) next_tok = c * CB + t < n_tok ? (tid < CB ? ec : wt)[(size_t)h * T + t_begin + c * CB + t] : 0.f;
+    };
+    auto keep = [&](int c) {
+        if (tid < 2 * CB) tok[(c & 1) * 2 * CB + tid] = next_tok;
+    };
+    ask(0);
 
     if (n_role) {
         // n and the divisors: a thread a dimension for the sums over tokens, a warp eight tokens for the products with q
         float* ns = red;
         float n = tid < DIM ? n_state[((size_t)slot * heads + h) * DIM + tid] : 0.f;
         fetch(0);
+        keep(0);
         for (int c = 0; c < nb; ++c) {
-            if (c + 1 < nb) { fetch(c + 1); cp_async_wait<1>(); }
+            const float decay = next_decay;
+            if (c + 1 < nb) { fetch(c + 1); ask(c + 1); cp_async_wait<1>(); }
             else cp_async_wait<0>();
             if (tid < DIM) ns[tid] = n;
             __syncthreads();
@@ -668,8 +725,9 @@ mlstm_chain_kernel(const Rows16 x, int q_off, int k_off, int v_off, float eps, i
 #pragma unroll 8
                 for (int s = 0; s < CB; ++s)
                     sum = fmaf(te[CB + s], __bfloat162float(*reinterpret_cast<const bf16*>(K + s * DIM * 2 + (((tid >> 3) ^ (s & 7)) << 4) + (tid & 7) * 2)), sum);
-                n = fmaf(block_decay[(size_t)(first + c) * heads + h], n, sum);
+                n = fmaf(decay, n, sum);
             }
+            if (c + 1 < nb) keep(c + 1);
             __syncthreads();
         }
         if (tid < DIM) n_state[((size_t)slot * heads + h) * DIM + tid] = n;
@@ -686,8 +744,10 @@ mlstm_chain_kernel(const Rows16 x, int q_off, int k_off, int v_off, float eps, i
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[j][e] = Sg[(size_t)(j * 8 + c0 + (e & 1)) * vdim + r0 + (e >> 1) * 8];
     fetch(0);
+    keep(0);
     for (int c = 0; c < nb; ++c) {
-        if (c + 1 < nb) { fetch(c + 1); cp_async_wait<1>(); }
+        const float decay = next_decay;
+        if (c + 1 < nb) { fetch(c + 1); ask(c + 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t qb = smem_addr(raw_sm + (c & 1) * Z::BUF), kb = qb + Z::QK, vb = kb + Z::QK, pb = vb + Z::V;
@@ -747,7 +807,6 @@ mlstm_chain_kernel(const Rows16 x, int q_off, int k_off, int v_off, float eps, i
             }
         }
         // the state after the block
-        const float decay = block_decay[(size_t)(first + c) * heads + h];
 #pragma unroll
         for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -777,6 +836,7 @@ mlstm_chain_kernel(const Rows16 x, int q_off, int k_off, int v_off, float eps, i
                     mma_bf16(st[2 * j + 1], a[i], kk[j][2], kk[j][3]);
                 }
         }
+        if (c + 1 < nb) keep(c + 1);              // (this place was last read before the block's first barrier)
         __syncthreads();                          // every part of the result is there, every tile has been read
         const int t0 = t_begin + c * CB, m = min(CB, n_tok - c * CB);
 #pragma unroll
@@ -829,9 +889,15 @@ extern "C" int rb_mlstm_step(const void* x, int x_dtype, int n_in, long long in_
     const size_t smem = (size_t)2 * dim * sizeof(float);
     const Cols<float> g{gates, g_n_in, (size_t)g_in_stride, g_row_stride};
 #define RB_MS(IT)                                                                                                             \
-    RB_LAUNCH((mlstm_step_kernel<IT>), grid, dim3(256), smem, (cudaStream_t)stream,                                           \
-              Cols<IT>{(const IT*)x, n_in, (size_t)in_stride, row_stride}, q_off, k_off, v_off, g, i_off, f_off, cap, q_scale, eps, \
-              heads, dim, vdim, S_state, n_state, m_state, seq_slot, cu_q, positions, out, ld_out, den)
+    do {                                                                                                                      \
+        const Cols<IT> c{(const IT*)x, n_in, (size_t)in_stride, row_stride};                                                  \
+        if (vdim % 4 == 0 && !((uintptr_t)S_state & 15))                                                                      \
+            RB_LAUNCH((mlstm_step_kernel<IT, 4>), grid, dim3(256), smem, (cudaStream_t)stream, c, q_off, k_off, v_off, g, i_off, f_off, \
+                      cap, q_scale, eps, heads, dim, vdim, S_state, n_state, m_state, seq_slot, cu_q, positions, out, ld_out, den); \
+        else                                                                                                                  \
+            RB_LAUNCH((mlstm_step_kernel<IT, 1>), grid, dim3(256), smem, (cudaStream_t)stream, c, q_off, k_off, v_off, g, i_off, f_off, \
+                      cap, q_scale, eps, heads, dim, vdim, S_state, n_state, m_state, seq_slot, cu_q, positions, out, ld_out, den); \
+    } while (0)
     if (x_dtype == RB_F32) RB_MS(float);
     else if (x_dtype == RB_BF16) RB_MS(__nv_bfloat16);
     else return RB_ERR_BAD_DTYPE;

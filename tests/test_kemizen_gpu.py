@@ -535,7 +535,8 @@ def test_every_mechanism_matters(model):
         m = L["mixer"]
         if L["type"] == "attention":
             if m.get("mask"):
-                paths.append((("layers", i, "mixer", "mask", "size"), m["mask"]["size"] + 1))
+                if m["mask"]["size"] < len(ids):
+                    paths.append((("layers", i, "mixer", "mask", "size"), m["mask"]["size"] + 1))
             if m.get("mask", {"size": 0})["size"] != 1:                 # (a window of one token leaves the scores no say)
                 paths.append((("layers", i, "mixer", "scale"), 0.5 * m["scale"]))
                 if m.get("softcap"):
