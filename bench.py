@@ -29,7 +29,9 @@ decoder (parallel layers with two norms, windowed attention that keeps the first
 in its denominator, values blended across layers), and ``--workload tibenex`` for the Tibenex decoder (layers that
 normalise after the sum, state-space mixers, latent attention with a rotated key part, attention with mixed heads), and
 ``--workload ravelorn`` for the Ravelorn decoder (norms on the sublayers' results only, the gated delta rule with a decay per
-key channel, and with a decay per head beside attention with a sink per head, routed experts with identity experts).  Sweeps, timelines and kernel
+key channel, and with a decay per head beside attention with a sink per head, routed experts with identity experts), and
+``--workload kemizen`` for the Kemizen decoder (a matrix memory with exponential gates, differential attention with a soft cap and
+shared keys and values, attention behind short convolutions beside a real-gated linear recurrent unit).  Sweeps, timelines and kernel
 measurements are ``python -m rocml_b200.measure``.
 
 The engine works on one GPU: for ``--gpus`` above 1 it says so and exits with 2.

@@ -703,23 +703,32 @@ mlstm_chain_kernel(const Rows16 x, int q_off, int k_off, int v_off, float eps, i
             const uint8_t* K = Q + Z::QK;
             const float* te = tok + (c & 1) * 2 * CB;
             const int t0 = t_begin + c * CB, m = min(CB, n_tok - c * CB);
-            for (int r = warp; r < m; r += 8) {
-                float acc = 0.f;
-                for (int d = lane * 8; d < DIM; d += 256) {
-                    const uint4 raw = *reinterpret_cast<const uint4*>(Q + r * DIM * 2 + (((d >> 3) ^ (r & 7)) << 4));
+            // eight tokens a warp, their sums side by side; lane u < 8 holds token u's divisor so far and its bound
+            const int mine_t = warp + 8 * lane;
+            float* dp = den + (size_t)(t0 + mine_t) * heads + h;
+            const bool has = lane < 8 && mine_t < m;
+            const float so_far = has ? *dp : 0.f, bound = has ? em[(size_t)h * T + t0 + mine_t] : 0.f;
+            float acc[8] = {};
+            for (int d = lane * 8; d < DIM; d += 256) {
+#pragma unroll
+                for (int r = 0; r < 8; ++r) {
+                    const int row = warp + 8 * r;
+                    const uint4 raw = *reinterpret_cast<const uint4*>(Q + row * DIM * 2 + (((d >> 3) ^ (row & 7)) << 4));
                     const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
                     for (int u = 0; u < 4; ++u) {
-                        acc = fmaf(__uint_as_float(w[u] << 16), ns[d + 2 * u], acc);
-                        acc = fmaf(__uint_as_float(w[u] & 0xFFFF0000u), ns[d + 2 * u + 1], acc);
+                        acc[r] = fmaf(__uint_as_float(w[u] << 16), ns[d + 2 * u], acc[r]);
+                        acc[r] = fmaf(__uint_as_float(w[u] & 0xFFFF0000u), ns[d + 2 * u + 1], acc[r]);
                     }
                 }
-                acc = warp_sum(acc);
-                if (lane == 0) {
-                    float* dp = den + (size_t)(t0 + r) * heads + h;
-                    *dp = fmaxf(fabsf(fmaf(te[r], acc, *dp)), em[(size_t)h * T + t0 + r]) + eps;
-                }
             }
+            float own = 0.f;
+#pragma unroll
+            for (int r = 0; r < 8; ++r) {
+                acc[r] = warp_sum(acc[r]);
+                if (lane == r) own = acc[r];
+            }
+            if (has) *dp = fmaxf(fabsf(fmaf(te[mine_t], own, so_far)), bound) + eps;
             if (tid < DIM) {
                 float sum = 0.f;
 #pragma unroll 8
